@@ -166,6 +166,16 @@ int32_t sp_cuda_engine_finalize(SpEngine* e);
  * names (crates/sapient-models/src/gguf_weights.rs:61-96,360-455), un-permute llama q/k rows (:114-154), split Phi
  * qkv (:273-330), create + finalize. max_ctx/max_batch 0 = file's context_length (capped at 8192) / 1. */
 int32_t sp_cuda_engine_from_gguf(const char* path, int32_t device, int32_t max_ctx, int32_t max_batch, SpEngine** out);
+/* Designs described by a configuration file instead of GGUF metadata (registry: sapient_b200/csrc/model_plan.h). The text of
+ * config.json names the architecture and every size and constant; compute_dtype is SP_BF16 (weights, matrix operands and
+ * cache in bf16 with f32 accumulation; the residual stream, norms, routing, angles and softmax in f32) or SP_F32
+ * (everything). Of *run only max_ctx, max_batch, max_tokens, device and kv_pages count. create_from_config is followed by
+ * sp_cuda_engine_set_tensor for every tensor (f32 / f16 / bf16, the file's names; a single number has dims {1}) and
+ * finalize; from_dir reads config.json and model.safetensors of a directory and returns a finalised engine.
+ * sp_cuda_arch_block: which block an architecture name runs with (0 Llama/Qwen, 1 Phi-2, 2 a layer plan). */
+int32_t sp_cuda_arch_block(const char* name, int32_t* block);
+int32_t sp_cuda_engine_create_from_config(const char* config_json, int32_t compute_dtype, const SpModelDesc* run, SpEngine** out);
+int32_t sp_cuda_engine_from_dir(const char* path, int32_t compute_dtype, const SpModelDesc* run, SpEngine** out);
 int32_t sp_cuda_engine_desc(const SpEngine* e, SpModelDesc* out);
 void sp_cuda_engine_destroy(SpEngine* e);
 /* Tensor parallelism (one process per GPU; Llama/Qwen block only). An engine created with tp_size > 1 keeps, of every
@@ -226,6 +236,11 @@ int32_t sp_cuda_forward_all_logits_cached(SpEngine* e, const uint32_t* ids, size
 /* Same for an explicit sequence slot (batched extension; the reference engine has exactly one sequence). */
 int32_t sp_cuda_forward_slot(SpEngine* e, int32_t slot, const uint32_t* ids, size_t n, int32_t all_positions,
                              float* logits_out);
+/* A mixed step: ids[i] is appended to slot slots[i] (a slot's tokens take consecutive positions in the order given), so
+ * portions of prompts and single decoded tokens run as one batch. rows[n_rows] (ascending token indices, may be empty)
+ * name the tokens whose logits[n_rows * vocab] / arg-max[n_rows] are written; either output may be NULL. */
+int32_t sp_cuda_forward_rows(SpEngine* e, const uint32_t* ids, const int32_t* slots, size_t n, const int32_t* rows, size_t n_rows,
+                             float* logits_out, uint32_t* argmax_out);
 /* One decode step for b sequences: ids[i] is appended to slot slots[i]. Either output may be NULL:
  * logits_out[b * vocab] (host) and/or argmax_out[b] (host; last-maximum tie rule). */
 int32_t sp_cuda_decode_batch(SpEngine* e, const uint32_t* ids, const int32_t* slots, int32_t b, float* logits_out,

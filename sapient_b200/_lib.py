@@ -77,6 +77,10 @@ SIGNATURES = {
     "sp_cuda_engine_set_tensor": (_i32, [_vp, C.c_char_p, _i32, _vp, _i32, _vp, _sz]),
     "sp_cuda_engine_finalize": (_i32, [_vp]),
     "sp_cuda_engine_from_gguf": (_i32, [C.c_char_p, _i32, _i32, _i32, C.POINTER(_vp)]),
+    "sp_cuda_arch_block": (_i32, [C.c_char_p, C.POINTER(_i32)]),
+    "sp_cuda_engine_create_from_config": (_i32, [C.c_char_p, _i32, C.POINTER(SpModelDesc), C.POINTER(_vp)]),
+    "sp_cuda_engine_from_dir": (_i32, [C.c_char_p, _i32, C.POINTER(SpModelDesc), C.POINTER(_vp)]),
+    "sp_cuda_forward_rows": (_i32, [_vp, _vp, _vp, _sz, _vp, _sz, _vp, _vp]),
     "sp_cuda_engine_desc": (_i32, [_vp, C.POINTER(SpModelDesc)]),
     "sp_cuda_engine_destroy": (None, [_vp]),
     "sp_cuda_engine_set_stream": (_i32, [_vp, _vp]),

@@ -10,6 +10,7 @@
 
 #include "batcher.h"
 #include "engine.h"
+#include "model_plan.h"
 #include "sp_common.cuh"
 
 using namespace sp;
@@ -29,6 +30,8 @@ struct SpEngine {
     Engine* e;
 };
 
+int sp_engine_from_config_impl(const char* text, size_t n, bool f32, const SpModelDesc& run, Engine** out);  // safetensors.cu
+int sp_engine_from_dir_impl(const char* dir, bool f32, const SpModelDesc& run, Engine** out);
 int sp_engine_from_gguf_impl(const char* path, int device, int max_ctx, int max_batch, Engine** out);  // gguf.cu
 namespace sp {
 int nccl_unique_id(const char* libpath, void* out, size_t cap);  // nccl_arm.cu
@@ -591,6 +594,56 @@ int32_t sp_cuda_engine_from_gguf(const char* path, int32_t device, int32_t max_c
     if (st != SP_OK) return st;
     *out = new SpEngine{eng};
     return SP_OK;
+    API_END
+}
+
+int32_t sp_cuda_arch_block(const char* name, int32_t* block) {
+    if (!name || !block) { set_error("null argument"); return SP_ERR_ARG; }
+    const ArchEntry* a = find_arch(name);
+    if (!a) { set_error(std::string("architecture '") + name + "' is not supported by the CUDA engine"); return SP_ERR_DTYPE; }
+    *block = a->block;
+    return SP_OK;
+}
+
+static int plan_compute_type(int32_t dtype, bool* f32) {
+    if (dtype != SP_F32 && dtype != SP_BF16) { set_error("the compute type is SP_BF16 or SP_F32"); return SP_ERR_DTYPE; }
+    *f32 = dtype == SP_F32;
+    return SP_OK;
+}
+
+int32_t sp_cuda_engine_create_from_config(const char* config_json, int32_t compute_dtype, const SpModelDesc* run, SpEngine** out) {
+    API_BEGIN
+    if (!config_json || !run || !out) { set_error("null argument"); return SP_ERR_ARG; }
+    bool f32 = false;
+    int st = plan_compute_type(compute_dtype, &f32);
+    if (st != SP_OK) return st;
+    Engine* eng = nullptr;
+    st = sp_engine_from_config_impl(config_json, std::strlen(config_json), f32, *run, &eng);
+    if (st != SP_OK) return st;
+    *out = new SpEngine{eng};
+    return SP_OK;
+    API_END
+}
+
+int32_t sp_cuda_engine_from_dir(const char* path, int32_t compute_dtype, const SpModelDesc* run, SpEngine** out) {
+    API_BEGIN
+    if (!path || !run || !out) { set_error("null argument"); return SP_ERR_ARG; }
+    bool f32 = false;
+    int st = plan_compute_type(compute_dtype, &f32);
+    if (st != SP_OK) return st;
+    Engine* eng = nullptr;
+    st = sp_engine_from_dir_impl(path, f32, *run, &eng);
+    if (st != SP_OK) return st;
+    *out = new SpEngine{eng};
+    return SP_OK;
+    API_END
+}
+
+int32_t sp_cuda_forward_rows(SpEngine* e, const uint32_t* ids, const int32_t* slots, size_t n, const int32_t* rows, size_t n_rows,
+                             float* logits_out, uint32_t* argmax_out) {
+    API_BEGIN
+    if (!e) { set_error("null engine"); return SP_ERR_ARG; }
+    return e->e->forward_rows(ids, slots, (int64_t)n, rows, (int64_t)n_rows, logits_out, argmax_out);
     API_END
 }
 

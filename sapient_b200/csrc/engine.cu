@@ -1,5 +1,6 @@
 // Resident CUDA engine for Llama/Qwen- and Phi-2-shaped quantized decoders (host side).
 #include "engine.h"
+#include "engine_plan.h"
 
 #include <algorithm>
 #include <cmath>
@@ -10,6 +11,12 @@
 #include "sp_common.cuh"
 
 namespace sp {
+
+#define SP_TRY(expr)                  \
+    do {                              \
+        int _s = (expr);              \
+        if (_s != SP_OK) return _s;   \
+    } while (0)
 
 static thread_local std::string g_err;
 void set_error(const std::string& msg) { g_err = msg; }
@@ -50,9 +57,31 @@ Engine::Engine(const SpModelDesc& desc) : d(desc) {
     seq_len.assign(d.max_batch, 0);
 }
 
+Engine::Engine(const SpModelDesc& desc, const ModelPlan& plan, bool f32) : Engine([&] {
+    SpModelDesc r = desc;
+    r.arch = ARCH_PLAN;
+    r.n_layers = (int32_t)plan.layers.size();
+    r.hidden = plan.width;
+    r.vocab = plan.vocab;
+    r.norm_eps = plan.eps;
+    // informative only: a plan's layers have sizes of their own
+    r.n_heads = plan.layers[0].mix.heads;
+    r.n_kv_heads = 1;
+    r.head_dim = plan.layers[0].mix.dim + plan.layers[0].mix.rot_dim;
+    r.rotary_dim = plan.layers[0].mix.rot_dim;
+    r.rope_theta = (float)plan.layers[0].mix.rot.base;
+    r.ffn = plan.layers[0].has_mlp ? plan.layers[0].mlp.expert.ff : 0;
+    return r;
+}()) {
+    plan_.reset(new PlanState());
+    plan_->plan = plan;
+    plan_->f32 = f32;
+}
+
 Engine::~Engine() {
     cudaSetDevice(d.device);
     if (stream) cudaStreamSynchronize(stream);
+    plan_release();
     for (auto& g : step_graphs_) cudaGraphExecDestroy(g.second);
     for (auto& r : prof_recs_) { cudaEventDestroy(r.a); cudaEventDestroy(r.b); }
     for (cudaEvent_t ev : prof_pool_) cudaEventDestroy(ev);
@@ -67,9 +96,9 @@ Engine::~Engine() {
     rows_.release();
     for (void* p : owned_) cudaFree(p);
     void* bufs[] = {kv_.pool, d_page_table_, x_, h_, qkv_, attn_, gu_, mid_, sel_, logits_, trace_, d_ids_, d_argmax_,
-                    d_tok_slot_, d_tok_pos_, cos_sin_};
+                    d_tok_slot_, d_tok_pos_, d_rows_, cos_sin_};
     for (void* p : bufs) if (p) cudaFree(p);
-    void* pinned[] = {p_ids_, p_slot_, p_pos_, p_logits_, p_argmax_};
+    void* pinned[] = {p_ids_, p_slot_, p_pos_, p_rows_, p_logits_, p_argmax_};
     for (void* p : pinned) if (p) cudaFreeHost(p);
     if (own_stream) cudaStreamDestroy(own_stream);
     release_staging();
@@ -149,7 +178,7 @@ int Engine::set_tensor_ex(const char* name, int dtype, const int64_t* dims, int 
         // Phi-3's fused `mlp.gate_up_proj` (rows 0..ffn gate, ffn..2 ffn up: forward/phi.rs:559-604) is kept as two
         // matrices: two row ranges of the caller's bytes, nothing is copied on the host
         const std::string nm(name);
-        const size_t at = nm.find("mlp.gate_up_proj.weight");
+        const size_t at = plan_ ? std::string::npos : nm.find("mlp.gate_up_proj.weight");
         if (at != std::string::npos && at + 23 == nm.size()) {
             const int bbq = block_bytes(dtype), beq = block_elems(dtype);
             if (ndim != 2 || bbq == 0 || dims[0] != 2 * (int64_t)g.ffn || dims[1] % beq != 0 ||
@@ -192,7 +221,7 @@ int Engine::set_tensor_ex(const char* name, int dtype, const int64_t* dims, int 
     const int64_t inner_l = t.dims.back();
     const bool skip = nm.find("norm") != std::string::npos || nm.find("bias") != std::string::npos ||
                       nm.find("embed") != std::string::npos || nm.find("lm_head") != std::string::npos;
-    if (ndim == 2 && !skip && (dtype == T_F16 || dtype == T_BF16) && t.numel() >= 32 && t.numel() % 32 == 0 &&
+    if (!plan_ && ndim == 2 && !skip && (dtype == T_F16 || dtype == T_BF16) && t.numel() >= 32 && t.numel() % 32 == 0 &&
         inner_l % 32 == 0) {
         // online Q8_0 quantisation, block by block along rows
         const int64_t n = t.numel();
@@ -305,6 +334,15 @@ int Engine::finalize() {
     SP_CUDA_TRY(cudaSetDevice(d.device));
     if (load_stream_) SP_CUDA_TRY(cudaStreamSynchronize(load_stream_));  // every weight has landed
     release_staging();
+    if (plan_) {
+        vocab_l_ = d.vocab;
+        int st = finalize_plan();
+        if (st == SP_OK) st = finalize_step_state();
+        if (st != SP_OK) return st;
+        SP_CUDA_TRY(cudaDeviceSynchronize());
+        finalized = true;
+        return SP_OK;
+    }
     if (d.tp_size > 1) {
         if (d.arch != 0) { set_error("tensor parallelism covers the Llama/Qwen block only"); return SP_ERR_ARG; }
         if (g.n_heads % d.tp_size || g.n_kv_heads % d.tp_size || g.ffn % d.tp_size || g.vocab % d.tp_size ||
@@ -394,7 +432,6 @@ int Engine::finalize() {
     // activations
     const size_t T = (size_t)d.max_tokens;
     const size_t qkv_ld = (size_t)(H + 2 * Hkv) * hd;
-    SP_CUDA_TRY(cudaMalloc((void**)&x_, T * hid * 4));
     SP_CUDA_TRY(cudaMalloc((void**)&h_, T * hid * 4));
     SP_CUDA_TRY(cudaMalloc((void**)&qkv_, T * qkv_ld * 4));
     SP_CUDA_TRY(cudaMalloc((void**)&attn_, T * (size_t)H * hd * 4));
@@ -402,23 +439,11 @@ int Engine::finalize() {
     SP_CUDA_TRY(cudaMalloc((void**)&mid_, T * (size_t)d.ffn * 4));
     SP_CUDA_TRY(cudaMalloc((void**)&sel_, T * hid * 4));
     SP_CUDA_TRY(cudaMalloc((void**)&att_scratch_, attention_scratch_floats(ATT_SPLIT_TOKENS, H, ATT_SPLITS, hd) * 4));
-    logit_rows_ = std::min<int>(32, d.max_tokens);
-    SP_CUDA_TRY(cudaMalloc((void**)&logits_, (size_t)logit_rows_ * vocab_l_ * 4));
-    SP_CUDA_TRY(cudaMalloc((void**)&d_ids_, T * 4));
-    SP_CUDA_TRY(cudaMalloc((void**)&d_argmax_, T * 4));
-    SP_CUDA_TRY(cudaMalloc(&argmax_scratch_, argmax_scratch_bytes()));
-    SP_CUDA_TRY(cudaMemset(argmax_scratch_, 0, argmax_scratch_bytes()));
-    SP_CUDA_TRY(cudaMalloc((void**)&d_tok_slot_, T * 4));
-    SP_CUDA_TRY(cudaMalloc((void**)&d_tok_pos_, T * 4));
-    SP_CUDA_TRY(cudaMallocHost((void**)&p_ids_, T * 4));
-    SP_CUDA_TRY(cudaMallocHost((void**)&p_slot_, T * 4));
-    SP_CUDA_TRY(cudaMallocHost((void**)&p_pos_, T * 4));
-    SP_CUDA_TRY(cudaMallocHost((void**)&p_logits_, (size_t)logit_rows_ * vocab_l_ * 4));
     {
         const int st = tp_alloc();
         if (st != SP_OK) return st;
     }
-    SP_CUDA_TRY(cudaMallocHost((void**)&p_argmax_, T * 4));
+    SP_TRY(finalize_step_state());
     // RoPE table: theta = pos / base^(2i/rotary_dim) in f32, as crates/sapient-backends/cpu/src/kernels/rope.rs:40-43,118-121.
     const int half = d.rotary_dim / 2;
     std::vector<float2> cs((size_t)d.max_ctx * half);
@@ -435,10 +460,31 @@ int Engine::finalize() {
     final_b_ = phi ? find_f32(fn + ".bias", hid) : nullptr;
     if (!final_w_) { set_error("missing final norm weight"); return SP_ERR_STATE; }
     lm_bias_ = phi ? find_f32("lm_head.bias", lm_head_->dims[0]) : nullptr;
-    SP_CUDA_TRY(cudaStreamCreateWithFlags(&own_stream, cudaStreamNonBlocking));
-    stream = own_stream;
     SP_CUDA_TRY(cudaDeviceSynchronize());
     finalized = true;
+    return SP_OK;
+}
+
+int Engine::finalize_step_state() {
+    const size_t T = (size_t)d.max_tokens;
+    SP_CUDA_TRY(cudaMalloc((void**)&x_, T * d.hidden * 4));
+    logit_rows_ = std::min<int>(32, d.max_tokens);
+    SP_CUDA_TRY(cudaMalloc((void**)&logits_, (size_t)logit_rows_ * vocab_l_ * 4));
+    SP_CUDA_TRY(cudaMalloc((void**)&d_ids_, T * 4));
+    SP_CUDA_TRY(cudaMalloc((void**)&d_argmax_, T * 4));
+    SP_CUDA_TRY(cudaMalloc(&argmax_scratch_, argmax_scratch_bytes()));
+    SP_CUDA_TRY(cudaMemset(argmax_scratch_, 0, argmax_scratch_bytes()));
+    SP_CUDA_TRY(cudaMalloc((void**)&d_tok_slot_, T * 4));
+    SP_CUDA_TRY(cudaMalloc((void**)&d_tok_pos_, T * 4));
+    SP_CUDA_TRY(cudaMalloc((void**)&d_rows_, T * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_rows_, T * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_ids_, T * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_slot_, T * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_pos_, T * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_logits_, (size_t)logit_rows_ * vocab_l_ * 4));
+    SP_CUDA_TRY(cudaMallocHost((void**)&p_argmax_, T * 4));
+    SP_CUDA_TRY(cudaStreamCreateWithFlags(&own_stream, cudaStreamNonBlocking));
+    stream = own_stream;
     return SP_OK;
 }
 

@@ -1,6 +1,8 @@
 // Host-side resident engine: device weights in raw ggml block layout, a paged fp16 KV
 // cache with per-slot page tables, and the per-layer launch sequence for Llama/Qwen
-// and Phi-2 shaped decoders. Mirrors the contract of the reference's resident GPU
+// and Phi-2 shaped decoders; designs described by a layer plan (model_plan.h) run on the
+// same slots, pages, step graphs and host API with their own weights and cache rows
+// (engine_plan.cu). Mirrors the contract of the reference's resident GPU
 // engine (crates/sapient-models/src/forward/wgpu_engine.rs:93-110,173-341,362-676)
 // behind ForwardEngine (crates/sapient-models/src/forward/mod.rs:381-506).
 #pragma once
@@ -8,6 +10,7 @@
 #include <cuda_runtime.h>
 
 #include <map>
+#include <memory>
 #include <string>
 #include <vector>
 
@@ -51,9 +54,16 @@ struct LayerW {
     const float *qb = nullptr, *kb = nullptr, *vb = nullptr, *ob = nullptr, *upb = nullptr, *downb = nullptr;
 };
 
+struct ModelPlan;
+struct PlanState;
+struct PlanMat;
+
 class Engine {
   public:
     explicit Engine(const SpModelDesc& d);
+    // A plan-driven engine; of `d` only the run-time fields count (max_ctx, max_batch, max_tokens, device, kv_pages).
+    // f32: weights, activations and cache in f32 instead of bf16.
+    Engine(const SpModelDesc& d, const ModelPlan& plan, bool f32);
     ~Engine();
     int set_tensor(const char* name, int dtype, const int64_t* dims, int ndim, const void* bytes, size_t nbytes);
     // The same with the rows of each head still in the GGUF llama order (row h*D + 2b + a holds HF row h*D + a*D/2 + b,
@@ -68,6 +78,10 @@ class Engine {
     // positions). want_all: logits for every token, else only for the last token. Either output may be null.
     int forward(const uint32_t* ids, const int32_t* slots, int64_t n, bool want_all, float* logits_out,
                 uint32_t* argmax_out);
+    // The same with the wanted logits named: rows[0..n_rows) are ascending token indices. Every slot's tokens may be a portion
+    // of a prompt or one decoded token; all of them run as one batch (in chunks of max_tokens rows).
+    int forward_rows(const uint32_t* ids, const int32_t* slots, int64_t n, const int32_t* rows, int64_t n_rows, float* logits_out,
+                     uint32_t* argmax_out);
     int reset(int slot);
     int truncate(int slot, size_t n, size_t* kept);
     int debug_layer_out(int layer, float* out, size_t cap, int32_t* n_tokens);
@@ -135,10 +149,10 @@ class Engine {
     uint64_t weight_bytes = 0, kv_bytes = 0;
 
   private:
-    int run_chunk(const uint32_t* ids, const int32_t* slots, int T, int rows_from, float* logits_out, uint32_t* argmax_out);
+    int run_chunk(const uint32_t* ids, int T, const std::vector<int32_t>& rows, float* logits_out, uint32_t* argmax_out);
     int enqueue_layers(int T);                       // embed + all layers for the staged token table
     // final norm is done by the caller; lm_head + argmax of rc rows (pre: digits of those rows already in the workspace)
-    int enqueue_head(int rows_from, int r0, int rc, const ImmaArgs* pre = nullptr);
+    int enqueue_head(int r0, int rc, const ImmaArgs* pre = nullptr);
     int enqueue_decode_step(int T);                  // embed, layers, final norm, lm_head, argmax for T <= logit_rows_ rows
     int launch_decode_step(int T);                   // the same through a cached CUDA graph when allowed
     void prof_begin(int fam);
@@ -217,6 +231,21 @@ class Engine {
     float* att_scratch_ = nullptr;
     int repack_weights();
 
+    // plan-driven models (engine_plan.cu)
+    friend struct PlanPacker;
+    std::unique_ptr<PlanState> plan_;
+    int finalize_plan();
+    void plan_release();
+    int plan_stage(int T);
+    int plan_layers(int T);
+    int plan_mixer(int layer, int T);
+    int plan_experts(int layer, int T);
+    int plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, int ldy, bool out_f32);
+    int plan_head(const int32_t* rows, int n);
+    int plan_ctx_bucket() const;
+    int plan_privatise_copy(int from, int to);
+    int finalize_step_state();  // host and device state of a step that every kind of model has
+
     // paged KV cache
     KvGeom kv_{};
     int32_t* d_page_table_ = nullptr;
@@ -228,13 +257,13 @@ class Engine {
           *logits_ = nullptr, *trace_ = nullptr;
     uint32_t *d_ids_ = nullptr, *d_argmax_ = nullptr;
     void* argmax_scratch_ = nullptr;  // candidates and arrival counters of the multi-block arg-max
-    int32_t *d_tok_slot_ = nullptr, *d_tok_pos_ = nullptr;
+    int32_t *d_tok_slot_ = nullptr, *d_tok_pos_ = nullptr, *d_rows_ = nullptr;
     float2* cos_sin_ = nullptr;
     int trace_tokens_ = 0;
     int logit_rows_ = 32;  // rows of the lm_head GEMV per pass
     // pinned staging
     uint32_t* p_ids_ = nullptr;
-    int32_t *p_slot_ = nullptr, *p_pos_ = nullptr;
+    int32_t *p_slot_ = nullptr, *p_pos_ = nullptr, *p_rows_ = nullptr;
     float* p_logits_ = nullptr;
     uint32_t* p_argmax_ = nullptr;
     // device-resident greedy loop

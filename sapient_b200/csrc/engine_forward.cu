@@ -6,6 +6,7 @@
 #include <cstring>
 
 #include "engine.h"
+#include "engine_plan.h"
 #include "sp_common.cuh"
 
 namespace sp {
@@ -45,6 +46,7 @@ int Engine::privatise_tail(int slot) {
     const int r = pages.privatise_tail(slot, seq_len[slot], &from, &to);
     if (r < 0) { set_error("KV page pool exhausted"); return SP_ERR_KV_FULL; }
     if (r == 0) return SP_OK;
+    if (plan_) return plan_privatise_copy(from, to);
     const size_t run = (size_t)2 * kv_.n_kv * KV_PAGE * kv_.head_dim * sizeof(__half);
     const size_t pitch = run * (size_t)kv_.n_pages;
     const uint8_t* base = reinterpret_cast<const uint8_t*>(kv_.pool);
@@ -82,6 +84,7 @@ int Engine::truncate(int slot, size_t n, size_t* kept) {
 }
 
 int Engine::enqueue_layers(int T) {
+    if (plan_) return plan_layers(T);
     const int hid = d.hidden;
     SP_LAUNCH(F_EMBED, launch_embed(embed_->dtype, embed_->d, hid, d_ids_, T, x_, stream));
     for (int l = 0; l < d.n_layers; ++l) {
@@ -95,8 +98,7 @@ int Engine::enqueue_layers(int T) {
 }
 
 // lm_head over rows [r0, r0+rc) of the normalised selection sel_, plus their argmax.
-int Engine::enqueue_head(int rows_from, int r0, int rc, const ImmaArgs* pre) {
-    (void)rows_from;
+int Engine::enqueue_head(int r0, int rc, const ImmaArgs* pre) {
     const int V = vocab_l_, hid = d.hidden;
     // lm_head rows beyond the vocabulary (if the table is larger) are not computed: n = V (this rank's slice under
     // tensor parallelism)
@@ -115,6 +117,7 @@ int Engine::enqueue_head(int rows_from, int r0, int rc, const ImmaArgs* pre) {
 int Engine::enqueue_decode_step(int T) {
     const int hid = d.hidden;
     SP_TRY(enqueue_layers(T));
+    if (plan_) return plan_head(nullptr, T);
     ImmaArgs ia;
     {
         DevTensor head = *lm_head_;
@@ -128,19 +131,17 @@ int Engine::enqueue_decode_step(int T) {
     }
     if (lm_head_->tiled && plan_digits(T, hid, ia)) {
         SP_LAUNCH(F_NORM, launch_norm_quant(x_, hid, final_w_, final_b_, d.arch == 1, d.norm_eps, nullptr, 0, ia, stream, tp_take()));
-        return enqueue_head(0, 0, T, &ia);
+        return enqueue_head(0, T, &ia);
     }
     SP_TRY(tp_resolve(T));
     if (d.arch == 1) SP_LAUNCH(F_NORM, launch_layer_norm(x_, final_w_, final_b_, T, hid, d.norm_eps, sel_, stream));
     else SP_LAUNCH(F_NORM, launch_rms_norm(x_, final_w_, T, hid, d.norm_eps, sel_, stream));
-    return enqueue_head(0, 0, T);
+    return enqueue_head(0, T);
 }
 
 // One chunk of T <= max_tokens tokens whose (slot, pos) are already staged in p_slot_/p_pos_.
-// Logits are produced for chunk rows [rows_from, T).
-int Engine::run_chunk(const uint32_t* ids, const int32_t* slots, int T, int rows_from, float* logits_out,
-                      uint32_t* argmax_out) {
-    (void)slots;
+// Logits are produced for the chunk rows named in `rows` (ascending).
+int Engine::run_chunk(const uint32_t* ids, int T, const std::vector<int32_t>& rows, float* logits_out, uint32_t* argmax_out) {
     std::memcpy(p_ids_, ids, (size_t)T * 4);
     SP_CUDA_TRY(cudaMemcpyAsync(d_ids_, p_ids_, (size_t)T * 4, cudaMemcpyHostToDevice, stream));
     SP_CUDA_TRY(cudaMemcpyAsync(d_tok_slot_, p_slot_, (size_t)T * 4, cudaMemcpyHostToDevice, stream));
@@ -148,9 +149,10 @@ int Engine::run_chunk(const uint32_t* ids, const int32_t* slots, int T, int rows
     SP_TRY(sync_page_table());
     const int hid = d.hidden, V = vocab_l_;
     if (trace_on && !trace_) SP_CUDA_TRY(cudaMalloc((void**)&trace_, (size_t)d.n_layers * d.max_tokens * hid * 4));
-    const int rows = T - rows_from;
-    const bool want = rows > 0 && (logits_out || argmax_out);
-    if (want && rows_from == 0 && T <= logit_rows_) {
+    if (plan_) SP_TRY(plan_stage(T));
+    const int n = (int)rows.size();
+    const bool want = n > 0 && (logits_out || argmax_out);
+    if (want && n == T && T <= logit_rows_) {
         // decode-shaped call: the whole step is one (graph) launch
         SP_TRY(launch_decode_step(T));
         if (argmax_out) SP_CUDA_TRY(cudaMemcpyAsync(p_argmax_, d_argmax_, (size_t)T * 4, cudaMemcpyDeviceToHost, stream));
@@ -164,12 +166,23 @@ int Engine::run_chunk(const uint32_t* ids, const int32_t* slots, int T, int rows
     SP_TRY(enqueue_layers(T));
     SP_TRY(tp_resolve(T));
     if (want) {
-        const float* src = x_ + (size_t)rows_from * hid;
-        if (d.arch == 1) SP_LAUNCH(F_NORM, launch_layer_norm(src, final_w_, final_b_, rows, hid, d.norm_eps, sel_, stream));
-        else SP_LAUNCH(F_NORM, launch_rms_norm(src, final_w_, rows, hid, d.norm_eps, sel_, stream));
-        for (int r0 = 0; r0 < rows; r0 += logit_rows_) {
-            const int rc = std::min(logit_rows_, rows - r0);
-            SP_TRY(enqueue_head(rows_from, r0, rc));
+        const bool run = rows.back() - rows.front() == n - 1;
+        if (!run || plan_) {
+            std::memcpy(p_rows_, rows.data(), (size_t)n * 4);
+            SP_CUDA_TRY(cudaMemcpyAsync(d_rows_, p_rows_, (size_t)n * 4, cudaMemcpyHostToDevice, stream));
+        }
+        if (!plan_) {
+            const float* src = x_ + (size_t)rows.front() * hid;
+            if (!run) {
+                SP_LAUNCH(F_ELEM, launch_gather_rows(x_, hid, d_rows_, n, hid, h_, stream));
+                src = h_;
+            }
+            if (d.arch == 1) SP_LAUNCH(F_NORM, launch_layer_norm(src, final_w_, final_b_, n, hid, d.norm_eps, sel_, stream));
+            else SP_LAUNCH(F_NORM, launch_rms_norm(src, final_w_, n, hid, d.norm_eps, sel_, stream));
+        }
+        for (int r0 = 0; r0 < n; r0 += logit_rows_) {
+            const int rc = std::min(logit_rows_, n - r0);
+            SP_TRY(plan_ ? plan_head(d_rows_ + r0, rc) : enqueue_head(r0, rc));
             if (argmax_out) SP_CUDA_TRY(cudaMemcpyAsync(p_argmax_, d_argmax_, (size_t)rc * 4, cudaMemcpyDeviceToHost, stream));
             if (logits_out) SP_CUDA_TRY(cudaMemcpyAsync(p_logits_, logits_, (size_t)rc * V * 4, cudaMemcpyDeviceToHost, stream));
             SP_CUDA_TRY(cudaStreamSynchronize(stream));
@@ -184,8 +197,23 @@ int Engine::run_chunk(const uint32_t* ids, const int32_t* slots, int T, int rows
 
 int Engine::forward(const uint32_t* ids, const int32_t* slots, int64_t n, bool want_all, float* logits_out,
                     uint32_t* argmax_out) {
+    if (n <= 0) { set_error("empty input"); return SP_ERR_ARG; }
+    std::vector<int32_t> rows;
+    if (want_all) {
+        rows.resize((size_t)n);
+        for (int64_t i = 0; i < n; ++i) rows[(size_t)i] = (int32_t)i;
+    } else {
+        rows.push_back((int32_t)(n - 1));
+    }
+    return forward_rows(ids, slots, n, rows.data(), (int64_t)rows.size(), logits_out, argmax_out);
+}
+
+int Engine::forward_rows(const uint32_t* ids, const int32_t* slots, int64_t n, const int32_t* rows, int64_t n_rows, float* logits_out,
+                         uint32_t* argmax_out) {
     if (!finalized) { set_error("engine not finalised"); return SP_ERR_STATE; }
-    if (!ids || !slots || n <= 0) { set_error("empty input"); return SP_ERR_ARG; }
+    if (!ids || !slots || n <= 0 || n > INT32_MAX || n_rows < 0 || (n_rows > 0 && !rows)) { set_error("empty input"); return SP_ERR_ARG; }
+    for (int64_t i = 0; i < n_rows; ++i)
+        if (rows[i] < 0 || rows[i] >= n || (i > 0 && rows[i] <= rows[i - 1])) { set_error("wanted rows must be ascending token indices"); return SP_ERR_ARG; }
     SP_CUDA_TRY(cudaSetDevice(d.device));
     SP_TRY(drain_async());
     // validate everything before touching any state
@@ -208,6 +236,8 @@ int Engine::forward(const uint32_t* ids, const int32_t* slots, int64_t n, bool w
     for (int s = 0; s < d.max_batch; ++s)
         if (add[s]) SP_TRY(privatise_tail(s));
     const int C = d.max_tokens;
+    int64_t next = 0;  // first wanted row not yet produced
+    std::vector<int32_t> here;
     for (int64_t c0 = 0; c0 < n; c0 += C) {
         const int T = (int)std::min<int64_t>(C, n - c0);
         for (int i = 0; i < T; ++i) {
@@ -218,19 +248,10 @@ int Engine::forward(const uint32_t* ids, const int32_t* slots, int64_t n, bool w
         }
         step_ctx_ = 0;
         for (int i = 0; i < T; ++i) step_ctx_ = std::max(step_ctx_, p_pos_[i] + 1);
-        const bool last_chunk = c0 + T >= n;
-        int rows_from;
-        float* lo = nullptr;
-        uint32_t* ao = nullptr;
-        if (want_all) {
-            rows_from = 0;
-            lo = logits_out ? logits_out + (size_t)c0 * vocab_l_ : nullptr;
-            ao = argmax_out ? argmax_out + c0 : nullptr;
-        } else {
-            rows_from = last_chunk ? T - 1 : T;
-            if (last_chunk) { lo = logits_out; ao = argmax_out; }
-        }
-        SP_TRY(run_chunk(ids + c0, slots + c0, T, rows_from, lo, ao));
+        here.clear();
+        const int64_t first = next;
+        for (; next < n_rows && rows[next] < c0 + T; ++next) here.push_back((int32_t)(rows[next] - c0));
+        SP_TRY(run_chunk(ids + c0, T, here, logits_out ? logits_out + (size_t)first * vocab_l_ : nullptr, argmax_out ? argmax_out + first : nullptr));
     }
     return SP_OK;
 }

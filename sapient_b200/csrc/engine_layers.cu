@@ -10,6 +10,7 @@
 #include <algorithm>
 
 #include "engine.h"
+#include "engine_plan.h"
 #include "sp_common.cuh"
 
 namespace sp {
@@ -236,6 +237,7 @@ static inline bool all_tiled(const DevTensor* a, const DevTensor* b = nullptr, c
 // keys the unsplit kernel is a chain of 260 dependent iterations per block (measured 6 ms of attention per step of the
 // 8B shape; the KV bytes need 0.7 ms). The count is a power of two up to 16 and part of the step graph's key.
 int Engine::step_splits(int T) const {
+    if (plan_) return plan_ctx_bucket();
     if (T <= ATT_SPLIT_TOKENS && attention_takes_mma(T, step_ctx_, d.n_heads, d.n_kv_heads, d.head_dim)) {
         // tensor-core kernel, a block per (KV head, token, split): enough blocks to fill the SMs three deep, but no range
         // shorter than 256 keys (4 pages per warp) — its fixed cost per block (query fragments, warp merge) is larger

@@ -41,6 +41,7 @@
 #include "kernels.h"
 #include "pdl.cuh"
 #include "sp_common.cuh"
+#include "tc5_ptx.cuh"
 
 namespace sp {
 
@@ -58,39 +59,15 @@ constexpr int TC5_BK = 128;                    // columns per stage = two 128-by
 constexpr int TC5_NB_MAX = 256;                // activation rows per CTA
 constexpr int TC5_SMEM_LIMIT = 192 * 1024;
 constexpr int TC5_SMEM_MIN = 120 * 1024;       // more than half an SM's shared memory: one CTA per SM, which owns all of its tensor memory
-constexpr int TC5_SPIN_LIMIT = 1 << 22;
 
 __device__ int g_tc5_timeout = 0;
-
-__device__ __forceinline__ uint32_t tc5_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-// Shared-memory matrix descriptor: K-major operand, 128-byte swizzle, rows of 128 B, 8-row groups 1024 B apart.
-__device__ __forceinline__ uint64_t tc5_desc(uint32_t saddr) {
-    uint64_t d = 0;
-    d |= (uint64_t)((saddr & 0x3FFFFu) >> 4);  // start address / 16
-    d |= (uint64_t)1 << 16;                    // leading-dimension byte offset / 16 (not used by swizzled K-major)
-    d |= (uint64_t)(1024 >> 4) << 32;          // stride-dimension byte offset / 16: next 8-row group
-    d |= (uint64_t)1 << 46;                    // descriptor version of this architecture
-    d |= (uint64_t)2 << 61;                    // 128-byte swizzle
-    return d;
-}
 
 // Instruction descriptor, kind::f16: fp16 A and B, fp32 D, both K-major, M = 128, N = nb.
 __device__ __forceinline__ uint32_t tc5_idesc(int nb) {
     return (1u << 4) | ((uint32_t)(nb >> 3) << 17) | ((uint32_t)(TC5_BM >> 4) << 24);
 }
 
-__device__ __forceinline__ void tc5_mma(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n"
-        ".reg .pred p;\n"
-        "setp.ne.b32 p, %4, 0;\n"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n"
-        "}\n" ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-
-// The same with the A operand (weights) read from tensor memory: lane = weight row, 8 columns = 16 fp16 along K.
+// tc5_mma with the A operand (weights) read from tensor memory: lane = weight row, 8 columns = 16 fp16 along K.
 __device__ __forceinline__ void tc5_mma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
     asm volatile(
         "{\n"
@@ -117,32 +94,6 @@ __device__ __forceinline__ void tc5_mma_ts_acc(uint32_t d_tmem, uint32_t a_tmem,
 __device__ __forceinline__ void tc5_tmem_st(uint32_t taddr, const uint32_t (&v)[4]) {
     asm volatile("tcgen05.st.sync.aligned.16x256b.x1.b32 [%0], {%1, %2, %3, %4};\n" ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3])
                  : "memory");
-}
-
-__device__ __forceinline__ void tc5_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n" ::"r"(tc5_smem_u32(bar)) : "memory");
-}
-
-__device__ __forceinline__ void tc5_arrive(uint64_t* bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(tc5_smem_u32(bar)) : "memory");
-}
-
-__device__ __forceinline__ bool tc5_wait(uint64_t* bar, uint32_t parity) {
-    const uint32_t a = tc5_smem_u32(bar);
-    for (int i = 0; i < TC5_SPIN_LIMIT; ++i) {
-        uint32_t done;
-        asm volatile(
-            "{\n"
-            ".reg .pred p;\n"
-            "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
-            "selp.u32 %0, 1, 0, p;\n"
-            "}\n"
-            : "=r"(done)
-            : "r"(a), "r"(parity)
-            : "memory");
-        if (done) return true;
-    }
-    return false;
 }
 
 __device__ __forceinline__ uint32_t pack_h2(float a, float b) {
@@ -771,10 +722,6 @@ cudaError_t launch_x_to_f16_hilo(const float* x, int ldx, int m, int k, __half* 
     return count_launch_and_check();
 }
 
-typedef CUresult (*PFN_encodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                    const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
 // Up to three matrices sharing the activations in one launch. res (added to segment 0) may alias its y. The items of the
 // grid's last, partial wave are split along K over as many CTAs as fill the SMs (see Tc5Args) when the caller provides
 // scratch for their partial tiles, unless there is a residual that is not in place.
@@ -830,12 +777,7 @@ cudaError_t launch_gemm_tc5_multi(const Tc5Seg* segs, int nseg, int k, const __h
         }
     }
     // TMA descriptor of the fp16 activations [m][k]: boxes of 64 columns x nb_max rows, 128-byte swizzle, zero fill
-    static const PFN_encodeTiled encode = [] {  // initialised once, thread-safe
-        void* fn = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres) != cudaSuccess) fn = nullptr;
-        return reinterpret_cast<PFN_encodeTiled>(fn);
-    }();
+    const PFN_encodeTiled encode = tensor_map_encoder();
     if (!encode) return cudaErrorNotSupported;
     CUtensorMap tmap;
     {

@@ -20,6 +20,7 @@
 #include <vector>
 
 #include "engine.h"
+#include "model_plan.h"
 #include "sp_common.cuh"
 
 namespace {
@@ -201,10 +202,10 @@ int sp_engine_from_gguf_impl(const char* path, int device, int max_ctx, int max_
     // Phi-3 / 3.5 / 4-mini: PhiForward's sequential block — RMSNorm, fused q|k|v, fused gate|up SwiGLU
     // (crates/sapient-models/src/forward/phi.rs:391-503,559-604) — which is the Llama block once the fused tensors are cut
     const bool is_phi3 = arch == "phi3";
-    const bool is_llama_family = is_phi3 || arch == "llama" || arch == "mistral" || arch == "qwen2" || arch == "qwen3" || arch == "idefics3";
-    if (!is_phi && !is_llama_family) { set_error("architecture '" + arch + "' is not supported by the CUDA engine"); return SP_ERR_DTYPE; }
+    const sp::ArchEntry* entry = sp::find_arch(arch);
+    if (!entry || !entry->gguf) { set_error("architecture '" + arch + "' is not supported by the CUDA engine"); return SP_ERR_DTYPE; }
     if (num("expert_count", 0) > 0) { set_error("MoE models are not supported by the CUDA engine"); return SP_ERR_DTYPE; }
-    d.arch = is_phi ? 1 : 0;
+    d.arch = entry->block;
     double vocab = 32000;
     if (has("vocab_size")) vocab = num("vocab_size", 32000);
     else if (meta.count("tokenizer.ggml.tokens")) vocab = (double)meta["tokenizer.ggml.tokens"].arr_len;

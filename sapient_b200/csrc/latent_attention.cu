@@ -1,0 +1,556 @@
+// Latent attention over a paged latent cache (plan_kernels.h).
+//
+// The cache keeps, per token and owning layer, a normed latent c and one rotated key part kr shared by the heads. With
+// k_h = W_uk,h c and v_h = W_uv,h c, a head's score is q_h . W_uk,h c + qr_h . kr = [W_uk,h^T q_h | qr_h] . [c | kr]: in
+// the ABSORBED form every head of a token attends to the same cached rows with a query of rank + rot coordinates, the
+// softmax mixes the latents, and W_uv,h is applied to the mixture. It reads each cached byte once per token (16 heads are
+// the rows of one mma tile) and rebuilds nothing: decode steps and short portions. The EXPANDED form rebuilds k_h and v_h
+// of a key range with one matrix product and attends with dim + rot and vdim coordinates, a third of the work per
+// (query, key) pair: prompts.
+// Scores, softmax and accumulation are f32 in both; a sliding window bounds the keys a block visits.
+#include "kernels.h"
+#include "pdl.cuh"
+#include "plan_common.cuh"
+#include "plan_kernels.h"
+#include "sp_common.cuh"
+
+namespace sp {
+
+cudaError_t count_launch_and_check();  // kernels.cu
+
+// ── rotation, latent norm, cache append ──
+constexpr int LA_THREADS = 128;
+
+template <typename T>
+__device__ __forceinline__ void rotate_pairs(const float* src, T* dst, const float2* cs, int rot, int rot16) {
+    for (int i = threadIdx.x; i < rot16 / 2; i += LA_THREADS) {
+        float u = 0.f, v = 0.f;
+        if (2 * i < rot) {
+            const float a = src[2 * i], b = src[2 * i + 1];
+            const float2 r = cs[i];
+            u = a * r.x - b * r.y;
+            v = b * r.x + a * r.y;
+        }
+        dst[2 * i] = from_f32<T>(u);
+        dst[2 * i + 1] = from_f32<T>(v);
+    }
+}
+
+// Block (token, y): y < heads: that head's query; y == heads: the cache row.
+template <typename T>
+__global__ void __launch_bounds__(LA_THREADS) latent_append_kernel(const float* __restrict__ proj, int ldp, const LatentShape s, const LatentCache c,
+                                                                   const float* __restrict__ norm_gain, float eps, const float2* __restrict__ cos_sin,
+                                                                   const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
+                                                                   T* __restrict__ qn, int ldqn, T* __restrict__ qabs, T* __restrict__ qf) {
+    __shared__ float sh[LA_THREADS / 32];
+    pdl_wait();
+    pdl_trigger();
+    const int t = blockIdx.x, h = blockIdx.y, pos = tok_pos[t];
+    const float2* cs = cos_sin + (int64_t)pos * (s.rot / 2);
+    if (h < s.heads) {
+        const float* q = proj + (int64_t)t * ldp + (int64_t)h * (s.dim + s.rot);
+        if (qn) {
+            T* d = qn + ((int64_t)t * s.heads + h) * ldqn;
+            for (int i = threadIdx.x; i < ldqn; i += LA_THREADS) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
+            T* r = qabs + ((int64_t)t * s.heads + h) * c.ld;
+            for (int i = c.rank + threadIdx.x; i < c.rank16; i += LA_THREADS) r[i] = from_f32<T>(0.f);
+            rotate_pairs<T>(q + s.dim, r + c.rank16, cs, s.rot, c.rot16);
+        } else {
+            const int dim16 = (s.dim + 15) & ~15;
+            T* d = qf + ((int64_t)t * s.heads + h) * (dim16 + c.rot16);
+            for (int i = threadIdx.x; i < dim16; i += LA_THREADS) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
+            rotate_pairs<T>(q + s.dim, d + dim16, cs, s.rot, c.rot16);
+        }
+        return;
+    }
+    const float* kv = proj + (int64_t)t * ldp + (int64_t)s.heads * (s.dim + s.rot);
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < c.rank; i += LA_THREADS) ss = fmaf(kv[i], kv[i], ss);
+    const float r = rsqrtf(block_sum<LA_THREADS / 32>(ss, sh) / (float)c.rank + eps);
+    const int page = c.page_table[(int64_t)tok_slot[t] * c.max_pages + pos / KV_PAGE];
+    T* row = reinterpret_cast<T*>(c.pool) + ((int64_t)page * KV_PAGE + pos % KV_PAGE) * c.ld;
+    for (int i = threadIdx.x; i < c.rank16; i += LA_THREADS) row[i] = from_f32<T>(i < c.rank ? kv[i] * r * norm_gain[i] : 0.f);
+    rotate_pairs<T>(kv + c.rank, row + c.rank16, cs, s.rot, c.rot16);
+}
+
+cudaError_t launch_latent_append(const float* proj, int ldp, const LatentShape& s, const LatentCache& c, bool own, const float* norm_gain,
+                                 float eps, const float2* cos_sin, const int32_t* tok_slot, const int32_t* tok_pos, void* qn, int ldqn,
+                                 void* qabs, void* qf, bool f32, int n_tok, cudaStream_t st) {
+    if (n_tok == 0) return cudaSuccess;
+    const dim3 grid(n_tok, s.heads + (own ? 1 : 0));
+    cudaError_t le = f32 ? launch_pdl(latent_append_kernel<float>, grid, dim3(LA_THREADS), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
+                                      tok_pos, (float*)qn, ldqn, (float*)qabs, (float*)qf)
+                         : launch_pdl(latent_append_kernel<bf16>, grid, dim3(LA_THREADS), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
+                                      tok_pos, (bf16*)qn, ldqn, (bf16*)qabs, (bf16*)qf);
+    if (le != cudaSuccess) return le;
+    return count_launch_and_check();
+}
+
+// ── absorbed attention ──
+// Key range of split sp of n_splits for a token at `pos`.
+__device__ __forceinline__ void key_range(int pos, int window, int sp, int n_splits, int& begin, int& end) {
+    const int lo = window > pos ? 0 : pos - window + 1, n = pos + 1 - lo;
+    const int per = (n + n_splits - 1) / n_splits;
+    begin = lo + sp * per;
+    end = min(pos + 1, begin + per);
+}
+
+// Any compute type and sizes up to rank 1024: block per (head, token, split), a warp per key.
+constexpr int LS_WARPS = 4, LS_MAX_PER_LANE = 32;
+template <typename T>
+__global__ void __launch_bounds__(LS_WARPS * 32) latent_attention_simple_kernel(const T* __restrict__ qabs, const LatentShape s, const LatentCache c,
+                                                                                const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
+                                                                                T* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
+    extern __shared__ float ls_smem[];  // query, then one output row per warp
+    __shared__ float sm[LS_WARPS], sl[LS_WARPS];
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int width = c.rank16 + c.rot16;
+    float *q = ls_smem, *os = ls_smem + width;
+    const T* qr = qabs + ((int64_t)t * s.heads + h) * c.ld;
+    for (int i = threadIdx.x; i < width; i += LS_WARPS * 32) q[i] = to_f32(qr[i]);
+    __syncthreads();
+    int begin, end;
+    key_range(tok_pos[t], s.window, blockIdx.z, n_splits, begin, end);
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    float o[LS_MAX_PER_LANE];
+#pragma unroll
+    for (int i = 0; i < LS_MAX_PER_LANE; ++i) o[i] = 0.f;
+    float m = -INFINITY, l = 0.f;
+    for (int key = begin + warp; key < end; key += LS_WARPS) {
+        const T* row = reinterpret_cast<const T*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld;
+        float dot = 0.f;
+        for (int i = lane; i < width; i += 32) dot = fmaf(q[i], to_f32(row[i]), dot);
+        const float sc = warp_sum(dot) * s.scale;
+        const float mn = fmaxf(m, sc), corr = expf(m - mn), p = expf(sc - mn);
+#pragma unroll
+        for (int i = 0; i < LS_MAX_PER_LANE; ++i)
+            if (lane + 32 * i < c.rank) o[i] = fmaf(p, to_f32(row[lane + 32 * i]), o[i] * corr);
+        l = fmaf(l, corr, p);
+        m = mn;
+    }
+    if (lane == 0) { sm[warp] = m; sl[warp] = l; }
+#pragma unroll
+    for (int i = 0; i < LS_MAX_PER_LANE; ++i)
+        if (lane + 32 * i < c.rank) os[warp * c.rank + lane + 32 * i] = o[i];
+    __syncthreads();
+    float M = -INFINITY, L = 0.f, cw[LS_WARPS];
+#pragma unroll
+    for (int w = 0; w < LS_WARPS; ++w) M = fmaxf(M, sm[w]);
+#pragma unroll
+    for (int w = 0; w < LS_WARPS; ++w) {
+        cw[w] = sm[w] == -INFINITY ? 0.f : expf(sm[w] - M);
+        L = fmaf(cw[w], sl[w], L);
+    }
+    float* pd = part + (((int64_t)t * s.heads + h) * n_splits + blockIdx.z) * (c.rank + 2);
+    const float inv = n_splits == 1 ? 1.0f / L : 1.f;
+    for (int e = threadIdx.x; e < c.rank; e += LS_WARPS * 32) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < LS_WARPS; ++w) v = fmaf(cw[w], os[w * c.rank + e], v);
+        if (n_splits == 1) out[((int64_t)t * s.heads + h) * ldo + e] = from_f32<T>(v * inv);
+        else pd[2 + e] = v;
+    }
+    if (n_splits > 1 && threadIdx.x == 0) { pd[0] = M; pd[1] = L; }
+}
+
+// bf16: block per (16 heads, token, split), 4 warps, key tiles of 32 double-buffered with cp.async. Scores: warp w takes
+// keys 8 w .. + 7 of the tile, all heads; mixture: warp w takes NT 8-column tiles of the latent, all keys.
+constexpr int LM_KEYS = 32, LM_WARPS = 4, LM_PLD = LM_KEYS + 8;
+template <int NT>
+__global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
+                                                                             const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
+                                                                             bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
+    extern __shared__ __align__(16) bf16 lm_smem[];
+    __shared__ float ss[16][LM_KEYS + 1], corr_s[16], l_s[16], m_s[16];
+    __shared__ __align__(16) bf16 ps[16][LM_PLD];
+    const int width = c.rank16 + c.rot16, LD = width + 8;
+    bf16* qs = lm_smem;
+    bf16* ks = lm_smem + 16 * LD;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int h0 = blockIdx.x * 16, t = blockIdx.y;
+    pdl_wait();
+    pdl_trigger();
+    int begin, end;
+    key_range(tok_pos[t], s.window, blockIdx.z, n_splits, begin, end);
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    const int pieces = width / 8;
+    for (int i = tid; i < 16 * pieces; i += LM_WARPS * 32) {
+        const int r = i / pieces, p = i - r * pieces;
+        const bool live = h0 + r < s.heads;
+        cp_async16(qs + r * LD + p * 8, qabs + ((int64_t)t * s.heads + (live ? h0 + r : h0)) * c.ld + p * 8, live ? 16 : 0);
+    }
+    auto fetch = [&](int k0, int buf) {
+        bf16* d = ks + buf * LM_KEYS * LD;
+        for (int i = tid; i < LM_KEYS * pieces; i += LM_WARPS * 32) {
+            const int r = i / pieces, p = i - r * pieces, key = min(k0 + r, end - 1);
+            const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld + p * 8;
+            cp_async16(d + r * LD + p * 8, src, k0 + r < end ? 16 : 0);
+        }
+    };
+    if (begin < end) fetch(begin, 0);
+    cp_async_commit();
+    float o[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    float m = -INFINITY, l = 0.f;  // of row tid / 8, the same in its eight threads
+    const int col0 = warp * NT * 8;
+    for (int k0 = begin, buf = 0; k0 < end; k0 += LM_KEYS, buf ^= 1) {
+        cp_async_wait<0>();
+        __syncthreads();  // this tile has landed for everyone, and everyone is done with the other buffer
+        if (k0 + LM_KEYS < end) fetch(k0 + LM_KEYS, buf ^ 1);
+        cp_async_commit();
+        const bf16* kt = ks + buf * LM_KEYS * LD;
+        {
+            float a0[4] = {}, a1[4] = {};
+            const uint32_t qa = smem_addr(qs + (lane & 15) * LD + (lane >> 4) * 8);
+            const uint32_t ka = smem_addr(kt + (8 * warp + (lane & 7)) * LD + (lane >> 3) * 8);
+            int k = 0;
+            for (; k + 32 <= width; k += 32) {
+                uint32_t q0[4], q1[4], b[4];
+                ldsm_x4(q0, qa + 2 * k);
+                ldsm_x4(q1, qa + 2 * (k + 16));
+                ldsm_x4(b, ka + 2 * k);
+                mma_bf16(a0, q0[0], q0[1], q0[2], q0[3], b[0], b[1]);
+                mma_bf16(a1, q1[0], q1[1], q1[2], q1[3], b[2], b[3]);
+            }
+            if (k < width) {
+                uint32_t q0[4], b[2];
+                ldsm_x4(q0, qa + 2 * k);
+                ldsm_x2(b, smem_addr(kt + (8 * warp + (lane & 7)) * LD + ((lane >> 3) & 1) * 8) + 2 * k);
+                mma_bf16(a0, q0[0], q0[1], q0[2], q0[3], b[0], b[1]);
+            }
+            const int key = 8 * warp + 2 * tq;
+            const bool v0 = k0 + key < end, v1 = k0 + key + 1 < end;
+            ss[g][key] = v0 ? (a0[0] + a1[0]) * s.scale : -INFINITY;
+            ss[g][key + 1] = v1 ? (a0[1] + a1[1]) * s.scale : -INFINITY;
+            ss[g + 8][key] = v0 ? (a0[2] + a1[2]) * s.scale : -INFINITY;
+            ss[g + 8][key + 1] = v1 ? (a0[3] + a1[3]) * s.scale : -INFINITY;
+        }
+        __syncthreads();
+        {
+            const int r = tid >> 3, q4 = (tid & 7) * 4;
+            float v[4], mx = m;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { v[i] = ss[r][q4 + i]; mx = fmaxf(mx, v[i]); }
+#pragma unroll
+            for (int off = 4; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
+            // the tile's first key is live, so mx is finite
+            const float cr = expf(m - mx);
+            float sum = 0.f;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
+#pragma unroll
+            for (int off = 4; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
+            *reinterpret_cast<uint2*>(&ps[r][q4]) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+            l = fmaf(l, cr, sum);
+            m = mx;
+            if ((tid & 7) == 0) corr_s[r] = cr;
+        }
+        __syncthreads();
+        const float c0 = corr_s[g], c1 = corr_s[g + 8];
+#pragma unroll
+        for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+#pragma unroll
+        for (int kk = 0; kk < LM_KEYS / 16; ++kk) {
+            uint32_t p[4];
+            ldsm_x4(p, smem_addr(&ps[lane & 15][kk * 16 + (lane >> 4) * 8]));
+            const uint32_t va = smem_addr(kt + (kk * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
+#pragma unroll
+            for (int i = 0; i < NT; i += 2) {
+                if (col0 + i * 8 < c.rank16) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, va + 2 * (col0 + i * 8));
+                    mma_bf16(o[i], p[0], p[1], p[2], p[3], b[0], b[1]);
+                    mma_bf16(o[i + 1], p[0], p[1], p[2], p[3], b[2], b[3]);
+                }
+            }
+        }
+    }
+    cp_async_wait<0>();
+    if ((tid & 7) == 0) { l_s[tid >> 3] = l; m_s[tid >> 3] = m; }
+    __syncthreads();
+#pragma unroll
+    for (int r2 = 0; r2 < 2; ++r2) {
+        const int r = g + 8 * r2, h = h0 + r;
+        if (h >= s.heads) continue;
+        if (n_splits == 1) {
+            const float inv = 1.0f / l_s[r];
+            bf16* d = out + ((int64_t)t * s.heads + h) * ldo;
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const int e = col0 + i * 8 + 2 * tq;
+                if (e < c.rank) d[e] = __float2bfloat16_rn(o[i][2 * r2] * inv);
+                if (e + 1 < c.rank) d[e + 1] = __float2bfloat16_rn(o[i][2 * r2 + 1] * inv);
+            }
+        } else {
+            float* d = part + (((int64_t)t * s.heads + h) * n_splits + blockIdx.z) * (c.rank + 2);
+            if (warp == 0 && tq == 0) { d[0] = m_s[r]; d[1] = l_s[r]; }
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const int e = col0 + i * 8 + 2 * tq;
+                if (e < c.rank) d[2 + e] = o[i][2 * r2];
+                if (e + 1 < c.rank) d[3 + e] = o[i][2 * r2 + 1];
+            }
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part, int heads, int n_splits, int rank, T* __restrict__ out, int ldo) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t th = (int64_t)blockIdx.y * heads + blockIdx.x;
+    const float* src = part + th * n_splits * (rank + 2);
+    float M = -INFINITY, L = 0.f;
+    for (int i = 0; i < n_splits; ++i) M = fmaxf(M, src[(int64_t)i * (rank + 2)]);
+    for (int i = 0; i < n_splits; ++i) {
+        const float m = src[(int64_t)i * (rank + 2)];
+        if (m != -INFINITY) L = fmaf(expf(m - M), src[(int64_t)i * (rank + 2) + 1], L);
+    }
+    const float inv = 1.0f / L;
+    for (int e = threadIdx.x; e < rank; e += 128) {
+        float v = 0.f;
+        for (int i = 0; i < n_splits; ++i) {
+            const float m = src[(int64_t)i * (rank + 2)];
+            if (m != -INFINITY) v = fmaf(expf(m - M), src[(int64_t)i * (rank + 2) + 2 + e], v);
+        }
+        out[th * ldo + e] = from_f32<T>(v * inv);
+    }
+}
+
+size_t latent_part_floats(int n_tok, int heads, int n_splits, int rank) { return n_splits > 1 ? (size_t)n_tok * heads * n_splits * (rank + 2) : 0; }
+
+cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, const LatentCache& c, const int32_t* tok_slot, const int32_t* tok_pos,
+                                    void* o, int ldo, float* part, int n_splits, bool f32, int n_tok, cudaStream_t st) {
+    if (n_tok == 0) return cudaSuccess;
+    if (n_splits < 1 || (n_splits > 1 && !part) || c.rank > 32 * LS_MAX_PER_LANE) return cudaErrorInvalidValue;
+    constexpr int CAP = 200 * 1024;
+    static PerDeviceOnce once;
+    cudaError_t le = once.run([] {
+        const void* fns[] = {(const void*)latent_attention_mma_kernel<2>, (const void*)latent_attention_mma_kernel<4>, (const void*)latent_attention_mma_kernel<8>,
+                             (const void*)latent_attention_mma_kernel<16>, (const void*)latent_attention_simple_kernel<float>, (const void*)latent_attention_simple_kernel<bf16>};
+        for (const void* f : fns) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
+    });
+    if (le != cudaSuccess) return le;
+    const int width = c.rank16 + c.rot16;
+    const size_t mma_smem = (size_t)(16 + 2 * LM_KEYS) * (width + 8) * 2;
+    const int per_warp = (c.rank16 + 8 * LM_WARPS - 1) / (8 * LM_WARPS);  // 8-column tiles each warp has to cover
+    if (!f32 && per_warp <= 16 && mma_smem <= CAP) {
+        const dim3 grid((s.heads + 15) / 16, n_tok, n_splits), block(LM_WARPS * 32);
+#define SP_LM(NT) le = launch_pdl(latent_attention_mma_kernel<NT>, grid, block, mma_smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
+        if (per_warp <= 2) SP_LM(2);
+        else if (per_warp <= 4) SP_LM(4);
+        else if (per_warp <= 8) SP_LM(8);
+        else SP_LM(16);
+#undef SP_LM
+    } else {
+        const dim3 grid(s.heads, n_tok, n_splits), block(LS_WARPS * 32);
+        const size_t smem = (size_t)(width + LS_WARPS * c.rank) * 4;
+        if (smem > CAP) return cudaErrorInvalidValue;
+        le = f32 ? launch_pdl(latent_attention_simple_kernel<float>, grid, block, smem, st, (const float*)qabs, s, c, tok_slot, tok_pos, (float*)o, ldo, part, n_splits)
+                 : launch_pdl(latent_attention_simple_kernel<bf16>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits);
+    }
+    if (le != cudaSuccess) return le;
+    le = count_launch_and_check();
+    if (le != cudaSuccess || n_splits == 1) return le;
+    le = f32 ? launch_pdl(latent_merge_kernel<float>, dim3(s.heads, n_tok), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (float*)o, ldo)
+             : launch_pdl(latent_merge_kernel<bf16>, dim3(s.heads, n_tok), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (bf16*)o, ldo);
+    if (le != cudaSuccess) return le;
+    return count_launch_and_check();
+}
+
+// ── expanded attention ──
+__global__ void latent_gather_kernel(const LatentCache c, const int32_t* __restrict__ key_slot, const int32_t* __restrict__ key_pos, uint4* __restrict__ dst) {
+    pdl_wait();
+    pdl_trigger();
+    const int pos = key_pos[blockIdx.x], page = c.page_table[(int64_t)key_slot[blockIdx.x] * c.max_pages + pos / KV_PAGE];
+    const int ld16 = c.ld / 8;
+    const uint4* src = reinterpret_cast<const uint4*>(c.pool) + ((int64_t)page * KV_PAGE + pos % KV_PAGE) * ld16;
+    for (int i = threadIdx.x; i < ld16; i += blockDim.x) dst[(int64_t)blockIdx.x * ld16 + i] = src[i];
+}
+
+cudaError_t launch_latent_gather(const LatentCache& c, const int32_t* key_slot, const int32_t* key_pos, int n_keys, void* dst, cudaStream_t st) {
+    if (n_keys == 0) return cudaSuccess;
+    cudaError_t le = launch_pdl(latent_gather_kernel, dim3(n_keys), dim3(64), 0, st, c, key_slot, key_pos, (uint4*)dst);
+    if (le != cudaSuccess) return le;
+    return count_launch_and_check();
+}
+
+// Block per (head, tile of 64 tokens), 4 warps x 16 query rows, key tiles of 64 double-buffered with cp.async.
+constexpr int LE_KEYS = 64, LE_WARPS = 4;
+static int le_smem(int dim16, int rot16, int vdim16) { return (3 * 64 * (dim16 + rot16 + 8) + 2 * LE_KEYS * (vdim16 + 8)) * 2; }
+bool latent_expanded_supported(int dim, int rot, int vdim) {
+    const int d = (dim + 15) & ~15, r = (rot + 15) & ~15, v = (vdim + 15) & ~15;
+    return v <= 256 && le_smem(d, r, v) <= 200 * 1024;
+}
+
+template <int VT>
+__global__ void __launch_bounds__(LE_WARPS * 32) latent_expanded_kernel(const bf16* __restrict__ qf, const bf16* __restrict__ kv, const bf16* __restrict__ lat,
+                                                                        const LatentShape s, int rank16, int rot16, int ldl, const LatentTile* __restrict__ tiles,
+                                                                        const float* __restrict__ gate, int ldgate, bf16* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) bf16 le_sm[];
+    pdl_wait();
+    pdl_trigger();
+    const int dim16 = (s.dim + 15) & ~15, vdim16 = (s.vdim + 15) & ~15, qw = dim16 + rot16, LQ = qw + 8, LV = vdim16 + 8, kvw = dim16 + vdim16;
+    bf16 *qs = le_sm, *ks = qs + 64 * LQ, *vs = ks + 2 * LE_KEYS * LQ;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int h = blockIdx.x;
+    const LatentTile tl = tiles[blockIdx.y];
+    for (int i = tid; i < 64 * (qw / 8); i += LE_WARPS * 32) {
+        const int r = i / (qw / 8), p = i - r * (qw / 8);
+        cp_async16(qs + r * LQ + p * 8, qf + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * qw + p * 8, 16);
+    }
+    const int hi = tl.pos0 + tl.n - 1, lo = s.window > tl.pos0 ? 0 : tl.pos0 - s.window + 1;
+    auto fetch = [&](int k0, int buf) {
+        bf16 *kd = ks + buf * LE_KEYS * LQ, *vd = vs + buf * LE_KEYS * LV;
+        const int pk = dim16 / 8, pr = rot16 / 8, pv = vdim16 / 8, per = pk + pr + pv;
+        for (int i = tid; i < LE_KEYS * per; i += LE_WARPS * 32) {
+            const int r = i / per, p = i - r * per, key = min(k0 + r, hi);
+            const int64_t row = tl.key_row + (key - tl.key_pos0);
+            const int bytes = k0 + r <= hi ? 16 : 0;
+            const bf16* kvr = kv + (row * s.heads + h) * kvw;
+            if (p < pk) cp_async16(kd + r * LQ + p * 8, kvr + p * 8, bytes);
+            else if (p < pk + pr) cp_async16(kd + r * LQ + p * 8, lat + row * ldl + rank16 + (p - pk) * 8, bytes);
+            else cp_async16(vd + r * LV + (p - pk - pr) * 8, kvr + dim16 + (p - pk - pr) * 8, bytes);
+        }
+    };
+    fetch(lo, 0);
+    cp_async_commit();
+    float o[VT][4];
+#pragma unroll
+    for (int i = 0; i < VT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const int r0 = warp * 16 + g, r1 = r0 + 8;
+    const int p0 = tl.pos0 + min(r0, tl.n - 1), p1 = tl.pos0 + min(r1, tl.n - 1);
+    for (int k0 = lo, buf = 0; k0 <= hi; k0 += LE_KEYS, buf ^= 1) {
+        cp_async_wait<0>();
+        __syncthreads();
+        if (k0 + LE_KEYS <= hi) fetch(k0 + LE_KEYS, buf ^ 1);
+        cp_async_commit();
+        const bf16 *kt = ks + buf * LE_KEYS * LQ, *vt = vs + buf * LE_KEYS * LV;
+        float sc[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+        const uint32_t qa = smem_addr(qs + (warp * 16 + (lane & 15)) * LQ + (lane >> 4) * 8);
+        const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8);
+        for (int k = 0; k < qw; k += 16) {
+            uint32_t q[4];
+            ldsm_x4(q, qa + 2 * k);
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                uint32_t b[4];
+                ldsm_x4(b, ka + 2 * (8 * j * LQ + k));
+                mma_bf16(sc[j], q[0], q[1], q[2], q[3], b[0], b[1]);
+                mma_bf16(sc[j + 1], q[0], q[1], q[2], q[3], b[2], b[3]);
+            }
+        }
+        float x0 = m0, x1 = m1;
+        // only the window's two ends need the mask
+        const bool edge = k0 + LE_KEYS - 1 > tl.pos0 || (int64_t)hi - k0 >= s.window;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int key = k0 + 8 * j + 2 * tq + e;
+                sc[j][e] = (!edge || (key <= p0 && p0 - key < s.window)) ? sc[j][e] * s.scale : -INFINITY;
+                sc[j][2 + e] = (!edge || (key <= p1 && p1 - key < s.window)) ? sc[j][2 + e] * s.scale : -INFINITY;
+                x0 = fmaxf(x0, sc[j][e]);
+                x1 = fmaxf(x1, sc[j][2 + e]);
+            }
+        }
+#pragma unroll
+        for (int off = 1; off < 4; off <<= 1) {
+            x0 = fmaxf(x0, __shfl_xor_sync(0xFFFFFFFFu, x0, off));
+            x1 = fmaxf(x1, __shfl_xor_sync(0xFFFFFFFFu, x1, off));
+        }
+        // a row that has seen no visible key yet keeps everything at zero
+        const float b0 = x0 == -INFINITY ? 0.f : x0, b1 = x1 == -INFINITY ? 0.f : x1;
+        const float c0 = expf(m0 - b0), c1 = expf(m1 - b1);
+        float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            sc[j][0] = __expf(sc[j][0] - b0); sc[j][1] = __expf(sc[j][1] - b0);
+            sc[j][2] = __expf(sc[j][2] - b1); sc[j][3] = __expf(sc[j][3] - b1);
+            s0 += sc[j][0] + sc[j][1];
+            s1 += sc[j][2] + sc[j][3];
+        }
+        l0 = fmaf(l0, c0, s0);
+        l1 = fmaf(l1, c1, s1);
+        m0 = x0;
+        m1 = x1;
+#pragma unroll
+        for (int i = 0; i < VT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            const uint32_t a0 = pack_bf16(sc[2 * kk][0], sc[2 * kk][1]), a1 = pack_bf16(sc[2 * kk][2], sc[2 * kk][3]);
+            const uint32_t a2 = pack_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1]), a3 = pack_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3]);
+            const uint32_t va = smem_addr(vt + (kk * 16 + (lane & 15)) * LV + (lane >> 4) * 8);
+#pragma unroll
+            for (int i = 0; i < VT; i += 2) {
+                if (i * 8 < vdim16) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, va + 2 * (i * 8));
+                    mma_bf16(o[i], a0, a1, a2, a3, b[0], b[1]);
+                    mma_bf16(o[i + 1], a0, a1, a2, a3, b[2], b[3]);
+                }
+            }
+        }
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int off = 1; off < 4; off <<= 1) {
+        l0 += __shfl_xor_sync(0xFFFFFFFFu, l0, off);
+        l1 += __shfl_xor_sync(0xFFFFFFFFu, l1, off);
+    }
+#pragma unroll
+    for (int r2 = 0; r2 < 2; ++r2) {
+        const int r = r2 ? r1 : r0;
+        if (r >= tl.n) continue;
+        const int64_t row = tl.row0 + r;
+        const float f = (gate ? sigmoid_f32(gate[row * ldgate + h]) : 1.f) / (r2 ? l1 : l0);
+        bf16* d = out + row * ldo + (int64_t)h * s.vdim;
+#pragma unroll
+        for (int i = 0; i < VT; ++i) {
+            const int e = i * 8 + 2 * tq;
+            if (e < s.vdim) d[e] = __float2bfloat16_rn(o[i][2 * r2] * f);
+            if (e + 1 < s.vdim) d[e + 1] = __float2bfloat16_rn(o[i][2 * r2 + 1] * f);
+        }
+    }
+}
+
+cudaError_t launch_latent_expanded(const void* qf, const void* kv, const void* lat, const LatentShape& s, const LatentCache& c,
+                                   const LatentTile* tiles, int n_tiles, const float* gate, int ldgate, void* out, int ldo, cudaStream_t st) {
+    if (n_tiles == 0) return cudaSuccess;
+    if (!latent_expanded_supported(s.dim, s.rot, s.vdim)) return cudaErrorInvalidValue;
+    constexpr int CAP = 200 * 1024;
+    static PerDeviceOnce once;
+    cudaError_t le = once.run([] {
+        const void* fns[] = {(const void*)latent_expanded_kernel<4>, (const void*)latent_expanded_kernel<8>, (const void*)latent_expanded_kernel<16>,
+                             (const void*)latent_expanded_kernel<32>};
+        for (const void* f : fns) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
+    });
+    if (le != cudaSuccess) return le;
+    const int vdim16 = (s.vdim + 15) & ~15;
+    const size_t smem = (size_t)le_smem((s.dim + 15) & ~15, c.rot16, vdim16);
+    const dim3 grid(s.heads, n_tiles), block(LE_WARPS * 32);
+#define SP_LE(VT) le = launch_pdl(latent_expanded_kernel<VT>, grid, block, smem, st, (const bf16*)qf, (const bf16*)kv, (const bf16*)lat, s, c.rank16, c.rot16, c.ld, tiles, gate, ldgate, (bf16*)out, ldo)
+    if (vdim16 <= 32) SP_LE(4);
+    else if (vdim16 <= 64) SP_LE(8);
+    else if (vdim16 <= 128) SP_LE(16);
+    else SP_LE(32);
+#undef SP_LE
+    if (le != cudaSuccess) return le;
+    return count_launch_and_check();
+}
+
+}  // namespace sp

@@ -1,0 +1,126 @@
+// Registry of architectures and the readers of their configuration files (model_plan.h).
+#include "model_plan.h"
+
+#include <climits>
+#include <cmath>
+
+#include "engine.h"
+
+namespace sp {
+
+namespace {
+
+// Typed access to a configuration object; the first problem is remembered with the path it was found at.
+struct Cfg {
+    const Json* j;
+    std::string at;
+    std::string* err;
+    Cfg sub(const char* key) const {
+        const Json* s = j ? j->get(key) : nullptr;
+        if (!s || s->type != Json::OBJ) fail(std::string(key) + " is missing or not an object");
+        return Cfg{s, at + key + ".", err};
+    }
+    bool has(const char* key) const { return j && j->get(key); }
+    void fail(const std::string& what) const {
+        if (err->empty()) *err = "config: " + at + what;
+    }
+    double num(const char* key) const {
+        const Json* s = j ? j->get(key) : nullptr;
+        if (!s || s->type != Json::NUM || !std::isfinite(s->num)) { fail(std::string(key) + " is missing or not a number"); return 0; }
+        return s->num;
+    }
+    int size(const char* key, int least = 1) const {
+        const double v = num(key);
+        if (err->empty() && (v != std::floor(v) || v < least || v > INT_MAX)) fail(std::string(key) + " is out of range");
+        return err->empty() ? (int)v : least;
+    }
+};
+
+ClampedExpertSpec read_expert(const Cfg& c) {
+    ClampedExpertSpec e;
+    e.ff = c.size("ff");
+    e.limit = (float)c.num("limit");
+    return e;
+}
+
+LatentAttentionSpec read_latent_attention(const Cfg& c, int layer, const ModelPlan& p) {
+    LatentAttentionSpec m;
+    m.heads = c.size("heads");
+    m.dim = c.size("dim");
+    m.rot_dim = c.size("rot_dim");
+    m.vdim = c.size("vdim");
+    m.kv_rank = c.size("kv_rank");
+    m.scale = (float)c.num("scale");
+    const Cfg rot = c.sub("rot");
+    m.rot.base = rot.num("base");
+    m.rot.dims = rot.has("dims") ? rot.size("dims") : m.rot_dim;
+    if (m.rot.dims != m.rot_dim || (m.rot_dim & 1) || m.rot.base <= 0) c.fail("rot does not fit rot_dim");
+    if (c.has("mask") && c.sub("mask").has("size")) m.window = c.sub("mask").size("size");
+    if (c.has("kv_from")) {
+        m.kv_from = c.size("kv_from", 0);
+        if (!c.err->empty()) return m;
+        if (m.kv_from >= layer) { c.fail("kv_from must name an earlier layer"); return m; }
+        const LatentAttentionSpec& o = p.layers[(size_t)m.kv_from].mix;
+        if (o.kv_from >= 0 || o.kv_rank != m.kv_rank || o.rot_dim != m.rot_dim || o.rot.base != m.rot.base)
+            c.fail("kv_from names a layer whose latent does not fit");
+    }
+    return m;
+}
+
+int read_lepalorn(const Json& cfg, ModelPlan* out) {
+    std::string err;
+    const Cfg c{&cfg, "", &err};
+    ModelPlan p;
+    p.name = "Lepalorn";
+    p.vocab = c.size("vocab");
+    p.width = c.size("width");
+    p.eps = (float)c.sub("norm").num("eps");
+    p.embed_scale = (float)c.sub("embedding").num("scale");
+    p.depth_average = true;
+    const Json* layers = cfg.get("layers");
+    if (!layers || layers->type != Json::ARR || layers->arr.empty()) c.fail("layers is missing or not a list");
+    for (size_t i = 0; err.empty() && i < layers->arr.size(); ++i) {
+        const std::string idx = std::to_string(i);
+        const Cfg lc{&layers->arr[i], "layers[" + idx + "].", &err};
+        LayerPlan l;
+        l.prefix = "l" + idx + ".";
+        const Json* type = lc.j->get("type");
+        if (!type || type->str != "latent_attention") { lc.fail("type is not a mixer of this design"); break; }
+        l.mix = read_latent_attention(lc.sub("mixer"), (int)i, p);
+        if (lc.has("mlp")) {
+            const Cfg m = lc.sub("mlp");
+            const Json* kind = m.j ? m.j->get("kind") : nullptr;
+            if (!kind || kind->str != "moe") { m.fail("kind is not a feed-forward of this design"); break; }
+            l.has_mlp = true;
+            l.mlp.experts = m.sub("router").size("experts");
+            l.mlp.top = m.sub("router").size("top");
+            l.mlp.expert = read_expert(m.sub("expert"));
+            if (m.has("shared")) {
+                l.mlp.has_shared = true;
+                l.mlp.shared = read_expert(m.sub("shared"));
+            }
+            if (l.mlp.top > l.mlp.experts) m.fail("router.top exceeds router.experts");
+        }
+        p.layers.push_back(l);
+    }
+    if (!err.empty()) { set_error(err); return SP_ERR_ARG; }
+    *out = std::move(p);
+    return SP_OK;
+}
+
+// GGUF names: crates/sapient-models/src/forward/mod.rs:223-316 (family dispatch of the reference's loader).
+const ArchEntry ARCHS[] = {
+    {"llama", ARCH_LLAMA, true, nullptr},   {"mistral", ARCH_LLAMA, true, nullptr}, {"qwen2", ARCH_LLAMA, true, nullptr},
+    {"qwen3", ARCH_LLAMA, true, nullptr},   {"idefics3", ARCH_LLAMA, true, nullptr}, {"phi3", ARCH_LLAMA, true, nullptr},
+    {"phi", ARCH_PHI2, true, nullptr},      {"phi2", ARCH_PHI2, true, nullptr},     {"Lepalorn", ARCH_PLAN, false, read_lepalorn},
+};
+
+}  // namespace
+
+const ArchEntry* find_arch(const std::string& name) {
+    for (const ArchEntry& a : ARCHS)
+        if (name == a.name) return &a;
+    return nullptr;
+}
+
+}  // namespace sp

@@ -7,6 +7,7 @@
 #include <cstring>
 
 #include "engine.h"
+#include "plan_kernels.h"
 #include "pdl.cuh"
 #include "sp_common.cuh"
 
@@ -277,9 +278,10 @@ int Engine::tp_reset() {
 }
 
 int Engine::device_check() {
-    const int a = tc5_take_timeout(), b = imma_take_timeout();
-    if (a < 0 || b < 0) { set_error("could not read the kernels' timeout flags"); return SP_ERR_CUDA; }
+    const int a = tc5_take_timeout(), b = imma_take_timeout(), c = mat_tc5_take_timeout();
+    if (a < 0 || b < 0 || c < 0) { set_error("could not read the kernels' timeout flags"); return SP_ERR_CUDA; }
     if (a > 0) { set_error("tcgen05 GEMM: a bounded mbarrier wait expired, the outputs of that launch are not valid"); return SP_ERR_CUDA; }
+    if (c > 0) { set_error("tcgen05 GEMM on bf16 weights: a bounded mbarrier wait expired, the outputs of that launch are not valid"); return SP_ERR_CUDA; }
     if (b > 0) { set_error("streaming GEMV: a bounded mbarrier wait expired, the outputs of that launch are not valid"); return SP_ERR_CUDA; }
     return tp_check();
 }

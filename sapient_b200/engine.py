@@ -48,7 +48,9 @@ class ForwardEngine:
         more on the tcgen05 GEMM with operands rounded to fp16 instead of the default exact-class mode (see
         set_large_m_gemm)."""
         d = SpModelDesc()
-        d.arch = 1 if cfg["arch"] in ("phi2", "phi") else 0
+        d.arch = cls.arch_block(cfg["arch"])
+        if d.arch == 2:
+            raise SapientCudaError(_lib.SP_ERR_ARG, "layer-plan architectures are built by from_config / from_pretrained")
         d.n_layers, d.hidden, d.n_heads, d.n_kv_heads = cfg["n_layers"], cfg["hidden"], cfg["n_heads"], cfg["n_kv_heads"]
         d.head_dim, d.ffn, d.vocab, d.max_ctx = cfg["head_dim"], cfg["ffn"], cfg["vocab"], cfg["max_ctx"]
         d.rotary_dim = cfg.get("rotary_dim") or cfg["head_dim"]
@@ -76,6 +78,63 @@ class ForwardEngine:
     def from_gguf(cls, path: str, device: int = 0, max_ctx: int = 0, max_batch: int = 1) -> "ForwardEngine":
         h = C.c_void_p()
         check(lib().sp_cuda_engine_from_gguf(str(path).encode(), device, max_ctx, max_batch, C.byref(h)))
+        d = SpModelDesc()
+        check(lib().sp_cuda_engine_desc(h, C.byref(d)))
+        return cls(h, d)
+
+    @staticmethod
+    def arch_block(name: str) -> int:
+        """Which block the registry runs an architecture with: 0 Llama/Qwen, 1 Phi-2, 2 a layer plan."""
+        b = C.c_int32()
+        check(lib().sp_cuda_arch_block(name.encode(), C.byref(b)))
+        return int(b.value)
+
+    @staticmethod
+    def _run_desc(device: int, max_ctx: int, max_batch: int, max_tokens: int, kv_pages: int) -> SpModelDesc:
+        d = SpModelDesc()
+        d.device, d.max_ctx, d.max_batch, d.max_tokens, d.kv_pages, d.tp_size = device, max_ctx, max_batch, max_tokens, kv_pages, 1
+        return d
+
+    COMPUTE = {"bfloat16": 30, "float32": 0}
+
+    @classmethod
+    def from_pretrained(cls, path: str, dtype: str = "bfloat16", device: int = 0, max_ctx: int = 4096, max_batch: int = 1,
+                        max_tokens: int = 1024, kv_pages: int = 0) -> "ForwardEngine":
+        """A model directory: config.json (its "architecture" chooses the model from the registry) and
+        model.safetensors. dtype: "bfloat16" (matrix operands and cache in bf16, f32 accumulation) or "float32"."""
+        run = cls._run_desc(device, max_ctx, max_batch, max_tokens, kv_pages)
+        h = C.c_void_p()
+        check(lib().sp_cuda_engine_from_dir(str(path).encode(), cls.COMPUTE[dtype], C.byref(run), C.byref(h)))
+        d = SpModelDesc()
+        check(lib().sp_cuda_engine_desc(h, C.byref(d)))
+        return cls(h, d)
+
+    @classmethod
+    def from_config(cls, cfg: dict, weights: dict, dtype: str = "bfloat16", device: int = 0, max_ctx: int = 4096, max_batch: int = 1,
+                    max_tokens: int = 1024, kv_pages: int = 0) -> "ForwardEngine":
+        """The same from a configuration dict and name -> array weights: float32 arrays (numpy or CPU torch), or torch
+        bfloat16 tensors."""
+        import json
+
+        run = cls._run_desc(device, max_ctx, max_batch, max_tokens, kv_pages)
+        h = C.c_void_p()
+        check(lib().sp_cuda_engine_create_from_config(json.dumps(cfg).encode(), cls.COMPUTE[dtype], C.byref(run), C.byref(h)))
+        try:
+            for name, w in weights.items():
+                if hasattr(w, "detach"):
+                    import torch
+
+                    w = w.detach().cpu().contiguous()
+                    ty, raw = (30, w.view(torch.int16).numpy()) if w.dtype == torch.bfloat16 else (0, w.float().numpy())
+                else:
+                    ty, raw = 0, np.ascontiguousarray(w, np.float32)
+                shape = tuple(raw.shape) or (1,)
+                dd = (C.c_int64 * len(shape))(*shape)
+                check(lib().sp_cuda_engine_set_tensor(h, name.encode(), ty, dd, len(shape), _p(raw), raw.nbytes))
+            check(lib().sp_cuda_engine_finalize(h))
+        except Exception:
+            lib().sp_cuda_engine_destroy(h)
+            raise
         d = SpModelDesc()
         check(lib().sp_cuda_engine_desc(h, C.byref(d)))
         return cls(h, d)
@@ -251,6 +310,23 @@ class ForwardEngine:
         out = np.empty((ids.size, self.vocab_local) if all_positions else (self.vocab_local,), np.float32)
         check(lib().sp_cuda_forward_slot(self._h, slot, _p(ids), ids.size, int(all_positions), _p(out)))
         return out
+
+    def forward_mixed(self, entries, want_argmax: bool = False):
+        """One step over several sequences: entries = [(slot, token ids, wanted places among them)], portions of prompts
+        beside single tokens. Returns logits [wanted, vocab] (or the greedy picks) in the order of entries and places."""
+        ids, slots, rows = [], [], []
+        for slot, toks, want in entries:
+            places = [int(w) for w in want]
+            if sorted(set(places)) != places:
+                raise SapientCudaError(_lib.SP_ERR_ARG, "wanted places must be ascending")
+            rows += [len(ids) + w for w in places]
+            ids += [int(t) for t in toks]
+            slots += [int(slot)] * len(toks)
+        i, s, r = _ids(ids), np.ascontiguousarray(slots, dtype=np.int32), np.ascontiguousarray(rows, dtype=np.int32)
+        lg = None if want_argmax else np.empty((r.size, self.vocab_local), np.float32)
+        am = np.empty(r.size, np.uint32) if want_argmax else None
+        check(lib().sp_cuda_forward_rows(self._h, _p(i), _p(s), i.size, _p(r), r.size, None if want_argmax else _p(lg), _p(am) if want_argmax else None))
+        return am if want_argmax else lg
 
     def decode_batch(self, input_ids, slots, want_logits: bool = True, want_argmax: bool = False):
         """One token per sequence slot. Returns (logits [b, vocab] or None, argmax [b] or None)."""
