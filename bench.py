@@ -283,12 +283,21 @@ def main() -> None:
     ap.add_argument("--quick", action="store_true", help="prefill + warm-up + timed device loop only (for profiler runs)")
     ap.add_argument("--no-batch32", action="store_true", help="skip the 32-sequence decode section")
     ap.add_argument("--no-sweep", action="store_true", help="skip the operator sweep section")
+    ap.add_argument("--design", default=None, help="instead of the default workload: prefill and decode throughput of a layer-plan design "
+                    "(Lepalorn) beside the Llama block at equal size, one JSON line per size")
+    ap.add_argument("--design-size", default=None, help="only this size")
+    ap.add_argument("--design-only", action="store_true", help="without the Llama block")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local = int(os.environ.get("LOCAL_RANK", "0"))
     if args.impl == "reference":
         run_reference(args, rank, world)
+        return
+    if args.design:
+        from sapient_b200 import design_bench
+
+        design_bench.run(args.design, measured_peaks()[0], [args.design_size] if args.design_size else None, designs_only=args.design_only)
         return
     args.warmup = max(args.warmup, 3)
 

@@ -1,0 +1,157 @@
+"""Throughput of layer-plan designs beside the framework's closest GGUF block at equal size (`bench.py --design NAME`).
+
+Per size: the design with random bf16 weights, and a Llama block of the same width, heads, layers and ACTIVE feed-forward
+width (chosen experts + shared expert) in Q8_0 — prefill of one prompt, greedy decode at batch 1 and 32, device time by
+CUDA events, and for each family of kernels of a decode step and of a prefill its device time, algorithmic bytes and flops
+and the fraction of the roofline max(bytes / copy bandwidth, flops / GEMM rate) that is. Weights exceed L2 at every size.
+"""
+from __future__ import annotations
+
+import json
+
+import numpy as np
+
+from . import synth
+from .configs_bench import _engine, _timed
+from .engine import ForwardEngine
+
+# name -> (design keywords)
+SIZES = {
+    "2b": dict(layers=6, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, experts=64, top=6, ff=1408, shared_ff=2816,
+               vocab=32768, shared_latent_from=3),
+    "8b": dict(layers=4, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, experts=32, top=4, ff=2048, shared_ff=2048,
+               vocab=32768, shared_latent_from=2),
+}
+
+
+def llama_like(s: dict) -> dict:
+    return dict(arch="llama", n_layers=s["layers"], hidden=s["width"], n_heads=s["heads"], n_kv_heads=s["heads"], head_dim=128,
+                ffn=s["top"] * s["ff"] + s["shared_ff"], vocab=s["vocab"], norm_eps=1e-5, rope_theta=1e4, tied=False)
+
+
+def design_engine(s: dict, **kw):
+    import torch
+
+    cfg = synth.lepalorn_config(**s)
+    W = {k: v.cpu() for k, v in synth.lepalorn_weights(cfg, seed=11, device="cuda").items()}
+    torch.cuda.empty_cache()
+    eng = ForwardEngine.from_config(cfg, W, **kw)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    eng.set_stream(stream.cuda_stream)
+    return eng, stream
+
+
+def llama_engine(s: dict, max_ctx: int, **kw):
+    import torch
+
+    cfg, W = synth.build_model(llama_like(s), seed=12, device="cuda", max_ctx=max_ctx, dtype=synth.Q8_0)
+    W = synth.weights_to_numpy(W)
+    torch.cuda.empty_cache()
+    eng, stream = _engine(cfg, W, **kw)
+    return eng, stream
+
+
+def _distinct(experts: int, top: int, rows: int) -> float:
+    """Expected number of experts that at least one of `rows` tokens chooses (uniform choice)."""
+    return experts * (1.0 - (1.0 - top / experts) ** rows)
+
+
+def _pairs(n: int, window: int) -> int:
+    """(query, key) pairs of a causal prompt of n tokens under a sliding window."""
+    w = min(n, window)
+    return w * (w + 1) // 2 + (n - w) * w
+
+
+def design_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    """Algorithmic (bytes, flops) of one step by kernel family. Prefill: one sequence of `rows` tokens; decode: `rows`
+    sequences with `ctx` cached tokens each."""
+    L, W, H, D, R, V, K, E = s["layers"], s["width"], s["heads"], s["dim"], s["rot"], s["vdim"], s["rank"], s["experts"]
+    own = s["shared_latent_from"] + 1 if s["shared_latent_from"] is not None else L
+    dense = L * (H * (D + R) * W + H * W + H * (D + V) * K + W * H * V + (E + 1) * W + 3 * s["shared_ff"] * W) + own * (K + R) * W
+    active = L * 3 * s["ff"] * W
+    used = _distinct(E, s["top"], rows)
+    head = s["vocab"] * W
+    keys = _pairs(rows, s["window"]) if prefill else rows * min(ctx, s["window"])
+    per_pair = 2 * H * (D + R + V) if prefill else 2 * H * (K + R + K)
+    return {"gemv": (2 * (dense + active * used + head), 2 * rows * (dense + active * s["top"]) + 2 * head * (1 if prefill else rows)),
+            "attention": (L * 2 * (K + R) * (rows if prefill else keys), L * per_pair * keys)}
+
+
+def llama_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    c = llama_like(s)
+    q = c["n_heads"] * c["head_dim"]
+    mats = c["n_layers"] * (4 * q * c["hidden"] + 3 * c["ffn"] * c["hidden"])
+    head = c["vocab"] * c["hidden"]
+    keys = _pairs(rows, 1 << 30) if prefill else rows * ctx
+    return {"gemv": (34 / 32 * (mats + head), 2 * rows * mats + 2 * head * (1 if prefill else rows)),
+            "attention": (c["n_layers"] * 2 * 2 * q * (rows if prefill else keys), c["n_layers"] * 4 * q * keys)}
+
+
+def _families(ms: dict, work: dict, peaks: dict) -> dict:
+    out = {}
+    for f, t in ms.items():
+        if t <= 0:
+            continue
+        out[f] = {"ms": round(t, 4)}
+        if f in work:
+            b, fl = work[f]
+            floor = max(b / (peaks["hbm_gbs"] * 1e9), fl / (peaks["bf16_tflops"] * 1e12)) * 1e3
+            out[f].update(roofline_ms=round(floor, 4), frac=round(floor / t, 3))
+    return out
+
+
+def measure(eng, stream, vocab: int, work, prompt: int, ctx: int, batch: int, steps: int, peaks: dict, fast: bool = False) -> dict:
+    rng = np.random.default_rng(0)
+    ids = rng.integers(0, vocab, prompt).astype(np.uint32)
+    if fast:
+        eng.set_large_m_gemm(1)
+    res = {}
+    for _ in range(3):
+        eng.reset_cache(0)
+        eng.forward_slot(0, ids)
+    times = []
+    for _ in range(5):
+        eng.reset_cache(0)
+        times.append(_timed(stream, lambda: eng.forward_slot(0, ids)))
+    ms = sorted(times)[len(times) // 2]
+    eng.reset_cache(0)
+    eng.profile_read()
+    eng.set_profile(True)
+    eng.forward_slot(0, ids)
+    fam = {k: v[0] for k, v in eng.profile_read().items()}
+    eng.set_profile(False)
+    res["prefill"] = {"tokens": prompt, "ms": round(ms, 3), "tokens_per_s": round(prompt / ms * 1e3), "families": _families(fam, work(prompt, 0, True), peaks)}
+    for b in (1, batch):
+        eng.reset_cache()
+        for i in range(b):
+            eng.forward_slot(i, rng.integers(0, vocab, ctx).astype(np.uint32))
+        slots = list(range(b))
+        first = rng.integers(0, vocab, b).astype(np.uint32)
+        toks = eng.decode_greedy(first, slots, 8)
+        ms = _timed(stream, lambda: eng.decode_greedy(toks[-1], slots, steps, fetch=False)) / steps
+        eng.synchronize()
+        fam = {f: eng.time_families(f, b, 20) for f in eng.PROFILE_FAMILIES}
+        res[f"decode_b{b}"] = {"ctx": ctx, "ms_per_step": round(ms, 4), "tokens_per_s": round(b / ms * 1e3), "families": _families(fam, work(b, ctx, False), peaks)}
+    return res
+
+
+def run(design: str, peaks: dict, sizes=None, prompt: int = 2048, ctx: int = 1024, batch: int = 32, steps: int = 32, designs_only: bool = False) -> dict:
+    if design.lower() != "lepalorn":
+        raise SystemExit(f"no such design: {design}")
+    out = {"design": "Lepalorn", "data": "synthetic random weights", "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
+    kw = dict(max_batch=batch, max_tokens=prompt, kv_pages=(max(prompt, 0) + batch * (ctx + 256)) // 16)
+    for name in sizes or SIZES:
+        s = SIZES[name]
+        r = {"config": s}
+        eng, stream = design_engine(s, max_ctx=prompt + ctx, **kw)
+        r["design"] = measure(eng, stream, s["vocab"], lambda a, c, p: design_work(s, a, c, p), prompt, ctx, batch, steps, peaks)
+        eng.close()
+        if not designs_only:
+            for tag, fast in (("llama_q8_0", False), ("llama_q8_0_fp16_operands", True)):
+                eng, stream = llama_engine(s, prompt + ctx, **kw)
+                r[tag] = measure(eng, stream, s["vocab"], lambda a, c, p: llama_work(s, a, c, p), prompt, ctx, batch, steps, peaks, fast)
+                eng.close()
+        out["sizes"][name] = r
+        print(json.dumps({name: r}), flush=True)
+    return out

@@ -199,12 +199,13 @@ def weight_dtype(cfg: dict, role: str, layer: int, k: int) -> int:
     return Q4_K
 
 
-def build_model(cfg: dict, seed: int, device: str = "cpu", max_ctx: int | None = None, embed_float=None) -> tuple[dict, dict]:
+def build_model(cfg: dict, seed: int, device: str = "cpu", max_ctx: int | None = None, embed_float=None, dtype: int | None = None) -> tuple[dict, dict]:
     """Random-init N(0, 0.02) weights quantised per block. Returns (cfg, weights) where
     weights maps HF-style names (the keys the reference's GGUF name map produces,
     crates/sapient-models/src/gguf_weights.rs:360-455) to (dtype, dims, uint8 tensor).
     embed_float: a [vocab, hidden] f32 tensor to quantise as the token embedding (and tied output head) instead of a
-    fresh random one."""
+    fresh random one. dtype: one block format for every matrix instead of the layout rule."""
+    force = dtype
     cfg = dict(cfg)
     cfg.setdefault("rotary_dim", cfg["head_dim"])
     cfg["max_ctx"] = max_ctx or cfg.get("max_ctx", 4096)
@@ -214,7 +215,7 @@ def build_model(cfg: dict, seed: int, device: str = "cpu", max_ctx: int | None =
     W: dict = {}
 
     def mat(name, n, k, role, layer=0, dtype=None):
-        dt = dtype if dtype is not None else weight_dtype(cfg, role, layer, k)
+        dt = next((x for x in (dtype, force) if x is not None), weight_dtype(cfg, role, layer, k))
         # quantise in row chunks to bound temporary memory on large matrices
         rows_per = max(1, (1 << 26) // k)
         parts = []
@@ -382,3 +383,86 @@ def write_gguf(path: str, cfg: dict, W: dict) -> None:
     wr.write_kv_data_to_file()
     wr.write_tensors_to_file()
     wr.close()
+
+
+# ── layer-plan designs: a configuration dict as in config.json, and name -> bf16 tensor weights ──
+def lepalorn_config(layers: int, width: int, heads: int, dim: int, rot: int, vdim: int, rank: int, window: int, experts: int, top: int, ff: int,
+                    shared_ff: int, vocab: int, shared_latent_from: int | None = None, limit: float = 7.0) -> dict:
+    """Equal layers; layers after `shared_latent_from` read that layer's latents instead of making their own."""
+    out = []
+    for i in range(layers):
+        mix = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5,
+               "mask": {"size": window}, "rot": {"base": 10000.0, "dims": rot}}
+        if shared_latent_from is not None and i > shared_latent_from:
+            mix["kv_from"] = shared_latent_from
+        mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": limit}}
+        if shared_ff:
+            mlp["shared"] = {"ff": shared_ff, "limit": limit}
+        out.append({"type": "latent_attention", "mixer": mix, "mlp": mlp})
+    return {"architecture": "Lepalorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": out}
+
+
+def lepalorn_weights(cfg: dict, seed: int, device: str = "cpu") -> dict:
+    """Random bf16 weights, rows scaled so that activations keep their magnitude; depth averages near the newest result."""
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W: dict = {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = (torch.randn(n, k, generator=g, device=device, dtype=torch.float32) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(name, values):
+        W[name] = torch.as_tensor(values, dtype=torch.float32, device=device).to(torch.bfloat16)
+
+    w = cfg["width"]
+    mat("embed", cfg["vocab"], w, w ** 0.5)
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp, p = layer["mixer"], layer.get("mlp"), f"l{i}."
+        H, D, R, V, K = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        vec(p + "norm1", 0.5)
+        mat(p + "mix.q", H * (D + R), w)
+        if m.get("kv_from") is None:
+            mat(p + "mix.dkv", K + R, w)
+            vec(p + "mix.dkv.norm", 1.0 + 0.1 * torch.randn(K, generator=g, device=device))
+        mat(p + "mix.uk", H * D, K)
+        mat(p + "mix.uv", H * V, K)
+        mat(p + "mix.g", H, w)
+        mat(p + "mix.o", w, H * V)
+        if mlp:
+            vec(p + "norm2", 0.5)
+            mat(p + "mlp.router", mlp["router"]["experts"], w)
+            vec(p + "mlp.router.b", 0.1 * torch.randn(mlp["router"]["experts"], generator=g, device=device))
+            parts = [(f"mlp.e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+            if mlp.get("shared"):
+                parts.append(("mlp.shared.", mlp["shared"]["ff"]))
+                mat(p + "mlp.shared.sg", 1, w)
+            for tag, ff in parts:
+                mat(p + tag + "gate", ff, w)
+                mat(p + tag + "up", ff, w)
+                mat(p + tag + "down", w, ff)
+        vec(p + "dwa", 0.2 * torch.randn(i + 2, generator=g, device=device) + torch.eye(i + 2, device=device)[-1])
+    vec("final.norm", 1.0)
+    mat("head", cfg["vocab"], w)
+    return W
+
+
+def write_safetensors(path: str, cfg: dict, W: dict) -> None:
+    """A model directory: config.json and model.safetensors (bf16 tensors)."""
+    import json
+    import os
+    import struct
+
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    head, at, blobs = {}, 0, []
+    for name, t in W.items():
+        b = t.detach().cpu().contiguous().view(torch.int16).numpy().tobytes()
+        head[name] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(b)]}
+        at += len(b)
+        blobs.append(b)
+    h = json.dumps(head).encode()
+    with open(os.path.join(path, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(h)) + h)
+        for b in blobs:
+            f.write(b)
