@@ -57,6 +57,7 @@ struct LayerW {
 struct ModelPlan;
 struct PlanState;
 struct PlanMat;
+struct MatArgs;
 
 class Engine {
   public:
@@ -241,6 +242,7 @@ class Engine {
     int plan_mixer(int layer, int T);
     int plan_experts(int layer, int T);
     int plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, int ldy, bool out_f32);
+    int plan_product(const MatArgs& a, int max_tiles);
     int plan_head(const int32_t* rows, int n);
     int plan_ctx_bucket() const;
     int plan_privatise_copy(int from, int to);

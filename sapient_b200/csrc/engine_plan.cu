@@ -4,7 +4,7 @@
 // A layer is ten to twelve launches whatever the row count: projections, rotation + cache append, [absorb,] attention
 // [, merge, value maps], output projection, norm + residual, router, choice, grouping, gate|up of the chosen and the
 // shared expert, down, mixture + norm + residual + depth average. Steps of up to PLAN_ROWS rows take the row kernels
-// (mat_rows.cu) and the absorbed attention and can be captured as a graph; longer ones the tcgen05 GEMM (mat_tc5.cu) and,
+// (mat_f32.cu) and the absorbed attention and can be captured as a graph; longer ones the tcgen05 GEMM (mat_tc5.cu) and,
 // where rebuilding the keys pays, the expanded attention.
 #include "engine_plan.h"
 
@@ -34,7 +34,7 @@ namespace sp {
         }                                 \
     } while (0)
 
-constexpr int PLAN_ROWS = 32;         // rows the row kernels take in one pass
+constexpr int PLAN_ROWS = MAT_GATHER_ROWS;  // rows of a decode-shaped step
 constexpr int PLAN_SPLIT_ROWS = 256;  // (rows x key splits) of the absorbed attention's partials
 
 namespace {
@@ -90,7 +90,7 @@ struct PlanPacker {
         m.groups = groups;
         m.n = (int)rows;
         m.kp = mat_kpad(k);
-        const size_t bytes = (size_t)groups * rows * m.kp * p.elem() + 1024;  // + slack for whole-vector reads
+        const size_t bytes = (size_t)groups * rows * m.kp * p.elem();
         if (cudaMalloc(&m.w, bytes) != cudaSuccess) return fail(SP_ERR_OOM, "cannot allocate packed weights");
         p.owned.push_back(m.w);
         if (cudaMemset(m.w, 0, bytes) != cudaSuccess) return fail(SP_ERR_CUDA, "cudaMemset failed");
@@ -288,6 +288,10 @@ int Engine::finalize_plan() {
     p.part = (float*)take((size_t)PLAN_SPLIT_ROWS * n_part * 4);
     p.history = (float*)take((size_t)(L + 1) * T * W * 4);
     p.fin = take((size_t)PLAN_ROWS * p.wp * el);
+    if (!p.f32) {
+        p.scratch.part = (float*)take(MatScratch::FLOATS * 4);
+        p.scratch.cnt = (unsigned*)take(MatScratch::ITEMS * 4);
+    }
     if (n_pairs) {
         p.act = take(T * n_act * el);
         p.act_shared = take(T * n_act_s * el);
@@ -376,6 +380,11 @@ int Engine::plan_stage(int T) {
     return SP_OK;
 }
 
+int Engine::plan_product(const MatArgs& a, int max_tiles) {
+    SP_LAUNCH(F_GEMV, a.f32 ? launch_mat_f32(a, stream) : launch_mat_tc5(a, max_tiles, plan_->scratch, stream));
+    return SP_OK;
+}
+
 int Engine::plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, int ldy, bool out_f32) {
     MatArgs a{};
     a.f32 = plan_->f32;
@@ -383,9 +392,7 @@ int Engine::plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, i
     a.nseg = 1;
     a.m = m;
     a.seg[0] = MatSeg{w.w, w.n, w.kp, 1, 0.f, 0.f, x, ldx, 0, y, ldy, 0};
-    if (m > PLAN_ROWS && mat_tc5_supported(a)) SP_LAUNCH(F_GEMV, launch_mat_tc5(a, m, 0, stream));
-    else SP_LAUNCH(F_GEMV, launch_mat_rows(a, stream));
-    return SP_OK;
+    return plan_product(a, 0);
 }
 
 int Engine::plan_mixer(int li, int T) {
@@ -409,13 +416,13 @@ int Engine::plan_mixer(int li, int T) {
         a.nseg = 1;
         a.m = T;
         a.seg[0] = MatSeg{l.uk_t.w, l.uk_t.n, l.uk_t.kp, H, 0.f, 0.f, p.qn, H * l.uk_t.kp, l.uk_t.kp, p.qabs, H * l.cache.ld, l.cache.ld};
-        SP_LAUNCH(F_GEMV, launch_mat_rows(a, stream));
+        SP_TRY(plan_product(a, 0));
         SP_LAUNCH(F_ATTN, launch_latent_attention(p.qabs, s, l.cache, d_tok_slot_, d_tok_pos_, p.olat, l.uv.kp, p.part,
                                                   plan_splits(l, p.f32, plan_ctx_bucket(), T), p.f32, T, stream));
         a.seg[0] = MatSeg{l.uv.w, l.uv.n, l.uv.kp, H, 0.f, 0.f, p.olat, H * l.uv.kp, l.uv.kp, p.attn, l.o.kp, s.vdim};
         a.gate = gate;
         a.ldgate = ldp;
-        SP_LAUNCH(F_GEMV, launch_mat_rows(a, stream));
+        SP_TRY(plan_product(a, 0));
     }
     return plan_mat(l.o, p.attn, l.o.kp, T, p.y, p.plan.width, true);
 }
@@ -439,39 +446,41 @@ int Engine::plan_experts(int li, int T) {
     const MatSeg sgu{l.shared_gu.w, s.shared.ff, l.shared_gu.kp, 1, s.shared.limit, s.shared.alpha, p.xb, p.wp, 0, p.act_shared, l.shared_down.kp, 0};
     const MatSeg dn{l.down.w, W, l.down.kp, E, 0.f, 0.f, p.act, l.down.kp, 0, p.y_expert, W, 0};
     const MatSeg sdn{l.shared_down.w, W, l.shared_down.kp, 1, 0.f, 0.f, p.act_shared, l.shared_down.kp, 0, p.y_shared, W, 0};
+    const int max_tiles = std::min(pairs / MOE_TILE + std::min(E, pairs), pairs);
     if (T <= PLAN_ROWS || p.f32) {
         a.gather = true;
         a.nseg = s.has_shared ? 2 : 1;
         a.seg[0] = gu;
         a.seg[1] = sgu;
-        SP_LAUNCH(F_GEMV, launch_mat_rows(a, stream));
+        SP_TRY(plan_product(a, max_tiles));
         a.gather = a.dual = false;
         a.out_f32 = true;
+        a.x_rows = pairs;
         a.seg[0] = dn;
         a.seg[1] = sdn;
-        SP_LAUNCH(F_GEMV, launch_mat_rows(a, stream));
-        return SP_OK;
+        return plan_product(a, max_tiles);
     }
-    const int max_tiles = std::min(pairs / MOE_TILE + std::min(E, pairs), pairs);
     SP_LAUNCH(F_ELEM, launch_gather_act(p.xb, p.moe.row_src, pairs, p.wp, p.f32, p.xs, stream));
     a.nseg = 1;
+    a.x_rows = pairs;
     a.seg[0] = gu;
     a.seg[0].x = p.xs;
-    SP_LAUNCH(F_GEMV, launch_mat_tc5(a, pairs, max_tiles, stream));
+    SP_TRY(plan_product(a, max_tiles));
     a.seg[0] = dn;
     a.dual = false;
     a.out_f32 = true;
-    SP_LAUNCH(F_GEMV, launch_mat_tc5(a, pairs, max_tiles, stream));
+    SP_TRY(plan_product(a, max_tiles));
     if (s.has_shared) {
         a.moe = false;
+        a.x_rows = 0;
         a.dual = true;
         a.out_f32 = false;
         a.seg[0] = sgu;
-        SP_LAUNCH(F_GEMV, launch_mat_tc5(a, T, 0, stream));
+        SP_TRY(plan_product(a, 0));
         a.dual = false;
         a.out_f32 = true;
         a.seg[0] = sdn;
-        SP_LAUNCH(F_GEMV, launch_mat_tc5(a, T, 0, stream));
+        SP_TRY(plan_product(a, 0));
     }
     return SP_OK;
 }

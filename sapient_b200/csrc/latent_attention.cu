@@ -176,17 +176,23 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(con
     key_range(tok_pos[t], s.window, blockIdx.z, n_splits, begin, end);
     const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
     const int pieces = width / 8;
-    for (int i = tid; i < 16 * pieces; i += LM_WARPS * 32) {
-        const int r = i / pieces, p = i - r * pieces;
+    for (int r = warp; r < 16; r += LM_WARPS) {
         const bool live = h0 + r < s.heads;
-        cp_async16(qs + r * LD + p * 8, qabs + ((int64_t)t * s.heads + (live ? h0 + r : h0)) * c.ld + p * 8, live ? 16 : 0);
+        const bf16* src = qabs + ((int64_t)t * s.heads + (live ? h0 + r : h0)) * c.ld;
+        for (int p = lane; p < pieces; p += 32) cp_async16(qs + r * LD + p * 8, src + p * 8, live ? 16 : 0);
     }
-    auto fetch = [&](int k0, int buf) {
+    auto fetch = [&](int k0, int buf) {  // warp w copies keys w, w + 4, ..: a row's address is found once
         bf16* d = ks + buf * LM_KEYS * LD;
-        for (int i = tid; i < LM_KEYS * pieces; i += LM_WARPS * 32) {
-            const int r = i / pieces, p = i - r * pieces, key = min(k0 + r, end - 1);
-            const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld + p * 8;
-            cp_async16(d + r * LD + p * 8, src, k0 + r < end ? 16 : 0);
+        const bf16* src[LM_KEYS / LM_WARPS];
+#pragma unroll
+        for (int i = 0; i < LM_KEYS / LM_WARPS; ++i) {
+            const int key = min(k0 + warp + LM_WARPS * i, end - 1);
+            src[i] = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld;
+        }
+#pragma unroll
+        for (int i = 0; i < LM_KEYS / LM_WARPS; ++i) {
+            const int r = warp + LM_WARPS * i, bytes = k0 + r < end ? 16 : 0;
+            for (int p = lane; p < pieces; p += 32) cp_async16(d + r * LD + p * 8, src[i] + p * 8, bytes);
         }
     };
     if (begin < end) fetch(begin, 0);
@@ -297,27 +303,32 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(con
     }
 }
 
+// Block (head, token, 128 columns).
+constexpr int LATENT_MAX_SPLITS = 16;
 template <typename T>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part, int heads, int n_splits, int rank, T* __restrict__ out, int ldo) {
+    __shared__ float w_s[LATENT_MAX_SPLITS];
     pdl_wait();
     pdl_trigger();
     const int64_t th = (int64_t)blockIdx.y * heads + blockIdx.x;
     const float* src = part + th * n_splits * (rank + 2);
-    float M = -INFINITY, L = 0.f;
-    for (int i = 0; i < n_splits; ++i) M = fmaxf(M, src[(int64_t)i * (rank + 2)]);
-    for (int i = 0; i < n_splits; ++i) {
-        const float m = src[(int64_t)i * (rank + 2)];
-        if (m != -INFINITY) L = fmaf(expf(m - M), src[(int64_t)i * (rank + 2) + 1], L);
+    const int e = blockIdx.z * 128 + threadIdx.x;
+    float v[LATENT_MAX_SPLITS];
+#pragma unroll
+    for (int i = 0; i < LATENT_MAX_SPLITS; ++i) v[i] = i < n_splits && e < rank ? src[(int64_t)i * (rank + 2) + 2 + e] : 0.f;
+    if (threadIdx.x < 32) {
+        const int i = threadIdx.x;
+        const float m = i < n_splits ? src[(int64_t)i * (rank + 2)] : -INFINITY, l = i < n_splits ? src[(int64_t)i * (rank + 2) + 1] : 0.f;
+        const float M = warp_max(m);
+        const float f = m == -INFINITY ? 0.f : expf(m - M);
+        const float L = warp_sum(f * l);
+        if (i < LATENT_MAX_SPLITS) w_s[i] = f / L;
     }
-    const float inv = 1.0f / L;
-    for (int e = threadIdx.x; e < rank; e += 128) {
-        float v = 0.f;
-        for (int i = 0; i < n_splits; ++i) {
-            const float m = src[(int64_t)i * (rank + 2)];
-            if (m != -INFINITY) v = fmaf(expf(m - M), src[(int64_t)i * (rank + 2) + 2 + e], v);
-        }
-        out[th * ldo + e] = from_f32<T>(v * inv);
-    }
+    __syncthreads();
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < LATENT_MAX_SPLITS; ++i) o = fmaf(w_s[i], v[i], o);
+    if (e < rank) out[th * ldo + e] = from_f32<T>(o);
 }
 
 size_t latent_part_floats(int n_tok, int heads, int n_splits, int rank) { return n_splits > 1 ? (size_t)n_tok * heads * n_splits * (rank + 2) : 0; }
@@ -325,7 +336,7 @@ size_t latent_part_floats(int n_tok, int heads, int n_splits, int rank) { return
 cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, const LatentCache& c, const int32_t* tok_slot, const int32_t* tok_pos,
                                     void* o, int ldo, float* part, int n_splits, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    if (n_splits < 1 || (n_splits > 1 && !part) || c.rank > 32 * LS_MAX_PER_LANE) return cudaErrorInvalidValue;
+    if (n_splits < 1 || n_splits > LATENT_MAX_SPLITS || (n_splits > 1 && !part) || c.rank > 32 * LS_MAX_PER_LANE) return cudaErrorInvalidValue;
     constexpr int CAP = 200 * 1024;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
@@ -359,8 +370,8 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
     if (le != cudaSuccess) return le;
     le = count_launch_and_check();
     if (le != cudaSuccess || n_splits == 1) return le;
-    le = f32 ? launch_pdl(latent_merge_kernel<float>, dim3(s.heads, n_tok), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (float*)o, ldo)
-             : launch_pdl(latent_merge_kernel<bf16>, dim3(s.heads, n_tok), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (bf16*)o, ldo);
+    le = f32 ? launch_pdl(latent_merge_kernel<float>, dim3(s.heads, n_tok, (c.rank + 127) / 128), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (float*)o, ldo)
+             : launch_pdl(latent_merge_kernel<bf16>, dim3(s.heads, n_tok, (c.rank + 127) / 128), dim3(128), 0, st, (const float*)part, s.heads, n_splits, c.rank, (bf16*)o, ldo);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
@@ -402,22 +413,25 @@ __global__ void __launch_bounds__(LE_WARPS * 32) latent_expanded_kernel(const bf
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int h = blockIdx.x;
     const LatentTile tl = tiles[blockIdx.y];
-    for (int i = tid; i < 64 * (qw / 8); i += LE_WARPS * 32) {
-        const int r = i / (qw / 8), p = i - r * (qw / 8);
-        cp_async16(qs + r * LQ + p * 8, qf + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * qw + p * 8, 16);
+    // copies: eight lanes per row, four rows per warp and instruction
+    const int l8 = lane & 7, lr = warp * 16 + (lane >> 3);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int r = lr + 4 * i;
+        const bf16* src = qf + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * qw;
+        for (int p = l8; p < qw / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
     }
     const int hi = tl.pos0 + tl.n - 1, lo = s.window > tl.pos0 ? 0 : tl.pos0 - s.window + 1;
     auto fetch = [&](int k0, int buf) {
         bf16 *kd = ks + buf * LE_KEYS * LQ, *vd = vs + buf * LE_KEYS * LV;
-        const int pk = dim16 / 8, pr = rot16 / 8, pv = vdim16 / 8, per = pk + pr + pv;
-        for (int i = tid; i < LE_KEYS * per; i += LE_WARPS * 32) {
-            const int r = i / per, p = i - r * per, key = min(k0 + r, hi);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = lr + 4 * i, key = min(k0 + r, hi), bytes = k0 + r <= hi ? 16 : 0;
             const int64_t row = tl.key_row + (key - tl.key_pos0);
-            const int bytes = k0 + r <= hi ? 16 : 0;
-            const bf16* kvr = kv + (row * s.heads + h) * kvw;
-            if (p < pk) cp_async16(kd + r * LQ + p * 8, kvr + p * 8, bytes);
-            else if (p < pk + pr) cp_async16(kd + r * LQ + p * 8, lat + row * ldl + rank16 + (p - pk) * 8, bytes);
-            else cp_async16(vd + r * LV + (p - pk - pr) * 8, kvr + dim16 + (p - pk - pr) * 8, bytes);
+            const bf16 *kvr = kv + (row * s.heads + h) * kvw, *rr = lat + row * ldl + rank16;
+            for (int p = l8; p < dim16 / 8; p += 8) cp_async16(kd + r * LQ + p * 8, kvr + p * 8, bytes);
+            for (int p = l8; p < rot16 / 8; p += 8) cp_async16(kd + r * LQ + dim16 + p * 8, rr + p * 8, bytes);
+            for (int p = l8; p < vdim16 / 8; p += 8) cp_async16(vd + r * LV + p * 8, kvr + dim16 + p * 8, bytes);
         }
     };
     fetch(lo, 0);

@@ -1,15 +1,20 @@
-// Many-row matrix products on bf16 weights with the 5th-generation tensor cores (tcgen05 + TMEM), dense or grouped by
-// expert, plain or as the gate / up pair of a clamped gated unit.
+// Matrix products on bf16 weights with the 5th-generation tensor cores (tcgen05 + TMEM), for one row or thousands: dense,
+// per head or grouped by expert, plain or as the gate / up pair of a clamped gated unit.
 //
-// y[r, n] = sum_k x[r, k] W[n, k]. A CTA owns 128 weight rows (the MMA's M; for a gated unit 128 gate rows and the 128 up
-// rows that belong to them, two accumulators) x up to BN activation rows (the MMA's N). Warp 1 lane 0 has TMA fetch, per
-// 64 columns of K, the weight tile(s) and the activation tile into a ring of shared-memory stages (128-byte swizzle, both
-// operands K-major; columns past a matrix arrive as zeros, rows past it as zeros or as rows nobody stores); warp 0 lane 0
-// issues four tcgen05.mma per tile and stage and commits them to the stage's `empty` mbarrier; four epilogue warps read
-// the accumulators back (one weight row per thread), apply the gated unit and store with n contiguous across the warp.
-// Tiles are kept small enough for two CTAs per SM where that fits (256 TMEM columns and ~100 KB each), so that one CTA's
-// epilogue runs under the other's MMAs. Every mbarrier wait is bounded; on expiry the kernel raises a flag, still frees
-// its tensor memory and returns.
+// y[r, n] = sum_k x[r, k] W[n, k]. A CTA owns 128 weight rows of one matrix (the MMA's M; for a gated unit 128 gate rows
+// and the 128 up rows that belong to them, two accumulators) x up to bn activation rows (the MMA's N), over all of K or a
+// part of it. Warp 1 lane 0 has TMA fetch, per 64 columns of K, the weight tile(s) and the activation tile into a ring of
+// shared-memory stages (128-byte swizzle, both operands K-major; columns past a matrix arrive as zeros, rows past it as
+// zeros or as rows nobody stores) — the weights of the first stages before the previous kernel is waited for, since no
+// kernel writes weights; warp 0 lane 0 issues four tcgen05.mma per tile and stage and commits them to the stage's `empty`
+// mbarrier; four epilogue warps read the accumulators back (one weight row per thread), apply the gated unit or the output
+// gate and store with n contiguous across the warp. Two CTAs per SM (256 TMEM columns and ~100 KB each), so that one
+// CTA's epilogue runs under the other's loads and MMAs.
+// Few rows: the same kernel with 16- or 32-row activation tiles is a weight stream (all of a stage's bytes are weights but
+// an eighth); K is split over CTAs until the SMs are busy, partial tiles meet in a scratch buffer and the CTA that arrives
+// last adds them in order. Experts of a small step (`gather`) multiply every row of the step, which costs nothing at this
+// tile size, and keep the rows that chose them: no gathered copy.
+// Every mbarrier wait is bounded; on expiry the kernel raises a flag, still frees its tensor memory and returns.
 #include <algorithm>
 #include <atomic>
 
@@ -26,36 +31,64 @@ cudaError_t count_launch_and_check();  // kernels.cu
 constexpr int MT_BM = 128, MT_BK = 64, MT_MAX_STAGES = 6;
 constexpr int MT_THREADS = 192;            // MMA warp, TMA warp, four epilogue warps
 constexpr int MT_A_BYTES = MT_BM * MT_BK * 2;
-constexpr int MT_SMEM_HALF = 100 * 1024;   // two CTAs per SM
-constexpr int MT_SMEM_FULL = 200 * 1024;
+constexpr int MT_SMEM = 100 * 1024;        // per CTA, two of which share an SM
+constexpr int MT_MAX_PARTS = 8;
 
 __device__ int g_mat_tc5_timeout = 0;
 
-struct MatTc5Args {
+struct MatTc5Seg {
     void* y;
-    int ldy, n, kp, m;
-    int bn;               // activation rows per tile (box height)
-    int stages, stage_bytes, tmem_cols;
-    bool dual, out_f32, moe;
+    int64_t ygs;
+    int xgs;              // elements between the inputs of consecutive groups
+    int ldy, n, kp;
     float limit, alpha;
+};
+struct MatTc5Args {
+    MatTc5Seg seg[2];
+    int slots0;           // blockIdx.y below this: seg[0]
+    int row_tiles;        // row tiles of a dense or per-head product (blockIdx.y = group * row_tiles + tile)
+    int m, bn;            // activation rows, rows per tile (box height)
+    int stages, stage_bytes, tmem_cols;
+    int parts;            // CTAs (blockIdx.z) that share a tile's K range
+    bool dual, out_f32, moe, gather;
     MoeRows rows;
+    const float* gate;
+    int ldgate;
+    float* part_buf;      // [item][part][accumulator][bn columns][128]
+    unsigned* part_cnt;
 };
 
-__global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w,
-                                                             const __grid_constant__ CUtensorMap map_x) {
+__global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
+                                                             const __grid_constant__ CUtensorMap map_x0, const __grid_constant__ CUtensorMap map_w1,
+                                                             const __grid_constant__ CUtensorMap map_x1) {
     extern __shared__ uint8_t mt_smem_raw[];
     __shared__ __align__(8) uint64_t full[MT_MAX_STAGES], empty[MT_MAX_STAGES], done_bar;
     __shared__ uint32_t tmem_slot;
+    __shared__ int dest[MAT_GATHER_ROWS];  // gather: output row of each of the step's rows, -1: not this expert's
+    __shared__ int last_part;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int si = (int)blockIdx.y >= a.slots0;
+    const MatTc5Seg& s = a.seg[si];
+    const int n0 = blockIdx.x * MT_BM;
+    const bool grouped = a.moe && si == 0;
+    const bool in_range = n0 < s.n;
+    // whose tile: known at once unless the routing step decides it
+    int g = 0, r0 = 0, rows = 0;
+    if (!grouped) {
+        const int slot = blockIdx.y - (si ? a.slots0 : 0);
+        g = slot / a.row_tiles;
+        r0 = (slot - g * a.row_tiles) * a.bn;
+        rows = min(a.bn, a.m - r0);
+    }
     uint8_t* smem = mt_smem_raw + ((1024u - (tc5_smem_u32(mt_smem_raw) & 1023u)) & 1023u);
     if (warp == 0) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(tc5_smem_u32(&tmem_slot)), "r"(a.tmem_cols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
-    if (tid == 0) {
-        for (int s = 0; s < a.stages; ++s) {
-            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&full[s])) : "memory");
-            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&empty[s])) : "memory");
+    if (tid == 32) {
+        for (int i = 0; i < a.stages; ++i) {
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&full[i])) : "memory");
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&empty[i])) : "memory");
         }
         asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&done_bar)) : "memory");
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
@@ -64,89 +97,139 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
     const uint32_t tmem = tmem_slot;
+    const int all_chunks = s.kp / MT_BK, part = blockIdx.z;
+    const int c_begin = part * all_chunks / a.parts, n_chunks_all = (part + 1) * all_chunks / a.parts - c_begin;
+    const CUtensorMap* mw = si ? &map_w1 : &map_w0;
+    const CUtensorMap* mx = si ? &map_x1 : &map_x0;
+    const int a_tiles = a.dual ? 2 : 1;
+    auto load_w = [&](int c, int st) {  // expects the whole stage, fetches its weight part
+        const uint32_t bar = tc5_smem_u32(&full[st]);
+        const uint32_t dst = tc5_smem_u32(smem + (size_t)st * a.stage_bytes);
+        const int wrow = g * a_tiles * s.n + n0;
+        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(a.stage_bytes) : "memory");
+        tc5_tma_2d(dst, mw, (c_begin + c) * MT_BK, wrow, bar);
+        if (a.dual) tc5_tma_2d(dst + MT_A_BYTES, mw, (c_begin + c) * MT_BK, wrow + s.n, bar);
+    };
+    const int early = (grouped || !in_range) ? 0 : min(a.stages, n_chunks_all);
+    if (warp == 1 && lane == 0)
+        for (int c = 0; c < early; ++c) load_w(c, c);
     pdl_wait();
     pdl_trigger();
-    // this CTA's tile: weight rows n0.. of matrix g, activation rows r0 .. r0 + rows - 1
-    const int n0 = blockIdx.x * MT_BM;
-    int g = 0, r0 = blockIdx.y * a.bn, rows;
-    bool live = true;
-    if (a.moe) {
-        live = (int)blockIdx.y < *a.rows.n_tiles;
+    bool live = in_range;
+    if (grouped) {
+        live = live && (int)blockIdx.y < *a.rows.n_tiles;
         if (live) {
             g = a.rows.tile_group[blockIdx.y];
             r0 = a.rows.tile_row[blockIdx.y];
             rows = min(a.bn, a.rows.row_off[g + 1] - r0);
-        } else {
-            rows = 0;
         }
-    } else {
-        rows = min(a.bn, a.m - r0);
     }
-    const int nb = (rows + 15) & ~15;
-    const int n_chunks = live ? a.kp / MT_BK : 0;
-    const int64_t wrow = (int64_t)g * (a.dual ? 2 : 1) * a.n + n0;
+    const bool by_index = grouped && a.gather;
+    const int cols = by_index ? a.m : rows;       // activation rows in the tile
+    const int nb = (cols + 15) & ~15;
+    const int x0 = by_index ? 0 : r0;
+    const int n_chunks = live ? n_chunks_all : 0;
     bool ok = true;
     if (warp == 0) {
         if (lane == 0 && live) {
             const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nb >> 3) << 17) | ((uint32_t)(MT_BM >> 4) << 24);  // bf16 x bf16 -> f32
-            for (int c = 0, s = 0, u = 0; c < n_chunks; ++c, ++s) {
-                if (s == a.stages) { s = 0; ++u; }
-                ok = ok && tc5_wait(&full[s], (uint32_t)(u & 1));
+            for (int c = 0, st = 0, u = 0; c < n_chunks; ++c, ++st) {
+                if (st == a.stages) { st = 0; ++u; }
+                ok = ok && tc5_wait(&full[st], (uint32_t)(u & 1));
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-                const uint32_t st = tc5_smem_u32(smem + (size_t)s * a.stage_bytes);
-                const uint64_t ad = tc5_desc(st), ad2 = tc5_desc(st + MT_A_BYTES), bd = tc5_desc(st + (a.dual ? 2 : 1) * MT_A_BYTES);
+                const uint32_t base = tc5_smem_u32(smem + (size_t)st * a.stage_bytes);
+                const uint64_t ad = tc5_desc(base), ad2 = tc5_desc(base + MT_A_BYTES), bd = tc5_desc(base + a_tiles * MT_A_BYTES);
 #pragma unroll
                 for (int i = 0; i < MT_BK / 16; ++i) {  // 16 columns: 32 bytes inside the swizzle row
                     tc5_mma(tmem, ad + 2u * i, bd + 2u * i, idesc, (uint32_t)(c > 0 || i > 0));
                     if (a.dual) tc5_mma(tmem + (uint32_t)a.bn, ad2 + 2u * i, bd + 2u * i, idesc, (uint32_t)(c > 0 || i > 0));
                 }
-                tc5_commit(&empty[s]);
+                tc5_commit(&empty[st]);
             }
             if (ok) tc5_commit(&done_bar);
         }
     } else if (warp == 1) {
         if (lane == 0 && live) {
-            for (int c = 0, s = 0, u = 0; c < n_chunks; ++c, ++s) {
-                if (s == a.stages) { s = 0; ++u; }
-                if (u > 0) ok = ok && tc5_wait(&empty[s], (uint32_t)((u - 1) & 1));
+            for (int c = 0, st = 0, u = 0; c < n_chunks; ++c, ++st) {
+                if (st == a.stages) { st = 0; ++u; }
+                if (u > 0) ok = ok && tc5_wait(&empty[st], (uint32_t)((u - 1) & 1));
                 if (!ok) break;
-                const uint32_t bar = tc5_smem_u32(&full[s]);
-                uint32_t dst = tc5_smem_u32(smem + (size_t)s * a.stage_bytes);
-                asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(a.stage_bytes) : "memory");
-                tc5_tma_2d(dst, &map_w, c * MT_BK, (int)wrow, bar);
-                dst += MT_A_BYTES;
-                if (a.dual) {
-                    tc5_tma_2d(dst, &map_w, c * MT_BK, (int)wrow + a.n, bar);
-                    dst += MT_A_BYTES;
-                }
-                tc5_tma_2d(dst, &map_x, c * MT_BK, r0, bar);
+                if (c >= early) load_w(c, st);
+                tc5_tma_2d(tc5_smem_u32(smem + (size_t)st * a.stage_bytes) + a_tiles * MT_A_BYTES, mx, g * s.xgs + (c_begin + c) * MT_BK, x0,
+                           tc5_smem_u32(&full[st]));
             }
         }
     } else if (live) {
+        const int q4 = warp & 3, n = n0 + 32 * q4 + lane;
+        if (by_index) {
+            // the four epilogue warps agree on where each of the step's rows goes
+            if (warp == 2) {
+                dest[lane] = -1;
+                __syncwarp();
+                for (int j = lane; j < rows; j += 32) dest[a.rows.row_src[r0 + j]] = r0 + j;
+            }
+            asm volatile("bar.sync 1, 128;\n" ::: "memory");
+        }
         ok = tc5_wait(&done_bar, 0u);
         ok = __all_sync(0xFFFFFFFFu, ok);  // one verdict for the warp: the loads below are warp-collective
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        auto store = [&](int c, float f, float up) {
+            const int row = by_index ? dest[c] : r0 + c;
+            if (row < 0) return;
+            if (a.dual) f = clamped_unit(f, up, s.limit, s.alpha);
+            if (a.gate) f *= sigmoid_f32(a.gate[(int64_t)row * a.ldgate + g]);
+            const int64_t at = (int64_t)row * s.ldy + (int64_t)g * s.ygs + n;
+            if (a.out_f32) reinterpret_cast<float*>(s.y)[at] = f;
+            else reinterpret_cast<bf16*>(s.y)[at] = __float2bfloat16_rn(f);
+        };
+        const int64_t item = (int64_t)blockIdx.y * gridDim.x + blockIdx.x;
+        const int64_t tile_floats = (int64_t)a_tiles * a.bn * MT_BM;
+        float* all = a.part_buf + item * a.parts * tile_floats;
         if (ok) {
-            const int q4 = warp & 3, n = n0 + 32 * q4 + lane;
             const uint32_t lanes = tmem + ((uint32_t)(32 * q4) << 16);
+            float* mine = all + part * tile_floats + 32 * q4 + lane;
             for (int c = 0; c < nb; c += 16) {
                 uint32_t v[16], up[16];
                 tc5_ld16(lanes + (uint32_t)c, v);
                 if (a.dual) tc5_ld16(lanes + (uint32_t)(a.bn + c), up);
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-                if (n < a.n) {
+                if (a.parts > 1) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        if (c + j < rows) {
-                            float f = __uint_as_float(v[j]);
-                            if (a.dual) f = clamped_unit(f, __uint_as_float(up[j]), a.limit, a.alpha);
-                            const int64_t at = (int64_t)(r0 + c + j) * a.ldy + n;
-                            if (a.out_f32) reinterpret_cast<float*>(a.y)[at] = f;
-                            else reinterpret_cast<bf16*>(a.y)[at] = __float2bfloat16_rn(f);
+                        if (c + j >= cols) continue;
+                        // (a short K may leave a part without chunks)
+                        __stcg(mine + (c + j) * MT_BM, n_chunks ? __uint_as_float(v[j]) : 0.f);
+                        if (a.dual) __stcg(mine + (a.bn + c + j) * MT_BM, n_chunks ? __uint_as_float(up[j]) : 0.f);
+                    }
+                } else if (n < s.n) {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        if (c + j < cols) store(c + j, __uint_as_float(v[j]), a.dual ? __uint_as_float(up[j]) : 0.f);
+                }
+            }
+        }
+        if (a.parts > 1) {
+            // every epilogue warp comes here whatever its `ok`; no CTA waits for another
+            __threadfence();
+            asm volatile("bar.sync 1, 128;\n" ::: "memory");
+            if (tid == 64) last_part = atomicAdd(&a.part_cnt[item], 1u) == (unsigned)(a.parts - 1);
+            asm volatile("bar.sync 1, 128;\n" ::: "memory");
+            if (last_part) {
+                __threadfence();
+                const float* src = all + 32 * q4 + lane;
+                if (n < s.n) {
+                    for (int c = 0; c < cols; ++c) {
+                        if (by_index && dest[c] < 0) continue;
+                        float f = 0.f, up = 0.f;
+                        for (int p = 0; p < a.parts; ++p) {
+                            f += __ldcg(src + p * tile_floats + c * MT_BM);
+                            if (a.dual) up += __ldcg(src + p * tile_floats + (a.bn + c) * MT_BM);
                         }
+                        store(c, f, up);
                     }
                 }
+                if (tid == 64) a.part_cnt[item] = 0u;  // ready for the next launch
             }
         }
     }
@@ -168,54 +251,68 @@ int mat_tc5_take_timeout() {
     return flag ? 1 : 0;
 }
 
-bool mat_tc5_supported(const MatArgs& a) {
-    const MatSeg& s = a.seg[0];
-    return !a.f32 && a.nseg == 1 && !a.gate && !a.gather && (a.moe || s.groups == 1) && s.ldx % 8 == 0 &&
-           (reinterpret_cast<uintptr_t>(s.x) & 15) == 0 && (reinterpret_cast<uintptr_t>(s.w) & 15) == 0 &&
-           (int64_t)s.groups * s.n * (a.dual ? 2 : 1) < (1ll << 31);
+// [rows][cols] bf16 with a row stride of ld elements, boxes of 64 columns x box_rows.
+static bool mat_map(CUtensorMap* map, const void* p, int64_t cols, int64_t rows, int64_t ld, int box_rows) {
+    const PFN_encodeTiled encode = tensor_map_encoder();
+    const cuuint64_t dim[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, stride[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {MT_BK, (cuuint32_t)box_rows}, estr[2] = {1u, 1u};
+    return encode && encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(p), dim, stride, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-cudaError_t launch_mat_tc5(const MatArgs& a, int x_rows, int max_tiles, cudaStream_t st) {
-    if (a.m <= 0 || x_rows <= 0) return cudaSuccess;
-    if (!mat_tc5_supported(a)) return cudaErrorInvalidValue;
-    const MatSeg& s = a.seg[0];
-    const int row_tiles = (s.n + MT_BM - 1) / MT_BM;
+cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc, cudaStream_t st) {
+    if (a.m <= 0) return cudaSuccess;
+    if (a.f32 || a.nseg < 1 || a.nseg > 2 || (a.nseg == 2 && a.seg[1].groups != 1) || (a.gather && (!a.moe || a.m > MAT_GATHER_ROWS))) return cudaErrorInvalidValue;
     MatTc5Args k{};
-    // activation rows per tile: as many as keep the SMs busy
-    int bn = a.moe ? MOE_TILE : (a.dual ? 128 : 256);
+    int n_max = 0, kp_max = 0;
+    for (int i = 0; i < a.nseg; ++i) {
+        const MatSeg& s = a.seg[i];
+        if (s.kp % MAT_KPAD != 0 || s.n <= 0 || s.ldx % 8 != 0 || s.xgs % 8 != 0 || (int64_t)s.groups * s.n * 2 >= (1ll << 31)) return cudaErrorInvalidValue;
+        k.seg[i] = MatTc5Seg{s.y, s.ygs, (int)s.xgs, s.ldy, s.n, s.kp, s.limit, s.alpha};
+        n_max = std::max(n_max, s.n);
+        kp_max = std::max(kp_max, s.kp);
+    }
+    const int row_blocks = (n_max + MT_BM - 1) / MT_BM, sms = device_sm_count();
+    const int groups = a.moe ? 1 : a.seg[0].groups;
+    // activation rows per tile: all of a small step, else as many as keep the SMs busy
+    int bn = a.m <= 16 ? 16 : a.m <= 32 ? 32 : a.moe ? MOE_TILE : a.dual ? 128 : 256;
     if (!a.moe)
-        while (bn > 32 && ((int64_t)row_tiles * ((a.m + bn - 1) / bn) < device_sm_count() || bn >= 2 * a.m)) bn >>= 1;
-    k.y = s.y; k.ldy = s.ldy; k.n = s.n; k.kp = s.kp; k.m = a.m;
+        while (bn > 32 && ((int64_t)row_blocks * groups * ((a.m + bn - 1) / bn) < sms || bn >= 2 * a.m)) bn >>= 1;
     k.bn = bn;
-    k.dual = a.dual; k.out_f32 = a.out_f32; k.moe = a.moe; k.limit = s.limit; k.alpha = s.alpha; k.rows = a.rows;
-    k.stage_bytes = (a.dual ? 2 : 1) * MT_A_BYTES + bn * MT_BK * 2;
-    k.tmem_cols = std::max(32, (a.dual ? 2 : 1) * bn);
-    k.stages = std::min(MT_MAX_STAGES, MT_SMEM_HALF / k.stage_bytes);
-    const int smem = k.stages * k.stage_bytes + 1024;
-    const PFN_encodeTiled encode = tensor_map_encoder();
-    if (!encode) return cudaErrorNotSupported;
-    CUtensorMap mw, mx;
-    const cuuint32_t estr[2] = {1u, 1u};
-    {
-        const cuuint64_t dim[2] = {(cuuint64_t)s.kp, (cuuint64_t)s.groups * (cuuint64_t)s.n * (a.dual ? 2 : 1)}, stride[1] = {(cuuint64_t)s.kp * 2};
-        const cuuint32_t box[2] = {MT_BK, MT_BM};
-        if (encode(&mw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(s.w), dim, stride, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-            return cudaErrorInvalidValue;
+    k.m = a.m;
+    k.row_tiles = (a.m + bn - 1) / bn;
+    k.slots0 = a.moe ? max_tiles : groups * k.row_tiles;
+    const int slots = k.slots0 + (a.nseg == 2 ? k.row_tiles : 0);
+    k.dual = a.dual; k.out_f32 = a.out_f32; k.moe = a.moe; k.gather = a.gather; k.rows = a.rows; k.gate = a.gate; k.ldgate = a.ldgate;
+    const int acc = a.dual ? 2 : 1;
+    k.stage_bytes = acc * MT_A_BYTES + bn * MT_BK * 2;
+    k.tmem_cols = std::max(32, acc * bn);
+    k.stages = std::min(MT_MAX_STAGES, MT_SMEM / k.stage_bytes);
+    k.parts = 1;
+    const int64_t items = (int64_t)row_blocks * slots;
+    int64_t busy = 0;  // tiles that exist
+    for (int i = 0; i < a.nseg; ++i) busy += (int64_t)((a.seg[i].n + MT_BM - 1) / MT_BM) * (i ? k.row_tiles : k.slots0);
+    if (bn <= 32 && sc.part && items <= MatScratch::ITEMS) {
+        // two CTAs per SM, but no part shorter than four chunks of K
+        while (k.parts < MT_MAX_PARTS && busy * k.parts < 2 * sms && kp_max / MT_BK >= 8 * k.parts &&
+               items * (2 * k.parts) * acc * bn * MT_BM <= (int64_t)MatScratch::FLOATS)
+            k.parts *= 2;
     }
-    {
-        const cuuint64_t dim[2] = {(cuuint64_t)std::min(s.kp, s.ldx), (cuuint64_t)x_rows}, stride[1] = {(cuuint64_t)s.ldx * 2};
-        const cuuint32_t box[2] = {MT_BK, (cuuint32_t)bn};
-        if (encode(&mx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(s.x), dim, stride, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-            return cudaErrorInvalidValue;
+    k.part_buf = sc.part;
+    k.part_cnt = sc.cnt;
+    CUtensorMap mw[2], mx[2];
+    for (int i = 0; i < a.nseg; ++i) {
+        const MatSeg& s = a.seg[i];
+        const int64_t x_rows = i == 0 && a.x_rows > 0 ? a.x_rows : a.m;
+        if (!mat_map(&mw[i], s.w, s.kp, (int64_t)s.groups * s.n * acc, s.kp, MT_BM) || !mat_map(&mx[i], s.x, s.ldx, x_rows, s.ldx, bn)) return cudaErrorInvalidValue;
     }
+    if (a.nseg == 1) { mw[1] = mw[0]; mx[1] = mx[0]; }
     static PerDeviceOnce once;
-    cudaError_t le = once.run([] { return cudaFuncSetAttribute(mat_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM_FULL + 1024); });
+    cudaError_t le = once.run([] { return cudaFuncSetAttribute(mat_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM + 1024); });
     if (le != cudaSuccess) return le;
     g_mat_tc5_launched[current_device_index()].store(1);
-    const dim3 grid((unsigned)row_tiles, (unsigned)(a.moe ? max_tiles : (a.m + bn - 1) / bn));
-    le = launch_pdl(mat_tc5_kernel, grid, dim3(MT_THREADS), (size_t)smem, st, k, mw, mx);
+    le = launch_pdl(mat_tc5_kernel, dim3((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), dim3(MT_THREADS), (size_t)(k.stages * k.stage_bytes + 1024), st, k,
+                    mw[0], mx[0], mw[1], mx[1]);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }

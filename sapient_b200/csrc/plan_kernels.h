@@ -49,18 +49,26 @@ struct MatArgs {
     bool gather;               // its x rows are tokens (row_src), not sorted rows
     MoeRows rows;
     int slots;                 // moe: upper bound of active experts
+    int x_rows;                // rows of seg[0].x when they are not the m rows (sorted rows)
     const float* gate;         // y *= sigmoid(gate[row * ldgate + group]) or null
     int ldgate;
 };
 
-// Any shape, few rows: each weight is read once per up to 32 rows (bf16: mma.sync with the weights as the row operand,
-// f32: fused multiply-adds).
-cudaError_t launch_mat_rows(const MatArgs& a, cudaStream_t st);
+// f32: plain fused multiply-adds on 32 x 32 tiles, any shape and row count.
+cudaError_t launch_mat_f32(const MatArgs& a, cudaStream_t st);
 
-// Many rows, bf16: tcgen05 / TMEM, both operands staged by TMA. One segment, no gather (x rows already in order);
-// moe: x rows are the sorted rows, tiles of MOE_TILE rows, max_tiles an upper bound of their number.
-bool mat_tc5_supported(const MatArgs& a);
-cudaError_t launch_mat_tc5(const MatArgs& a, int x_rows, int max_tiles, cudaStream_t st);
+// bf16: tcgen05 / TMEM, both operands staged by TMA, any shape and row count. Launches whose tiles leave SMs idle split K
+// over several CTAs through `sc` (partial tiles, summed in order by the last to arrive). Grouped by expert: with `gather`
+// (at most MAT_GATHER_ROWS rows) every expert multiplies all rows and keeps its own; otherwise the x rows are the sorted
+// rows. max_tiles: upper bound of the row tiles of a grouped launch.
+constexpr int MAT_GATHER_ROWS = 32;
+struct MatScratch {            // owned by whoever owns the stream
+    float* part = nullptr;
+    unsigned* cnt = nullptr;   // zero between launches
+    static constexpr int ITEMS = 4096;
+    static constexpr size_t FLOATS = 8u << 20;
+};
+cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc, cudaStream_t st);
 int mat_tc5_take_timeout();    // as tc5_take_timeout (kernels.h)
 
 // ── the stream between the products ──

@@ -10,9 +10,25 @@ namespace sp {
 
 cudaError_t count_launch_and_check();  // kernels.cu
 
-#define SP_BY_TYPE(f32, K, ...) ((f32) ? launch_pdl(K<float>, __VA_ARGS__) : launch_pdl(K<bf16>, __VA_ARGS__))
+constexpr int ST_WARPS = 16, ST_THREADS = 32 * ST_WARPS;
 
-constexpr int ST_WARPS = 8, ST_THREADS = 32 * ST_WARPS;
+// V consecutive elements of a row (V = 4 where the width allows it).
+template <int V> struct Row;
+template <> struct Row<1> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[1]) { v[0] = *p; }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; }
+    static __device__ __forceinline__ void store(bf16* p, const float (&v)[1]) { *p = __float2bfloat16_rn(v[0]); }
+};
+template <> struct Row<4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+    static __device__ __forceinline__ void store(bf16* p, const float (&v)[4]) {
+        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+    }
+};
 
 template <typename T>
 __global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __restrict__ table, int ldt, const uint32_t* __restrict__ ids, int width,
@@ -37,7 +53,7 @@ cudaError_t launch_embed_scaled(const void* table, int ldt, bool f32, const uint
     return count_launch_and_check();
 }
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(ST_THREADS) norm_residual_kernel(const float* __restrict__ y, int ldy, const float* __restrict__ gain, float eps,
                                                                    const float* x, float* x_out, T* __restrict__ xb, int ldb, int width) {
     __shared__ float sh[ST_WARPS];
@@ -45,80 +61,142 @@ __global__ void __launch_bounds__(ST_THREADS) norm_residual_kernel(const float* 
     pdl_trigger();
     const int64_t t = blockIdx.x;
     const float* yr = y + t * ldy;
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < width; c += ST_THREADS) ss = fmaf(yr[c], yr[c], ss);
-    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps) * *gain;
-    for (int c = threadIdx.x; c < ldb; c += ST_THREADS) {
-        float v = 0.f;
-        if (c < width) {
-            v = fmaf(yr[c], r, x[t * width + c]);
-            x_out[t * width + c] = v;
-        }
-        xb[t * ldb + c] = from_f32<T>(v);
+    const float g = *gain;
+    float ss = 0.f, v[V], o[V];
+    for (int c = V * threadIdx.x; c < width; c += V * ST_THREADS) {
+        Row<V>::load(yr + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
     }
+    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps) * g;
+    for (int c = V * threadIdx.x; c < ldb; c += V * ST_THREADS) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) o[i] = 0.f;
+        if (c < width) {
+            Row<V>::load(yr + c, v);
+            Row<V>::load(x + t * width + c, o);
+#pragma unroll
+            for (int i = 0; i < V; ++i) o[i] = fmaf(v[i], r, o[i]);
+            Row<V>::store(x_out + t * width + c, o);
+        }
+        Row<V>::store(xb + t * ldb + c, o);
+    }
+}
+
+template <typename T>
+static cudaError_t norm_residual_by_width(const float* y, int ldy, const float* gain, float eps, const float* x, float* x_out, void* xb, int ldb,
+                                          int n_tok, int width, cudaStream_t st) {
+    return width % 4 == 0 && ldy % 4 == 0
+               ? launch_pdl(norm_residual_kernel<T, 4>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (T*)xb, ldb, width)
+               : launch_pdl(norm_residual_kernel<T, 1>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (T*)xb, ldb, width);
 }
 
 cudaError_t launch_norm_residual(const float* y, int ldy, const float* gain, float eps, const float* x, float* x_out, void* xb, int ldb, bool f32,
                                  int n_tok, int width, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    cudaError_t le = f32 ? launch_pdl(norm_residual_kernel<float>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (float*)xb, ldb, width)
-                         : launch_pdl(norm_residual_kernel<bf16>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (bf16*)xb, ldb, width);
+    cudaError_t le = f32 ? norm_residual_by_width<float>(y, ldy, gain, eps, x, x_out, xb, ldb, n_tok, width, st)
+                         : norm_residual_by_width<bf16>(y, ldy, gain, eps, x, x_out, xb, ldb, n_tok, width, st);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
 
-// One block per token. The feed-forward's sum lives in shared memory between the two passes over the width.
-template <typename T>
+// One block per token. Shared memory: the feed-forward's sum between the two passes over the width, the weights and rows
+// of the chosen experts, the depth coefficients.
+template <typename T, int V>
 __global__ void __launch_bounds__(ST_THREADS) combine_kernel(const CombineArgs a, int width) {
-    extern __shared__ float ff[];
+    extern __shared__ __align__(16) float ff[];
     __shared__ float sh[ST_WARPS];
+    float* w_s = ff + (a.y ? (width + 3) / 4 * 4 : 0);
+    int* row_s = reinterpret_cast<int*>(w_s + a.top);
+    float* dwa_s = w_s + 2 * a.top;
     pdl_wait();
     pdl_trigger();
     const int64_t t = blockIdx.x;
+    for (int k = threadIdx.x; k < a.top; k += ST_THREADS) {
+        w_s[k] = a.weight[t * a.top + k];
+        row_s[k] = a.slot_of[t * a.top + k];
+    }
+    if (a.dwa)
+        for (int j = threadIdx.x; j <= a.depth; j += ST_THREADS) dwa_s[j] = a.dwa[j];
+    const float sg = a.shared_gate ? sigmoid_f32(a.shared_gate[t * a.ld_gate]) : 0.f;
+    __syncthreads();
     float r = 0.f;
     if (a.y) {
-        const float sg = a.shared_gate ? sigmoid_f32(a.shared_gate[t * a.ld_gate]) : 0.f;
+        const float gain = *a.gain;
         float ss = 0.f;
-        for (int c = threadIdx.x; c < width; c += ST_THREADS) {
-            float v = 0.f;
-            for (int k = 0; k < a.top; ++k) v = fmaf(a.weight[t * a.top + k], a.y[(int64_t)a.slot_of[t * a.top + k] * a.ldy + c], v);
-            if (a.y_shared) v = fmaf(sg, a.y_shared[t * a.ldy + c], v);
-            ff[c] = v;
-            ss = fmaf(v, v, ss);
+        for (int c = V * threadIdx.x; c < width; c += V * ST_THREADS) {
+            float s[V], q[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) s[i] = 0.f;
+#pragma unroll 4
+            for (int k = 0; k < a.top; ++k) {
+                Row<V>::load(a.y + (int64_t)row_s[k] * a.ldy + c, q);
+#pragma unroll
+                for (int i = 0; i < V; ++i) s[i] = fmaf(w_s[k], q[i], s[i]);
+            }
+            if (a.y_shared) {
+                Row<V>::load(a.y_shared + t * a.ldy + c, q);
+#pragma unroll
+                for (int i = 0; i < V; ++i) s[i] = fmaf(sg, q[i], s[i]);
+            }
+            Row<V>::store(ff + c, s);
+#pragma unroll
+            for (int i = 0; i < V; ++i) ss = fmaf(s[i], s[i], ss);
         }
-        r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + a.eps) * *a.gain;
+        r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + a.eps) * gain;
     }
     float* mine = a.history + (int64_t)a.depth * a.hist_stride + t * width;
-    for (int c = threadIdx.x; c < a.ldb; c += ST_THREADS) {
-        float v = 0.f;
+    for (int c = V * threadIdx.x; c < a.ldb; c += V * ST_THREADS) {
+        float v[V], q[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = 0.f;
         if (c < width) {
-            v = a.x[t * width + c];
-            if (a.y) v = fmaf(ff[c], r, v);  // written above by this same thread
-            mine[c] = v;
-            if (a.dwa) {
-                float s = 0.f;
-                const float* h = a.history + t * width + c;
-#pragma unroll 8
-                for (int j = 0; j < a.depth; ++j) s = fmaf(a.dwa[j], h[(int64_t)j * a.hist_stride], s);
-                v = fmaf(a.dwa[a.depth], v, s);
+            Row<V>::load(a.x + t * width + c, v);
+            if (a.y) {
+                Row<V>::load(ff + c, q);  // written above by this same thread
+#pragma unroll
+                for (int i = 0; i < V; ++i) v[i] = fmaf(q[i], r, v[i]);
             }
-            a.x_out[t * width + c] = v;
+            Row<V>::store(mine + c, v);
+            if (a.dwa) {
+                const float* h = a.history + t * width + c;
+                float s[V];
+#pragma unroll
+                for (int i = 0; i < V; ++i) s[i] = 0.f;
+#pragma unroll 8
+                for (int j = 0; j < a.depth; ++j) {
+                    Row<V>::load(h + (int64_t)j * a.hist_stride, q);
+#pragma unroll
+                    for (int i = 0; i < V; ++i) s[i] = fmaf(dwa_s[j], q[i], s[i]);
+                }
+#pragma unroll
+                for (int i = 0; i < V; ++i) v[i] = fmaf(dwa_s[a.depth], v[i], s[i]);
+            }
+            Row<V>::store(a.x_out + t * width + c, v);
         }
-        reinterpret_cast<T*>(a.xb)[t * a.ldb + c] = from_f32<T>(v);
+        Row<V>::store(reinterpret_cast<T*>(a.xb) + t * a.ldb + c, v);
     }
 }
 
 cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    const size_t smem = a.y ? (size_t)width * 4 : 0;
-    if (smem > 200 * 1024) return cudaErrorInvalidValue;
+    const size_t smem = ((size_t)(a.y ? (width + 3) / 4 * 4 : 0) + 2 * (size_t)a.top + (a.dwa ? a.depth + 1 : 0)) * 4;
+    constexpr int CAP = 200 * 1024;
+    if (smem > CAP) return cudaErrorInvalidValue;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
-        cudaError_t e = cudaFuncSetAttribute(combine_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        return e != cudaSuccess ? e : cudaFuncSetAttribute(combine_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        const void* fns[] = {(const void*)combine_kernel<float, 1>, (const void*)combine_kernel<float, 4>, (const void*)combine_kernel<bf16, 1>,
+                             (const void*)combine_kernel<bf16, 4>};
+        for (const void* f : fns) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
     });
     if (le != cudaSuccess) return le;
-    le = SP_BY_TYPE(a.f32, combine_kernel, dim3(n_tok), dim3(ST_THREADS), smem, st, a, width);
+    const dim3 grid(n_tok), block(ST_THREADS);
+    if (width % 4 == 0) le = a.f32 ? launch_pdl(combine_kernel<float, 4>, grid, block, smem, st, a, width) : launch_pdl(combine_kernel<bf16, 4>, grid, block, smem, st, a, width);
+    else le = a.f32 ? launch_pdl(combine_kernel<float, 1>, grid, block, smem, st, a, width) : launch_pdl(combine_kernel<bf16, 1>, grid, block, smem, st, a, width);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
