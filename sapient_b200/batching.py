@@ -35,6 +35,7 @@ class ContinuousBatcher:
         self._h = C.c_void_p()
         self._engine = engine  # keeps the engine alive
         check(lib().sp_cuda_batcher_create(engine._h, int(prefill_chunk), int(bool(prefix_cache)), C.byref(self._h)))
+        engine._batchers.append(self._h)  # an engine that is closed first (a failed caller's clean-up) closes its batchers
 
     @classmethod
     def selftest(cls, vocab: int, max_slots: int, max_ctx: int, n_pages: int, prefill_chunk: int = 64, prefix_cache: bool = True):
@@ -49,7 +50,7 @@ class ContinuousBatcher:
     def close(self):
         if getattr(self, "_h", None) and self._h.value:
             lib().sp_cuda_batcher_destroy(self._h)
-            self._h = C.c_void_p()
+            self._h.value = None
 
     def __del__(self):
         try:

@@ -3,9 +3,9 @@
 //
 // A layer is ten to twelve launches whatever the row count: projections, rotation + cache append, [absorb,] attention
 // [, merge, value maps], output projection, norm + residual, router, choice, grouping, gate|up of the chosen and the
-// shared expert, down, mixture + norm + residual + depth average. Steps of up to PLAN_ROWS rows take the row kernels
-// (mat_f32.cu) and the absorbed attention and can be captured as a graph; longer ones the tcgen05 GEMM (mat_tc5.cu) and,
-// where rebuilding the keys pays, the expanded attention.
+// shared expert, down, mixture + norm + residual + depth average. bf16 products run on the tcgen05 kernel (mat_tc5.cu) at
+// every row count, f32 ones on mat_f32.cu. Steps of up to PLAN_ROWS rows take the absorbed attention and can be captured as
+// a graph; longer ones, where rebuilding the keys pays, the expanded attention.
 #include "engine_plan.h"
 
 #include <algorithm>

@@ -8,7 +8,7 @@
 // zeros or as rows nobody stores) — the weights of the first stages before the previous kernel is waited for, since no
 // kernel writes weights; warp 0 lane 0 issues four tcgen05.mma per tile and stage and commits them to the stage's `empty`
 // mbarrier; four epilogue warps read the accumulators back (one weight row per thread), apply the gated unit or the output
-// gate and store with n contiguous across the warp. Two CTAs per SM (256 TMEM columns and ~100 KB each), so that one
+// gate and store with n contiguous across the warp. Two CTAs per SM (256 TMEM columns and 109 KB each), so that one
 // CTA's epilogue runs under the other's loads and MMAs.
 // Few rows: the same kernel with 16- or 32-row activation tiles is a weight stream (all of a stage's bytes are weights but
 // an eighth); K is split over CTAs until the SMs are busy, partial tiles meet in a scratch buffer and the CTA that arrives
@@ -17,6 +17,7 @@
 // Every mbarrier wait is bounded; on expiry the kernel raises a flag, still frees its tensor memory and returns.
 #include <algorithm>
 #include <atomic>
+#include <type_traits>
 
 #include "kernels.h"
 #include "pdl.cuh"
@@ -31,7 +32,7 @@ cudaError_t count_launch_and_check();  // kernels.cu
 constexpr int MT_BM = 128, MT_BK = 64, MT_MAX_STAGES = 6;
 constexpr int MT_THREADS = 192;            // MMA warp, TMA warp, four epilogue warps
 constexpr int MT_A_BYTES = MT_BM * MT_BK * 2;
-constexpr int MT_SMEM = 100 * 1024;        // per CTA, two of which share an SM
+constexpr int MT_SMEM = 108 * 1024;        // per CTA, two of which share an SM
 constexpr int MT_MAX_PARTS = 8;
 
 __device__ int g_mat_tc5_timeout = 0;
@@ -50,7 +51,7 @@ struct MatTc5Args {
     int m, bn;            // activation rows, rows per tile (box height)
     int stages, stage_bytes, tmem_cols;
     int parts;            // CTAs (blockIdx.z) that share a tile's K range
-    bool dual, out_f32, moe, gather;
+    bool moe, gather;
     MoeRows rows;
     const float* gate;
     int ldgate;
@@ -58,6 +59,7 @@ struct MatTc5Args {
     unsigned* part_cnt;
 };
 
+template <bool DUAL, bool OUT_F32>
 __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
                                                              const __grid_constant__ CUtensorMap map_x0, const __grid_constant__ CUtensorMap map_w1,
                                                              const __grid_constant__ CUtensorMap map_x1) {
@@ -86,6 +88,8 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
     if (tid == 32) {
+        tc5_prefetch_map(si ? &map_w1 : &map_w0);
+        tc5_prefetch_map(si ? &map_x1 : &map_x0);
         for (int i = 0; i < a.stages; ++i) {
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&full[i])) : "memory");
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(tc5_smem_u32(&empty[i])) : "memory");
@@ -101,14 +105,14 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
     const int c_begin = part * all_chunks / a.parts, n_chunks_all = (part + 1) * all_chunks / a.parts - c_begin;
     const CUtensorMap* mw = si ? &map_w1 : &map_w0;
     const CUtensorMap* mx = si ? &map_x1 : &map_x0;
-    const int a_tiles = a.dual ? 2 : 1;
+    constexpr int a_tiles = DUAL ? 2 : 1;
     auto load_w = [&](int c, int st) {  // expects the whole stage, fetches its weight part
         const uint32_t bar = tc5_smem_u32(&full[st]);
         const uint32_t dst = tc5_smem_u32(smem + (size_t)st * a.stage_bytes);
         const int wrow = g * a_tiles * s.n + n0;
         asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(a.stage_bytes) : "memory");
         tc5_tma_2d(dst, mw, (c_begin + c) * MT_BK, wrow, bar);
-        if (a.dual) tc5_tma_2d(dst + MT_A_BYTES, mw, (c_begin + c) * MT_BK, wrow + s.n, bar);
+        if (DUAL) tc5_tma_2d(dst + MT_A_BYTES, mw, (c_begin + c) * MT_BK, wrow + s.n, bar);
     };
     const int early = (grouped || !in_range) ? 0 : min(a.stages, n_chunks_all);
     if (warp == 1 && lane == 0)
@@ -143,7 +147,7 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
 #pragma unroll
                 for (int i = 0; i < MT_BK / 16; ++i) {  // 16 columns: 32 bytes inside the swizzle row
                     tc5_mma(tmem, ad + 2u * i, bd + 2u * i, idesc, (uint32_t)(c > 0 || i > 0));
-                    if (a.dual) tc5_mma(tmem + (uint32_t)a.bn, ad2 + 2u * i, bd + 2u * i, idesc, (uint32_t)(c > 0 || i > 0));
+                    if (DUAL) tc5_mma(tmem + (uint32_t)a.bn, ad2 + 2u * i, bd + 2u * i, idesc, (uint32_t)(c > 0 || i > 0));
                 }
                 tc5_commit(&empty[st]);
             }
@@ -174,14 +178,12 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
         ok = tc5_wait(&done_bar, 0u);
         ok = __all_sync(0xFFFFFFFFu, ok);  // one verdict for the warp: the loads below are warp-collective
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        auto store = [&](int c, float f, float up) {
-            const int row = by_index ? dest[c] : r0 + c;
-            if (row < 0) return;
-            if (a.dual) f = clamped_unit(f, up, s.limit, s.alpha);
+        using Out = typename std::conditional<OUT_F32, float, bf16>::type;
+        Out* const yn = reinterpret_cast<Out*>(s.y) + (int64_t)g * s.ygs + n;
+        auto finish = [&](int row, float f, float up) {
+            if (DUAL) f = clamped_unit(f, up, s.limit, s.alpha);
             if (a.gate) f *= sigmoid_f32(a.gate[(int64_t)row * a.ldgate + g]);
-            const int64_t at = (int64_t)row * s.ldy + (int64_t)g * s.ygs + n;
-            if (a.out_f32) reinterpret_cast<float*>(s.y)[at] = f;
-            else reinterpret_cast<bf16*>(s.y)[at] = __float2bfloat16_rn(f);
+            yn[(int64_t)row * s.ldy] = from_f32<Out>(f);
         };
         const int64_t item = (int64_t)blockIdx.y * gridDim.x + blockIdx.x;
         const int64_t tile_floats = (int64_t)a_tiles * a.bn * MT_BM;
@@ -192,7 +194,7 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
             for (int c = 0; c < nb; c += 16) {
                 uint32_t v[16], up[16];
                 tc5_ld16(lanes + (uint32_t)c, v);
-                if (a.dual) tc5_ld16(lanes + (uint32_t)(a.bn + c), up);
+                if (DUAL) tc5_ld16(lanes + (uint32_t)(a.bn + c), up);
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
                 if (a.parts > 1) {
 #pragma unroll
@@ -200,12 +202,24 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
                         if (c + j >= cols) continue;
                         // (a short K may leave a part without chunks)
                         __stcg(mine + (c + j) * MT_BM, n_chunks ? __uint_as_float(v[j]) : 0.f);
-                        if (a.dual) __stcg(mine + (a.bn + c + j) * MT_BM, n_chunks ? __uint_as_float(up[j]) : 0.f);
+                        if (DUAL) __stcg(mine + (a.bn + c + j) * MT_BM, n_chunks ? __uint_as_float(up[j]) : 0.f);
                     }
                 } else if (n < s.n) {
+                    if (by_index || a.gate || c + 16 > cols) {
 #pragma unroll
-                    for (int j = 0; j < 16; ++j)
-                        if (c + j < cols) store(c + j, __uint_as_float(v[j]), a.dual ? __uint_as_float(up[j]) : 0.f);
+                        for (int j = 0; j < 16; ++j) {
+                            const int row = c + j < cols ? (by_index ? dest[c + j] : r0 + c + j) : -1;
+                            if (row >= 0) finish(row, __uint_as_float(v[j]), DUAL ? __uint_as_float(up[j]) : 0.f);
+                        }
+                    } else {
+                        Out* d = yn + (int64_t)(r0 + c) * s.ldy;
+#pragma unroll
+                        for (int j = 0; j < 16; ++j, d += s.ldy) {
+                            float f = __uint_as_float(v[j]);
+                            if (DUAL) f = clamped_unit(f, __uint_as_float(up[j]), s.limit, s.alpha);
+                            *d = from_f32<Out>(f);
+                        }
+                    }
                 }
             }
         }
@@ -220,13 +234,17 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
                 const float* src = all + 32 * q4 + lane;
                 if (n < s.n) {
                     for (int c = 0; c < cols; ++c) {
-                        if (by_index && dest[c] < 0) continue;
-                        float f = 0.f, up = 0.f;
-                        for (int p = 0; p < a.parts; ++p) {
-                            f += __ldcg(src + p * tile_floats + c * MT_BM);
-                            if (a.dual) up += __ldcg(src + p * tile_floats + (a.bn + c) * MT_BM);
+                        const int row = by_index ? dest[c] : r0 + c;
+                        if (row < 0) continue;
+                        float f[MT_MAX_PARTS], up[MT_MAX_PARTS];
+#pragma unroll
+                        for (int p = 0; p < MT_MAX_PARTS; ++p) {
+                            f[p] = p < a.parts ? __ldcg(src + p * tile_floats + c * MT_BM) : 0.f;
+                            up[p] = DUAL && p < a.parts ? __ldcg(src + p * tile_floats + (a.bn + c) * MT_BM) : 0.f;
                         }
-                        store(c, f, up);
+#pragma unroll
+                        for (int p = 1; p < MT_MAX_PARTS; ++p) { f[0] += f[p]; up[0] += up[p]; }
+                        finish(row, f[0], up[0]);
                     }
                 }
                 if (tid == 64) a.part_cnt[item] = 0u;  // ready for the next launch
@@ -283,7 +301,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc
     k.row_tiles = (a.m + bn - 1) / bn;
     k.slots0 = a.moe ? max_tiles : groups * k.row_tiles;
     const int slots = k.slots0 + (a.nseg == 2 ? k.row_tiles : 0);
-    k.dual = a.dual; k.out_f32 = a.out_f32; k.moe = a.moe; k.gather = a.gather; k.rows = a.rows; k.gate = a.gate; k.ldgate = a.ldgate;
+    k.moe = a.moe; k.gather = a.gather; k.rows = a.rows; k.gate = a.gate; k.ldgate = a.ldgate;
     const int acc = a.dual ? 2 : 1;
     k.stage_bytes = acc * MT_A_BYTES + bn * MT_BK * 2;
     k.tmem_cols = std::max(32, acc * bn);
@@ -292,9 +310,9 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc
     const int64_t items = (int64_t)row_blocks * slots;
     int64_t busy = 0;  // tiles that exist
     for (int i = 0; i < a.nseg; ++i) busy += (int64_t)((a.seg[i].n + MT_BM - 1) / MT_BM) * (i ? k.row_tiles : k.slots0);
-    if (bn <= 32 && sc.part && items <= MatScratch::ITEMS) {
-        // two CTAs per SM, but no part shorter than four chunks of K
-        while (k.parts < MT_MAX_PARTS && busy * k.parts < 2 * sms && kp_max / MT_BK >= 8 * k.parts &&
+    if (a.m <= 32 && sc.part && items <= MatScratch::ITEMS) {
+        // a CTA per SM, but no part shorter than four chunks of K
+        while (k.parts < MT_MAX_PARTS && busy * k.parts < sms && kp_max / MT_BK >= 8 * k.parts &&
                items * (2 * k.parts) * acc * bn * MT_BM <= (int64_t)MatScratch::FLOATS)
             k.parts *= 2;
     }
@@ -308,11 +326,23 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc
     }
     if (a.nseg == 1) { mw[1] = mw[0]; mx[1] = mx[0]; }
     static PerDeviceOnce once;
-    cudaError_t le = once.run([] { return cudaFuncSetAttribute(mat_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM + 1024); });
+    cudaError_t le = once.run([] {
+        const void* fns[] = {(const void*)mat_tc5_kernel<false, false>, (const void*)mat_tc5_kernel<false, true>, (const void*)mat_tc5_kernel<true, false>,
+                             (const void*)mat_tc5_kernel<true, true>};
+        for (const void* f : fns) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM + 1024);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
+    });
     if (le != cudaSuccess) return le;
     g_mat_tc5_launched[current_device_index()].store(1);
-    le = launch_pdl(mat_tc5_kernel, dim3((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), dim3(MT_THREADS), (size_t)(k.stages * k.stage_bytes + 1024), st, k,
-                    mw[0], mx[0], mw[1], mx[1]);
+    const dim3 grid((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), block(MT_THREADS);
+    const size_t smem = (size_t)(k.stages * k.stage_bytes + 1024);
+#define SP_MT(DUAL, F32) le = launch_pdl(mat_tc5_kernel<DUAL, F32>, grid, block, smem, st, k, mw[0], mx[0], mw[1], mx[1])
+    if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
+    else { if (a.out_f32) SP_MT(false, true); else SP_MT(false, false); }
+#undef SP_MT
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }

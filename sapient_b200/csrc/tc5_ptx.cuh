@@ -66,6 +66,11 @@ __device__ __forceinline__ void tc5_tma_2d(uint32_t dst, const CUtensorMap* map,
         : "memory");
 }
 
+// Brings a tensor map (a kernel parameter) into the descriptor cache ahead of its first copy.
+__device__ __forceinline__ void tc5_prefetch_map(const CUtensorMap* map) {
+    asm volatile("prefetch.tensormap [%0];\n" ::"l"(map) : "memory");
+}
+
 // 16 consecutive tensor-memory columns of the warp's 32 lanes, one lane per thread.
 __device__ __forceinline__ void tc5_ld16(uint32_t taddr, uint32_t (&r)[16]) {
     asm volatile(

@@ -37,6 +37,7 @@ class ForwardEngine:
         check(lib().sp_cuda_engine_vocab_local(handle, C.byref(rows), C.byref(first)))
         self.vocab_local, self.vocab_first = int(rows.value), int(first.value)  # this rank's slice of the logits
         self._tp_group = None
+        self._batchers = []  # handles of live batchers, destroyed before the engine
 
     # ── construction ────────────────────────────────────────────────────────
     @classmethod
@@ -141,6 +142,10 @@ class ForwardEngine:
 
     def close(self) -> None:
         if getattr(self, "_h", None):
+            for b in getattr(self, "_batchers", ()):
+                if b.value:
+                    lib().sp_cuda_batcher_destroy(b)
+                    b.value = None
             lib().sp_cuda_engine_destroy(self._h)
             self._h = None
 
