@@ -14,6 +14,7 @@
 #include <map>
 
 #include "engine.h"
+#include "pdl.cuh"
 #include "plan_common.cuh"
 #include "sp_common.cuh"
 
@@ -288,10 +289,6 @@ int Engine::finalize_plan() {
     p.part = (float*)take((size_t)PLAN_SPLIT_ROWS * n_part * 4);
     p.history = (float*)take((size_t)(L + 1) * T * W * 4);
     p.fin = take((size_t)PLAN_ROWS * p.wp * el);
-    if (!p.f32) {
-        p.scratch.part = (float*)take(MatScratch::FLOATS * 4);
-        p.scratch.cnt = (unsigned*)take(MatScratch::ITEMS * 4);
-    }
     if (n_pairs) {
         p.act = take(T * n_act * el);
         p.act_shared = take(T * n_act_s * el);
@@ -346,9 +343,10 @@ int Engine::plan_ctx_bucket() const {
 
 static int plan_splits(const PlanLayer& l, bool f32, int bucket, int T) {
     if (T > PLAN_ROWS) return 1;
-    const int keys = std::min(1 << bucket, l.shape.window), blocks = (f32 ? l.shape.heads : (l.shape.heads + 15) / 16) * T;
+    const int keys = std::min(1 << bucket, l.shape.window), blocks = (f32 ? l.shape.heads : (l.shape.heads + 31) / 32) * T;
+    const int slots = (f32 || l.shape.heads <= 16 ? 2 : 1) * device_sm_count();  // blocks the device holds at once
     int s = 1;
-    while (s < 16 && blocks * s < 296 && keys >= 64 * 2 * s && T * 2 * s <= PLAN_SPLIT_ROWS) s <<= 1;
+    while (s < 16 && blocks * 2 * s <= slots && keys >= 64 * 2 * s && T * 2 * s <= PLAN_SPLIT_ROWS) s <<= 1;
     return s;
 }
 
@@ -381,7 +379,7 @@ int Engine::plan_stage(int T) {
 }
 
 int Engine::plan_product(const MatArgs& a, int max_tiles) {
-    SP_LAUNCH(F_GEMV, a.f32 ? launch_mat_f32(a, stream) : launch_mat_tc5(a, max_tiles, plan_->scratch, stream));
+    SP_LAUNCH(F_GEMV, a.f32 ? launch_mat_f32(a, stream) : launch_mat_tc5(a, max_tiles, stream));
     return SP_OK;
 }
 

@@ -48,7 +48,6 @@ struct PlanState {
     float *proj = nullptr, *y = nullptr, *y_expert = nullptr, *y_shared = nullptr, *logit = nullptr, *weight = nullptr, *part = nullptr, *history = nullptr;
     int32_t *pick = nullptr, *tables = nullptr, *host_tiles = nullptr, *dev_tiles = nullptr;
     MoeTables moe{};
-    MatScratch scratch{};
     int keys_cap = 0;          // gathered keys a step may hold
     // the expanded form of the current step (0 tiles: absorbed)
     int n_tiles = 0, n_keys = 0;

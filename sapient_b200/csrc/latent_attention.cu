@@ -155,107 +155,136 @@ __global__ void __launch_bounds__(LS_WARPS * 32) latent_attention_simple_kernel(
     if (n_splits > 1 && threadIdx.x == 0) { pd[0] = M; pd[1] = L; }
 }
 
-// bf16: block per (16 heads, token, split), 4 warps, key tiles of 32 double-buffered with cp.async. Scores: warp w takes
-// keys 8 w .. + 7 of the tile, all heads; mixture: warp w takes NT 8-column tiles of the latent, all keys.
-constexpr int LM_KEYS = 32, LM_WARPS = 4, LM_PLD = LM_KEYS + 8;
-template <int NT>
-__global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
-                                                                             const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
-                                                                             bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
-    extern __shared__ __align__(16) bf16 lm_smem[];
-    __shared__ float ss[16][LM_KEYS + 1], corr_s[16], l_s[16], m_s[16];
-    __shared__ __align__(16) bf16 ps[16][LM_PLD];
+// bf16: block per (HG groups of 16 heads, token, split), 8 warps per group, key tiles of 32 double-buffered with cp.async and
+// shared by the groups. Scores: a warp owns an eighth of the coordinates (its query fragments stay in registers) for all
+// keys of the tile, the partial sums meet in shared memory; mixture: a warp owns NT 8-column tiles of the latent.
+constexpr int LM_KEYS = 32, LM_WARPS = 8, LM_PLD = LM_KEYS + 8, LM_SLD = LM_KEYS + 1;
+constexpr int LM_ROW_THREADS = LM_WARPS * 2, LM_ROW_KEYS = LM_KEYS / LM_ROW_THREADS;  // of the softmax: threads per query, keys per thread
+constexpr int LM_MAX_STEPS = 5;   // 16-coordinate steps per warp: rank + rot up to 640
+static size_t lm_smem(int width, int hg) { return (size_t)2 * LM_KEYS * (width + 8) * 2 + (size_t)hg * LM_WARPS * 16 * LM_SLD * 4; }
+__device__ __forceinline__ void group_sync(int grp) { asm volatile("bar.sync %0, %1;\n" ::"r"(grp + 1), "n"(LM_WARPS * 32) : "memory"); }
+
+template <int NT, int HG>
+__global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
+                                                                                  const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
+                                                                                  bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
+    extern __shared__ __align__(16) bf16 lm_smem_raw[];
+    __shared__ float corr_s[HG][16], l_s[HG][16], m_s[HG][16];
+    __shared__ __align__(16) bf16 ps_all[HG][16][LM_PLD];
     const int width = c.rank16 + c.rot16, LD = width + 8;
-    bf16* qs = lm_smem;
-    bf16* ks = lm_smem + 16 * LD;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-    const int h0 = blockIdx.x * 16, t = blockIdx.y;
+    const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+    const int grp = HG > 1 ? wid / LM_WARPS : 0, warp = wid % LM_WARPS, tid = threadIdx.x % (LM_WARPS * 32);
+    bf16* ks = lm_smem_raw;
+    float* ss = reinterpret_cast<float*>(ks + 2 * LM_KEYS * LD) + grp * LM_WARPS * 16 * LM_SLD;
+    bf16(*ps)[LM_PLD] = ps_all[grp];
+    const int h0 = (blockIdx.x * HG + grp) * 16, t = blockIdx.y;
     pdl_wait();
     pdl_trigger();
     int begin, end;
     key_range(tok_pos[t], s.window, blockIdx.z, n_splits, begin, end);
     const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
     const int pieces = width / 8;
-    for (int r = warp; r < 16; r += LM_WARPS) {
-        const bool live = h0 + r < s.heads;
-        const bf16* src = qabs + ((int64_t)t * s.heads + (live ? h0 + r : h0)) * c.ld;
-        for (int p = lane; p < pieces; p += 32) cp_async16(qs + r * LD + p * 8, src + p * 8, live ? 16 : 0);
-    }
-    auto fetch = [&](int k0, int buf) {  // warp w copies keys w, w + 4, ..: a row's address is found once
+    auto fetch = [&](int k0, int buf) {  // a warp copies every (8 HG)-th key: a row's address is found once
         bf16* d = ks + buf * LM_KEYS * LD;
-        const bf16* src[LM_KEYS / LM_WARPS];
+        constexpr int PER = LM_KEYS / (LM_WARPS * HG);
+        const bf16* src[PER];
 #pragma unroll
-        for (int i = 0; i < LM_KEYS / LM_WARPS; ++i) {
-            const int key = min(k0 + warp + LM_WARPS * i, end - 1);
+        for (int i = 0; i < PER; ++i) {
+            const int key = min(k0 + wid + LM_WARPS * HG * i, end - 1);
             src[i] = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld;
         }
 #pragma unroll
-        for (int i = 0; i < LM_KEYS / LM_WARPS; ++i) {
-            const int r = warp + LM_WARPS * i, bytes = k0 + r < end ? 16 : 0;
+        for (int i = 0; i < PER; ++i) {
+            const int r = wid + LM_WARPS * HG * i, bytes = k0 + r < end ? 16 : 0;
             for (int p = lane; p < pieces; p += 32) cp_async16(d + r * LD + p * 8, src[i] + p * 8, bytes);
         }
     };
+    // two tiles in flight from the start; a buffer is refilled as soon as everyone is done with it
     if (begin < end) fetch(begin, 0);
     cp_async_commit();
+    if (begin + LM_KEYS < end) fetch(begin + LM_KEYS, 1);
+    cp_async_commit();
+    // this warp's coordinates of the 16 queries
+    const int steps = width / 16, per = (steps + LM_WARPS - 1) / LM_WARPS, s0 = warp * per, my = max(0, min(per, steps - s0));
+    uint32_t qf[LM_MAX_STEPS][4];
+    {
+        const int ha = h0 + g, hb = h0 + g + 8;
+        const uint32_t* qa = reinterpret_cast<const uint32_t*>(qabs + ((int64_t)t * s.heads + min(ha, s.heads - 1)) * c.ld);
+        const uint32_t* qb = reinterpret_cast<const uint32_t*>(qabs + ((int64_t)t * s.heads + min(hb, s.heads - 1)) * c.ld);
+#pragma unroll
+        for (int i = 0; i < LM_MAX_STEPS; ++i) {
+            const int k = (s0 + i) * 8 + tq;  // in pairs
+            const bool on = i < my;
+            qf[i][0] = on && ha < s.heads ? qa[k] : 0u;
+            qf[i][1] = on && hb < s.heads ? qb[k] : 0u;
+            qf[i][2] = on && ha < s.heads ? qa[k + 4] : 0u;
+            qf[i][3] = on && hb < s.heads ? qb[k + 4] : 0u;
+        }
+    }
     float o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    float m = -INFINITY, l = 0.f;  // of row tid / 8, the same in its eight threads
+    float m = -INFINITY, l = 0.f;  // of row tid / LM_ROW_THREADS, the same in all its threads
     const int col0 = warp * NT * 8;
     for (int k0 = begin, buf = 0; k0 < end; k0 += LM_KEYS, buf ^= 1) {
-        cp_async_wait<0>();
-        __syncthreads();  // this tile has landed for everyone, and everyone is done with the other buffer
-        if (k0 + LM_KEYS < end) fetch(k0 + LM_KEYS, buf ^ 1);
-        cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();  // this tile has landed for everyone
         const bf16* kt = ks + buf * LM_KEYS * LD;
         {
-            float a0[4] = {}, a1[4] = {};
-            const uint32_t qa = smem_addr(qs + (lane & 15) * LD + (lane >> 4) * 8);
-            const uint32_t ka = smem_addr(kt + (8 * warp + (lane & 7)) * LD + (lane >> 3) * 8);
-            int k = 0;
-            for (; k + 32 <= width; k += 32) {
-                uint32_t q0[4], q1[4], b[4];
-                ldsm_x4(q0, qa + 2 * k);
-                ldsm_x4(q1, qa + 2 * (k + 16));
-                ldsm_x4(b, ka + 2 * k);
-                mma_bf16(a0, q0[0], q0[1], q0[2], q0[3], b[0], b[1]);
-                mma_bf16(a1, q1[0], q1[1], q1[2], q1[3], b[2], b[3]);
+            float a[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
+            const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8 + s0 * 16);
+#pragma unroll
+            for (int i = 0; i < LM_MAX_STEPS; ++i) {
+                if (i < my) {
+                    uint32_t b0[4], b1[4];
+                    ldsm_x4(b0, ka + 2 * (16 * i));
+                    ldsm_x4(b1, ka + 2 * (16 * LD + 16 * i));
+                    mma_bf16(a[0], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b0[0], b0[1]);
+                    mma_bf16(a[1], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b0[2], b0[3]);
+                    mma_bf16(a[2], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b1[0], b1[1]);
+                    mma_bf16(a[3], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b1[2], b1[3]);
+                }
             }
-            if (k < width) {
-                uint32_t q0[4], b[2];
-                ldsm_x4(q0, qa + 2 * k);
-                ldsm_x2(b, smem_addr(kt + (8 * warp + (lane & 7)) * LD + ((lane >> 3) & 1) * 8) + 2 * k);
-                mma_bf16(a0, q0[0], q0[1], q0[2], q0[3], b[0], b[1]);
+            float* d = ss + (warp * 16 + g) * LM_SLD + 2 * tq;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                d[8 * j] = a[j][0];
+                d[8 * j + 1] = a[j][1];
+                d[8 * LM_SLD + 8 * j] = a[j][2];
+                d[8 * LM_SLD + 8 * j + 1] = a[j][3];
             }
-            const int key = 8 * warp + 2 * tq;
-            const bool v0 = k0 + key < end, v1 = k0 + key + 1 < end;
-            ss[g][key] = v0 ? (a0[0] + a1[0]) * s.scale : -INFINITY;
-            ss[g][key + 1] = v1 ? (a0[1] + a1[1]) * s.scale : -INFINITY;
-            ss[g + 8][key] = v0 ? (a0[2] + a1[2]) * s.scale : -INFINITY;
-            ss[g + 8][key + 1] = v1 ? (a0[3] + a1[3]) * s.scale : -INFINITY;
         }
-        __syncthreads();
+        group_sync(grp);
         {
-            const int r = tid >> 3, q4 = (tid & 7) * 4;
-            float v[4], mx = m;
+            const int r = tid / LM_ROW_THREADS, key = tid % LM_ROW_THREADS * LM_ROW_KEYS;
+            float v[LM_ROW_KEYS], mx = m;
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { v[i] = ss[r][q4 + i]; mx = fmaxf(mx, v[i]); }
+            for (int i = 0; i < LM_ROW_KEYS; ++i) {
+                float z = 0.f;
 #pragma unroll
-            for (int off = 4; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
+                for (int w = 0; w < LM_WARPS; ++w) z += ss[(w * 16 + r) * LM_SLD + key + i];
+                v[i] = k0 + key + i < end ? z * s.scale : -INFINITY;
+                mx = fmaxf(mx, v[i]);
+            }
+#pragma unroll
+            for (int off = LM_ROW_THREADS / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
             // the tile's first key is live, so mx is finite
             const float cr = expf(m - mx);
             float sum = 0.f;
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
+            for (int i = 0; i < LM_ROW_KEYS; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
 #pragma unroll
-            for (int off = 4; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
-            *reinterpret_cast<uint2*>(&ps[r][q4]) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+            for (int off = LM_ROW_THREADS / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
+            static_assert(LM_ROW_KEYS == 2, "the softmax weights are stored in pairs");
+            *reinterpret_cast<uint32_t*>(&ps[r][key]) = pack_bf16(v[0], v[1]);
             l = fmaf(l, cr, sum);
             m = mx;
-            if ((tid & 7) == 0) corr_s[r] = cr;
+            if (tid % LM_ROW_THREADS == 0) corr_s[grp][r] = cr;
         }
-        __syncthreads();
-        const float c0 = corr_s[g], c1 = corr_s[g + 8];
+        group_sync(grp);
+        const float c0 = corr_s[grp][g], c1 = corr_s[grp][g + 8];
 #pragma unroll
         for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
 #pragma unroll
@@ -273,16 +302,19 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(con
                 }
             }
         }
+        __syncthreads();
+        if (k0 + 2 * LM_KEYS < end) fetch(k0 + 2 * LM_KEYS, buf);
+        cp_async_commit();
     }
     cp_async_wait<0>();
-    if ((tid & 7) == 0) { l_s[tid >> 3] = l; m_s[tid >> 3] = m; }
-    __syncthreads();
+    if (tid % LM_ROW_THREADS == 0) { l_s[grp][tid / LM_ROW_THREADS] = l; m_s[grp][tid / LM_ROW_THREADS] = m; }
+    group_sync(grp);
 #pragma unroll
     for (int r2 = 0; r2 < 2; ++r2) {
         const int r = g + 8 * r2, h = h0 + r;
         if (h >= s.heads) continue;
         if (n_splits == 1) {
-            const float inv = 1.0f / l_s[r];
+            const float inv = 1.0f / l_s[grp][r];
             bf16* d = out + ((int64_t)t * s.heads + h) * ldo;
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
@@ -292,7 +324,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(con
             }
         } else {
             float* d = part + (((int64_t)t * s.heads + h) * n_splits + blockIdx.z) * (c.rank + 2);
-            if (warp == 0 && tq == 0) { d[0] = m_s[r]; d[1] = l_s[r]; }
+            if (warp == 0 && tq == 0) { d[0] = m_s[grp][r]; d[1] = l_s[grp][r]; }
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
                 const int e = col0 + i * 8 + 2 * tq;
@@ -340,8 +372,10 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
     constexpr int CAP = 200 * 1024;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
-        const void* fns[] = {(const void*)latent_attention_mma_kernel<2>, (const void*)latent_attention_mma_kernel<4>, (const void*)latent_attention_mma_kernel<8>,
-                             (const void*)latent_attention_mma_kernel<16>, (const void*)latent_attention_simple_kernel<float>, (const void*)latent_attention_simple_kernel<bf16>};
+        const void* fns[] = {(const void*)latent_attention_mma_kernel<2, 1>, (const void*)latent_attention_mma_kernel<4, 1>, (const void*)latent_attention_mma_kernel<8, 1>,
+                             (const void*)latent_attention_mma_kernel<2, 2>, (const void*)latent_attention_mma_kernel<4, 2>,
+                             (const void*)latent_attention_mma_kernel<8, 2>,
+                             (const void*)latent_attention_simple_kernel<float>, (const void*)latent_attention_simple_kernel<bf16>};
         for (const void* f : fns) {
             const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
             if (e != cudaSuccess) return e;
@@ -350,15 +384,17 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
     });
     if (le != cudaSuccess) return le;
     const int width = c.rank16 + c.rot16;
-    const size_t mma_smem = (size_t)(16 + 2 * LM_KEYS) * (width + 8) * 2;
     const int per_warp = (c.rank16 + 8 * LM_WARPS - 1) / (8 * LM_WARPS);  // 8-column tiles each warp has to cover
-    if (!f32 && per_warp <= 16 && mma_smem <= CAP) {
-        const dim3 grid((s.heads + 15) / 16, n_tok, n_splits), block(LM_WARPS * 32);
-#define SP_LM(NT) le = launch_pdl(latent_attention_mma_kernel<NT>, grid, block, mma_smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
+    const int hg = s.heads > 16 ? 2 : 1;
+    const size_t smem = lm_smem(width, hg);
+    if (!f32 && per_warp <= 8 && width <= 16 * LM_WARPS * LM_MAX_STEPS && smem <= CAP) {
+        const dim3 grid((s.heads + 16 * hg - 1) / (16 * hg), n_tok, n_splits), block(LM_WARPS * 32 * hg);
+#define SP_LM(NT)                                                                                                                                  \
+    le = hg == 1 ? launch_pdl(latent_attention_mma_kernel<NT, 1>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits) \
+                 : launch_pdl(latent_attention_mma_kernel<NT, 2>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
         if (per_warp <= 2) SP_LM(2);
         else if (per_warp <= 4) SP_LM(4);
-        else if (per_warp <= 8) SP_LM(8);
-        else SP_LM(16);
+        else SP_LM(8);
 #undef SP_LM
     } else {
         const dim3 grid(s.heads, n_tok, n_splits), block(LS_WARPS * 32);

@@ -11,8 +11,8 @@
 // gate and store with n contiguous across the warp. Two CTAs per SM (256 TMEM columns and 109 KB each), so that one
 // CTA's epilogue runs under the other's loads and MMAs.
 // Few rows: the same kernel with 16- or 32-row activation tiles is a weight stream (all of a stage's bytes are weights but
-// an eighth); K is split over CTAs until the SMs are busy, partial tiles meet in a scratch buffer and the CTA that arrives
-// last adds them in order. Experts of a small step (`gather`) multiply every row of the step, which costs nothing at this
+// an eighth); K is split over the CTAs of a cluster until the SMs are busy, and they add each other's partial tiles in a fixed
+// order through distributed shared memory. Experts of a small step (`gather`) multiply every row of the step, which costs nothing at this
 // tile size, and keep the rows that chose them: no gathered copy.
 // Every mbarrier wait is bounded; on expiry the kernel raises a flag, still frees its tensor memory and returns.
 #include <algorithm>
@@ -37,6 +37,21 @@ constexpr int MT_MAX_PARTS = 8;
 
 __device__ int g_mat_tc5_timeout = 0;
 
+// A barrier of all threads of the cluster; shared-memory writes before it are visible to the peers after it.
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release;\nbarrier.cluster.wait.acquire;\n" ::: "memory");
+}
+__device__ __forceinline__ uint32_t peer_smem(uint32_t addr, int rank) {
+    uint32_t r;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(r) : "r"(addr), "r"(rank));
+    return r;
+}
+__device__ __forceinline__ float ld_peer(uint32_t addr) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(addr) : "memory");
+    return v;
+}
+
 struct MatTc5Seg {
     void* y;
     int64_t ygs;
@@ -50,24 +65,21 @@ struct MatTc5Args {
     int row_tiles;        // row tiles of a dense or per-head product (blockIdx.y = group * row_tiles + tile)
     int m, bn;            // activation rows, rows per tile (box height)
     int stages, stage_bytes, tmem_cols;
-    int parts;            // CTAs (blockIdx.z) that share a tile's K range
+    int parts;            // CTAs (blockIdx.z, one cluster) that share a tile's K range
     bool moe, gather;
     MoeRows rows;
     const float* gate;
     int ldgate;
-    float* part_buf;      // [item][part][accumulator][bn columns][128]
-    unsigned* part_cnt;
 };
 
 template <bool DUAL, bool OUT_F32>
-__global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
+__global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
                                                              const __grid_constant__ CUtensorMap map_x0, const __grid_constant__ CUtensorMap map_w1,
                                                              const __grid_constant__ CUtensorMap map_x1) {
     extern __shared__ uint8_t mt_smem_raw[];
     __shared__ __align__(8) uint64_t full[MT_MAX_STAGES], empty[MT_MAX_STAGES], done_bar;
     __shared__ uint32_t tmem_slot;
     __shared__ int dest[MAT_GATHER_ROWS];  // gather: output row of each of the step's rows, -1: not this expert's
-    __shared__ int last_part;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int si = (int)blockIdx.y >= a.slots0;
     const MatTc5Seg& s = a.seg[si];
@@ -133,6 +145,7 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
     const int nb = (cols + 15) & ~15;
     const int x0 = by_index ? 0 : r0;
     const int n_chunks = live ? n_chunks_all : 0;
+    float* const partial = reinterpret_cast<float*>(smem);  // [accumulator][bn columns][128], once the ring has drained
     bool ok = true;
     if (warp == 0) {
         if (lane == 0 && live) {
@@ -180,17 +193,16 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         using Out = typename std::conditional<OUT_F32, float, bf16>::type;
         Out* const yn = reinterpret_cast<Out*>(s.y) + (int64_t)g * s.ygs + n;
-        auto finish = [&](int row, float f, float up) {
+        // gate: what the output gate's logit of (row, g) is; the callers load a batch of them before the first store
+        auto gate_of = [&](int row) { return a.gate[(int64_t)row * a.ldgate + g]; };
+        auto finish = [&](int row, float f, float up, float gate) {
             if (DUAL) f = clamped_unit(f, up, s.limit, s.alpha);
-            if (a.gate) f *= sigmoid_f32(a.gate[(int64_t)row * a.ldgate + g]);
+            if (a.gate) f *= sigmoid_f32(gate);
             yn[(int64_t)row * s.ldy] = from_f32<Out>(f);
         };
-        const int64_t item = (int64_t)blockIdx.y * gridDim.x + blockIdx.x;
-        const int64_t tile_floats = (int64_t)a_tiles * a.bn * MT_BM;
-        float* all = a.part_buf + item * a.parts * tile_floats;
         if (ok) {
             const uint32_t lanes = tmem + ((uint32_t)(32 * q4) << 16);
-            float* mine = all + part * tile_floats + 32 * q4 + lane;
+            float* mine = partial + 32 * q4 + lane;
             for (int c = 0; c < nb; c += 16) {
                 uint32_t v[16], up[16];
                 tc5_ld16(lanes + (uint32_t)c, v);
@@ -201,16 +213,21 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
                     for (int j = 0; j < 16; ++j) {
                         if (c + j >= cols) continue;
                         // (a short K may leave a part without chunks)
-                        __stcg(mine + (c + j) * MT_BM, n_chunks ? __uint_as_float(v[j]) : 0.f);
-                        if (DUAL) __stcg(mine + (a.bn + c + j) * MT_BM, n_chunks ? __uint_as_float(up[j]) : 0.f);
+                        mine[(c + j) * MT_BM] = n_chunks ? __uint_as_float(v[j]) : 0.f;
+                        if (DUAL) mine[(a.bn + c + j) * MT_BM] = n_chunks ? __uint_as_float(up[j]) : 0.f;
                     }
                 } else if (n < s.n) {
                     if (by_index || a.gate || c + 16 > cols) {
+                        int row[16];
+                        float gt[16];
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
-                            const int row = c + j < cols ? (by_index ? dest[c + j] : r0 + c + j) : -1;
-                            if (row >= 0) finish(row, __uint_as_float(v[j]), DUAL ? __uint_as_float(up[j]) : 0.f);
+                            row[j] = c + j < cols ? (by_index ? dest[c + j] : r0 + c + j) : -1;
+                            gt[j] = a.gate && row[j] >= 0 ? gate_of(row[j]) : 0.f;
                         }
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            if (row[j] >= 0) finish(row[j], __uint_as_float(v[j]), DUAL ? __uint_as_float(up[j]) : 0.f, gt[j]);
                     } else {
                         Out* d = yn + (int64_t)(r0 + c) * s.ldy;
 #pragma unroll
@@ -224,32 +241,42 @@ __global__ void __launch_bounds__(MT_THREADS) mat_tc5_kernel(const MatTc5Args a,
             }
         }
         if (a.parts > 1) {
-            // every epilogue warp comes here whatever its `ok`; no CTA waits for another
-            __threadfence();
-            asm volatile("bar.sync 1, 128;\n" ::: "memory");
-            if (tid == 64) last_part = atomicAdd(&a.part_cnt[item], 1u) == (unsigned)(a.parts - 1);
-            asm volatile("bar.sync 1, 128;\n" ::: "memory");
-            if (last_part) {
-                __threadfence();
-                const float* src = all + 32 * q4 + lane;
-                if (n < s.n) {
-                    for (int c = 0; c < cols; ++c) {
-                        const int row = by_index ? dest[c] : r0 + c;
-                        if (row < 0) continue;
-                        float f[MT_MAX_PARTS], up[MT_MAX_PARTS];
+            // the cluster's CTAs share out the columns; each adds its columns' partials in part order
+            cluster_sync();
+            if (n < s.n) {
+                constexpr int NC = 4;
+                const uint32_t my_row = tc5_smem_u32(partial + 32 * q4 + lane);
+                for (int c0 = part; c0 < cols; c0 += NC * a.parts) {
+                    int row[NC];
+                    float f[NC], up[NC], gt[NC];
 #pragma unroll
-                        for (int p = 0; p < MT_MAX_PARTS; ++p) {
-                            f[p] = p < a.parts ? __ldcg(src + p * tile_floats + c * MT_BM) : 0.f;
-                            up[p] = DUAL && p < a.parts ? __ldcg(src + p * tile_floats + (a.bn + c) * MT_BM) : 0.f;
-                        }
-#pragma unroll
-                        for (int p = 1; p < MT_MAX_PARTS; ++p) { f[0] += f[p]; up[0] += up[p]; }
-                        finish(row, f[0], up[0]);
+                    for (int j = 0; j < NC; ++j) {
+                        const int c = c0 + j * a.parts;
+                        row[j] = c < cols ? (by_index ? dest[c] : r0 + c) : -1;
+                        gt[j] = a.gate && row[j] >= 0 ? gate_of(row[j]) : 0.f;
+                        f[j] = up[j] = 0.f;
                     }
+#pragma unroll 4
+                    for (int p = 0; p < a.parts; ++p) {
+                        const uint32_t peer = peer_smem(my_row, p);
+#pragma unroll
+                        for (int j = 0; j < NC; ++j) {
+                            if (row[j] < 0) continue;
+                            const int c = c0 + j * a.parts;
+                            f[j] += ld_peer(peer + (uint32_t)c * MT_BM * 4);
+                            if (DUAL) up[j] += ld_peer(peer + (uint32_t)(a.bn + c) * MT_BM * 4);
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < NC; ++j)
+                        if (row[j] >= 0) finish(row[j], f[j], up[j], gt[j]);
                 }
-                if (tid == 64) a.part_cnt[item] = 0u;  // ready for the next launch
             }
         }
+    }
+    if (a.parts > 1 && live) {
+        if (warp < 2) { __syncwarp(); cluster_sync(); }  // the service warps' share of the cluster's first barrier
+        cluster_sync();                                  // nobody leaves while its partials are being read
     }
     if (!ok) atomicExch(&g_mat_tc5_timeout, 1);
     asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -278,7 +305,7 @@ static bool mat_map(CUtensorMap* map, const void* p, int64_t cols, int64_t rows,
                             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc, cudaStream_t st) {
+cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     if (a.m <= 0) return cudaSuccess;
     if (a.f32 || a.nseg < 1 || a.nseg > 2 || (a.nseg == 2 && a.seg[1].groups != 1) || (a.gather && (!a.moe || a.m > MAT_GATHER_ROWS))) return cudaErrorInvalidValue;
     MatTc5Args k{};
@@ -307,17 +334,11 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc
     k.tmem_cols = std::max(32, acc * bn);
     k.stages = std::min(MT_MAX_STAGES, MT_SMEM / k.stage_bytes);
     k.parts = 1;
-    const int64_t items = (int64_t)row_blocks * slots;
     int64_t busy = 0;  // tiles that exist
     for (int i = 0; i < a.nseg; ++i) busy += (int64_t)((a.seg[i].n + MT_BM - 1) / MT_BM) * (i ? k.row_tiles : k.slots0);
-    if (a.m <= 32 && sc.part && items <= MatScratch::ITEMS) {
-        // a CTA per SM, but no part shorter than four chunks of K
-        while (k.parts < MT_MAX_PARTS && busy * k.parts < sms && kp_max / MT_BK >= 8 * k.parts &&
-               items * (2 * k.parts) * acc * bn * MT_BM <= (int64_t)MatScratch::FLOATS)
-            k.parts *= 2;
-    }
-    k.part_buf = sc.part;
-    k.part_cnt = sc.cnt;
+    // a CTA per SM, but no part shorter than four chunks of K
+    if (a.m <= 32)
+        while (k.parts < MT_MAX_PARTS && busy * k.parts < sms && kp_max / MT_BK >= 8 * k.parts) k.parts *= 2;
     CUtensorMap mw[2], mx[2];
     for (int i = 0; i < a.nseg; ++i) {
         const MatSeg& s = a.seg[i];
@@ -339,7 +360,20 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc
     g_mat_tc5_launched[current_device_index()].store(1);
     const dim3 grid((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), block(MT_THREADS);
     const size_t smem = (size_t)(k.stages * k.stage_bytes + 1024);
-#define SP_MT(DUAL, F32) le = launch_pdl(mat_tc5_kernel<DUAL, F32>, grid, block, smem, st, k, mw[0], mx[0], mw[1], mx[1])
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = attr[1].val.clusterDim.y = 1;
+    attr[1].val.clusterDim.z = (unsigned)k.parts;
+    cfg.attrs = attr;
+    cfg.numAttrs = k.parts > 1 ? 2 : 1;
+#define SP_MT(DUAL, F32) le = cudaLaunchKernelEx(&cfg, mat_tc5_kernel<DUAL, F32>, k, mw[0], mx[0], mw[1], mx[1])
     if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
     else { if (a.out_f32) SP_MT(false, true); else SP_MT(false, false); }
 #undef SP_MT

@@ -62,13 +62,7 @@ cudaError_t launch_mat_f32(const MatArgs& a, cudaStream_t st);
 // (at most MAT_GATHER_ROWS rows) every expert multiplies all rows and keeps its own; otherwise the x rows are the sorted
 // rows. max_tiles: upper bound of the row tiles of a grouped launch.
 constexpr int MAT_GATHER_ROWS = 32;
-struct MatScratch {            // owned by whoever owns the stream
-    float* part = nullptr;
-    unsigned* cnt = nullptr;   // zero between launches
-    static constexpr int ITEMS = 4096;
-    static constexpr size_t FLOATS = 8u << 20;
-};
-cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, const MatScratch& sc, cudaStream_t st);
+cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st);
 int mat_tc5_take_timeout();    // as tc5_take_timeout (kernels.h)
 
 // ── the stream between the products ──
