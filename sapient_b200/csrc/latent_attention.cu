@@ -19,11 +19,11 @@ namespace sp {
 cudaError_t count_launch_and_check();  // kernels.cu
 
 // ── rotation, latent norm, cache append ──
-constexpr int LA_THREADS = 128;
+constexpr int LA_WARPS = 4;
 
 template <typename T>
 __device__ __forceinline__ void rotate_pairs(const float* src, T* dst, const float2* cs, int rot, int rot16) {
-    for (int i = threadIdx.x; i < rot16 / 2; i += LA_THREADS) {
+    for (int i = threadIdx.x & 31; i < rot16 / 2; i += 32) {
         float u = 0.f, v = 0.f;
         if (2 * i < rot) {
             const float a = src[2 * i], b = src[2 * i + 1];
@@ -36,40 +36,41 @@ __device__ __forceinline__ void rotate_pairs(const float* src, T* dst, const flo
     }
 }
 
-// Block (token, y): y < heads: that head's query; y == heads: the cache row.
+// A warp per (token, part): parts 0 .. heads - 1 are the heads' queries, part `heads` the cache row.
 template <typename T>
-__global__ void __launch_bounds__(LA_THREADS) latent_append_kernel(const float* __restrict__ proj, int ldp, const LatentShape s, const LatentCache c,
+__global__ void __launch_bounds__(LA_WARPS * 32) latent_append_kernel(const float* __restrict__ proj, int ldp, const LatentShape s, const LatentCache c,
                                                                    const float* __restrict__ norm_gain, float eps, const float2* __restrict__ cos_sin,
                                                                    const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
-                                                                   T* __restrict__ qn, int ldqn, T* __restrict__ qabs, T* __restrict__ qf) {
-    __shared__ float sh[LA_THREADS / 32];
+                                                                   T* __restrict__ qn, int ldqn, T* __restrict__ qabs, T* __restrict__ qf, int parts) {
     pdl_wait();
     pdl_trigger();
-    const int t = blockIdx.x, h = blockIdx.y, pos = tok_pos[t];
+    const int t = blockIdx.x, h = blockIdx.y * LA_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (h >= parts) return;
+    const int pos = tok_pos[t];
     const float2* cs = cos_sin + (int64_t)pos * (s.rot / 2);
     if (h < s.heads) {
         const float* q = proj + (int64_t)t * ldp + (int64_t)h * (s.dim + s.rot);
         if (qn) {
             T* d = qn + ((int64_t)t * s.heads + h) * ldqn;
-            for (int i = threadIdx.x; i < ldqn; i += LA_THREADS) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
+            for (int i = lane; i < ldqn; i += 32) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
             T* r = qabs + ((int64_t)t * s.heads + h) * c.ld;
-            for (int i = c.rank + threadIdx.x; i < c.rank16; i += LA_THREADS) r[i] = from_f32<T>(0.f);
+            for (int i = c.rank + lane; i < c.rank16; i += 32) r[i] = from_f32<T>(0.f);
             rotate_pairs<T>(q + s.dim, r + c.rank16, cs, s.rot, c.rot16);
         } else {
             const int dim16 = (s.dim + 15) & ~15;
             T* d = qf + ((int64_t)t * s.heads + h) * (dim16 + c.rot16);
-            for (int i = threadIdx.x; i < dim16; i += LA_THREADS) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
+            for (int i = lane; i < dim16; i += 32) d[i] = from_f32<T>(i < s.dim ? q[i] : 0.f);
             rotate_pairs<T>(q + s.dim, d + dim16, cs, s.rot, c.rot16);
         }
         return;
     }
     const float* kv = proj + (int64_t)t * ldp + (int64_t)s.heads * (s.dim + s.rot);
     float ss = 0.f;
-    for (int i = threadIdx.x; i < c.rank; i += LA_THREADS) ss = fmaf(kv[i], kv[i], ss);
-    const float r = rsqrtf(block_sum<LA_THREADS / 32>(ss, sh) / (float)c.rank + eps);
+    for (int i = lane; i < c.rank; i += 32) ss = fmaf(kv[i], kv[i], ss);
+    const float r = rsqrtf(warp_sum(ss) / (float)c.rank + eps);
     const int page = c.page_table[(int64_t)tok_slot[t] * c.max_pages + pos / KV_PAGE];
     T* row = reinterpret_cast<T*>(c.pool) + ((int64_t)page * KV_PAGE + pos % KV_PAGE) * c.ld;
-    for (int i = threadIdx.x; i < c.rank16; i += LA_THREADS) row[i] = from_f32<T>(i < c.rank ? kv[i] * r * norm_gain[i] : 0.f);
+    for (int i = lane; i < c.rank16; i += 32) row[i] = from_f32<T>(i < c.rank ? kv[i] * r * norm_gain[i] : 0.f);
     rotate_pairs<T>(kv + c.rank, row + c.rank16, cs, s.rot, c.rot16);
 }
 
@@ -77,11 +78,12 @@ cudaError_t launch_latent_append(const float* proj, int ldp, const LatentShape& 
                                  float eps, const float2* cos_sin, const int32_t* tok_slot, const int32_t* tok_pos, void* qn, int ldqn,
                                  void* qabs, void* qf, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    const dim3 grid(n_tok, s.heads + (own ? 1 : 0));
-    cudaError_t le = f32 ? launch_pdl(latent_append_kernel<float>, grid, dim3(LA_THREADS), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
-                                      tok_pos, (float*)qn, ldqn, (float*)qabs, (float*)qf)
-                         : launch_pdl(latent_append_kernel<bf16>, grid, dim3(LA_THREADS), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
-                                      tok_pos, (bf16*)qn, ldqn, (bf16*)qabs, (bf16*)qf);
+    const int parts = s.heads + (own ? 1 : 0);
+    const dim3 grid(n_tok, (parts + LA_WARPS - 1) / LA_WARPS);
+    cudaError_t le = f32 ? launch_pdl(latent_append_kernel<float>, grid, dim3(LA_WARPS * 32), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
+                                      tok_pos, (float*)qn, ldqn, (float*)qabs, (float*)qf, parts)
+                         : launch_pdl(latent_append_kernel<bf16>, grid, dim3(LA_WARPS * 32), 0, st, proj, ldp, s, c, norm_gain, eps, cos_sin, tok_slot,
+                                      tok_pos, (bf16*)qn, ldqn, (bf16*)qabs, (bf16*)qf, parts);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
@@ -155,55 +157,63 @@ __global__ void __launch_bounds__(LS_WARPS * 32) latent_attention_simple_kernel(
     if (n_splits > 1 && threadIdx.x == 0) { pd[0] = M; pd[1] = L; }
 }
 
-// bf16: block per (HG groups of 16 heads, token, split), 8 warps per group, key tiles of 32 double-buffered with cp.async and
-// shared by the groups. Scores: a warp owns an eighth of the coordinates (its query fragments stay in registers) for all
+// bf16: block per (HG groups of 16 heads, token, split), 8 warps per group, a ring of ST tiles of KEYS keys filled by
+// cp.async and shared by the groups. Scores: a warp owns an eighth of the coordinates (its query fragments stay in registers) for all
 // keys of the tile, the partial sums meet in shared memory; mixture: a warp owns NT 8-column tiles of the latent.
-constexpr int LM_KEYS = 32, LM_WARPS = 8, LM_PLD = LM_KEYS + 8, LM_SLD = LM_KEYS + 1;
-constexpr int LM_ROW_THREADS = LM_WARPS * 2, LM_ROW_KEYS = LM_KEYS / LM_ROW_THREADS;  // of the softmax: threads per query, keys per thread
+constexpr int LM_WARPS = 8, LM_PAGES = 256;
+constexpr int LM_ROW_THREADS = LM_WARPS * 2;  // of the softmax: threads per query
+constexpr int LM_COPY = 3;       // 16-byte pieces of a row per lane: rank + rot up to 640, as
 constexpr int LM_MAX_STEPS = 5;   // 16-coordinate steps per warp: rank + rot up to 640
-static size_t lm_smem(int width, int hg) { return (size_t)2 * LM_KEYS * (width + 8) * 2 + (size_t)hg * LM_WARPS * 16 * LM_SLD * 4; }
+static size_t lm_smem(int width, int hg, int keys, int st) { return (size_t)st * keys * (width + 8) * 2 + (size_t)hg * LM_WARPS * 16 * (keys + 1) * 4; }
 __device__ __forceinline__ void group_sync(int grp) { asm volatile("bar.sync %0, %1;\n" ::"r"(grp + 1), "n"(LM_WARPS * 32) : "memory"); }
 
-template <int NT, int HG>
+template <int NT, int HG, int KEYS, int ST>
 __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
                                                                                   const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
                                                                                   bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
+    constexpr int PLD = KEYS + 8, SLD = KEYS + 1, ROW_KEYS = KEYS / LM_ROW_THREADS;
     extern __shared__ __align__(16) bf16 lm_smem_raw[];
+    __shared__ int pages_s[LM_PAGES];
     __shared__ float corr_s[HG][16], l_s[HG][16], m_s[HG][16];
-    __shared__ __align__(16) bf16 ps_all[HG][16][LM_PLD];
+    __shared__ __align__(16) bf16 ps_all[HG][16][PLD];
     const int width = c.rank16 + c.rot16, LD = width + 8;
     const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
     const int grp = HG > 1 ? wid / LM_WARPS : 0, warp = wid % LM_WARPS, tid = threadIdx.x % (LM_WARPS * 32);
     bf16* ks = lm_smem_raw;
-    float* ss = reinterpret_cast<float*>(ks + 2 * LM_KEYS * LD) + grp * LM_WARPS * 16 * LM_SLD;
-    bf16(*ps)[LM_PLD] = ps_all[grp];
+    float* ss = reinterpret_cast<float*>(ks + ST * KEYS * LD) + grp * LM_WARPS * 16 * SLD;
+    bf16(*ps)[PLD] = ps_all[grp];
     const int h0 = (blockIdx.x * HG + grp) * 16, t = blockIdx.y;
     pdl_wait();
     pdl_trigger();
     int begin, end;
     key_range(tok_pos[t], s.window, blockIdx.z, n_splits, begin, end);
     const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
-    const int pieces = width / 8;
+    const int pieces = width / 8, page0 = begin / KV_PAGE;
+    // the range's page numbers, so that a copy does not wait for its own
+    const bool listed = (end - 1) / KV_PAGE - page0 < LM_PAGES;
+    if (listed)
+        for (int i = threadIdx.x; begin < end && i <= (end - 1) / KV_PAGE - page0; i += LM_WARPS * 32 * HG) pages_s[i] = pt[page0 + i];
+    __syncthreads();
     auto fetch = [&](int k0, int buf) {  // a warp copies every (8 HG)-th key: a row's address is found once
-        bf16* d = ks + buf * LM_KEYS * LD;
-        constexpr int PER = LM_KEYS / (LM_WARPS * HG);
-        const bf16* src[PER];
+        constexpr int PER = KEYS / (LM_WARPS * HG);
+        const uint32_t d0 = smem_addr(ks + (buf * KEYS + wid) * LD + lane * 8);
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
-            const int key = min(k0 + wid + LM_WARPS * HG * i, end - 1);
-            src[i] = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[key / KV_PAGE] * KV_PAGE + key % KV_PAGE) * c.ld;
-        }
+            const int key = k0 + wid + LM_WARPS * HG * i, at = min(key, end - 1), bytes = key < end ? 16 : 0;
+            const int page = listed ? pages_s[at / KV_PAGE - page0] : pt[at / KV_PAGE];
+            const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)page * KV_PAGE + at % KV_PAGE) * c.ld + lane * 8;
+            const uint32_t d = d0 + (uint32_t)(2 * LM_WARPS * HG * i * LD);
 #pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const int r = wid + LM_WARPS * HG * i, bytes = k0 + r < end ? 16 : 0;
-            for (int p = lane; p < pieces; p += 32) cp_async16(d + r * LD + p * 8, src[i] + p * 8, bytes);
+            for (int p = 0; p < LM_COPY; ++p)
+                if (lane + 32 * p < pieces) cp_async16_at(d + 512 * p, src + 256 * p, bytes);
         }
     };
-    // two tiles in flight from the start; a buffer is refilled as soon as everyone is done with it
-    if (begin < end) fetch(begin, 0);
-    cp_async_commit();
-    if (begin + LM_KEYS < end) fetch(begin + LM_KEYS, 1);
-    cp_async_commit();
+    // the ring is full from the start; a stage is refilled as soon as everyone is done with it
+#pragma unroll
+    for (int i = 0; i < ST; ++i) {
+        if (begin + i * KEYS < end) fetch(begin + i * KEYS, i);
+        cp_async_commit();
+    }
     // this warp's coordinates of the 16 queries
     const int steps = width / 16, per = (steps + LM_WARPS - 1) / LM_WARPS, s0 = warp * per, my = max(0, min(per, steps - s0));
     uint32_t qf[LM_MAX_STEPS][4];
@@ -226,45 +236,45 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
     for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m = -INFINITY, l = 0.f;  // of row tid / LM_ROW_THREADS, the same in all its threads
     const int col0 = warp * NT * 8;
-    for (int k0 = begin, buf = 0; k0 < end; k0 += LM_KEYS, buf ^= 1) {
-        cp_async_wait<1>();
+    for (int k0 = begin, buf = 0; k0 < end; k0 += KEYS, buf = buf + 1 == ST ? 0 : buf + 1) {
+        cp_async_wait<ST - 1>();
         __syncthreads();  // this tile has landed for everyone
-        const bf16* kt = ks + buf * LM_KEYS * LD;
+        const bf16* kt = ks + buf * KEYS * LD;
         {
-            float a[4][4];
+            float a[KEYS / 8][4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
+            for (int j = 0; j < KEYS / 8; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
             const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8 + s0 * 16);
 #pragma unroll
             for (int i = 0; i < LM_MAX_STEPS; ++i) {
                 if (i < my) {
-                    uint32_t b0[4], b1[4];
-                    ldsm_x4(b0, ka + 2 * (16 * i));
-                    ldsm_x4(b1, ka + 2 * (16 * LD + 16 * i));
-                    mma_bf16(a[0], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b0[0], b0[1]);
-                    mma_bf16(a[1], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b0[2], b0[3]);
-                    mma_bf16(a[2], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b1[0], b1[1]);
-                    mma_bf16(a[3], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b1[2], b1[3]);
+#pragma unroll
+                    for (int j = 0; j < KEYS / 8; j += 2) {
+                        uint32_t b[4];
+                        ldsm_x4(b, ka + 2 * (8 * j * LD + 16 * i));
+                        mma_bf16(a[j], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[0], b[1]);
+                        mma_bf16(a[j + 1], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[2], b[3]);
+                    }
                 }
             }
-            float* d = ss + (warp * 16 + g) * LM_SLD + 2 * tq;
+            float* d = ss + (warp * 16 + g) * SLD + 2 * tq;
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < KEYS / 8; ++j) {
                 d[8 * j] = a[j][0];
                 d[8 * j + 1] = a[j][1];
-                d[8 * LM_SLD + 8 * j] = a[j][2];
-                d[8 * LM_SLD + 8 * j + 1] = a[j][3];
+                d[8 * SLD + 8 * j] = a[j][2];
+                d[8 * SLD + 8 * j + 1] = a[j][3];
             }
         }
         group_sync(grp);
         {
-            const int r = tid / LM_ROW_THREADS, key = tid % LM_ROW_THREADS * LM_ROW_KEYS;
-            float v[LM_ROW_KEYS], mx = m;
+            const int r = tid / LM_ROW_THREADS, key = tid % LM_ROW_THREADS * ROW_KEYS;
+            float v[ROW_KEYS], mx = m;
 #pragma unroll
-            for (int i = 0; i < LM_ROW_KEYS; ++i) {
+            for (int i = 0; i < ROW_KEYS; ++i) {
                 float z = 0.f;
 #pragma unroll
-                for (int w = 0; w < LM_WARPS; ++w) z += ss[(w * 16 + r) * LM_SLD + key + i];
+                for (int w = 0; w < LM_WARPS; ++w) z += ss[(w * 16 + r) * SLD + key + i];
                 v[i] = k0 + key + i < end ? z * s.scale : -INFINITY;
                 mx = fmaxf(mx, v[i]);
             }
@@ -274,11 +284,11 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
             const float cr = expf(m - mx);
             float sum = 0.f;
 #pragma unroll
-            for (int i = 0; i < LM_ROW_KEYS; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
+            for (int i = 0; i < ROW_KEYS; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
 #pragma unroll
             for (int off = LM_ROW_THREADS / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
-            static_assert(LM_ROW_KEYS == 2, "the softmax weights are stored in pairs");
-            *reinterpret_cast<uint32_t*>(&ps[r][key]) = pack_bf16(v[0], v[1]);
+            if (ROW_KEYS == 2) *reinterpret_cast<uint32_t*>(&ps[r][key]) = pack_bf16(v[0], v[ROW_KEYS - 1]);
+            else ps[r][key] = __float2bfloat16_rn(v[0]);
             l = fmaf(l, cr, sum);
             m = mx;
             if (tid % LM_ROW_THREADS == 0) corr_s[grp][r] = cr;
@@ -288,7 +298,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
 #pragma unroll
         for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
 #pragma unroll
-        for (int kk = 0; kk < LM_KEYS / 16; ++kk) {
+        for (int kk = 0; kk < KEYS / 16; ++kk) {
             uint32_t p[4];
             ldsm_x4(p, smem_addr(&ps[lane & 15][kk * 16 + (lane >> 4) * 8]));
             const uint32_t va = smem_addr(kt + (kk * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
@@ -303,7 +313,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
             }
         }
         __syncthreads();
-        if (k0 + 2 * LM_KEYS < end) fetch(k0 + 2 * LM_KEYS, buf);
+        if (k0 + ST * KEYS < end) fetch(k0 + ST * KEYS, buf);
         cp_async_commit();
     }
     cp_async_wait<0>();
@@ -325,11 +335,17 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
         } else {
             float* d = part + (((int64_t)t * s.heads + h) * n_splits + blockIdx.z) * (c.rank + 2);
             if (warp == 0 && tq == 0) { d[0] = m_s[grp][r]; d[1] = l_s[grp][r]; }
+            d += 2 + col0 + 2 * tq;
+            if (col0 + NT * 8 <= c.rank && c.rank % 2 == 0) {
 #pragma unroll
-            for (int i = 0; i < NT; ++i) {
-                const int e = col0 + i * 8 + 2 * tq;
-                if (e < c.rank) d[2 + e] = o[i][2 * r2];
-                if (e + 1 < c.rank) d[3 + e] = o[i][2 * r2 + 1];
+                for (int i = 0; i < NT; ++i) *reinterpret_cast<float2*>(d + 8 * i) = make_float2(o[i][2 * r2], o[i][2 * r2 + 1]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < NT; ++i) {
+                    const int e = col0 + i * 8 + 2 * tq;
+                    if (e < c.rank) d[8 * i] = o[i][2 * r2];
+                    if (e + 1 < c.rank) d[8 * i + 1] = o[i][2 * r2 + 1];
+                }
             }
         }
     }
@@ -372,9 +388,9 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
     constexpr int CAP = 200 * 1024;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
-        const void* fns[] = {(const void*)latent_attention_mma_kernel<2, 1>, (const void*)latent_attention_mma_kernel<4, 1>, (const void*)latent_attention_mma_kernel<8, 1>,
-                             (const void*)latent_attention_mma_kernel<2, 2>, (const void*)latent_attention_mma_kernel<4, 2>,
-                             (const void*)latent_attention_mma_kernel<8, 2>,
+        const void* fns[] = {(const void*)latent_attention_mma_kernel<2, 1, 32, 2>, (const void*)latent_attention_mma_kernel<4, 1, 32, 2>,
+                             (const void*)latent_attention_mma_kernel<8, 1, 32, 2>, (const void*)latent_attention_mma_kernel<2, 2, 32, 4>,
+                             (const void*)latent_attention_mma_kernel<4, 2, 32, 4>, (const void*)latent_attention_mma_kernel<8, 2, 32, 4>,
                              (const void*)latent_attention_simple_kernel<float>, (const void*)latent_attention_simple_kernel<bf16>};
         for (const void* f : fns) {
             const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
@@ -386,12 +402,13 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
     const int width = c.rank16 + c.rot16;
     const int per_warp = (c.rank16 + 8 * LM_WARPS - 1) / (8 * LM_WARPS);  // 8-column tiles each warp has to cover
     const int hg = s.heads > 16 ? 2 : 1;
-    const size_t smem = lm_smem(width, hg);
+    // one head group: two blocks per SM; two groups: one block of 16 warps and a deeper ring
+    const size_t smem = lm_smem(width, hg, 32, hg == 1 ? 2 : 4);
     if (!f32 && per_warp <= 8 && width <= 16 * LM_WARPS * LM_MAX_STEPS && smem <= CAP) {
         const dim3 grid((s.heads + 16 * hg - 1) / (16 * hg), n_tok, n_splits), block(LM_WARPS * 32 * hg);
 #define SP_LM(NT)                                                                                                                                  \
-    le = hg == 1 ? launch_pdl(latent_attention_mma_kernel<NT, 1>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits) \
-                 : launch_pdl(latent_attention_mma_kernel<NT, 2>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
+    le = hg == 1 ? launch_pdl(latent_attention_mma_kernel<NT, 1, 32, 2>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits) \
+                 : launch_pdl(latent_attention_mma_kernel<NT, 2, 32, 4>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
         if (per_warp <= 2) SP_LM(2);
         else if (per_warp <= 4) SP_LM(4);
         else SP_LM(8);

@@ -75,7 +75,10 @@ def design_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
     keys = _pairs(rows, s["window"]) if prefill else rows * min(ctx, s["window"])
     per_pair = 2 * H * (D + R + V) if prefill else 2 * H * (K + R + K)
     return {"gemv": (2 * (dense + active * used + head), 2 * rows * (dense + active * s["top"]) + 2 * head * (1 if prefill else rows)),
-            "attention": (L * 2 * (K + R) * (rows if prefill else keys), L * per_pair * keys)}
+            "attention": (L * 2 * (K + R) * (rows if prefill else keys), L * per_pair * keys),
+            # residual + norm after the mixer; mixture, norm, residual and depth average (all results so far) after the experts
+            "norm": (rows * W * sum(14 + 4 * s["top"] + 18 + 4 * (i + 1) for i in range(L)), 0),
+            "rope_kv": (rows * 6 * (L * H * (D + R) + own * (K + R)), 0)}
 
 
 def llama_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
@@ -85,7 +88,8 @@ def llama_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
     head = c["vocab"] * c["hidden"]
     keys = _pairs(rows, 1 << 30) if prefill else rows * ctx
     return {"gemv": (34 / 32 * (mats + head), 2 * rows * mats + 2 * head * (1 if prefill else rows)),
-            "attention": (c["n_layers"] * 2 * 2 * q * (rows if prefill else keys), c["n_layers"] * 4 * q * keys)}
+            "attention": (c["n_layers"] * 2 * 2 * q * (rows if prefill else keys), c["n_layers"] * 4 * q * keys),
+            "norm": (rows * c["hidden"] * c["n_layers"] * 2 * 8, 0), "rope_kv": (rows * c["n_layers"] * q * (12 + 4 + 4), 0)}
 
 
 def _families(ms: dict, work: dict, peaks: dict) -> dict:
