@@ -431,8 +431,7 @@ int Engine::plan_experts(int li, int T) {
     const MoeSpec& s = p.plan.layers[(size_t)li].mlp;
     const int W = p.plan.width, E = s.experts, pairs = T * s.top;
     SP_TRY(plan_mat(l.router, p.xb, p.wp, T, p.logit, l.router.n, true));
-    SP_LAUNCH(F_ELEM, launch_moe_topk(p.logit, l.router.n, l.router_b, T, E, s.top, p.pick, p.weight, stream));
-    SP_LAUNCH(F_ELEM, launch_moe_group(p.pick, T, E, s.top, p.moe, stream));
+    SP_LAUNCH(F_ELEM, launch_moe_route(p.logit, l.router.n, l.router_b, T, E, s.top, p.pick, p.weight, p.moe, stream));
     MatArgs a{};
     a.f32 = p.f32;
     a.m = T;

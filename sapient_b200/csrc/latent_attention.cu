@@ -164,14 +164,15 @@ constexpr int LM_WARPS = 8, LM_PAGES = 256;
 constexpr int LM_ROW_THREADS = LM_WARPS * 2;  // of the softmax: threads per query
 constexpr int LM_COPY = 3;       // 16-byte pieces of a row per lane: rank + rot up to 640, as
 constexpr int LM_MAX_STEPS = 5;   // 16-coordinate steps per warp: rank + rot up to 640
-static size_t lm_smem(int width, int hg, int keys, int st) { return (size_t)st * keys * (width + 8) * 2 + (size_t)hg * LM_WARPS * 16 * (keys + 1) * 4; }
+static size_t lm_smem(int width, int hg, int keys, int st) { return (size_t)st * keys * (width + 8) * 2 + (size_t)hg * LM_WARPS * 16 * (keys + 8) * 4; }
 __device__ __forceinline__ void group_sync(int grp) { asm volatile("bar.sync %0, %1;\n" ::"r"(grp + 1), "n"(LM_WARPS * 32) : "memory"); }
 
 template <int NT, int HG, int KEYS, int ST>
 __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
                                                                                   const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
                                                                                   bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
-    constexpr int PLD = KEYS + 8, SLD = KEYS + 1, ROW_KEYS = KEYS / LM_ROW_THREADS;
+    constexpr int PLD = KEYS + 8, SLD = KEYS + 8;
+    static_assert(KEYS == 2 * LM_ROW_THREADS, "the softmax gives every thread two keys");
     extern __shared__ __align__(16) bf16 lm_smem_raw[];
     __shared__ int pages_s[LM_PAGES];
     __shared__ float corr_s[HG][16], l_s[HG][16], m_s[HG][16];
@@ -260,22 +261,23 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
             float* d = ss + (warp * 16 + g) * SLD + 2 * tq;
 #pragma unroll
             for (int j = 0; j < KEYS / 8; ++j) {
-                d[8 * j] = a[j][0];
-                d[8 * j + 1] = a[j][1];
-                d[8 * SLD + 8 * j] = a[j][2];
-                d[8 * SLD + 8 * j + 1] = a[j][3];
+                *reinterpret_cast<float2*>(d + 8 * j) = make_float2(a[j][0], a[j][1]);  // rows 40 floats apart: no bank conflicts in pairs
+                *reinterpret_cast<float2*>(d + 8 * SLD + 8 * j) = make_float2(a[j][2], a[j][3]);
             }
         }
         group_sync(grp);
         {
-            const int r = tid / LM_ROW_THREADS, key = tid % LM_ROW_THREADS * ROW_KEYS;
-            float v[ROW_KEYS], mx = m;
+            const int r = tid / LM_ROW_THREADS, key = tid % LM_ROW_THREADS * 2;
+            float v[2] = {0.f, 0.f}, mx = m;
 #pragma unroll
-            for (int i = 0; i < ROW_KEYS; ++i) {
-                float z = 0.f;
+            for (int w = 0; w < LM_WARPS; ++w) {
+                const float2 z = *reinterpret_cast<const float2*>(ss + (w * 16 + r) * SLD + key);
+                v[0] += z.x;
+                v[1] += z.y;
+            }
 #pragma unroll
-                for (int w = 0; w < LM_WARPS; ++w) z += ss[(w * 16 + r) * SLD + key + i];
-                v[i] = k0 + key + i < end ? z * s.scale : -INFINITY;
+            for (int i = 0; i < 2; ++i) {
+                v[i] = k0 + key + i < end ? v[i] * s.scale : -INFINITY;
                 mx = fmaxf(mx, v[i]);
             }
 #pragma unroll
@@ -284,11 +286,10 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
             const float cr = expf(m - mx);
             float sum = 0.f;
 #pragma unroll
-            for (int i = 0; i < ROW_KEYS; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
+            for (int i = 0; i < 2; ++i) { v[i] = expf(v[i] - mx); sum += v[i]; }
 #pragma unroll
             for (int off = LM_ROW_THREADS / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
-            if (ROW_KEYS == 2) *reinterpret_cast<uint32_t*>(&ps[r][key]) = pack_bf16(v[0], v[ROW_KEYS - 1]);
-            else ps[r][key] = __float2bfloat16_rn(v[0]);
+            *reinterpret_cast<uint32_t*>(&ps[r][key]) = pack_bf16(v[0], v[1]);
             l = fmaf(l, cr, sum);
             m = mx;
             if (tid % LM_ROW_THREADS == 0) corr_s[grp][r] = cr;

@@ -28,7 +28,7 @@ struct MatSeg {
     int64_t ygs;
 };
 
-// Rows of a step sorted by expert, made on the device by launch_moe_group.
+// Rows of a step sorted by expert, made on the device by launch_moe_route.
 struct MoeRows {
     const int32_t* row_off;    // [experts + 1] first sorted row of each expert
     const int32_t* row_src;    // token of each sorted row
@@ -100,14 +100,14 @@ cudaError_t launch_final_norm(const float* x, const int32_t* rows, int n_rows, i
                               cudaStream_t st);
 
 // ── experts ──
-// Per token the `top` largest of logits[t][0..experts) + bias (ties: the lower index), softmax over the chosen ones.
-cudaError_t launch_moe_topk(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
-                            cudaStream_t st);
-// Sorts the (token, choice) pairs by expert: MoeRows tables and slot_of[t][k] = sorted row of a pair.
+// Per token the `top` largest of logits[t][0..experts) + bias (ties: the lower index) with the softmax over the chosen ones
+// as weight[t][top], and the (token, choice) pairs sorted by expert: MoeRows tables and slot_of[t][k] = sorted row of a
+// pair. pick[t][top] is scratch.
 struct MoeTables {
     int32_t *row_off, *row_src, *active, *n_active, *tile_group, *tile_row, *n_tiles, *slot_of;
 };
-cudaError_t launch_moe_group(const int32_t* pick, int n_tok, int experts, int top, const MoeTables& t, cudaStream_t st);
+cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
+                             const MoeTables& t, cudaStream_t st);
 // dst[i] = src[row_src[i]] for n rows of ld elements of the compute type (ld * element size a multiple of 16).
 cudaError_t launch_gather_act(const void* src, const int32_t* row_src, int n, int ld, bool f32, void* dst, cudaStream_t st);
 

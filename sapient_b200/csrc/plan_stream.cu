@@ -224,17 +224,11 @@ cudaError_t launch_final_norm(const float* x, const int32_t* rows, int n_rows, i
 }
 
 // ── experts ──
-// One warp per token; the logits wait in shared memory and a chosen one is struck out.
-constexpr int TK_WARPS = 4;
-__global__ void __launch_bounds__(TK_WARPS * 32) moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok,
-                                                                 int experts, int top, int32_t* __restrict__ pick, float* __restrict__ weight) {
-    extern __shared__ float tk_smem[];
-    pdl_wait();
-    pdl_trigger();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * TK_WARPS + warp;
-    if (t >= n_tok) return;
-    float* z = tk_smem + warp * experts;
-    for (int e = lane; e < experts; e += 32) z[e] = logits[(int64_t)t * ld + e] + (bias ? bias[e] : 0.f);
+// One warp's choice for token t: its logits wait in shared memory (z, `experts` floats) and a chosen one is struck out.
+__device__ __forceinline__ void choose_experts(const float* __restrict__ logits, const float* __restrict__ bias, int experts, int top, float* z,
+                                               int32_t* pick, float* weight) {
+    const int lane = threadIdx.x & 31;
+    for (int e = lane; e < experts; e += 32) z[e] = logits[e] + (bias ? bias[e] : 0.f);
     __syncwarp();
     float best0 = 0.f, sum = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -253,33 +247,30 @@ __global__ void __launch_bounds__(TK_WARPS * 32) moe_topk_kernel(const float* __
         const float ex = expf(v - best0);
         sum += ex;
         if (lane == 0) {
-            pick[(int64_t)t * top + k] = at;
-            weight[(int64_t)t * top + k] = ex;
+            pick[k] = at;
+            weight[k] = ex;
             z[at] = -INFINITY;
         }
         __syncwarp();
     }
-    for (int k = lane; k < top; k += 32) weight[(int64_t)t * top + k] /= sum;
+    for (int k = lane; k < top; k += 32) weight[k] /= sum;
 }
 
-cudaError_t launch_moe_topk(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
-                            cudaStream_t st) {
-    if (n_tok == 0) return cudaSuccess;
-    const size_t smem = (size_t)TK_WARPS * experts * 4;
-    if (smem > 48 * 1024) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(moe_topk_kernel, dim3((n_tok + TK_WARPS - 1) / TK_WARPS), dim3(TK_WARPS * 32), smem, st, logits, ld, bias, n_tok, experts,
-                                top, pick, weight);
-    if (le != cudaSuccess) return le;
-    return count_launch_and_check();
+constexpr int TK_WARPS = 4;
+__global__ void __launch_bounds__(TK_WARPS * 32) moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok,
+                                                                 int experts, int top, int32_t* __restrict__ pick, float* __restrict__ weight) {
+    extern __shared__ float tk_smem[];
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, t = blockIdx.x * TK_WARPS + warp;
+    if (t >= n_tok) return;
+    choose_experts(logits + (int64_t)t * ld, bias, experts, top, tk_smem + warp * experts, pick + (int64_t)t * top, weight + (int64_t)t * top);
 }
 
 // One block: counts per expert, prefix sums, the tables. Within an expert the rows come in no particular order (every row
 // is computed by itself and found again through slot_of).
-__global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restrict__ pick, int n_pairs, int experts, int top, const MoeTables t) {
-    extern __shared__ int mg_smem[];
+__device__ __forceinline__ void group_rows(const int32_t* pick, int n_pairs, int experts, int top, const MoeTables& t, int* mg_smem) {
     int *cnt = mg_smem, *off = mg_smem + experts;
-    pdl_wait();
-    pdl_trigger();
     for (int e = threadIdx.x; e < experts; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
     for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&cnt[pick[i]], 1);
@@ -325,13 +316,44 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
     }
 }
 
-cudaError_t launch_moe_group(const int32_t* pick, int n_tok, int experts, int top, const MoeTables& t, cudaStream_t st) {
+__global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restrict__ pick, int n_pairs, int experts, int top, const MoeTables t) {
+    extern __shared__ int mg_smem[];
+    pdl_wait();
+    pdl_trigger();
+    group_rows(pick, n_pairs, experts, top, t, mg_smem);
+}
+
+// Choice and grouping of up to 8 tokens in one block, a warp per token.
+__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok, int experts,
+                                                         int top, float* __restrict__ weight, const MoeTables t) {
+    extern __shared__ int mr_smem[];  // counts and offsets, the choices, a row of logits per warp
+    pdl_wait();
+    pdl_trigger();
+    int* pick = mr_smem + 2 * experts;
+    float* z = reinterpret_cast<float*>(pick + n_tok * top);
+    const int warp = threadIdx.x >> 5;
+    if (warp < n_tok) choose_experts(logits + (int64_t)warp * ld, bias, experts, top, z + warp * experts, pick + warp * top, weight + (int64_t)warp * top);
+    __syncthreads();
+    group_rows(pick, n_tok * top, experts, top, t, mr_smem);
+}
+
+cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
+                             const MoeTables& t, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    const size_t smem = (size_t)experts * 8;
-    if (smem > 48 * 1024) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(moe_group_kernel, dim3(1), dim3(n_tok * top > 256 ? 1024 : 256), smem, st, pick, n_tok * top, experts, top, t);
+    constexpr size_t CAP = 48 * 1024;
+    const size_t small = ((size_t)(2 + n_tok) * experts + (size_t)n_tok * top) * 4;
+    if (n_tok <= 8 && small <= CAP) {
+        const cudaError_t le = launch_pdl(moe_route_kernel, dim3(1), dim3(256), small, st, logits, ld, bias, n_tok, experts, top, weight, t);
+        return le != cudaSuccess ? le : count_launch_and_check();
+    }
+    const size_t rows = (size_t)TK_WARPS * experts * 4, counts = (size_t)experts * 8;
+    if (rows > CAP || counts > CAP) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(moe_topk_kernel, dim3((n_tok + TK_WARPS - 1) / TK_WARPS), dim3(TK_WARPS * 32), rows, st, logits, ld, bias, n_tok, experts, top,
+                                pick, weight);
+    if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
-    return count_launch_and_check();
+    le = launch_pdl(moe_group_kernel, dim3(1), dim3(1024), counts, st, (const int32_t*)pick, n_tok * top, experts, top, t);
+    return le != cudaSuccess ? le : count_launch_and_check();
 }
 
 __global__ void gather_act_kernel(const uint4* __restrict__ src, const int32_t* __restrict__ row_src, int ld16, uint4* __restrict__ dst) {
