@@ -14,7 +14,6 @@
 #include <map>
 
 #include "engine.h"
-#include "pdl.cuh"
 #include "plan_common.cuh"
 #include "sp_common.cuh"
 
@@ -343,10 +342,8 @@ int Engine::plan_ctx_bucket() const {
 
 static int plan_splits(const PlanLayer& l, bool f32, int bucket, int T) {
     if (T > PLAN_ROWS) return 1;
-    const int keys = std::min(1 << bucket, l.shape.window), blocks = (f32 ? l.shape.heads : (l.shape.heads + 31) / 32) * T;
-    const int slots = (f32 || l.shape.heads <= 16 ? 2 : 1) * device_sm_count();  // blocks the device holds at once
-    int s = 1;
-    while (s < 16 && blocks * 2 * s <= slots && keys >= 64 * 2 * s && T * 2 * s <= PLAN_SPLIT_ROWS) s <<= 1;
+    int s = latent_attention_splits(l.shape.heads, T, std::min(1 << bucket, l.shape.window), f32);
+    while (s > 1 && T * s > PLAN_SPLIT_ROWS) s >>= 1;
     return s;
 }
 

@@ -160,7 +160,7 @@ __global__ void __launch_bounds__(LS_WARPS * 32) latent_attention_simple_kernel(
 // bf16: block per (HG groups of 16 heads, token, split), 8 warps per group, a ring of ST tiles of KEYS keys filled by
 // cp.async and shared by the groups. Scores: a warp owns an eighth of the coordinates (its query fragments stay in registers) for all
 // keys of the tile, the partial sums meet in shared memory; mixture: a warp owns NT 8-column tiles of the latent.
-constexpr int LM_WARPS = 8, LM_PAGES = 256;
+constexpr int LM_WARPS = 8, LM_PAGES = 256, LM_MAX_SPLITS = 16;  // splits are blocks of a cluster
 constexpr int LM_ROW_THREADS = LM_WARPS * 2;  // of the softmax: threads per query
 constexpr int LM_COPY = 3;       // 16-byte pieces of a row per lane: rank + rot up to 640, as
 constexpr int LM_MAX_STEPS = 5;   // 16-coordinate steps per warp: rank + rot up to 640
@@ -170,12 +170,12 @@ __device__ __forceinline__ void group_sync(int grp) { asm volatile("bar.sync %0,
 template <int NT, int HG, int KEYS, int ST>
 __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kernel(const bf16* __restrict__ qabs, const LatentShape s, const LatentCache c,
                                                                                   const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
-                                                                                  bf16* __restrict__ out, int ldo, float* __restrict__ part, int n_splits) {
+                                                                                  bf16* __restrict__ out, int ldo, int n_splits) {
     constexpr int PLD = KEYS + 8, SLD = KEYS + 8;
     static_assert(KEYS == 2 * LM_ROW_THREADS, "the softmax gives every thread two keys");
     extern __shared__ __align__(16) bf16 lm_smem_raw[];
     __shared__ int pages_s[LM_PAGES];
-    __shared__ float corr_s[HG][16], l_s[HG][16], m_s[HG][16];
+    __shared__ float corr_s[HG][16], l_s[HG][16], m_s[HG][16], share_s[HG * 16][LM_MAX_SPLITS];
     __shared__ __align__(16) bf16 ps_all[HG][16][PLD];
     const int width = c.rank16 + c.rot16, LD = width + 8;
     const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
@@ -319,37 +319,73 @@ __global__ void __launch_bounds__(LM_WARPS * 32 * HG) latent_attention_mma_kerne
     }
     cp_async_wait<0>();
     if (tid % LM_ROW_THREADS == 0) { l_s[grp][tid / LM_ROW_THREADS] = l; m_s[grp][tid / LM_ROW_THREADS] = m; }
-    group_sync(grp);
+    if (n_splits == 1) {
+        group_sync(grp);
 #pragma unroll
-    for (int r2 = 0; r2 < 2; ++r2) {
-        const int r = g + 8 * r2, h = h0 + r;
-        if (h >= s.heads) continue;
-        if (n_splits == 1) {
+        for (int r2 = 0; r2 < 2; ++r2) {
+            const int r = g + 8 * r2, h = h0 + r;
+            if (h >= s.heads) continue;
             const float inv = 1.0f / l_s[grp][r];
-            bf16* d = out + ((int64_t)t * s.heads + h) * ldo;
+            bf16* d = out + ((int64_t)t * s.heads + h) * ldo + col0 + 2 * tq;
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
                 const int e = col0 + i * 8 + 2 * tq;
-                if (e < c.rank) d[e] = __float2bfloat16_rn(o[i][2 * r2] * inv);
-                if (e + 1 < c.rank) d[e + 1] = __float2bfloat16_rn(o[i][2 * r2 + 1] * inv);
-            }
-        } else {
-            float* d = part + (((int64_t)t * s.heads + h) * n_splits + blockIdx.z) * (c.rank + 2);
-            if (warp == 0 && tq == 0) { d[0] = m_s[grp][r]; d[1] = l_s[grp][r]; }
-            d += 2 + col0 + 2 * tq;
-            if (col0 + NT * 8 <= c.rank && c.rank % 2 == 0) {
-#pragma unroll
-                for (int i = 0; i < NT; ++i) *reinterpret_cast<float2*>(d + 8 * i) = make_float2(o[i][2 * r2], o[i][2 * r2 + 1]);
-            } else {
-#pragma unroll
-                for (int i = 0; i < NT; ++i) {
-                    const int e = col0 + i * 8 + 2 * tq;
-                    if (e < c.rank) d[8 * i] = o[i][2 * r2];
-                    if (e + 1 < c.rank) d[8 * i + 1] = o[i][2 * r2 + 1];
-                }
+                if (e + 1 < c.rank) *reinterpret_cast<uint32_t*>(d + 8 * i) = pack_bf16(o[i][2 * r2] * inv, o[i][2 * r2 + 1] * inv);
+                else if (e < c.rank) d[8 * i] = __float2bfloat16_rn(o[i][2 * r2] * inv);
             }
         }
+        return;
     }
+    // The splits are the blocks of a cluster: each leaves its mixtures (relative to its own maxima) where the key ring was
+    // and adds up a share of the columns of all of them, in split order.
+    __syncthreads();
+    const int LDO = c.rank16 + 8;
+    float* mix = reinterpret_cast<float*>(lm_smem_raw);  // [HG * 16][LDO]
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        if (col0 + i * 8 < c.rank16) {
+            float* d = mix + (grp * 16 + g) * LDO + col0 + i * 8 + 2 * tq;
+            *reinterpret_cast<float2*>(d) = make_float2(o[i][0], o[i][1]);
+            *reinterpret_cast<float2*>(d + 8 * LDO) = make_float2(o[i][2], o[i][3]);
+        }
+    }
+    cluster_sync();
+    {
+        // a thread per (head, split)
+        static_assert(LM_WARPS * 32 == 16 * LM_MAX_SPLITS, "16 heads x 16 splits per group");
+        const int hh = threadIdx.x / LM_MAX_SPLITS, p = threadIdx.x % LM_MAX_SPLITS;
+        const bool on = p < n_splits;
+        const float mp = on ? ld_peer(peer_smem(smem_addr(&m_s[0][0] + hh), p)) : -INFINITY, lp = on ? ld_peer(peer_smem(smem_addr(&l_s[0][0] + hh), p)) : 0.f;
+        float M = mp;
+#pragma unroll
+        for (int off = LM_MAX_SPLITS / 2; off > 0; off >>= 1) M = fmaxf(M, __shfl_xor_sync(0xFFFFFFFFu, M, off));
+        const float f = mp == -INFINITY ? 0.f : expf(mp - M);
+        float L = f * lp;
+#pragma unroll
+        for (int off = LM_MAX_SPLITS / 2; off > 0; off >>= 1) L += __shfl_xor_sync(0xFFFFFFFFu, L, off);
+        share_s[hh][p] = f / L;
+    }
+    __syncthreads();
+    const int pairs = (c.rank + 1) / 2, rows = min(HG * 16, s.heads - (int)blockIdx.x * HG * 16);
+    for (int idx = blockIdx.z * blockDim.x + threadIdx.x; idx < rows * pairs; idx += n_splits * blockDim.x) {
+        const int r = idx / pairs, e = 2 * (idx - r * pairs);
+        const uint32_t at = smem_addr(mix + r * LDO + e);
+        float x = 0.f, y = 0.f;
+        for (int p0 = 0; p0 < n_splits; p0 += 4) {  // n_splits is a power of two
+            float2 v[4];
+#pragma unroll
+            for (int p = 0; p < 4; ++p) v[p] = p0 + p < n_splits ? ld_peer2(peer_smem(at, p0 + p)) : make_float2(0.f, 0.f);
+#pragma unroll
+            for (int p = 0; p < 4; ++p) {
+                x = fmaf(share_s[r][p0 + p], v[p].x, x);
+                y = fmaf(share_s[r][p0 + p], v[p].y, y);
+            }
+        }
+        bf16* d = out + ((int64_t)t * s.heads + blockIdx.x * HG * 16 + r) * ldo + e;
+        if (e + 1 < c.rank) *reinterpret_cast<uint32_t*>(d) = pack_bf16(x, y);
+        else d[0] = __float2bfloat16_rn(x);
+    }
+    cluster_sync();  // nobody leaves while its mixtures are being read
 }
 
 // Block (head, token, 128 columns).
@@ -380,6 +416,19 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
     if (e < rank) out[th * ldo + e] = from_f32<T>(o);
 }
 
+// Two head groups share a block's keys once there are tokens enough to fill the device without splitting the heads up.
+static int latent_head_groups(int heads, int n_tok) { return heads > 16 && n_tok >= 8 ? 2 : 1; }
+
+int latent_attention_splits(int heads, int n_tok, int keys, bool f32) {
+    const int hg = f32 ? 1 : latent_head_groups(heads, n_tok);
+    const int blocks = (f32 ? heads : (heads + 16 * hg - 1) / (16 * hg)) * n_tok;
+    const int slots = (hg == 1 ? 2 : 1) * device_sm_count();  // blocks the device holds at once
+    const int most = hg == 1 ? LM_MAX_SPLITS : 8;             // (a cluster of 16 needs the small blocks)
+    int n = 1;
+    while (n < most && blocks * 2 * n <= slots && keys >= 64 * 2 * n) n <<= 1;
+    return n;
+}
+
 size_t latent_part_floats(int n_tok, int heads, int n_splits, int rank) { return n_splits > 1 ? (size_t)n_tok * heads * n_splits * (rank + 2) : 0; }
 
 cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, const LatentCache& c, const int32_t* tok_slot, const int32_t* tok_pos,
@@ -397,23 +446,30 @@ cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, cons
             const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
             if (e != cudaSuccess) return e;
         }
+        const void* wide[] = {(const void*)latent_attention_mma_kernel<2, 1, 32, 2>, (const void*)latent_attention_mma_kernel<4, 1, 32, 2>,
+                              (const void*)latent_attention_mma_kernel<8, 1, 32, 2>};
+        for (const void* f : wide) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+            if (e != cudaSuccess) return e;
+        }
         return cudaSuccess;
     });
     if (le != cudaSuccess) return le;
     const int width = c.rank16 + c.rot16;
     const int per_warp = (c.rank16 + 8 * LM_WARPS - 1) / (8 * LM_WARPS);  // 8-column tiles each warp has to cover
-    const int hg = s.heads > 16 ? 2 : 1;
+    const int hg = latent_head_groups(s.heads, n_tok);
     // one head group: two blocks per SM; two groups: one block of 16 warps and a deeper ring
     const size_t smem = lm_smem(width, hg, 32, hg == 1 ? 2 : 4);
-    if (!f32 && per_warp <= 8 && width <= 16 * LM_WARPS * LM_MAX_STEPS && smem <= CAP) {
+    if (!f32 && per_warp <= 8 && width <= 16 * LM_WARPS * LM_MAX_STEPS && smem <= CAP && n_splits <= (hg == 1 ? LM_MAX_SPLITS : 8)) {
         const dim3 grid((s.heads + 16 * hg - 1) / (16 * hg), n_tok, n_splits), block(LM_WARPS * 32 * hg);
 #define SP_LM(NT)                                                                                                                                  \
-    le = hg == 1 ? launch_pdl(latent_attention_mma_kernel<NT, 1, 32, 2>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits) \
-                 : launch_pdl(latent_attention_mma_kernel<NT, 2, 32, 4>, grid, block, smem, st, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, part, n_splits)
+    le = hg == 1 ? launch_pdl_cluster(latent_attention_mma_kernel<NT, 1, 32, 2>, grid, block, smem, st, n_splits, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, n_splits) \
+                 : launch_pdl_cluster(latent_attention_mma_kernel<NT, 2, 32, 4>, grid, block, smem, st, n_splits, (const bf16*)qabs, s, c, tok_slot, tok_pos, (bf16*)o, ldo, n_splits)
         if (per_warp <= 2) SP_LM(2);
         else if (per_warp <= 4) SP_LM(4);
         else SP_LM(8);
 #undef SP_LM
+        return le != cudaSuccess ? le : count_launch_and_check();
     } else {
         const dim3 grid(s.heads, n_tok, n_splits), block(LS_WARPS * 32);
         const size_t smem = (size_t)(width + LS_WARPS * c.rank) * 4;

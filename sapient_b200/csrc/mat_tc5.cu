@@ -37,21 +37,6 @@ constexpr int MT_MAX_PARTS = 8;
 
 __device__ int g_mat_tc5_timeout = 0;
 
-// A barrier of all threads of the cluster; shared-memory writes before it are visible to the peers after it.
-__device__ __forceinline__ void cluster_sync() {
-    asm volatile("barrier.cluster.arrive.release;\nbarrier.cluster.wait.acquire;\n" ::: "memory");
-}
-__device__ __forceinline__ uint32_t peer_smem(uint32_t addr, int rank) {
-    uint32_t r;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(r) : "r"(addr), "r"(rank));
-    return r;
-}
-__device__ __forceinline__ float ld_peer(uint32_t addr) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(addr) : "memory");
-    return v;
-}
-
 struct MatTc5Seg {
     void* y;
     int64_t ygs;
@@ -360,20 +345,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     g_mat_tc5_launched[current_device_index()].store(1);
     const dim3 grid((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), block(MT_THREADS);
     const size_t smem = (size_t)(k.stages * k.stage_bytes + 1024);
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = st;
-    cudaLaunchAttribute attr[2];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
-    attr[1].id = cudaLaunchAttributeClusterDimension;
-    attr[1].val.clusterDim.x = attr[1].val.clusterDim.y = 1;
-    attr[1].val.clusterDim.z = (unsigned)k.parts;
-    cfg.attrs = attr;
-    cfg.numAttrs = k.parts > 1 ? 2 : 1;
-#define SP_MT(DUAL, F32) le = cudaLaunchKernelEx(&cfg, mat_tc5_kernel<DUAL, F32>, k, mw[0], mx[0], mw[1], mx[1])
+#define SP_MT(DUAL, F32) le = launch_pdl_cluster(mat_tc5_kernel<DUAL, F32>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1])
     if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
     else { if (a.out_f32) SP_MT(false, true); else SP_MT(false, false); }
 #undef SP_MT

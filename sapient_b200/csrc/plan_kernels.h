@@ -133,8 +133,10 @@ cudaError_t launch_latent_append(const float* proj, int ldp, const LatentShape& 
                                  float eps, const float2* cos_sin, const int32_t* tok_slot, const int32_t* tok_pos, void* qn, int ldqn,
                                  void* qabs, void* qf, bool f32, int n_tok, cudaStream_t st);
 // Absorbed attention: scores and values straight from the latent rows. o[t][heads][ldo] (compute type) = normalised
-// mixture of latents; n_splits > 1 splits the keys over blocks through `part`
+// mixture of latents. n_splits > 1 splits the keys over blocks (latent_attention_splits of the longest range to visit, or
+// fewer): bf16 over a cluster, f32 and ranks beyond the tensor-core kernel through `part`
 // (latent_part_floats(n_tok, heads, splits, rank) floats).
+int latent_attention_splits(int heads, int n_tok, int keys, bool f32);
 size_t latent_part_floats(int n_tok, int heads, int n_splits, int rank);
 cudaError_t launch_latent_attention(const void* qabs, const LatentShape& s, const LatentCache& c, const int32_t* tok_slot, const int32_t* tok_pos,
                                     void* o, int ldo, float* part, int n_splits, bool f32, int n_tok, cudaStream_t st);
