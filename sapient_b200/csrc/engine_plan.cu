@@ -1,9 +1,10 @@
 // Plan-driven models (model_plan.h) on the resident engine: weights packed once into the shapes the kernels read, a paged
 // latent cache behind the same page pool, and the launch sequence of a step.
 //
-// A layer is ten to twelve launches whatever the row count: projections, rotation + cache append, [absorb,] attention
-// [, merge, value maps], output projection, norm + residual, router, choice, grouping, gate|up of the chosen and the
-// shared expert, down, mixture + norm + residual + depth average. bf16 products run on the tcgen05 kernel (mat_tc5.cu) at
+// A layer is ten to fifteen launches: projections, rotation + cache append, then either queries to latent space, absorbed
+// attention and value maps or gather, rebuilt keys and values and expanded attention; output projection, norm + residual,
+// router, choice and grouping, gate|up of the chosen and the shared expert, down, mixture + norm + residual + depth
+// average. bf16 products run on the tcgen05 kernel (mat_tc5.cu) at
 // every row count, f32 ones on mat_f32.cu. Steps of up to PLAN_ROWS rows take the absorbed attention and can be captured as
 // a graph; longer ones, where rebuilding the keys pays, the expanded attention.
 #include "engine_plan.h"
