@@ -65,12 +65,13 @@ Engine::Engine(const SpModelDesc& desc, const ModelPlan& plan, bool f32) : Engin
     r.vocab = plan.vocab;
     r.norm_eps = plan.eps;
     // informative only: a plan's layers have sizes of their own
-    r.n_heads = plan.layers[0].mix.heads;
-    r.n_kv_heads = 1;
-    r.head_dim = plan.layers[0].mix.dim + plan.layers[0].mix.rot_dim;
-    r.rotary_dim = plan.layers[0].mix.rot_dim;
-    r.rope_theta = (float)plan.layers[0].mix.rot.base;
-    r.ffn = plan.layers[0].has_mlp ? plan.layers[0].mlp.expert.ff : 0;
+    const LayerPlan& l = plan.layers[0];
+    r.n_heads = l.mixer == MIX_LATENT ? l.latent.heads : l.mixer == MIX_GROUPED ? l.grouped.heads : l.state.heads;
+    r.n_kv_heads = l.mixer == MIX_LATENT ? 1 : l.mixer == MIX_GROUPED ? l.grouped.kv_heads : l.state.heads;
+    r.head_dim = l.mixer == MIX_LATENT ? l.latent.dim + l.latent.rot_dim : l.mixer == MIX_GROUPED ? l.grouped.dim : l.state.dim;
+    r.rotary_dim = l.mixer == MIX_LATENT ? l.latent.rot_dim : l.mixer == MIX_GROUPED ? l.grouped.rot.dims : 0;
+    r.rope_theta = l.mixer == MIX_LATENT ? (float)l.latent.rot.base : l.mixer == MIX_GROUPED ? (float)l.grouped.rot.base : 0.f;
+    r.ffn = l.mlp == MLP_MOE ? l.moe.expert.ff : l.mlp == MLP_DENSE ? l.dense.ff : 0;
     return r;
 }()) {
     plan_.reset(new PlanState());

@@ -84,13 +84,18 @@ class Engine {
     int forward_rows(const uint32_t* ids, const int32_t* slots, int64_t n, const int32_t* rows, int64_t n_rows, float* logits_out,
                      uint32_t* argmax_out);
     int reset(int slot);
+    // Keeps the first n tokens of a slot. A model with recurrent states can only go back to a length whose state it still
+    // has: *kept <= n tells how far it went, and the tokens from there on are fed again.
     int truncate(int slot, size_t n, size_t* kept);
+    // Remembers the slot's states at its present length, so that truncate can come back to it (models without: nothing to do).
+    int checkpoint(int slot);
+    bool keeps_state() const;
     int debug_layer_out(int layer, float* out, size_t cap, int32_t* n_tokens);
     // `steps` greedy decode steps for b slots with no host work in between: step 0 consumes first_ids, every
     // later step consumes the device-side argmax of the previous one. tokens_out[steps * b] (host) may be null.
     int decode_greedy(const uint32_t* first_ids, const int32_t* slots, int b, int steps, uint32_t* tokens_out);
     // Per-kernel-family device time of profiled forwards (ms, accumulated) and launch counts.
-    enum Family { F_GEMV = 0, F_ATTN, F_NORM, F_ROPE, F_ELEM, F_EMBED, F_ARGMAX, F_COUNT };
+    enum Family { F_GEMV = 0, F_ATTN, F_NORM, F_ROPE, F_ELEM, F_EMBED, F_ARGMAX, F_STATE, F_COUNT };
     // Device time of one decode step of T tokens restricted to the kernel families in fam_mask (bit i = family i):
     // the step is captured with the other launches left out and replayed `reps` times between two events.
     // Activations and the KV entries of the last staged positions are undefined afterwards.
@@ -239,8 +244,14 @@ class Engine {
     void plan_release();
     int plan_stage(int T);
     int plan_layers(int T);
-    int plan_mixer(int layer, int T);
+    void plan_stage_latent(int T);
+    int plan_layer_post_norm(int layer, int T);
+    int plan_layer_parallel(int layer, int T);
+    int plan_latent(int layer, int T);
+    int plan_grouped(int layer, int T);
+    int plan_state(int layer, int T);
     int plan_experts(int layer, int T);
+    int plan_rollback(int slot, int n, int* kept);
     int plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, int ldy, bool out_f32);
     int plan_product(const MatArgs& a, int max_tiles);
     int plan_head(const int32_t* rows, int n);

@@ -57,6 +57,7 @@ int Engine::privatise_tail(int slot) {
 
 int Engine::adopt_prefix(int slot, const int32_t* page_ids, int n) {
     if (slot < 0 || slot >= d.max_batch || n < 0 || (n > 0 && !page_ids)) { set_error("adopt_prefix: bad argument"); return SP_ERR_ARG; }
+    if (n > 0 && keeps_state()) { set_error("adopt_prefix: the model keeps states that pages do not hold"); return SP_ERR_STATE; }
     if (seq_len[slot] != 0 || !pages.adopt(slot, page_ids, n)) { set_error("adopt_prefix: the slot is not empty or a page is not live"); return SP_ERR_STATE; }
     seq_len[slot] = n * KV_PAGE;
     return SP_OK;
@@ -75,7 +76,8 @@ int Engine::reset(int slot) {
 // O(1): the page-table tail is returned to the pool, the kept pages stay where they are.
 int Engine::truncate(int slot, size_t n, size_t* kept) {
     if (slot < 0 || slot >= d.max_batch) { set_error("slot out of range"); return SP_ERR_ARG; }
-    const int k = (int)std::min<size_t>(n, (size_t)seq_len[slot]);
+    int k = (int)std::min<size_t>(n, (size_t)seq_len[slot]);
+    if (keeps_state()) SP_TRY(plan_rollback(slot, k, &k));
     seq_len[slot] = k;
     const int keep_pages = (k + KV_PAGE - 1) / KV_PAGE;
     pages.shrink(slot, keep_pages);

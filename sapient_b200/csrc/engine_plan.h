@@ -1,7 +1,15 @@
-// State of a plan-driven engine (engine_plan.cu): the packed weights of every layer, the latent cache and the buffers of
-// a step. Owned by Engine, which keeps the sequence slots, the page tables, the step graphs and the host API.
+// State of a plan-driven engine: the packed weights of every layer, the cache and state pools and the buffers of a step.
+// Owned by Engine, which keeps the sequence slots, the page tables, the step graphs and the host API. engine_plan.cu has
+// what every plan shares, engine_plan_latent.cu latent attention and experts, engine_plan_parallel.cu the parallel layer
+// form with grouped attention, state mixers and dense feed-forwards.
 #pragma once
+#include <algorithm>
+#include <map>
+#include <string>
+#include <utility>
 #include <vector>
+
+#include "engine.h"
 
 #include "model_plan.h"
 #include "plan_kernels.h"
@@ -14,13 +22,32 @@ struct PlanMat {
     int n = 0, kp = 0, groups = 1;
 };
 
+constexpr int PLAN_ROWS = MAT_GATHER_ROWS;  // rows of a decode-shaped step
+static_assert(PLAN_ROWS <= STATE_STEP_ROWS, "a decode-shaped step runs the state mixers' step kernel");
+
+#define SP_TRY(expr)                  \
+    do {                              \
+        int _s = (expr);              \
+        if (_s != SP_OK) return _s;   \
+    } while (0)
+
+#define SP_LAUNCH(fam, expr)              \
+    do {                                  \
+        if (fam_mask & (1u << (fam))) {   \
+            prof_begin(fam);              \
+            SP_CUDA_TRY(expr);            \
+            prof_end(fam);                \
+        }                                 \
+    } while (0)
+
 struct PlanLayer {
-    PlanMat proj;              // q | latent and rotated key part (own cache only) | output gate
+    PlanMat proj;              // everything that reads the mixer's input. Latent: q | latent and rotated key part (own cache only) |
+                               // output gate. Parallel form: the mixer's f32 rows | low-rank rows | feed-forward up
     int gate_col = 0;          // first gate column of the projection's output
     PlanMat uk_t;              // per head, transposed: query -> latent space
     PlanMat uv;                // per head: latent -> value
     PlanMat kv;                // per head key rows then value rows, each padded to 16: the expanded form
-    PlanMat o;
+    PlanMat o;                 // output projection; parallel form: [W_o | W_down] over [mixer output | activation]
     const float *norm1 = nullptr, *norm2 = nullptr, *dkv_norm = nullptr, *dwa = nullptr;
     PlanMat router;            // experts rows, then the shared expert's gate row
     const float* router_b = nullptr;
@@ -29,6 +56,24 @@ struct PlanLayer {
     LatentCache cache{};       // the layer's own, or the one it borrows
     bool own = true, expand = false;
     const float2* cos_sin = nullptr;
+    // parallel form
+    int mix_rows = 0, silu_rows = 0, low_rows = 0, ff = 0;  // of proj: f32 rows, of which silu_rows come first, ...
+    int act_col = 0;           // first column of the activation in o's input
+    GroupedShape grouped{};
+    GroupedCache kv_cache{};
+    const float2 *cs_key = nullptr, *cs_val = nullptr;
+    StateShape state_shape{};
+    size_t state_at = 0;       // of a slot's floats
+    PlanMat w2;
+    const float *decay = nullptr, *a_bias = nullptr, *w0 = nullptr, *gain = nullptr;
+};
+
+// Elements per row that the step's buffers need: the largest of all layers.
+struct PlanSizes {
+    size_t proj = 0, qn = 0, qabs = 0, qf = 0, olat = 0, mixed = 0, act = 0, act_shared = 0, pairs = 0, kv = 0, lat = 0, part = 0, low = 0,
+           wlogit = 0, state_out = 0, q = 0;
+    int experts = 0;
+    static void most(size_t& a, size_t b) { a = std::max(a, b); }
 };
 
 struct PlanState {
@@ -40,18 +85,52 @@ struct PlanState {
     const float* final_norm = nullptr;
     int wp = 0;                // padded width
     size_t page_bytes = 0;     // all layers' rows of one page
-    std::vector<size_t> cache_run, cache_base;  // per owning layer: bytes of a page, offset of its slice
+    std::vector<size_t> cache_run, cache_base;  // per layer: bytes of a page (0: none of its own), offset of its slice
+    size_t cache_bytes = 0;
     void* cache = nullptr;
     // buffers of a step
+    PlanSizes need;
+    bool has_latent = false, has_grouped = false, has_state = false;
     void *xb = nullptr, *qn = nullptr, *qabs = nullptr, *qf = nullptr, *olat = nullptr, *attn = nullptr, *act = nullptr, *act_shared = nullptr,
-         *xs = nullptr, *kvx = nullptr, *lat = nullptr, *fin = nullptr;
-    float *proj = nullptr, *y = nullptr, *y_expert = nullptr, *y_shared = nullptr, *logit = nullptr, *weight = nullptr, *part = nullptr, *history = nullptr;
+         *xs = nullptr, *kvx = nullptr, *lat = nullptr, *fin = nullptr, *q = nullptr, *low = nullptr;
+    float *proj = nullptr, *y = nullptr, *y_expert = nullptr, *y_shared = nullptr, *logit = nullptr, *weight = nullptr, *part = nullptr, *history = nullptr, *wlogit = nullptr, *state_out = nullptr;
     int32_t *pick = nullptr, *tables = nullptr, *host_tiles = nullptr, *dev_tiles = nullptr;
+    // sections of host_tiles / dev_tiles, in ints
+    size_t keys_at = 0, grouped_at = 0, seg_at = 0, order_at = 0, table_ints = 0;
     MoeTables moe{};
     int keys_cap = 0;          // gathered keys a step may hold
-    // the expanded form of the current step (0 tiles: absorbed)
-    int n_tiles = 0, n_keys = 0;
+    // the current step, when it is longer than PLAN_ROWS
+    int n_tiles = 0, n_keys = 0;        // latent attention: tiles and gathered keys of the expanded form (0 tiles: absorbed)
+    int n_grouped = 0, n_seg = 0;       // grouped attention: tiles; state mixers: segments
+    // states [slot][layer][heads][vdim][dim_pad] and what checkpoint() keeps of each slot
+    float *states = nullptr, *checkpoints = nullptr;
+    size_t slot_state = 0;              // floats per slot
+    std::vector<int> checkpoint_len;    // per slot: tokens the kept state has seen, -1: none
+    std::map<std::pair<double, int>, const float2*> angles;
     std::vector<void*> owned;
+};
+
+size_t plan_latent_part_rows();  // engine_plan_latent.cu
+
+// Builds packed matrices out of the uploaded tensors.
+struct PlanPacker {
+    Engine& e;
+    PlanState& p;
+    int status = SP_OK;
+
+    bool fail(int st, const std::string& msg);
+    const DevTensor* need(const std::string& name, int64_t rows, int64_t cols);
+    int64_t rows_of(const std::string& name);            // first dimension of a tensor whose size only its shape tells
+    const float* vec(const std::string& name, int64_t n);
+    bool alloc(PlanMat& m, int groups, int64_t rows, int k);
+    // rows [r0, r0 + rows) of source tensor t to packed rows starting at `to` (counted over all groups), columns at c0
+    bool put(PlanMat& m, int64_t to, const DevTensor* t, int64_t r0, int64_t rows, int k, bool transpose = false, int c0 = 0);
+    // cos and sin of position * base^(-2 i / dims), i < dims / 2, for every position: computed in double, rounded once
+    const float2* angles(double base, int dims);
+    void cache_slice(size_t page_bytes);                 // the next layer's share of the cache
+    void latent_layer(int i);
+    void experts(int i);
+    void parallel_layer(int i);
 };
 
 }  // namespace sp

@@ -40,6 +40,14 @@ __device__ __forceinline__ bool mat_work(const MatArgs& a, int slot, MatWork& w)
 }
 
 __device__ __forceinline__ void mat_store(const MatArgs& a, const MatSeg& s, const MatWork& w, int row, int n, float v) {
+    if (a.n_outs) {
+        int i = 0;
+        while (n >= a.outs[i].n_end) ++i;
+        float* y = reinterpret_cast<float*>(a.outs[i].y) + row * a.outs[i].ldy + n - (i ? a.outs[i - 1].n_end : 0);
+        v = mat_act(a.outs[i].act, v, a.scale, a.cap);
+        *y = a.outs[i].add ? *y + v : v;
+        return;
+    }
     if (a.gate) v *= sigmoid_f32(a.gate[(int64_t)row * a.ldgate + w.g]);
     reinterpret_cast<float*>(s.y)[(int64_t)row * s.ldy + (int64_t)w.g * s.ygs + n] = v;
 }
@@ -92,6 +100,7 @@ __global__ void __launch_bounds__(256) mat_f32_kernel(const MatArgs a) {
 cudaError_t launch_mat_f32(const MatArgs& a, cudaStream_t st) {
     if (a.m <= 0) return cudaSuccess;
     if (!a.f32 || a.nseg < 1 || a.nseg > 2) return cudaErrorInvalidValue;
+    if (!mat_outs_valid(a)) return cudaErrorInvalidValue;
     int n_max = 0, slots = a.moe ? a.slots : a.seg[0].groups;
     for (int i = 0; i < a.nseg; ++i) {
         if (a.seg[i].kp % MAT_KPAD != 0 || a.seg[i].n <= 0) return cudaErrorInvalidValue;

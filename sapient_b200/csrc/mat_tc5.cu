@@ -55,9 +55,13 @@ struct MatTc5Args {
     MoeRows rows;
     const float* gate;
     int ldgate;
+    int n_outs;
+    MatOut outs[MAT_MAX_OUTS];
+    float scale, cap;
 };
 
-template <bool DUAL, bool OUT_F32>
+// OUTS: a plain product whose weight rows go where a.outs says (OUT_F32 then has no meaning).
+template <bool DUAL, bool OUT_F32, bool OUTS = false>
 __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
                                                              const __grid_constant__ CUtensorMap map_x0, const __grid_constant__ CUtensorMap map_w1,
                                                              const __grid_constant__ CUtensorMap map_x1) {
@@ -185,6 +189,28 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
             if (a.gate) f *= sigmoid_f32(gate);
             yn[(int64_t)row * s.ldy] = from_f32<Out>(f);
         };
+        // OUTS: this thread's range
+        int act = MAT_ID;
+        int64_t oldd = 0;
+        float* of = nullptr;   // f32 destination of row 0
+        bf16* ob = nullptr;    // or bf16
+        bool add = false;
+        if (OUTS && n < s.n) {
+            int i = 0;
+            while (n >= a.outs[i].n_end) ++i;
+            const int col = n - (i ? a.outs[i - 1].n_end : 0);
+            act = a.outs[i].act;
+            oldd = a.outs[i].ldy;
+            add = a.outs[i].add;
+            if (a.outs[i].f32) of = reinterpret_cast<float*>(a.outs[i].y) + col;
+            else ob = reinterpret_cast<bf16*>(a.outs[i].y) + col;
+        }
+        auto held = [&](int row) { return add ? of[row * oldd] : 0.f; };
+        auto put = [&](int row, float f, float before) {
+            f = mat_act(act, f, a.scale, a.cap);
+            if (of) of[row * oldd] = add ? before + f : f;
+            else ob[row * oldd] = __float2bfloat16_rn(f);
+        };
         if (ok) {
             const uint32_t lanes = tmem + ((uint32_t)(32 * q4) << 16);
             float* mine = partial + 32 * q4 + lane;
@@ -200,6 +226,15 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
                         // (a short K may leave a part without chunks)
                         mine[(c + j) * MT_BM] = n_chunks ? __uint_as_float(v[j]) : 0.f;
                         if (DUAL) mine[(a.bn + c + j) * MT_BM] = n_chunks ? __uint_as_float(up[j]) : 0.f;
+                    }
+                } else if (OUTS) {
+                    if (n < s.n) {
+                        float before[16];
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) before[j] = c + j < cols ? held(r0 + c + j) : 0.f;
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            if (c + j < cols) put(r0 + c + j, __uint_as_float(v[j]), before[j]);
                     }
                 } else if (n < s.n) {
                     if (by_index || a.gate || c + 16 > cols) {
@@ -238,7 +273,7 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
                     for (int j = 0; j < NC; ++j) {
                         const int c = c0 + j * a.parts;
                         row[j] = c < cols ? (by_index ? dest[c] : r0 + c) : -1;
-                        gt[j] = a.gate && row[j] >= 0 ? gate_of(row[j]) : 0.f;
+                        gt[j] = row[j] < 0 ? 0.f : OUTS ? held(row[j]) : a.gate ? gate_of(row[j]) : 0.f;
                         f[j] = up[j] = 0.f;
                     }
 #pragma unroll 4
@@ -254,7 +289,10 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
                     }
 #pragma unroll
                     for (int j = 0; j < NC; ++j)
-                        if (row[j] >= 0) finish(row[j], f[j], up[j], gt[j]);
+                        if (row[j] >= 0) {
+                            if (OUTS) put(row[j], f[j], gt[j]);
+                            else finish(row[j], f[j], up[j], gt[j]);
+                        }
                 }
             }
         }
@@ -293,6 +331,7 @@ static bool mat_map(CUtensorMap* map, const void* p, int64_t cols, int64_t rows,
 cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     if (a.m <= 0) return cudaSuccess;
     if (a.f32 || a.nseg < 1 || a.nseg > 2 || (a.nseg == 2 && a.seg[1].groups != 1) || (a.gather && (!a.moe || a.m > MAT_GATHER_ROWS))) return cudaErrorInvalidValue;
+    if (!mat_outs_valid(a)) return cudaErrorInvalidValue;
     MatTc5Args k{};
     int n_max = 0, kp_max = 0;
     for (int i = 0; i < a.nseg; ++i) {
@@ -314,6 +353,8 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     k.slots0 = a.moe ? max_tiles : groups * k.row_tiles;
     const int slots = k.slots0 + (a.nseg == 2 ? k.row_tiles : 0);
     k.moe = a.moe; k.gather = a.gather; k.rows = a.rows; k.gate = a.gate; k.ldgate = a.ldgate;
+    k.n_outs = a.n_outs; k.scale = a.scale; k.cap = a.cap;
+    std::copy(a.outs, a.outs + MAT_MAX_OUTS, k.outs);
     const int acc = a.dual ? 2 : 1;
     k.stage_bytes = acc * MT_A_BYTES + bn * MT_BK * 2;
     k.tmem_cols = std::max(32, acc * bn);
@@ -334,7 +375,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
         const void* fns[] = {(const void*)mat_tc5_kernel<false, false>, (const void*)mat_tc5_kernel<false, true>, (const void*)mat_tc5_kernel<true, false>,
-                             (const void*)mat_tc5_kernel<true, true>};
+                             (const void*)mat_tc5_kernel<true, true>, (const void*)mat_tc5_kernel<false, true, true>};
         for (const void* f : fns) {
             const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM + 1024);
             if (e != cudaSuccess) return e;
@@ -346,7 +387,8 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     const dim3 grid((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), block(MT_THREADS);
     const size_t smem = (size_t)(k.stages * k.stage_bytes + 1024);
 #define SP_MT(DUAL, F32) le = launch_pdl_cluster(mat_tc5_kernel<DUAL, F32>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1])
-    if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
+    if (a.n_outs) le = launch_pdl_cluster(mat_tc5_kernel<false, true, true>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1]);
+    else if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
     else { if (a.out_f32) SP_MT(false, true); else SP_MT(false, false); }
 #undef SP_MT
     if (le != cudaSuccess) return le;

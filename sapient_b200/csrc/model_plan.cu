@@ -60,11 +60,97 @@ LatentAttentionSpec read_latent_attention(const Cfg& c, int layer, const ModelPl
         m.kv_from = c.size("kv_from", 0);
         if (!c.err->empty()) return m;
         if (m.kv_from >= layer) { c.fail("kv_from must name an earlier layer"); return m; }
-        const LatentAttentionSpec& o = p.layers[(size_t)m.kv_from].mix;
+        const LatentAttentionSpec& o = p.layers[(size_t)m.kv_from].latent;
         if (o.kv_from >= 0 || o.kv_rank != m.kv_rank || o.rot_dim != m.rot_dim || o.rot.base != m.rot.base)
             c.fail("kv_from names a layer whose latent does not fit");
     }
     return m;
+}
+
+GroupedAttentionSpec read_grouped_attention(const Cfg& c, bool rotate_values) {
+    GroupedAttentionSpec m;
+    m.heads = c.size("heads");
+    m.kv_heads = c.size("kv_heads");
+    m.dim = c.size("dim");
+    m.vdim = c.size("vdim");
+    m.scale = (float)c.num("scale");
+    const Cfg rot = c.sub("rot");
+    m.rot.base = rot.num("base");
+    m.rot.dims = rot.size("dims", 0);
+    m.rotate_values = rotate_values;
+    if (c.has("mask") && c.sub("mask").has("size")) m.window = c.sub("mask").size("size");
+    if (!c.err->empty()) return m;
+    if (m.heads % m.kv_heads) c.fail("heads is no multiple of kv_heads");
+    if ((m.rot.dims & 1) || m.rot.dims > m.dim || m.rot.base <= 0) c.fail("rot does not fit dim");
+    if (rotate_values && (m.vdim & 1)) c.fail("vdim must be even");
+    return m;
+}
+
+StateMixerSpec read_state_mixer(const Cfg& c, StateRule rule) {
+    StateMixerSpec m;
+    m.rule = rule;
+    m.heads = c.size("heads");
+    m.dim = c.size("dim");
+    m.vdim = rule == STATE_DELTA ? m.dim : c.size("vdim");
+    if (rule == STATE_DECAY) {
+        const Json* d = c.j ? c.j->get("decay") : nullptr;
+        if (!d || d->type != Json::ARR || (c.err->empty() && (int)d->arr.size() != m.heads)) { c.fail("decay must list a number per head"); return m; }
+        for (const Json& v : d->arr) {
+            if (v.type != Json::NUM || !std::isfinite(v.num)) { c.fail("decay must list a number per head"); return m; }
+            m.decay.push_back((float)v.num);
+        }
+    }
+    if (c.err->empty() && m.dim > STATE_MAX_DIM) c.fail("dim is above " + std::to_string(STATE_MAX_DIM));
+    return m;
+}
+
+// A layer's entry is null or has no "mlp": no feed-forward.
+void read_dense(const Cfg& lc, LayerPlan* l) {
+    if (!lc.has("mlp")) return;
+    const Cfg c = lc.sub("mlp");
+    const Json* kind = c.j ? c.j->get("kind") : nullptr;
+    if (!kind || kind->str != "dense") { c.fail("kind is not a feed-forward of this design"); return; }
+    l->mlp = MLP_DENSE;
+    l->dense.ff = c.size("ff");
+}
+
+int read_tedelix(const Json& cfg, ModelPlan* out) {
+    std::string err;
+    const Cfg c{&cfg, "", &err};
+    ModelPlan p;
+    p.name = "Tedelix";
+    p.vocab = c.size("vocab");
+    p.width = c.size("width");
+    p.eps = (float)c.sub("norm").num("eps");
+    p.form = FORM_PARALLEL;
+    p.tied_head = true;
+    if (c.has("logit_scale")) p.logit_scale = (float)c.num("logit_scale");
+    if (c.has("logit_softcap")) p.logit_softcap = (float)c.num("logit_softcap");
+    const Json* layers = cfg.get("layers");
+    if (!layers || layers->type != Json::ARR || layers->arr.empty()) c.fail("layers is missing or not a list");
+    for (size_t i = 0; err.empty() && i < layers->arr.size(); ++i) {
+        const std::string idx = std::to_string(i);
+        const Cfg lc{&layers->arr[i], "layers[" + idx + "].", &err};
+        LayerPlan l;
+        l.prefix = "l" + idx + ".";
+        const Json* type = lc.j->get("type");
+        const std::string t = type ? type->str : "";
+        if (t == "attention") {
+            l.mixer = MIX_GROUPED;
+            l.grouped = read_grouped_attention(lc.sub("mixer"), true);
+        } else if (t == "lightning" || t == "general_delta") {
+            l.mixer = MIX_STATE;
+            l.state = read_state_mixer(lc.sub("mixer"), t == "lightning" ? STATE_DECAY : STATE_DELTA);
+        } else {
+            lc.fail("type is not a mixer of this design");
+            break;
+        }
+        read_dense(lc, &l);
+        p.layers.push_back(l);
+    }
+    if (!err.empty()) { set_error(err); return SP_ERR_ARG; }
+    *out = std::move(p);
+    return SP_OK;
 }
 
 int read_lepalorn(const Json& cfg, ModelPlan* out) {
@@ -86,20 +172,20 @@ int read_lepalorn(const Json& cfg, ModelPlan* out) {
         l.prefix = "l" + idx + ".";
         const Json* type = lc.j->get("type");
         if (!type || type->str != "latent_attention") { lc.fail("type is not a mixer of this design"); break; }
-        l.mix = read_latent_attention(lc.sub("mixer"), (int)i, p);
+        l.latent = read_latent_attention(lc.sub("mixer"), (int)i, p);
         if (lc.has("mlp")) {
             const Cfg m = lc.sub("mlp");
             const Json* kind = m.j ? m.j->get("kind") : nullptr;
             if (!kind || kind->str != "moe") { m.fail("kind is not a feed-forward of this design"); break; }
-            l.has_mlp = true;
-            l.mlp.experts = m.sub("router").size("experts");
-            l.mlp.top = m.sub("router").size("top");
-            l.mlp.expert = read_expert(m.sub("expert"));
+            l.mlp = MLP_MOE;
+            l.moe.experts = m.sub("router").size("experts");
+            l.moe.top = m.sub("router").size("top");
+            l.moe.expert = read_expert(m.sub("expert"));
             if (m.has("shared")) {
-                l.mlp.has_shared = true;
-                l.mlp.shared = read_expert(m.sub("shared"));
+                l.moe.has_shared = true;
+                l.moe.shared = read_expert(m.sub("shared"));
             }
-            if (l.mlp.top > l.mlp.experts) m.fail("router.top exceeds router.experts");
+            if (l.moe.top > l.moe.experts) m.fail("router.top exceeds router.experts");
         }
         p.layers.push_back(l);
     }
@@ -113,6 +199,7 @@ const ArchEntry ARCHS[] = {
     {"llama", ARCH_LLAMA, true, nullptr},   {"mistral", ARCH_LLAMA, true, nullptr}, {"qwen2", ARCH_LLAMA, true, nullptr},
     {"qwen3", ARCH_LLAMA, true, nullptr},   {"idefics3", ARCH_LLAMA, true, nullptr}, {"phi3", ARCH_LLAMA, true, nullptr},
     {"phi", ARCH_PHI2, true, nullptr},      {"phi2", ARCH_PHI2, true, nullptr},     {"Lepalorn", ARCH_PLAN, false, read_lepalorn},
+    {"Tedelix", ARCH_PLAN, false, read_tedelix},
 };
 
 }  // namespace

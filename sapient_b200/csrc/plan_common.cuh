@@ -4,6 +4,7 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "plan_kernels.h"
 #include "sp_common.cuh"
 
 namespace sp {
@@ -22,6 +23,19 @@ __device__ __forceinline__ float clamped_unit(float g, float u, float limit, flo
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g * sigmoid_f32(alpha * g) * (u + 1.0f);
+}
+
+__device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
+
+// The activation of a product's output range (plan_kernels.h: MatOut).
+__device__ __forceinline__ float mat_act(int act, float z, float scale, float cap) {
+    switch (act) {
+        case MAT_RELU2: z = fmaxf(z, 0.f); return z * z;
+        case MAT_TANH: return tanhf(z);
+        case MAT_SILU: return silu_f32(z);
+        case MAT_SOFTCAP: return cap > 0.f ? cap * tanhf(z * scale / cap) : z * scale;
+        default: return z;
+    }
 }
 
 // Sum over the block, the same value in every thread. sh: one float per warp.

@@ -28,6 +28,18 @@ struct MatSeg {
     int64_t ygs;
 };
 
+// Where a range of a matrix's rows goes: output elements [previous n_end, n_end) of every activation row to y (column 0 is
+// the range's first), through an activation, as f32 or in the compute type; `add`: y (f32) += instead of =.
+enum MatAct : int { MAT_ID = 0, MAT_RELU2, MAT_TANH, MAT_SILU, MAT_SOFTCAP };  // softcap: cap * tanh(scale * z / cap)
+struct MatOut {
+    int n_end;
+    void* y;
+    int64_t ldy;
+    MatAct act;
+    bool f32, add;
+};
+constexpr int MAT_MAX_OUTS = 4;
+
 // Rows of a step sorted by expert, made on the device by launch_moe_route.
 struct MoeRows {
     const int32_t* row_off;    // [experts + 1] first sorted row of each expert
@@ -52,7 +64,22 @@ struct MatArgs {
     int x_rows;                // rows of seg[0].x when they are not the m rows (sorted rows)
     const float* gate;         // y *= sigmoid(gate[row * ldgate + group]) or null
     int ldgate;
+    int n_outs;                // > 0: one plain product whose rows go where outs[] says (seg[0].y is not used)
+    MatOut outs[MAT_MAX_OUTS];
+    float scale, cap;          // of MAT_SOFTCAP
 };
+
+// The ranges cover the matrix, and the product is a plain one.
+inline bool mat_outs_valid(const MatArgs& a) {
+    if (a.n_outs == 0) return true;
+    if (a.n_outs < 0 || a.n_outs > MAT_MAX_OUTS || a.nseg != 1 || a.seg[0].groups != 1 || a.moe || a.dual || a.gate) return false;
+    int n = 0;
+    for (int i = 0; i < a.n_outs; ++i) {
+        if (a.outs[i].n_end <= n || !a.outs[i].y || (a.outs[i].add && !a.outs[i].f32 && !a.f32)) return false;
+        n = a.outs[i].n_end;
+    }
+    return n == a.seg[0].n;
+}
 
 // f32: plain fused multiply-adds on 32 x 32 tiles, any shape and row count.
 cudaError_t launch_mat_f32(const MatArgs& a, cudaStream_t st);
@@ -66,7 +93,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st);
 int mat_tc5_take_timeout();    // as tc5_take_timeout (kernels.h)
 
 // ── the stream between the products ──
-// x0[t] = table[ids[t]] * scale (f32), xb = the same in the compute type (row stride ldb, padding zeroed).
+// x0[t] = table[ids[t]] * scale (f32), xb (or null) = the same in the compute type (row stride ldb, padding zeroed).
 cudaError_t launch_embed_scaled(const void* table, int ldt, bool f32, const uint32_t* ids, int n_tok, int width, float scale, float* x0, void* xb,
                                 int ldb, cudaStream_t st);
 // x += rms_norm(y) * gain (one number), f32; xb as above.
@@ -95,9 +122,9 @@ struct CombineArgs {
     float eps;
 };
 cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStream_t st);
-// out (compute type) = rms_norm(x[rows[i] or i]) * gain.
-cudaError_t launch_final_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, float eps, void* out, int ldo, bool f32,
-                              cudaStream_t st);
+// out (compute type) = rms_norm(x[rows[i] or i]) * gain; gain: one number, or one per coordinate (per_coord).
+cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, bool per_coord, float eps, void* out,
+                            int ldo, bool f32, cudaStream_t st);
 
 // ── experts ──
 // Per token the `top` largest of logits[t][0..experts) + bias (ties: the lower index) with the softmax over the chosen ones
@@ -155,5 +182,81 @@ constexpr int LATENT_Q_TILE = 64;
 // head by head, times sigmoid(gate[t * ldgate + head]).
 cudaError_t launch_latent_expanded(const void* qf, const void* kv, const void* lat, const LatentShape& s, const LatentCache& c,
                                    const LatentTile* tiles, int n_tiles, const float* gate, int ldgate, void* out, int ldo, cudaStream_t st);
+
+// ── grouped attention ──
+// One layer's slice of the paged cache: [page][kv head][16 tokens][dim16 | vdim16] of the compute type, keys and values
+// rotated, padded with zeros to multiples of 16.
+struct GroupedCache {
+    void* pool;
+    const int32_t* page_table;
+    int max_pages;
+    int dim16, vdim16;
+};
+struct GroupedShape {
+    int heads, kv_heads, dim, vdim, rot;
+    int window;
+    float scale;
+};
+// proj[t] (f32, row stride ldp): queries head by head, keys, values. Rotates queries and keys by cs_key[pos][rot / 2] and,
+// where cs_val[pos][vdim / 2] is given, values; q[t][heads][dim16] in the compute type, keys and values to the cache.
+cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const float2* cs_key, const float2* cs_val,
+                                  const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st);
+// out[t][ldo] (compute type), head by head vdim values: the mixtures, turned back by cs_val (or null). Any sizes up to
+// GROUPED_MAX_VDIM. n_splits > 1 (bf16: grouped_attention_splits of the longest range to visit) splits the keys over the
+// blocks of a cluster.
+constexpr int GROUPED_MAX_VDIM = 1024;
+bool grouped_mma_supported(const GroupedShape& s);
+int grouped_attention_splits(const GroupedShape& s, int n_tok, int keys, bool f32);
+cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const int32_t* tok_slot,
+                                     const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st);
+// bf16, many rows: tiles of up to GROUPED_Q_TILE consecutive tokens of one sequence.
+struct GroupedTile {
+    int32_t row0, n;           // token rows
+    int32_t pos0;              // position of the first
+    int32_t slot;
+};
+constexpr int GROUPED_Q_TILE = 64;
+cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const GroupedTile* tiles,
+                                   int n_tiles, void* out, int ldo, cudaStream_t st);
+
+// ── mixers with a state matrix (model_plan.h: StateMixerSpec) ──
+// State of a slot: [heads][vdim][dim_pad] f32, slots slot_stride floats apart (a value column's keys are contiguous). A sequence's first token (position 0)
+// starts from zeros, whatever the slot held.
+struct StateShape {
+    int heads, dim, vdim;
+    int rule;                  // StateRule
+    int dim_pad;               // state_dim_pad(dim)
+    float eps;
+};
+int state_dim_pad(int dim);
+struct StateArgs {
+    StateShape s;
+    float* state;
+    int64_t slot_stride;
+    const float* decay;        // STATE_DECAY: [heads]
+    // STATE_DECAY: proj[t] = q | k | v (silu applied) | gate logits. STATE_DELTA: r | k | v | removal logits | gate logits.
+    float* proj;
+    int ldp;
+    const float* a_bias;       // STATE_DELTA: [heads * dim]
+    const float* w0;           // STATE_DELTA: decay logit = w0 + W2 low[t]
+    const void* w2;            // compute type, [heads * dim][ldlow]
+    const void* low;           // compute type, [t][ldlow]
+    int ldlow;
+    float* wlogit;             // many rows: W2 low[t] (f32, [t][heads * dim]), overwritten with the decays
+    float* o;                  // many rows: [t][heads * vdim] f32
+    const float* gain;         // [heads * vdim]
+    const int32_t *tok_slot, *tok_pos;
+    void* out;                 // compute type, [t][ldo]
+    int ldo;
+    bool f32;
+};
+// Up to STATE_STEP_ROWS rows: gates, recurrence, norm and output gate in one launch. Rows of one slot are taken in order.
+constexpr int STATE_STEP_ROWS = 32;
+cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st);
+// Any number of rows: a segment is the n rows order[begin .. begin + n) of one slot; row0 >= 0: they are row0, row0 + 1, ...
+struct StateSegment {
+    int32_t begin, n, slot, fresh, row0;  // fresh: starts at position 0
+};
+cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* order, int n_tok, cudaStream_t st);
 
 }  // namespace sp

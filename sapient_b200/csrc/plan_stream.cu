@@ -40,7 +40,7 @@ __global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __res
     for (int c = threadIdx.x; c < ldb; c += ST_THREADS) {
         const float v = c < width ? to_f32(row[c]) * scale : 0.f;
         if (c < width) x0[(int64_t)t * width + c] = v;
-        xb[(int64_t)t * ldb + c] = from_f32<T>(v);
+        if (xb) xb[(int64_t)t * ldb + c] = from_f32<T>(v);
     }
 }
 
@@ -201,24 +201,41 @@ cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStrea
     return count_launch_and_check();
 }
 
-template <typename T>
-__global__ void __launch_bounds__(ST_THREADS) final_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, int width,
-                                                                const float* __restrict__ gain, float eps, T* __restrict__ out, int ldo) {
+template <typename T, int V>
+__global__ void __launch_bounds__(ST_THREADS) row_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, int width,
+                                                              const float* __restrict__ gain, bool per_coord, float eps, T* __restrict__ out, int ldo) {
     __shared__ float sh[ST_WARPS];
     pdl_wait();
     pdl_trigger();
     const float* xr = x + (int64_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * width;
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < width; c += ST_THREADS) ss = fmaf(xr[c], xr[c], ss);
-    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps) * *gain;
-    for (int c = threadIdx.x; c < ldo; c += ST_THREADS) out[(int64_t)blockIdx.x * ldo + c] = from_f32<T>(c < width ? xr[c] * r : 0.f);
+    float ss = 0.f, v[V], g[V];
+    for (int c = V * threadIdx.x; c < width; c += V * ST_THREADS) {
+        Row<V>::load(xr + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
+    }
+    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps);
+    for (int c = V * threadIdx.x; c < ldo; c += V * ST_THREADS) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = 0.f;
+        if (c < width) {
+            Row<V>::load(xr + c, v);
+            if (per_coord) Row<V>::load(gain + c, g);
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = v[i] * r * (per_coord ? g[i] : *gain);
+        }
+        Row<V>::store(out + (int64_t)blockIdx.x * ldo + c, v);
+    }
 }
 
-cudaError_t launch_final_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, float eps, void* out, int ldo, bool f32,
-                              cudaStream_t st) {
+cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, bool per_coord, float eps, void* out,
+                            int ldo, bool f32, cudaStream_t st) {
     if (n_rows == 0) return cudaSuccess;
-    cudaError_t le = f32 ? launch_pdl(final_norm_kernel<float>, dim3(n_rows), dim3(ST_THREADS), 0, st, x, rows, width, gain, eps, (float*)out, ldo)
-                         : launch_pdl(final_norm_kernel<bf16>, dim3(n_rows), dim3(ST_THREADS), 0, st, x, rows, width, gain, eps, (bf16*)out, ldo);
+    const bool wide = width % 4 == 0 && ldo % 4 == 0 && (!per_coord || (reinterpret_cast<uintptr_t>(gain) & 15) == 0);
+    const dim3 grid(n_rows), block(ST_THREADS);
+#define SP_RN(T, V) launch_pdl(row_norm_kernel<T, V>, grid, block, 0, st, x, rows, width, gain, per_coord, eps, (T*)out, ldo)
+    const cudaError_t le = f32 ? (wide ? SP_RN(float, 4) : SP_RN(float, 1)) : (wide ? SP_RN(bf16, 4) : SP_RN(bf16, 1));
+#undef SP_RN
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
