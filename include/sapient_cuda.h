@@ -341,9 +341,14 @@ int32_t sp_cuda_engine_set_profile(SpEngine* e, int32_t on);
  * CUDA graph `reps` times between two events. Activations and the newest KV entries are undefined afterwards. */
 int32_t sp_cuda_engine_time_families(SpEngine* e, uint32_t family_mask, int32_t n_tokens, int32_t reps, float* ms_per_step);
 int32_t sp_cuda_engine_profile_read(SpEngine* e, double* ms, uint64_t* launches, int32_t cap, int32_t reset);
-/* reset_cache / truncate_cache (forward/mod.rs:381-414): kept = min(n, current). slot < 0 = all slots. */
+/* reset_cache / truncate_cache (forward/mod.rs:381-414): kept = min(n, current). slot < 0 = all slots.
+ * A model with recurrent states (a layer plan with state mixers) can only go back to a length whose states it still has:
+ * the current length, the one sp_cuda_engine_checkpoint last recorded for the slot, or 0. *kept is then the longest such
+ * length of at most n, and the caller feeds the tokens from there on again. checkpoint costs one copy of the slot's states
+ * and does nothing for other models. */
 int32_t sp_cuda_reset_cache(SpEngine* e, int32_t slot);
 int32_t sp_cuda_truncate_cache(SpEngine* e, int32_t slot, size_t n, size_t* kept);
+int32_t sp_cuda_engine_checkpoint(SpEngine* e, int32_t slot);
 int32_t sp_cuda_seq_len(const SpEngine* e, int32_t slot, size_t* len);
 /* backend_label (forward/mod.rs:482-494) -> "cuda"; is_hybrid is always false. */
 int32_t sp_cuda_backend_label(const SpEngine* e, char* buf, size_t cap);

@@ -101,6 +101,7 @@ SIGNATURES = {
     "sp_cuda_engine_time_families": (_i32, [_vp, C.c_uint32, _i32, _i32, C.POINTER(C.c_float)]),
     "sp_cuda_reset_cache": (_i32, [_vp, _i32]),
     "sp_cuda_truncate_cache": (_i32, [_vp, _i32, _sz, C.POINTER(_sz)]),
+    "sp_cuda_engine_checkpoint": (_i32, [_vp, _i32]),
     "sp_cuda_seq_len": (_i32, [_vp, _i32, C.POINTER(_sz)]),
     "sp_cuda_backend_label": (_i32, [_vp, C.c_char_p, _sz]),
     "sp_cuda_engine_set_trace": (_i32, [_vp, _i32]),

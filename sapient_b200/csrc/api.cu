@@ -977,6 +977,14 @@ int32_t sp_cuda_truncate_cache(SpEngine* e, int32_t slot, size_t n, size_t* kept
     API_END
 }
 
+int32_t sp_cuda_engine_checkpoint(SpEngine* e, int32_t slot) {
+    API_BEGIN
+    if (!e) { set_error("null engine"); return SP_ERR_ARG; }
+    if (!e->e->finalized) { set_error("engine not finalised"); return SP_ERR_STATE; }
+    return e->e->checkpoint(slot);
+    API_END
+}
+
 int32_t sp_cuda_seq_len(const SpEngine* e, int32_t slot, size_t* len) {
     if (!e || !len || slot < 0 || slot >= e->e->d.max_batch) { set_error("bad argument"); return SP_ERR_ARG; }
     *len = (size_t)e->e->seq_len[slot];

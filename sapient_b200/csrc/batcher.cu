@@ -25,7 +25,7 @@ uint64_t Batcher::chain(uint64_t parent, const uint32_t* tok) {
     return h ? h : 1;
 }
 
-Batcher::Batcher(SeqBackend* be, int prefill_chunk, bool prefix_cache) : be_(be), chunk_(std::max(1, prefill_chunk)), use_prefix_(prefix_cache) {
+Batcher::Batcher(SeqBackend* be, int prefill_chunk, bool prefix_cache) : be_(be), chunk_(std::max(1, prefill_chunk)), use_prefix_(prefix_cache && be->shares_prefixes()) {
     for (int s = be_->max_slots() - 1; s >= 0; --s) free_slots_.push_back(s);
 }
 
@@ -306,6 +306,7 @@ class EngineBackend : public SeqBackend {
         return e_->forward(ids, slots, b, true, nullptr, argmax);
     }
     int release(int slot) override { size_t kept; return e_->truncate(slot, 0, &kept); }
+    bool shares_prefixes() const override { return !e_->keeps_state(); }
     int adopt_prefix(int slot, const int32_t* pages, int n) override { return e_->adopt_prefix(slot, pages, n); }
 
   private:

@@ -35,6 +35,7 @@ class SeqBackend {
     // One token for each of b distinct slots; argmax[b] receives the picks.
     virtual int decode(const uint32_t* ids, const int32_t* slots, int b, uint32_t* argmax) = 0;
     virtual int release(int slot) = 0;  // truncate to 0
+    virtual bool shares_prefixes() const { return true; }  // pages are all there is to a prefix
     virtual int adopt_prefix(int slot, const int32_t* pages, int n) = 0;
 };
 

@@ -207,7 +207,8 @@ int Engine::finalize_plan() {
     }
     if (long_steps) {
         p.wlogit = (float*)take(T * n.wlogit * 4);
-        p.state_out = (float*)take(T * n.state_out * 4);
+        p.groups_cap = p.has_state ? T / state_group(p.f32) + std::min<size_t>(T, (size_t)d.max_batch) + 1 : 0;
+        p.state_rec = (float*)take(p.groups_cap * n.state_rec * 4);
     }
     if (n.pairs) {
         p.act = take(T * n.act * el);
@@ -240,8 +241,8 @@ int Engine::finalize_plan() {
         p.keys_at = p.has_latent ? T * (sizeof(LatentTile) / 4) : 0;
         p.grouped_at = p.keys_at + 2 * (size_t)p.keys_cap;
         p.seg_at = p.grouped_at + (p.has_grouped ? T * (sizeof(GroupedTile) / 4) : 0);
-        p.order_at = p.seg_at + (p.has_state ? T * (sizeof(StateSegment) / 4) : 0);
-        p.table_ints = p.order_at + (p.has_state ? T : 0);
+        p.groups_at = (p.seg_at + (p.has_state ? (size_t)d.max_batch * (sizeof(StateSegment) / 4) : 0) + 3) / 4 * 4;
+        p.table_ints = p.groups_at + p.groups_cap * state_group(p.f32);
         p.dev_tiles = (int32_t*)take(p.table_ints * 4);
         if (p.table_ints) SP_CUDA_TRY(cudaMallocHost((void**)&p.host_tiles, p.table_ints * 4));
     }
@@ -269,7 +270,7 @@ int Engine::plan_ctx_bucket() const {
 // Tables of the staged tokens, for steps longer than PLAN_ROWS. Host data only: called outside graphs.
 int Engine::plan_stage(int T) {
     PlanState& p = *plan_;
-    p.n_tiles = p.n_keys = p.n_grouped = p.n_seg = 0;
+    p.n_tiles = p.n_keys = p.n_grouped = p.n_seg = p.n_groups = 0;
     if (T <= PLAN_ROWS) return SP_OK;
     if (p.has_latent && !p.f32) plan_stage_latent(T);
     if (p.has_grouped && !p.f32) {
@@ -283,22 +284,19 @@ int Engine::plan_stage(int T) {
     }
     if (p.has_state) {
         StateSegment* seg = reinterpret_cast<StateSegment*>(p.host_tiles + p.seg_at);
-        int32_t* order = p.host_tiles + p.order_at;
-        std::vector<int> count((size_t)d.max_batch, 0), first((size_t)d.max_batch, -1), last((size_t)d.max_batch, -1);
-        for (int i = 0; i < T; ++i) {
-            const int s = p_slot_[i];
-            if (count[s]++ == 0) first[s] = i;
-            last[s] = i;
-        }
-        std::vector<int> at((size_t)d.max_batch, 0);
-        int begin = 0;
+        int32_t* groups = p.host_tiles + p.groups_at;
+        const int group = state_group(p.f32);
+        std::vector<int> count((size_t)d.max_batch, 0), next((size_t)d.max_batch, 0);
+        for (int i = 0; i < T; ++i) ++count[p_slot_[i]];
         for (int s = 0; s < d.max_batch; ++s) {
             if (!count[s]) continue;
-            at[s] = begin;
-            seg[p.n_seg++] = StateSegment{begin, count[s], s, p_pos_[first[s]] == 0, last[s] - first[s] + 1 == count[s] ? first[s] : -1};
-            begin += count[s];
+            const int n = (count[s] + group - 1) / group;
+            next[s] = p.n_groups * group;
+            std::fill(groups + next[s], groups + next[s] + n * group, -1);
+            seg[p.n_seg++] = StateSegment{p.n_groups, n, s, seq_len[s] == count[s]};
+            p.n_groups += n;
         }
-        for (int i = 0; i < T; ++i) order[at[p_slot_[i]]++] = i;
+        for (int i = 0; i < T; ++i) groups[next[p_slot_[i]]++] = i;
     }
     if (p.table_ints) SP_CUDA_TRY(cudaMemcpyAsync(p.dev_tiles, p.host_tiles, p.table_ints * 4, cudaMemcpyHostToDevice, stream));
     return SP_OK;

@@ -71,7 +71,7 @@ struct PlanLayer {
 // Elements per row that the step's buffers need: the largest of all layers.
 struct PlanSizes {
     size_t proj = 0, qn = 0, qabs = 0, qf = 0, olat = 0, mixed = 0, act = 0, act_shared = 0, pairs = 0, kv = 0, lat = 0, part = 0, low = 0,
-           wlogit = 0, state_out = 0, q = 0;
+           wlogit = 0, state_rec = 0, q = 0;
     int experts = 0;
     static void most(size_t& a, size_t b) { a = std::max(a, b); }
 };
@@ -93,19 +93,21 @@ struct PlanState {
     bool has_latent = false, has_grouped = false, has_state = false;
     void *xb = nullptr, *qn = nullptr, *qabs = nullptr, *qf = nullptr, *olat = nullptr, *attn = nullptr, *act = nullptr, *act_shared = nullptr,
          *xs = nullptr, *kvx = nullptr, *lat = nullptr, *fin = nullptr, *q = nullptr, *low = nullptr;
-    float *proj = nullptr, *y = nullptr, *y_expert = nullptr, *y_shared = nullptr, *logit = nullptr, *weight = nullptr, *part = nullptr, *history = nullptr, *wlogit = nullptr, *state_out = nullptr;
+    float *proj = nullptr, *y = nullptr, *y_expert = nullptr, *y_shared = nullptr, *logit = nullptr, *weight = nullptr, *part = nullptr, *history = nullptr, *wlogit = nullptr, *state_rec = nullptr;
     int32_t *pick = nullptr, *tables = nullptr, *host_tiles = nullptr, *dev_tiles = nullptr;
     // sections of host_tiles / dev_tiles, in ints
-    size_t keys_at = 0, grouped_at = 0, seg_at = 0, order_at = 0, table_ints = 0;
+    size_t keys_at = 0, grouped_at = 0, seg_at = 0, groups_at = 0, table_ints = 0;
     MoeTables moe{};
     int keys_cap = 0;          // gathered keys a step may hold
     // the current step, when it is longer than PLAN_ROWS
     int n_tiles = 0, n_keys = 0;        // latent attention: tiles and gathered keys of the expanded form (0 tiles: absorbed)
-    int n_grouped = 0, n_seg = 0;       // grouped attention: tiles; state mixers: segments
+    int n_grouped = 0;                  // grouped attention: tiles
+    int n_seg = 0, n_groups = 0;        // state mixers: segments and groups of tokens
     // states [slot][layer][heads][vdim][dim_pad] and what checkpoint() keeps of each slot
     float *states = nullptr, *checkpoints = nullptr;
     size_t slot_state = 0;              // floats per slot
     std::vector<int> checkpoint_len;    // per slot: tokens the kept state has seen, -1: none
+    size_t groups_cap = 0;              // groups a step may have
     std::map<std::pair<double, int>, const float2*> angles;
     std::vector<void*> owned;
 };

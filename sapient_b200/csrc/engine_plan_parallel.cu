@@ -62,7 +62,7 @@ void PlanPacker::parallel_layer(int i) {
             if (cudaMemcpy(q, m.decay.data(), (size_t)H * 4, cudaMemcpyHostToDevice) != cudaSuccess) { fail(SP_ERR_CUDA, "cudaMemcpy failed"); return; }
             l.decay = (const float*)q;
         }
-        PlanSizes::most(n.state_out, (size_t)hv);
+        PlanSizes::most(n.state_rec, state_record_floats(l.state_shape, p.f32));
     }
     cache_slice(page);
     for (const Part& part : parts) l.mix_rows += part.rows;
@@ -112,7 +112,7 @@ int Engine::plan_state(int li, int T) {
     a.low = p.low;
     a.ldlow = l.w2.kp;
     a.wlogit = p.wlogit;
-    a.o = p.state_out;
+    a.rec = p.state_rec;
     a.gain = l.gain;
     a.tok_slot = d_tok_slot_;
     a.tok_pos = d_tok_pos_;
@@ -124,7 +124,7 @@ int Engine::plan_state(int li, int T) {
         return SP_OK;
     }
     if (l.low_rows) SP_TRY(plan_mat(l.w2, p.low, l.w2.kp, T, p.wlogit, l.w2.n, true));
-    SP_LAUNCH(F_STATE, launch_state_scan(a, (const StateSegment*)(p.dev_tiles + p.seg_at), p.n_seg, p.dev_tiles + p.order_at, T, stream));
+    SP_LAUNCH(F_STATE, launch_state_scan(a, (const StateSegment*)(p.dev_tiles + p.seg_at), p.n_seg, p.dev_tiles + p.groups_at, p.n_groups, stream));
     return SP_OK;
 }
 

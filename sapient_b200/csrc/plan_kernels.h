@@ -235,15 +235,15 @@ struct StateArgs {
     int64_t slot_stride;
     const float* decay;        // STATE_DECAY: [heads]
     // STATE_DECAY: proj[t] = q | k | v (silu applied) | gate logits. STATE_DELTA: r | k | v | removal logits | gate logits.
-    float* proj;
+    const float* proj;
     int ldp;
     const float* a_bias;       // STATE_DELTA: [heads * dim]
     const float* w0;           // STATE_DELTA: decay logit = w0 + W2 low[t]
     const void* w2;            // compute type, [heads * dim][ldlow]
     const void* low;           // compute type, [t][ldlow]
     int ldlow;
-    float* wlogit;             // many rows: W2 low[t] (f32, [t][heads * dim]), overwritten with the decays
-    float* o;                  // many rows: [t][heads * vdim] f32
+    const float* wlogit;       // many rows: W2 low[t] (f32, [t][heads * dim])
+    float* rec;                // many rows: scratch, state_record_floats per group
     const float* gain;         // [heads * vdim]
     const int32_t *tok_slot, *tok_pos;
     void* out;                 // compute type, [t][ldo]
@@ -253,10 +253,14 @@ struct StateArgs {
 // Up to STATE_STEP_ROWS rows: gates, recurrence, norm and output gate in one launch. Rows of one slot are taken in order.
 constexpr int STATE_STEP_ROWS = 32;
 cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st);
-// Any number of rows: a segment is the n rows order[begin .. begin + n) of one slot; row0 >= 0: they are row0, row0 + 1, ...
+// Any number of rows, in groups of up to state_group() tokens of one slot, in order: groups[i][] names their rows (-1 behind the
+// last). A segment is a slot's run of groups.
+constexpr int STATE_GROUP_F32 = 4, STATE_CHUNK = 16;
+inline int state_group(bool f32) { return f32 ? STATE_GROUP_F32 : STATE_CHUNK; }
 struct StateSegment {
-    int32_t begin, n, slot, fresh, row0;  // fresh: starts at position 0
+    int32_t group0, n_groups, slot, fresh;  // fresh: starts at position 0
 };
-cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* order, int n_tok, cudaStream_t st);
+size_t state_record_floats(const StateShape& s, bool f32);  // of a group
+cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* groups, int n_groups, cudaStream_t st);
 
 }  // namespace sp

@@ -11,7 +11,8 @@
 //   * target: ONE forward of the k + 1 rows [pending, d1 .. dk] — each weight matrix is streamed once for all rows —
 //     returning only the k + 1 arg-max ids a0 .. ak (last maximum wins, sampler.rs:161-168);
 //   * accept the longest prefix with d(i+1) == a(i); commit those drafts and a(n), which becomes the next `pending`;
-//   * roll both caches back to the committed tokens (truncate is O(1) on the paged cache); when every draft was
+//   * roll both caches back to the committed tokens (truncate is O(1) on the paged cache; recurrent states come back to a
+//     checkpoint made before the round and take the committed tokens again); when every draft was
 //     accepted the draft model consumes dk, which it had produced but not read.
 // The committed stream equals the target's own greedy decoding token for token; per round the host sees k + (k + 1)
 // token ids instead of 2k + 2 logit vectors.
@@ -21,6 +22,16 @@
 #include "engine.h"
 
 namespace sp {
+
+// Cuts slot 0 to n tokens. A model with recurrent states may come back further than that (to its checkpoint at length
+// `from`) and is fed the tokens in between again: tokens[i] is the one at position from + i.
+static int rewind(Engine* e, int from, int n, const uint32_t* tokens, const std::vector<int32_t>& zeros) {
+    size_t kept = 0;
+    const int st = e->truncate(0, (size_t)n, &kept);
+    if (st != SP_OK || (int)kept == n) return st;
+    if ((int)kept < from) { set_error("spec_greedy: the state at the round's start is gone"); return SP_ERR_STATE; }
+    return e->forward(tokens + (kept - (size_t)from), zeros.data(), n - (int)kept, false, nullptr, nullptr);
+}
 
 int spec_greedy(Engine* target, Engine* draft, const uint32_t* prompt, size_t n_prompt, int k, size_t max_new, const uint32_t* eos,
                 int n_eos, uint32_t* tokens_out, size_t* n_out, uint64_t* stats) {
@@ -48,6 +59,7 @@ int spec_greedy(Engine* target, Engine* draft, const uint32_t* prompt, size_t n_
         // room for pending + k drafts in both windows, else a shorter round
         int kk = std::min<int>(k, std::min(target->d.max_ctx, draft->d.max_ctx) - L - 1);
         if (kk < 1) { set_error("spec_greedy: KV cache full"); *n_out = count; return SP_ERR_KV_FULL; }
+        if ((st = target->checkpoint(0)) != SP_OK || (st = draft->checkpoint(0)) != SP_OK) return st;
         if ((st = draft->decode_greedy(&pending, &slot0, 1, kk, d.data())) != SP_OK) return st;
         rows[0] = pending;
         for (int i = 0; i < kk; ++i) rows[(size_t)i + 1] = d[(size_t)i];
@@ -64,10 +76,9 @@ int spec_greedy(Engine* target, Engine* draft, const uint32_t* prompt, size_t n_
             stop = is_eos(t);
         }
         pending = picks[(size_t)n];
-        size_t kept = 0;
-        if ((st = target->truncate(0, (size_t)(L + 1 + n), &kept)) != SP_OK) return st;
+        if ((st = rewind(target, L, L + 1 + n, rows.data(), zeros)) != SP_OK) return st;
         if (n < kk) {
-            if ((st = draft->truncate(0, (size_t)(L + 1 + n), &kept)) != SP_OK) return st;
+            if ((st = rewind(draft, L, L + 1 + n, rows.data(), zeros)) != SP_OK) return st;
         } else if (!stop && count < max_new) {
             // every draft accepted: the draft model has produced dk but not consumed it
             if ((st = draft->forward(&d[(size_t)kk - 1], zeros.data(), 1, false, nullptr, nullptr)) != SP_OK) return st;

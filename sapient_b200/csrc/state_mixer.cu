@@ -6,8 +6,8 @@
 //   Step (few rows): a block has a whole head, so gates, recurrence, norm and output gate are one launch; where the norm runs
 //   over all heads the blocks of a row are a cluster and exchange their sums of squares. The state is requested before the
 //   previous kernel is waited for: no kernel of the last two before this one writes it.
-//   Scan (many rows): a block has a few columns of a head and walks the tokens, whose vectors arrive in tiles by cp.async; gates
-//   come before and norms after it as kernels of their own.
+//   Scan (many rows): gates and what a group of four tokens owes to itself are made in parallel, then a block with a few columns
+//   of a head walks the groups, then come norm and output gate.
 #include <algorithm>
 
 #include "kernels.h"
@@ -15,6 +15,7 @@
 #include "pdl.cuh"
 #include "plan_common.cuh"
 #include "plan_kernels.h"
+#include "state_common.cuh"
 
 namespace sp {
 
@@ -25,18 +26,6 @@ int state_dim_pad(int dim) {
     while (p < dim) p <<= 1;
     return p;
 }
-
-// Columns of a projection row.
-struct StateCols {
-    int r, k, v, a, g;
-};
-__host__ __device__ __forceinline__ StateCols state_cols(const StateShape& s) {
-    const int hd = s.heads * s.dim, hv = s.heads * s.vdim;
-    return s.rule == STATE_DELTA ? StateCols{0, hd, 2 * hd, 3 * hd, 4 * hd} : StateCols{0, hd, 2 * hd, 0, 2 * hd + hv};
-}
-
-constexpr float EXP_MINUS_HALF = 0.60653065971263342f;
-__device__ __forceinline__ float channel_decay(float logit) { return expf(-EXP_MINUS_HALF * sigmoid_f32(logit)); }
 
 template <int L> __device__ __forceinline__ float lanes_sum(float v) {
 #pragma unroll
@@ -250,116 +239,268 @@ cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st) {
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
-// ── many rows ──
-// A warp per (token, head): decays from their logits (in place), removal rates times the key's inverse square length.
-constexpr int SG_WARPS = 4;
-__global__ void __launch_bounds__(SG_WARPS * 32) state_gates_kernel(const StateArgs a) {
-    pdl_wait();
-    pdl_trigger();
-    const int64_t t = blockIdx.x;
-    const int h = blockIdx.y * SG_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = a.s.dim;
-    if (h >= a.s.heads) return;
-    const StateCols co = state_cols(a.s);
-    float* pr = a.proj + t * a.ldp + h * D;
-    float* wl = a.wlogit + (t * a.s.heads + h) * D;
-    float ss = 0.f;
-    for (int c = lane; c < D; c += 32) ss = fmaf(pr[co.k + c], pr[co.k + c], ss);
-    const float inv = 1.0f / (warp_sum(ss) + 1e-6f);
-    for (int c = lane; c < D; c += 32) {
-        wl[c] = channel_decay(wl[c] + a.w0[h * D + c]);
-        pr[co.a + c] = sigmoid_f32(pr[co.a + c] + a.a_bias[h * D + c]) * inv;
-    }
+// ── many rows, f32 engines (bf16 ones: state_chunk.cu) ──
+// Plain fused multiply-adds. Tokens go in groups of four of one sequence. With c(s, t) the product of the decays of tokens s + 1 .. t (per key channel)
+// and S the state before the group,
+//   d_t = U_t . S + sum_{s < t} Auk[t][s] v_s - Aub[t][s] d_s      what the unit key u_t finds (delta rule)
+//   o_t = R_t . S + sum_{s <= t} Ark[t][s] v_s - Arb[t][s] d_s
+//   S  <- c(0, 4) S + sum_s K_s v_s - B_s d_s
+// where U_t = c(0, t - 1) u_t, R_t = c(0, t) r_t, K_s = c(s, 4) k_s, B_s = c(s, 4) a_s u_s and, summed over the channels,
+// Auk = u_t c(s, t - 1) k_s, Aub = u_t c(s, t - 1) a_s u_s, Ark = r_t c(s, t) k_s, Arb = r_t c(s, t) a_s u_s. So the scan's
+// chain of reductions has a link per group, not per token. Everything but d, o and S is made by a kernel that is parallel
+// over groups and heads; a sequence's last group is filled up with tokens that change nothing (k = r = a = 0, decay 1).
+// Per (group, head) a record: U | R | K | B as [4][dim_pad] each, c(0, 4) (delta; the decaying sum has R | K only), the
+// coefficients, and the values [4][v_pad], where the scan leaves the outputs.
+constexpr int SGRP = STATE_GROUP_F32, A_UB = 8, A_RK = 16, A_RB = 32, A_FLOATS = 48;  // Auk at 0: (t, s < t) in order of t
+struct StateRecord {
+    int k, b, c, a, v, v_pad, floats;  // offsets of U (or R) = 0, ...
+    int r;
+};
+__host__ __device__ __forceinline__ StateRecord state_record(const StateShape& s) {
+    StateRecord r;
+    const int m = SGRP * s.dim_pad;
+    const bool delta = s.rule == STATE_DELTA;
+    r.r = delta ? m : 0;
+    r.k = r.r + m;
+    r.b = r.k + m;
+    r.c = delta ? r.b + m : r.b;
+    r.a = delta ? r.c + s.dim_pad : r.c;
+    r.v = r.a + A_FLOATS;
+    r.v_pad = (s.vdim + 3) & ~3;
+    r.floats = r.v + SGRP * r.v_pad;
+    return r;
 }
+static StateRecordView state_view(const StateShape& s, bool f32) {
+    const StateRecord r = state_record(s);
+    return f32 ? StateRecordView{r.v, r.v_pad, r.floats} : state_chunk_view(s);
+}
+size_t state_record_floats(const StateShape& s, bool f32) { return (size_t)s.heads * state_view(s, f32).floats; }
 
-// A block per token: norms of the heads (delta) or of all of them together, gain, gate.
-constexpr int SN_WARPS = 8;
-template <typename T>
-__global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateArgs a) {
-    __shared__ float sh[SN_WARPS];
-    pdl_wait();
-    pdl_trigger();
-    const int64_t t = blockIdx.x;
-    const int H = a.s.heads, V = a.s.vdim, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const float *o = a.o + t * H * V, *g = a.proj + t * a.ldp + state_cols(a.s).g;
-    T* out = reinterpret_cast<T*>(a.out) + t * a.ldo;
-    auto finish = [&](int i, float r) { out[i] = from_f32<T>(o[i] * r * a.gain[i] * sigmoid_f32(g[i])); };
-    if (a.s.rule == STATE_DELTA) {
-        for (int h = warp; h < H; h += SN_WARPS) {
-            float ss = 0.f;
-            for (int i = lane; i < V; i += 32) ss = fmaf(o[h * V + i], o[h * V + i], ss);
-            const float r = rsqrtf(warp_sum(ss) / (float)V + a.s.eps);
-            for (int i = lane; i < V; i += 32) finish(h * V + i, r);
+// Sums p[i] over the warp for all i at once: lane i receives the sum of p[i].
+__device__ __forceinline__ float warp_sums(float (&p)[32]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) {
+        const bool up = lane & m;
+#pragma unroll
+        for (int i = 0; i < m; ++i) {
+            const float send = up ? p[i] : p[i + m], keep = up ? p[i + m] : p[i];
+            p[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, m);
         }
-        return;
     }
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < H * V; i += SN_WARPS * 32) ss = fmaf(o[i], o[i], ss);
-    const float r = rsqrtf(block_sum<SN_WARPS>(ss, sh) / (float)(H * V) + a.s.eps);
-    for (int i = threadIdx.x; i < H * V; i += SN_WARPS * 32) finish(i, r);
+    return p[0];
 }
 
-__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_addr(dst)), "l"(src) : "memory");
+// A warp per (group, head).
+constexpr int SG_WARPS = 4;
+template <bool DELTA>
+__global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const StateArgs a, const int4* __restrict__ groups) {
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y * SG_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = a.s.dim, DP = a.s.dim_pad, V = a.s.vdim, H = a.s.heads;
+    if (h >= H) return;
+    const StateCols co = state_cols(a.s);
+    const StateRecord rec = state_record(a.s);
+    float* out = a.rec + ((int64_t)blockIdx.x * H + h) * rec.floats;
+    const int4 g4 = groups[blockIdx.x];
+    const int row[SGRP] = {g4.x, g4.y, g4.z, g4.w};
+    const float* pr[SGRP];
+#pragma unroll
+    for (int t = 0; t < SGRP; ++t) pr[t] = a.proj + (int64_t)max(row[t], 0) * a.ldp;
+    float inv[SGRP] = {};  // 1 / |k|
+    if (DELTA) {
+        for (int c = lane; c < D; c += 32)
+#pragma unroll
+            for (int t = 0; t < SGRP; ++t) {
+                const float k = pr[t][co.k + h * D + c];
+                inv[t] = fmaf(k, k, inv[t]);
+            }
+#pragma unroll
+        for (int t = 0; t < SGRP; ++t) inv[t] = 1.0f / sqrtf(warp_sum(inv[t]) + 1e-6f);
+    }
+    const float decay = DELTA ? 0.f : a.decay[h];
+    float p[32];  // Auk, Aub (t, s < t), then Ark, Arb (t, s <= t); the decaying sum: Ark alone
+#pragma unroll
+    for (int i = 0; i < 32; ++i) p[i] = 0.f;
+    float whole = 1.f;
+    for (int c = lane; c < DP; c += 32) {
+        const bool on = c < D;
+        const int hc = h * D + min(c, D - 1);
+        float k[SGRP], r[SGRP], w[SGRP], u[SGRP], b[SGRP];
+#pragma unroll
+        for (int t = 0; t < SGRP; ++t) {
+            const bool live = on && row[t] >= 0;
+            k[t] = live ? pr[t][co.k + hc] : 0.f;
+            r[t] = live ? pr[t][co.r + hc] : 0.f;
+            w[t] = row[t] < 0 ? 1.f : decay;
+            if (DELTA) {
+                w[t] = live ? channel_decay(a.wlogit[(int64_t)row[t] * H * D + hc] + a.w0[hc]) : 1.f;
+                u[t] = k[t] * inv[t];
+                b[t] = live ? u[t] * sigmoid_f32(pr[t][co.a + hc] + a.a_bias[hc]) : 0.f;
+            }
+        }
+        int i = 0;
+        if (DELTA) {
+#pragma unroll
+            for (int t = 1; t < SGRP; ++t)
+#pragma unroll
+                for (int s = 0; s < t; ++s, ++i) {
+                    float q = u[t];
+#pragma unroll
+                    for (int j = s + 1; j < t; ++j) q *= w[j];
+                    p[i] = fmaf(q, k[s], p[i]);
+                    p[6 + i] = fmaf(q, b[s], p[6 + i]);
+                }
+            i = 12;
+        }
+#pragma unroll
+        for (int t = 0; t < SGRP; ++t)
+#pragma unroll
+            for (int s = 0; s <= t; ++s, ++i) {
+                float q = r[t];
+#pragma unroll
+                for (int j = s + 1; j <= t; ++j) q *= w[j];
+                p[i] = fmaf(q, k[s], p[i]);
+                if (DELTA) p[10 + i] = fmaf(q, b[s], p[10 + i]);
+            }
+        float before = 1.f, after = 1.f;
+#pragma unroll
+        for (int t = 0; t < SGRP; ++t) {
+            if (DELTA) out[t * DP + c] = before * u[t];
+            before *= w[t];
+            out[rec.r + t * DP + c] = before * r[t];
+        }
+#pragma unroll
+        for (int t = SGRP - 1; t >= 0; --t) {
+            out[rec.k + t * DP + c] = after * k[t];
+            if (DELTA) out[rec.b + t * DP + c] = after * b[t];
+            after *= w[t];
+        }
+        if (DELTA) out[rec.c + c] = before;
+        whole = before;
+    }
+    const float sum = warp_sums(p);
+    // lane -> (t, s) of its coefficient; the upper triangles stay zero
+    float* A = out + rec.a;
+    for (int i = lane; i < A_FLOATS; i += 32) A[i] = 0.f;
+    __syncwarp();
+    const int first = DELTA ? 12 : 0;
+    if (DELTA && lane < 12) A[lane < 6 ? lane : A_UB + lane - 6] = sum;
+    else if (lane >= first && lane < first + (DELTA ? 20 : 10)) {
+        const int i = lane - first, q = i % 10, t = q >= 6 ? 3 : q >= 3 ? 2 : q >= 1 ? 1 : 0;
+        A[(i >= 10 ? A_RB : A_RK) + 4 * t + q - t * (t + 1) / 2] = sum;
+    }
+    if (!DELTA && lane == 0) A[0] = whole;
+    for (int c = lane; c < rec.v_pad; c += 32)
+#pragma unroll
+        for (int t = 0; t < SGRP; ++t) out[rec.v + t * rec.v_pad + c] = c < V && row[t] >= 0 ? pr[t][co.v + h * V + c] : 0.f;
 }
 
-// Block (columns, head, segment). Tiles of tb tokens in two stages: per token the vectors k, r (, w, a) of dim_pad floats and
-// the block's values.
-constexpr int SC_WARPS = 4, SC_THREADS = SC_WARPS * 32;
+// Block (SC_COLS columns, head, segment); records arrive in tiles of tg groups, two stages of cp.async.
+constexpr int SC_COLS = 16;
 template <int L, int R, bool DELTA>
-__global__ void __launch_bounds__(SC_THREADS) state_scan_kernel(const StateArgs a, const StateSegment* __restrict__ segs, const int32_t* __restrict__ order, int tb) {
+__global__ void __launch_bounds__(SC_COLS * L) state_scan_kernel(const StateArgs a, const StateSegment* __restrict__ segs, int tg) {
     extern __shared__ __align__(16) float sc_smem[];
-    constexpr int DP = 4 * L * R, NV = DELTA ? 4 : 2, COLS = SC_THREADS / L, TOK = NV * DP + COLS;  // floats per token
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, l = tid % L, H = a.s.heads, D = a.s.dim, V = a.s.vdim;
-    const int h = blockIdx.y, col0 = blockIdx.x * COLS, col = col0 + tid / L;
-    for (int i = tid; i < 2 * tb * TOK; i += SC_THREADS) sc_smem[i] = 0.f;  // the padding stays zero
+    constexpr int DP = 4 * L * R, THREADS = SC_COLS * L;
+    const int tid = threadIdx.x, l = tid % L, cl = tid / L, H = a.s.heads, V = a.s.vdim, h = blockIdx.y, col0 = blockIdx.x * SC_COLS, col = col0 + cl;
+    const StateRecord rec = state_record(a.s);
+    const int stage = rec.v + SGRP * SC_COLS;  // floats of a group in shared memory: the record with this block's values only
     pdl_wait();
     pdl_trigger();
     const StateSegment sg = segs[blockIdx.z];
-    const StateCols co = state_cols(a.s);
     float* state = a.state + sg.slot * a.slot_stride + ((int64_t)h * V + col) * DP + 4 * l;
     float4 st[R];
 #pragma unroll
-    for (int i = 0; i < R; ++i) st[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (col < V && !sg.fresh)
-#pragma unroll
-        for (int i = 0; i < R; ++i) st[i] = *reinterpret_cast<const float4*>(state + 4 * L * i);
-    const float decay = DELTA ? 0.f : a.decay[h];
-    const bool wide = D % 4 == 0 && a.ldp % 4 == 0, wide_v = wide && V % 4 == 0;
-    auto row_of = [&](int i) { return (int64_t)(sg.row0 >= 0 ? sg.row0 + i : order[sg.begin + i]); };
-    const int nv = min(COLS, V - col0);
-    auto fetch = [&](int i0, int buf) {
-        for (int k = warp; k < tb && i0 + k < sg.n; k += SC_WARPS) {
-            const int64_t row = row_of(i0 + k);
-            const float* pr = a.proj + row * a.ldp;
-            float* d = sc_smem + (buf * tb + k) * TOK;
-            const float* src[4] = {pr + co.k + h * D, pr + co.r + h * D, DELTA ? a.wlogit + (row * H + h) * D : nullptr, DELTA ? pr + co.a + h * D : nullptr};
-            const float* v = pr + co.v + h * V + col0;
-#pragma unroll
-            for (int q = 0; q < NV; ++q) {
-                if (wide)
-                    for (int c = 4 * lane; c < D; c += 128) cp_async16(d + q * DP + c, src[q] + c, 16);
-                else
-                    for (int c = lane; c < D; c += 32) cp_async4(d + q * DP + c, src[q] + c);
-            }
-            if (wide_v)
-                for (int c = 4 * lane; c < nv; c += 128) cp_async16(d + NV * DP + c, v + c, 16);
-            else
-                for (int c = lane; c < nv; c += 32) cp_async4(d + NV * DP + c, v + c);
+    for (int i = 0; i < R; ++i) st[i] = col < V && !sg.fresh ? *reinterpret_cast<const float4*>(state + 4 * L * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float* const first = a.rec + ((int64_t)sg.group0 * H + h) * rec.floats;
+    const int64_t step = (int64_t)H * rec.floats;
+    const int v_pieces = min(SC_COLS, rec.v_pad - col0) / 4;
+    auto fetch = [&](int g0, int buf) {
+        for (int k = 0; k < tg && g0 + k < sg.n_groups; ++k) {
+            const float* src = first + (g0 + k) * step;
+            float* d = sc_smem + (buf * tg + k) * stage;
+            for (int i = 4 * tid; i < rec.v; i += 4 * THREADS) cp_async16(d + i, src + i, 16);
+            const int t = tid / (SC_COLS / 4), q = tid % (SC_COLS / 4);
+            if (t < SGRP && q < v_pieces) cp_async16(d + rec.v + t * SC_COLS + 4 * q, src + rec.v + t * rec.v_pad + col0 + 4 * q, 16);
         }
     };
-    __syncthreads();
     fetch(0, 0);
     cp_async_commit();
-    for (int i0 = 0, buf = 0; i0 < sg.n; i0 += tb, buf ^= 1) {
-        if (i0 + tb < sg.n) fetch(i0 + tb, buf ^ 1);
+    // the token whose output this lane finishes, after the exchange below
+    const int mine = 2 * (l & 1) + ((l >> 1) & 1);
+    for (int g0 = 0, buf = 0; g0 < sg.n_groups; g0 += tg, buf ^= 1) {
+        if (g0 + tg < sg.n_groups) fetch(g0 + tg, buf ^ 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        const float* d = sc_smem + buf * tb * TOK;
-        const int n = min(tb, sg.n - i0);
-        for (int k = 0; k < n; ++k, d += TOK) {
-            const float o = state_token<L, R, DELTA>(st, d, d + DP, d + 2 * DP, d + 3 * DP, decay, d[NV * DP + tid / L], l);
-            if (l == 0 && col < V) a.o[(row_of(i0 + k) * H + h) * V + col] = o;
+        const int n = min(tg, sg.n_groups - g0);
+        for (int k = 0; k < n; ++k) {
+            const float* d = sc_smem + (buf * tg + k) * stage;
+            const float* A = d + rec.a;
+            float v[SGRP], e[SGRP] = {}, f[SGRP] = {};
+#pragma unroll
+            for (int t = 0; t < SGRP; ++t) v[t] = d[rec.v + t * SC_COLS + cl];
+#pragma unroll
+            for (int i = 0; i < R; ++i) {
+                const int at = 4 * (l + L * i);
+#pragma unroll
+                for (int t = 0; t < SGRP; ++t) {
+                    if (DELTA) {
+                        const float4 u = *reinterpret_cast<const float4*>(d + t * DP + at);
+                        e[t] = fmaf(u.x, st[i].x, fmaf(u.y, st[i].y, fmaf(u.z, st[i].z, fmaf(u.w, st[i].w, e[t]))));
+                    }
+                    const float4 r = *reinterpret_cast<const float4*>(d + rec.r + t * DP + at);
+                    f[t] = fmaf(r.x, st[i].x, fmaf(r.y, st[i].y, fmaf(r.z, st[i].z, fmaf(r.w, st[i].w, f[t]))));
+                }
+            }
+            if (DELTA) {
+#pragma unroll
+                for (int t = 0; t < SGRP; ++t) e[t] = lanes_sum<L>(e[t]);
+                const float4 k0 = *reinterpret_cast<const float4*>(A), b0 = *reinterpret_cast<const float4*>(A + A_UB);
+                const float2 k1 = *reinterpret_cast<const float2*>(A + 4), b1 = *reinterpret_cast<const float2*>(A + A_UB + 4);
+                e[1] = fmaf(k0.x, v[0], fmaf(-b0.x, e[0], e[1]));
+                e[2] = fmaf(k0.y, v[0], fmaf(k0.z, v[1], fmaf(-b0.y, e[0], fmaf(-b0.z, e[1], e[2]))));
+                e[3] = fmaf(k0.w, v[0], fmaf(k1.x, v[1], fmaf(k1.y, v[2], fmaf(-b0.w, e[0], fmaf(-b1.x, e[1], fmaf(-b1.y, e[2], e[3]))))));
+            }
+            const float whole = DELTA ? 0.f : A[0];
+#pragma unroll
+            for (int i = 0; i < R; ++i) {
+                const int at = 4 * (l + L * i);
+                float4 c = make_float4(whole, whole, whole, whole);
+                if (DELTA) c = *reinterpret_cast<const float4*>(d + rec.c + at);
+                st[i].x *= c.x; st[i].y *= c.y; st[i].z *= c.z; st[i].w *= c.w;
+#pragma unroll
+                for (int t = 0; t < SGRP; ++t) {
+                    const float4 q = *reinterpret_cast<const float4*>(d + rec.k + t * DP + at);
+                    st[i].x = fmaf(q.x, v[t], st[i].x);
+                    st[i].y = fmaf(q.y, v[t], st[i].y);
+                    st[i].z = fmaf(q.z, v[t], st[i].z);
+                    st[i].w = fmaf(q.w, v[t], st[i].w);
+                    if (DELTA) {
+                        const float4 b = *reinterpret_cast<const float4*>(d + rec.b + t * DP + at);
+                        st[i].x = fmaf(-b.x, e[t], st[i].x);
+                        st[i].y = fmaf(-b.y, e[t], st[i].y);
+                        st[i].z = fmaf(-b.z, e[t], st[i].z);
+                        st[i].w = fmaf(-b.w, e[t], st[i].w);
+                    }
+                }
+            }
+            // the lanes of a column share out the four outputs while they sum them
+            {
+                const bool up = l & 1, up2 = l & 2;
+                const float x = (up ? f[2] : f[0]) + __shfl_xor_sync(0xFFFFFFFFu, up ? f[0] : f[2], 1);
+                const float y = (up ? f[3] : f[1]) + __shfl_xor_sync(0xFFFFFFFFu, up ? f[1] : f[3], 1);
+                float o = (up2 ? y : x) + __shfl_xor_sync(0xFFFFFFFFu, up2 ? x : y, 2);
+#pragma unroll
+                for (int m = 4; m < L; m <<= 1) o += __shfl_xor_sync(0xFFFFFFFFu, o, m);
+                const float4 q = *reinterpret_cast<const float4*>(A + A_RK + 4 * mine);
+                o = fmaf(q.x, v[0], fmaf(q.y, v[1], fmaf(q.z, v[2], fmaf(q.w, v[3], o))));
+                if (DELTA) {
+                    const float4 b = *reinterpret_cast<const float4*>(A + A_RB + 4 * mine);
+                    o = fmaf(-b.x, e[0], fmaf(-b.y, e[1], fmaf(-b.z, e[2], fmaf(-b.w, e[3], o))));
+                }
+                if (l < 4 && col < V) first[(g0 + k) * step + rec.v + mine * rec.v_pad + col] = o;
+            }
         }
         __syncthreads();
     }
@@ -369,42 +510,90 @@ __global__ void __launch_bounds__(SC_THREADS) state_scan_kernel(const StateArgs 
         for (int i = 0; i < R; ++i) *reinterpret_cast<float4*>(state + 4 * L * i) = st[i];
 }
 
+// Norms of the scan's outputs, gain, gate. Delta: a warp per (token, head); else a block per token, for the norm is over all heads.
+constexpr int SN_WARPS = 8, SN_KEEP = 4;  // values a lane keeps in registers
+template <typename T, bool DELTA>
+__global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateArgs a, const StateRecordView rec, const int32_t* __restrict__ groups, int group) {
+    __shared__ float sh[SN_WARPS];
+    pdl_wait();
+    pdl_trigger();
+    const int H = a.s.heads, V = a.s.vdim, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x % group;
+    const int64_t row = groups[blockIdx.x];
+    if (row < 0) return;
+    const float *o = a.rec + (int64_t)(blockIdx.x / group) * H * rec.floats + rec.v + t * rec.v_pad, *g = a.proj + row * a.ldp + state_cols(a.s).g;
+    T* out = reinterpret_cast<T*>(a.out) + row * a.ldo;
+    auto finish = [&](int h, int i, float v, float r) { out[h * V + i] = from_f32<T>(v * r * a.gain[h * V + i] * sigmoid_f32(g[h * V + i])); };
+    if (DELTA) {
+        const int h = blockIdx.y * SN_WARPS + warp;
+        if (h >= H) return;
+        const float* oh = o + (int64_t)h * rec.floats;
+        float v[SN_KEEP], ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < SN_KEEP; ++j) {
+            v[j] = lane + 32 * j < V ? oh[lane + 32 * j] : 0.f;
+            ss = fmaf(v[j], v[j], ss);
+        }
+        for (int i = lane + 32 * SN_KEEP; i < V; i += 32) ss = fmaf(oh[i], oh[i], ss);
+        const float r = rsqrtf(warp_sum(ss) / (float)V + a.s.eps);
+#pragma unroll
+        for (int j = 0; j < SN_KEEP; ++j)
+            if (lane + 32 * j < V) finish(h, lane + 32 * j, v[j], r);
+        for (int i = lane + 32 * SN_KEEP; i < V; i += 32) finish(h, i, oh[i], r);
+        return;
+    }
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H * V; i += SN_WARPS * 32) {
+        const float v = o[(int64_t)(i / V) * rec.floats + i % V];
+        ss = fmaf(v, v, ss);
+    }
+    const float r = rsqrtf(block_sum<SN_WARPS>(ss, sh) / (float)(H * V) + a.s.eps);
+    for (int i = threadIdx.x; i < H * V; i += SN_WARPS * 32) finish(i / V, i % V, o[(int64_t)(i / V) * rec.floats + i % V], r);
+}
+
 template <int L, int R, bool DELTA>
-static cudaError_t state_scan_launch(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* order, cudaStream_t st) {
-    constexpr int COLS = SC_THREADS / L, TOK = (DELTA ? 4 : 2) * 4 * L * R + COLS, CAP = 96 * 1024;
-    int tb = 16;
-    while (tb > 2 && 2 * tb * TOK * 4 > CAP) tb >>= 1;
+static cudaError_t state_scan_launch(const StateArgs& a, const StateSegment* seg, int n_seg, cudaStream_t st) {
+    constexpr int CAP = 96 * 1024;
+    const size_t group = (size_t)(state_record(a.s).v + SGRP * SC_COLS) * 4;
+    int tg = 4;
+    while (tg > 1 && 2 * tg * group > CAP) tg >>= 1;
     static PerDeviceOnce once;
     const cudaError_t le = once.run([] { return cudaFuncSetAttribute(state_scan_kernel<L, R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP); });
     if (le != cudaSuccess) return le;
-    return launch_pdl(state_scan_kernel<L, R, DELTA>, dim3((a.s.vdim + COLS - 1) / COLS, a.s.heads, n_seg), dim3(SC_THREADS), (size_t)2 * tb * TOK * 4, st, a, seg,
-                      order, tb);
+    return launch_pdl(state_scan_kernel<L, R, DELTA>, dim3((a.s.vdim + SC_COLS - 1) / SC_COLS, a.s.heads, n_seg), dim3(SC_COLS * L), 2 * tg * group, st, a, seg, tg);
 }
 
-cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* order, int n_tok, cudaStream_t st) {
-    if (n_tok == 0 || n_seg == 0) return cudaSuccess;
-    if (a.s.dim > STATE_MAX_DIM || a.s.dim_pad != state_dim_pad(a.s.dim)) return cudaErrorInvalidValue;
+static cudaError_t launch_state_groups(const StateArgs& a, const StateSegment* seg, int n_seg, const int4* groups, int n_groups, cudaStream_t st) {
     const bool delta = a.s.rule == STATE_DELTA;
-    cudaError_t le = cudaSuccess;
-    if (delta) {
-        le = launch_pdl(state_gates_kernel, dim3(n_tok, (a.s.heads + SG_WARPS - 1) / SG_WARPS), dim3(SG_WARPS * 32), 0, st, a);
-        if (le == cudaSuccess) le = count_launch_and_check();
-        if (le != cudaSuccess) return le;
-    }
+    const dim3 pg(n_groups, (a.s.heads + SG_WARPS - 1) / SG_WARPS);
+    cudaError_t le = delta ? launch_pdl(state_prepare_kernel<true>, pg, dim3(SG_WARPS * 32), 0, st, a, groups) : launch_pdl(state_prepare_kernel<false>, pg, dim3(SG_WARPS * 32), 0, st, a, groups);
+    if (le == cudaSuccess) le = count_launch_and_check();
+    if (le != cudaSuccess) return le;
     le = cudaErrorInvalidValue;
-#define SP_SC(L, R) le = delta ? state_scan_launch<L, R, true>(a, seg, n_seg, order, st) : state_scan_launch<L, R, false>(a, seg, n_seg, order, st)
+#define SP_SC(L, R) le = delta ? state_scan_launch<L, R, true>(a, seg, n_seg, st) : state_scan_launch<L, R, false>(a, seg, n_seg, st)
     switch (a.s.dim_pad) {
         case 16: SP_SC(4, 1); break;
-        case 32: SP_SC(4, 2); break;
+        case 32: SP_SC(8, 1); break;
         case 64: SP_SC(8, 2); break;
-        case 128: SP_SC(8, 4); break;
+        case 128: SP_SC(16, 2); break;
         case 256: SP_SC(16, 4); break;
         case 512: SP_SC(32, 4); break;
     }
 #undef SP_SC
-    if (le == cudaSuccess) le = count_launch_and_check();
+    return le != cudaSuccess ? le : count_launch_and_check();
+}
+
+cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n_seg, const int32_t* groups, int n_groups, cudaStream_t st) {
+    if (n_groups == 0 || n_seg == 0) return cudaSuccess;
+    if (a.s.dim > STATE_MAX_DIM || a.s.dim_pad != state_dim_pad(a.s.dim)) return cudaErrorInvalidValue;
+    cudaError_t le = a.f32 ? launch_state_groups(a, seg, n_seg, reinterpret_cast<const int4*>(groups), n_groups, st) : launch_state_chunks(a, seg, n_seg, groups, n_groups, st);
     if (le != cudaSuccess) return le;
-    le = a.f32 ? launch_pdl(state_norm_kernel<float>, dim3(n_tok), dim3(SN_WARPS * 32), 0, st, a) : launch_pdl(state_norm_kernel<bf16>, dim3(n_tok), dim3(SN_WARPS * 32), 0, st, a);
+    const bool delta = a.s.rule == STATE_DELTA;
+    const int group = state_group(a.f32);
+    const dim3 grid(n_groups * group, delta ? (a.s.heads + SN_WARPS - 1) / SN_WARPS : 1), block(SN_WARPS * 32);
+    const StateRecordView rec = state_view(a.s, a.f32);
+#define SP_SN(T, D) launch_pdl(state_norm_kernel<T, D>, grid, block, 0, st, a, rec, groups, group)
+    le = a.f32 ? (delta ? SP_SN(float, true) : SP_SN(float, false)) : (delta ? SP_SN(bf16, true) : SP_SN(bf16, false));
+#undef SP_SN
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 

@@ -1,7 +1,7 @@
 """Throughput of layer-plan designs beside the framework's closest GGUF block at equal size (`bench.py --design NAME`).
 
 Per size: the design with random bf16 weights, and a Llama block of the same width, heads, layers and ACTIVE feed-forward
-width (chosen experts + shared expert) in Q8_0 — prefill of one prompt, greedy decode at batch 1 and 32, device time by
+weights in Q8_0 — prefill of one prompt, greedy decode at batch 1 and 32, device time by
 CUDA events, and for each family of kernels of a decode step and of a prefill its device time, algorithmic bytes and flops
 and the fraction of the roofline max(bytes / copy bandwidth, flops / GEMM rate) that is. Weights exceed L2 at every size.
 """
@@ -15,25 +15,50 @@ from . import synth
 from .configs_bench import _engine, _timed
 from .engine import ForwardEngine
 
-# name -> (design keywords)
-SIZES = {
+# design -> size -> keywords of its configuration
+LEPALORN = {
     "2b": dict(layers=6, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, experts=64, top=6, ff=1408, shared_ff=2816,
                vocab=32768, shared_latent_from=3),
     "8b": dict(layers=4, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, experts=32, top=4, ff=2048, shared_ff=2048,
                vocab=32768, shared_latent_from=2),
 }
+_PATTERN = ["general_delta", "general_delta", "attention", "lightning"]
+TEDELIX = {
+    "2b": dict(layers=_PATTERN * 2, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, state_heads=32, state_dim=64, state_vdim=64, window=1024, ff=6144, vocab=32768),
+    "8b": dict(layers=_PATTERN, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, state_heads=64, state_dim=64, state_vdim=64, window=2048, ff=12288, vocab=32768),
+}
+TEDELIX_RANK = 64  # of the decay logits
 
 
-def llama_like(s: dict) -> dict:
-    return dict(arch="llama", n_layers=s["layers"], hidden=s["width"], n_heads=s["heads"], n_kv_heads=s["heads"], head_dim=128,
-                ffn=s["top"] * s["ff"] + s["shared_ff"], vocab=s["vocab"], norm_eps=1e-5, rope_theta=1e4, tied=False)
+def lepalorn_llama(s: dict) -> dict:
+    """Same width, heads, layers and active feed-forward width."""
+    return _llama(s, s["layers"], s["heads"], s["top"] * s["ff"] + s["shared_ff"])
 
 
-def design_engine(s: dict, **kw):
+def tedelix_llama(s: dict) -> dict:
+    """Same width, heads, layers and feed-forward weights (three matrices for two)."""
+    return _llama(s, len(s["layers"]), s["kv_heads"], 2 * s["ff"] // 3)
+
+
+def _llama(s: dict, layers: int, kv_heads: int, ffn: int) -> dict:
+    return dict(arch="llama", n_layers=layers, hidden=s["width"], n_heads=s["heads"], n_kv_heads=kv_heads, head_dim=128, ffn=ffn, vocab=s["vocab"],
+                norm_eps=1e-5, rope_theta=1e4, tied=False)
+
+
+def lepalorn_model(s: dict):
+    cfg = synth.lepalorn_config(**s)
+    return cfg, synth.lepalorn_weights(cfg, seed=11, device="cuda")
+
+
+def tedelix_model(s: dict):
+    cfg = synth.tedelix_config(**s)
+    return cfg, synth.tedelix_weights(cfg, seed=11, rank=TEDELIX_RANK, device="cuda")
+
+
+def design_engine(cfg: dict, W: dict, **kw):
     import torch
 
-    cfg = synth.lepalorn_config(**s)
-    W = {k: v.cpu() for k, v in synth.lepalorn_weights(cfg, seed=11, device="cuda").items()}
+    W = {k: v.cpu() for k, v in W.items()}
     torch.cuda.empty_cache()
     eng = ForwardEngine.from_config(cfg, W, **kw)
     stream = torch.cuda.Stream()
@@ -42,10 +67,10 @@ def design_engine(s: dict, **kw):
     return eng, stream
 
 
-def llama_engine(s: dict, max_ctx: int, **kw):
+def llama_engine(shape: dict, max_ctx: int, **kw):
     import torch
 
-    cfg, W = synth.build_model(llama_like(s), seed=12, device="cuda", max_ctx=max_ctx, dtype=synth.Q8_0)
+    cfg, W = synth.build_model(shape, seed=12, device="cuda", max_ctx=max_ctx, dtype=synth.Q8_0)
     W = synth.weights_to_numpy(W)
     torch.cuda.empty_cache()
     eng, stream = _engine(cfg, W, **kw)
@@ -63,7 +88,7 @@ def _pairs(n: int, window: int) -> int:
     return w * (w + 1) // 2 + (n - w) * w
 
 
-def design_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+def lepalorn_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
     """Algorithmic (bytes, flops) of one step by kernel family. Prefill: one sequence of `rows` tokens; decode: `rows`
     sequences with `ctx` cached tokens each."""
     L, W, H, D, R, V, K, E = s["layers"], s["width"], s["heads"], s["dim"], s["rot"], s["vdim"], s["rank"], s["experts"]
@@ -81,15 +106,37 @@ def design_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
             "rope_kv": (rows * 6 * (L * H * (D + R) + own * (K + R)), 0)}
 
 
-def llama_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
-    c = llama_like(s)
-    q = c["n_heads"] * c["head_dim"]
-    mats = c["n_layers"] * (4 * q * c["hidden"] + 3 * c["ffn"] * c["hidden"])
+def tedelix_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    """The same. State mixers: what enters them (f32 rows) and leaves, and the states read and written once per step; bytes only,
+    their arithmetic is not tensor-core work."""
+    W, H, G, D, V, HS, DS, VS, F = (s[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "state_heads", "state_dim", "state_vdim", "ff"))
+    n = {t: s["layers"].count(t) for t in ("attention", "lightning", "general_delta")}
+    L, hd, hv, R = len(s["layers"]), HS * DS, HS * VS, TEDELIX_RANK
+    mats = 2 * L * F * W + n["attention"] * (H * D + G * (D + V) + H * V) * W + n["lightning"] * (2 * hd + 3 * hv) * W
+    mats += n["general_delta"] * ((6 * hd + R) * W + hd * R)
+    head = s["vocab"] * W
+    keys = _pairs(rows, s["window"]) if prefill else rows * min(ctx, s["window"])
+    seqs = 1 if prefill else rows
+    states = 8 * seqs * (n["lightning"] * HS * DS * VS + n["general_delta"] * HS * DS * DS)
+    return {"gemv": (2 * (mats + head), 2 * rows * mats + 2 * head * (1 if prefill else rows)),
+            "attention": (n["attention"] * 2 * (G * (D + V) * (rows if prefill else keys) + rows * H * (D + V)), n["attention"] * 2 * H * (D + V) * keys),
+            "state": (states + rows * (n["lightning"] * (4 * (2 * hd + 2 * hv) + 2 * hv) + n["general_delta"] * (4 * 5 * hd + 2 * hd)), 0),
+            "norm": (rows * W * 6 * L, 0), "rope_kv": (rows * n["attention"] * 6 * (H * D + G * (D + V)), 0)}
+
+
+def llama_work(c: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    q, kv = c["n_heads"] * c["head_dim"], c["n_kv_heads"] * c["head_dim"]
+    mats = c["n_layers"] * (2 * (q + kv) * c["hidden"] + 3 * c["ffn"] * c["hidden"])
     head = c["vocab"] * c["hidden"]
     keys = _pairs(rows, 1 << 30) if prefill else rows * ctx
     return {"gemv": (34 / 32 * (mats + head), 2 * rows * mats + 2 * head * (1 if prefill else rows)),
-            "attention": (c["n_layers"] * 2 * 2 * q * (rows if prefill else keys), c["n_layers"] * 4 * q * keys),
-            "norm": (rows * c["hidden"] * c["n_layers"] * 2 * 8, 0), "rope_kv": (rows * c["n_layers"] * q * (12 + 4 + 4), 0)}
+            "attention": (c["n_layers"] * 2 * 2 * kv * (rows if prefill else keys), c["n_layers"] * 4 * q * keys),
+            "norm": (rows * c["hidden"] * c["n_layers"] * 2 * 8, 0), "rope_kv": (rows * c["n_layers"] * (8 * q + 6 * 2 * kv), 0)}
+
+
+# design -> (sizes, model of a size, its work, the Llama block of equal size)
+DESIGNS = {"lepalorn": ("Lepalorn", LEPALORN, lepalorn_model, lepalorn_work, lepalorn_llama),
+           "tedelix": ("Tedelix", TEDELIX, tedelix_model, tedelix_work, tedelix_llama)}
 
 
 def _families(ms: dict, work: dict, peaks: dict) -> dict:
@@ -135,26 +182,29 @@ def measure(eng, stream, vocab: int, work, prompt: int, ctx: int, batch: int, st
         toks = eng.decode_greedy(first, slots, 8)
         ms = _timed(stream, lambda: eng.decode_greedy(toks[-1], slots, steps, fetch=False)) / steps
         eng.synchronize()
-        fam = {f: eng.time_families(f, b, 20) for f in eng.PROFILE_FAMILIES}
-        res[f"decode_b{b}"] = {"ctx": ctx, "ms_per_step": round(ms, 4), "tokens_per_s": round(b / ms * 1e3), "families": _families(fam, work(b, ctx, False), peaks)}
+        todo = work(b, ctx, False)
+        fam = {f: eng.time_families(f, b, 20) for f in eng.PROFILE_FAMILIES if f != "state" or f in todo}
+        res[f"decode_b{b}"] = {"ctx": ctx, "ms_per_step": round(ms, 4), "tokens_per_s": round(b / ms * 1e3), "families": _families(fam, todo, peaks)}
     return res
 
 
 def run(design: str, peaks: dict, sizes=None, prompt: int = 2048, ctx: int = 1024, batch: int = 32, steps: int = 32, designs_only: bool = False) -> dict:
-    if design.lower() != "lepalorn":
+    if design.lower() not in DESIGNS:
         raise SystemExit(f"no such design: {design}")
-    out = {"design": "Lepalorn", "data": "synthetic random weights", "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
+    title, all_sizes, model, design_work, llama_like = DESIGNS[design.lower()]
+    out = {"design": title, "data": "synthetic random weights", "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
     kw = dict(max_batch=batch, max_tokens=prompt, kv_pages=(max(prompt, 0) + batch * (ctx + 256)) // 16)
-    for name in sizes or SIZES:
-        s = SIZES[name]
+    for name in sizes or all_sizes:
+        s = all_sizes[name]
         r = {"config": s}
-        eng, stream = design_engine(s, max_ctx=prompt + ctx, **kw)
+        eng, stream = design_engine(*model(s), max_ctx=prompt + ctx, **kw)
         r["design"] = measure(eng, stream, s["vocab"], lambda a, c, p: design_work(s, a, c, p), prompt, ctx, batch, steps, peaks)
         eng.close()
         if not designs_only:
+            shape = llama_like(s)
             for tag, fast in (("llama_q8_0", False), ("llama_q8_0_fp16_operands", True)):
-                eng, stream = llama_engine(s, prompt + ctx, **kw)
-                r[tag] = measure(eng, stream, s["vocab"], lambda a, c, p: llama_work(s, a, c, p), prompt, ctx, batch, steps, peaks, fast)
+                eng, stream = llama_engine(shape, prompt + ctx, **kw)
+                r[tag] = measure(eng, stream, s["vocab"], lambda a, c, p: llama_work(shape, a, c, p), prompt, ctx, batch, steps, peaks, fast)
                 eng.close()
         out["sizes"][name] = r
         print(json.dumps({name: r}), flush=True)

@@ -276,9 +276,16 @@ class ForwardEngine:
         check(lib().sp_cuda_reset_cache(self._h, slot))
 
     def truncate_cache(self, n: int, slot: int = 0) -> int:
+        """Keeps the first n tokens; returns how many were kept. With recurrent states that is n, the checkpoint's length
+        or 0, and the tokens from there on are fed again."""
         kept = C.c_size_t()
         check(lib().sp_cuda_truncate_cache(self._h, slot, n, C.byref(kept)))
         return int(kept.value)
+
+    def checkpoint(self, slot: int = 0) -> None:
+        """Remembers the slot's recurrent states at its present length, so that truncate_cache can come back to it.
+        Models without such states can be cut anywhere and need none."""
+        check(lib().sp_cuda_engine_checkpoint(self._h, slot))
 
     def backend_label(self) -> str:
         buf = C.create_string_buffer(64)
@@ -382,7 +389,7 @@ class ForwardEngine:
         separate producers."""
         check(lib().sp_cuda_engine_set_ring(self._h, int(on)))
 
-    PROFILE_FAMILIES = ("gemv", "attention", "norm", "rope_kv", "elementwise", "embed", "argmax")
+    PROFILE_FAMILIES = ("gemv", "attention", "norm", "rope_kv", "elementwise", "embed", "argmax", "state")
 
     def set_profile(self, on: bool) -> None:
         check(lib().sp_cuda_engine_set_profile(self._h, int(on)))

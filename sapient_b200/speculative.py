@@ -70,6 +70,20 @@ class SpecState:
     history: list = field(default_factory=list)  # (drafted, committed) per round
 
 
+def _checkpoint(*engines) -> None:
+    """Before a round: engines with recurrent states remember them (the others, and engines without the call, need not)."""
+    for e in engines:
+        if hasattr(e, "checkpoint"):
+            e.checkpoint()
+
+
+def _rewind(engine, n: int, tokens: Sequence[int]) -> None:
+    """The engine's sequence becomes tokens[:n]; what its states could not be cut to is fed again."""
+    kept = engine.truncate_cache(n)
+    if kept is not None and kept < n:
+        engine.forward_logits(list(tokens[kept:n]), True)
+
+
 def spec_prefill(target, draft, prompt: Sequence[int]) -> SpecState:
     prompt = [int(t) for t in prompt]
     if not prompt:
@@ -85,6 +99,7 @@ def spec_round(target, draft, state: SpecState, k: int, sample: Callable = greed
     if rand is None:
         raise ValueError("spec_round needs a uniform random source")
     l = state.committed_len
+    _checkpoint(target, draft)
     # 1. draft up to k tokens, extending the draft cache
     drafts: List[int] = []
     dprobs: List[np.ndarray] = []
@@ -134,13 +149,13 @@ def spec_round(target, draft, state: SpecState, k: int, sample: Callable = greed
     # 5. reconcile the caches with the committed context
     if not hit_eos:
         if rejected:
-            target.truncate_cache(l + n_acc - 1)
+            _rewind(target, l + n_acc - 1, state.all_tokens + accepted)
         state.target_next = np.asarray(target.forward_logits([accepted[-1]], True), dtype=np.float32)
         # The reference rewinds the draft to l and replays every committed token one by one (:612-618). The
         # draft cache already holds drafts[0 .. m-2]; the accepted ones among them stay, the rest of the
         # committed tokens go through in one call — same committed context, one forward instead of n_acc.
         keep = min(n_draft_ok, m - 1)
-        draft.truncate_cache(l + keep)
+        _rewind(draft, l + keep, state.all_tokens + accepted)
         state.draft_next = np.asarray(draft.forward_logits(accepted[keep:], True), dtype=np.float32)
     state.all_tokens.extend(accepted)
     state.committed_len = l + n_acc
@@ -195,7 +210,9 @@ def generate_greedy(target, draft, prompt: Sequence[int], max_new_tokens: int, k
     out: List[int] = [pending] if max_new_tokens > 0 else []
     stop = max_new_tokens == 0 or pending in eos_ids
     length = len(prompt)  # committed tokens held by both caches
+    committed = list(prompt)
     while not stop and len(out) < max_new_tokens:
+        _checkpoint(target, draft)
         drafts: List[int] = []
         tok = pending
         for _ in range(k):
@@ -214,10 +231,11 @@ def generate_greedy(target, draft, prompt: Sequence[int], max_new_tokens: int, k
                 break
             out.append(t)
             stop = t in eos_ids
-        pending = picks[n]
-        target.truncate_cache(length + 1 + n)
+        fed, pending = pending, picks[n]
+        committed += [fed] + drafts[:n]
+        _rewind(target, length + 1 + n, committed)
         if n < k:
-            draft.truncate_cache(length + 1 + n)
+            _rewind(draft, length + 1 + n, committed)
         elif not stop and len(out) < max_new_tokens:
             draft.forward_logits([drafts[-1]], True)
         length += 1 + n

@@ -446,6 +446,62 @@ def lepalorn_weights(cfg: dict, seed: int, device: str = "cpu") -> dict:
     return W
 
 
+def tedelix_config(layers, width: int, heads: int, kv_heads: int, dim: int, vdim: int, state_heads: int, state_dim: int, state_vdim: int, window: int,
+                   ff: int, vocab: int, rot: int | None = None) -> dict:
+    """layers: the types in order; layers of one type are equal."""
+    mixers = {
+        "attention": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": window},
+                      "rot": {"base": 10000.0, "dims": dim if rot is None else rot}},
+        "lightning": {"heads": state_heads, "dim": state_dim, "vdim": state_vdim, "decay": [1.0 - 2.0 ** (-1 - 7.0 * i / max(1, state_heads - 1)) for i in range(state_heads)]},
+        "general_delta": {"heads": state_heads, "dim": state_dim},
+    }
+    return {"architecture": "Tedelix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.7, "logit_softcap": 40.0,
+            "layers": [{"type": t, "mixer": dict(mixers[t]), "mlp": {"kind": "dense", "ff": ff}} for t in layers]}
+
+
+def tedelix_weights(cfg: dict, seed: int, rank: int = 64, device: str = "cpu") -> dict:
+    """Random bf16 weights, rows scaled so that activations keep their magnitude. rank: of the decay logits' low-rank product."""
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W: dict = {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = (torch.randn(n, k, generator=g, device=device, dtype=torch.float32) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(name, n, mean=0.0, spread=0.1):
+        W[name] = (mean + spread * torch.randn(n, generator=g, device=device)).to(torch.bfloat16)
+
+    w = cfg["width"]
+    mat("embed", cfg["vocab"], w, w ** 0.5)
+    for i, layer in enumerate(cfg["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        H, D = m["heads"], m["dim"]
+        V = m.get("vdim", D)
+        vec(f"l{i}.norm1", w, 1.0)
+        if layer["type"] == "attention":
+            mat(p + "q", H * D, w)
+            mat(p + "k", m["kv_heads"] * D, w)
+            mat(p + "v", m["kv_heads"] * V, w)
+        else:
+            mat(p + ("q" if layer["type"] == "lightning" else "r"), H * D, w)
+            mat(p + "k", H * D, w)
+            mat(p + "v", H * V, w)
+            mat(p + "g", H * V, w)
+            vec(p + "norm", H * V, 1.0)
+            if layer["type"] == "general_delta":
+                mat(p + "a", H * D, w)
+                vec(p + "a.b", H * D)
+                mat(p + "w1", rank, w)
+                mat(p + "w2", H * D, rank)
+                vec(p + "w0", H * D, -3.0, 1.0)
+        mat(p + "o", w, H * V, 0.5)
+        if layer.get("mlp"):
+            mat(f"l{i}.mlp.up", layer["mlp"]["ff"], w)
+            mat(f"l{i}.mlp.down", w, layer["mlp"]["ff"], 0.5)
+    vec("final.norm", w, 1.0)
+    return W
+
+
 def write_safetensors(path: str, cfg: dict, W: dict) -> None:
     """A model directory: config.json and model.safetensors (bf16 tensors)."""
     import json
