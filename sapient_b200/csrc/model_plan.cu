@@ -76,7 +76,7 @@ GroupedAttentionSpec read_grouped_attention(const Cfg& c, bool rotate_values) {
     m.scale = (float)c.num("scale");
     const Cfg rot = c.sub("rot");
     m.rot.base = rot.num("base");
-    m.rot.dims = rot.size("dims", 0);
+    m.rot.dims = rot.has("dims") ? rot.size("dims", 0) : m.dim;
     m.rotate_values = rotate_values;
     if (c.has("mask") && c.sub("mask").has("size")) m.window = c.sub("mask").size("size");
     if (!c.err->empty()) return m;
