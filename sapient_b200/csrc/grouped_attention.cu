@@ -134,9 +134,9 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* 
 
 // ── few rows, bf16 ──
 // Block per (cached head, 16 of its query heads; token; split of the keys), the splits being the blocks of a cluster. Each of
-// the four warps walks pages of 16 keys of its own with two stages of cp.async; with up to eight query heads the remainders
+// the four warps walks pages of 16 keys of its own with three stages of cp.async; with up to eight query heads the remainders
 // of the softmax weights fill the other eight rows of the tile, else they are a second product.
-constexpr int GD_WARPS = 4, GD_STAGES = 2, GD_MAX_SPLITS = 8;
+constexpr int GD_WARPS = 4, GD_STAGES = 3, GD_MAX_SPLITS = 8;
 static size_t gd_smem(int dim16, int vdim16) { return (size_t)(GD_WARPS * GD_STAGES * KV_PAGE * (dim16 + vdim16 + 8) + 16 * (dim16 + 8)) * 2; }
 
 template <int VT, bool PACKED>
@@ -182,7 +182,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
     for (int i = 0; i < VT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const uint32_t qa = smem_addr(qs + (lane & 15) * LQ + (lane >> 4) * 8);
-    for (int page = page0, st = 0; page <= page_end; page += stride, st ^= 1) {
+    for (int page = page0, st = 0; page <= page_end; page += stride, st = st + 1 == GD_STAGES ? 0 : st + 1) {
         cp_async_wait<GD_STAGES - 1>();
         __syncwarp();
         const bf16* kt = ring + st * KV_PAGE * LD;
@@ -358,7 +358,7 @@ cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const
                                      const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
     if (n_splits < 1 || n_splits > GD_MAX_SPLITS || (n_splits & (n_splits - 1)) || s.vdim > GROUPED_MAX_VDIM) return cudaErrorInvalidValue;
-    constexpr int CAP = 200 * 1024;
+    constexpr int CAP = 220 * 1024;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
         const void* fns[] = {(const void*)grouped_decode_kernel<4, true>, (const void*)grouped_decode_kernel<8, true>, (const void*)grouped_decode_kernel<16, true>,

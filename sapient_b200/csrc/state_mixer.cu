@@ -527,17 +527,19 @@ __global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateAr
         const int h = blockIdx.y * SN_WARPS + warp;
         if (h >= H) return;
         const float* oh = o + (int64_t)h * rec.floats;
-        float v[SN_KEEP], ss = 0.f;
+        float v[SN_KEEP], f[SN_KEEP], ss = 0.f;  // outputs, gain and gate
 #pragma unroll
         for (int j = 0; j < SN_KEEP; ++j) {
-            v[j] = lane + 32 * j < V ? oh[lane + 32 * j] : 0.f;
+            const int i = lane + 32 * j;
+            v[j] = i < V ? oh[i] : 0.f;
+            f[j] = i < V ? a.gain[h * V + i] * sigmoid_f32(g[h * V + i]) : 0.f;
             ss = fmaf(v[j], v[j], ss);
         }
         for (int i = lane + 32 * SN_KEEP; i < V; i += 32) ss = fmaf(oh[i], oh[i], ss);
         const float r = rsqrtf(warp_sum(ss) / (float)V + a.s.eps);
 #pragma unroll
         for (int j = 0; j < SN_KEEP; ++j)
-            if (lane + 32 * j < V) finish(h, lane + 32 * j, v[j], r);
+            if (lane + 32 * j < V) out[h * V + lane + 32 * j] = from_f32<T>(v[j] * r * f[j]);
         for (int i = lane + 32 * SN_KEEP; i < V; i += 32) finish(h, i, oh[i], r);
         return;
     }
