@@ -395,7 +395,7 @@ def main() -> None:
     # ── per-family device time: each family's launches of one step replayed alone as a CUDA graph ──
     P = 20
     # (single GPU only: under tensor parallelism a subset would separate the producers of an exchange from its consumers)
-    fam_ms = {f: eng.time_families(f, 1, P) for f in eng.PROFILE_FAMILIES} if world == 1 else {}
+    fam_ms = {f: eng.time_families(f, 1, P) for f in eng.PROFILE_FAMILIES if f != "state"} if world == 1 else {}
     fam_ms["all"] = eng.time_families("all", 1, P)
     gemv_ms = fam_ms.get("gemv", 0.0) * P
     gemv_n = (4 * cfg["n_layers"] + 1) * P
