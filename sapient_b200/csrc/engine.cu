@@ -64,6 +64,7 @@ Engine::Engine(const SpModelDesc& desc, const ModelPlan& plan, bool f32) : Engin
     r.hidden = plan.width;
     r.vocab = plan.vocab;
     r.norm_eps = plan.eps;
+    if (plan.max_positions > 0) r.max_ctx = std::min(r.max_ctx, plan.max_positions);
     // informative only: a plan's layers have sizes of their own
     const LayerPlan& l = plan.layers[0];
     r.n_heads = l.mixer == MIX_LATENT ? l.latent.heads : l.mixer == MIX_GROUPED ? l.grouped.heads : l.state.heads;

@@ -251,6 +251,7 @@ class Engine {
     int plan_grouped(int layer, int T);
     int plan_state(int layer, int T);
     int plan_experts(int layer, int T);
+    int plan_dense(int layer, int T);
     int plan_rollback(int slot, int n, int* kept);
     int plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, int ldy, bool out_f32);
     int plan_product(const MatArgs& a, int max_tiles);

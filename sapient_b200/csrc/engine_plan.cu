@@ -1,6 +1,6 @@
 // Plan-driven models (model_plan.h) on the resident engine: what every plan shares — weights packed once into the shapes
 // the kernels read, a paged cache behind the same page pool, state pools, the buffers and tables of a step, the output head.
-// The layers themselves are in engine_plan_latent.cu and engine_plan_parallel.cu. bf16 products run on the tcgen05 kernel
+// The layers themselves are in engine_plan_post_norm.cu and engine_plan_parallel.cu. bf16 products run on the tcgen05 kernel
 // (mat_tc5.cu) at every row count, f32 ones on mat_f32.cu. Steps of up to PLAN_ROWS rows can be captured as a graph.
 #include "engine_plan.h"
 
@@ -52,6 +52,41 @@ const float* PlanPacker::vec(const std::string& name, int64_t n) {
     const float* f = e.find_f32(name, n);
     if (!f) fail(SP_ERR_OOM, "cannot convert '" + name + "'");
     return f;
+}
+
+RowGain PlanPacker::gain(const std::string& name) {
+    const int W = p.plan.width;
+    if (p.plan.norm_gain == GAIN_SCALAR) return RowGain{vec(name, 1), false};
+    if (p.plan.norm_gain == GAIN_COORD) return RowGain{vec(name, W), true};
+    std::vector<float> g = host(name, 1, W);
+    for (float& v : g) v += 1.f;
+    return RowGain{upload(g), true};
+}
+
+std::vector<float> PlanPacker::host(const std::string& name, int64_t rows, int64_t cols) {
+    const DevTensor* t = need(name, rows, cols);
+    const int64_t n = rows * cols;
+    float* f = nullptr;
+    std::vector<float> out;
+    if (!t) return out;
+    if (t->dtype != T_F32 && cudaMalloc((void**)&f, (size_t)n * 4) != cudaSuccess) { fail(SP_ERR_OOM, "cannot convert '" + name + "'"); return out; }
+    out.resize((size_t)n);
+    if ((f && launch_dequant(t->dtype, t->d, 1, n, f, 0) != cudaSuccess) ||
+        cudaMemcpy(out.data(), f ? f : (const float*)t->d, (size_t)n * 4, cudaMemcpyDeviceToHost) != cudaSuccess) {
+        fail(SP_ERR_CUDA, "cannot convert '" + name + "'");
+        out.clear();
+    }
+    if (f) cudaFree(f);
+    return out;
+}
+
+const float* PlanPacker::upload(const std::vector<float>& v) {
+    void* q = nullptr;
+    if (v.empty()) return nullptr;
+    if (cudaMalloc(&q, v.size() * 4) != cudaSuccess) { fail(SP_ERR_OOM, "cannot allocate a table"); return nullptr; }
+    p.owned.push_back(q);
+    if (cudaMemcpy(q, v.data(), v.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) { fail(SP_ERR_CUDA, "cudaMemcpy failed"); return nullptr; }
+    return (const float*)q;
 }
 
 bool PlanPacker::alloc(PlanMat& m, int groups, int64_t rows, int k) {
@@ -128,7 +163,8 @@ int Engine::finalize_plan() {
     if (pk.alloc(p.embed, 1, mp.vocab, W)) pk.put(p.embed, 0, pk.need("embed", mp.vocab, W), 0, mp.vocab, W);
     if (mp.tied_head) p.head = p.embed;
     else if (pk.alloc(p.head, 1, mp.vocab, W)) pk.put(p.head, 0, pk.need("head", mp.vocab, W), 0, mp.vocab, W);
-    p.final_norm = pk.vec("final.norm", mp.form == FORM_PARALLEL ? W : 1);
+    if (mp.max_positions > 0 && pk.alloc(p.pos, 1, mp.max_positions, W)) pk.put(p.pos, 0, pk.need("pos", mp.max_positions, W), 0, mp.max_positions, W);
+    p.final_norm = pk.gain("final.norm");
     // pages first: the layers' cache slices are laid out one after another
     const int pages_per_seq = (d.max_ctx + KV_PAGE - 1) / KV_PAGE;
     const int64_t n_pages = d.kv_pages > 0 ? d.kv_pages : (int64_t)d.max_batch * pages_per_seq;
@@ -139,12 +175,8 @@ int Engine::finalize_plan() {
     kv_.max_pages = pages_per_seq;
     kv_.page_table = d_page_table_;
     for (int i = 0; i < L && pk.status == SP_OK; ++i) {
-        if (mp.form == FORM_PARALLEL) {
-            pk.parallel_layer(i);
-        } else {
-            pk.latent_layer(i);
-            if (pk.status == SP_OK && mp.layers[(size_t)i].mlp == MLP_MOE) pk.experts(i);
-        }
+        if (mp.form == FORM_PARALLEL) pk.parallel_layer(i);
+        else pk.post_norm_layer(i);
     }
     if (pk.status != SP_OK) return pk.status;
     SP_CUDA_TRY(cudaDeviceSynchronize());
@@ -203,15 +235,15 @@ int Engine::finalize_plan() {
     p.low = take(T * n.low * el);
     if (mp.form == FORM_POST_NORM) {
         p.y = (float*)take(T * W * 4);
-        p.history = (float*)take((size_t)(L + 1) * T * W * 4);
+        if (mp.depth_average) p.history = (float*)take((size_t)(L + 1) * T * W * 4);
     }
+    p.act = take(T * n.act * el);
     if (long_steps) {
         p.wlogit = (float*)take(T * n.wlogit * 4);
         p.groups_cap = p.has_state ? T / state_group(p.f32) + std::min<size_t>(T, (size_t)d.max_batch) + 1 : 0;
         p.state_rec = (float*)take(p.groups_cap * n.state_rec * 4);
     }
     if (n.pairs) {
-        p.act = take(T * n.act * el);
         p.act_shared = take(T * n.act_shared * el);
         p.y_expert = (float*)take(T * n.pairs * W * 4);
         p.y_shared = (float*)take(T * W * 4);
@@ -313,7 +345,7 @@ int Engine::plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, i
     a.out_f32 = out_f32;
     a.nseg = 1;
     a.m = m;
-    a.seg[0] = MatSeg{w.w, w.n, w.kp, 1, 0.f, 0.f, x, ldx, 0, y, ldy, 0};
+    a.seg[0] = MatSeg{w.w, w.n, w.kp, 1, MatUnit{}, x, ldx, 0, y, ldy, 0};
     return plan_product(a, 0);
 }
 
@@ -321,8 +353,8 @@ int Engine::plan_layers(int T) {
     PlanState& p = *plan_;
     const int W = p.plan.width, L = (int)p.layers.size();
     const bool parallel = p.plan.form == FORM_PARALLEL;
-    SP_LAUNCH(F_EMBED, launch_embed_scaled(p.embed.w, p.embed.kp, p.f32, d_ids_, T, W, p.plan.embed_scale, parallel ? x_ : p.history, parallel ? nullptr : p.xb,
-                                           p.wp, stream));
+    SP_LAUNCH(F_EMBED, launch_embed_scaled(p.embed.w, p.pos.w, p.embed.kp, p.f32, d_ids_, d_tok_pos_, T, W, p.plan.embed_scale, p.history ? p.history : x_,
+                                           parallel ? nullptr : p.xb, p.wp, stream));
     for (int i = 0; i < L; ++i) {
         SP_TRY(parallel ? plan_layer_parallel(i, T) : plan_layer_post_norm(i, T));
         if (trace_on) SP_CUDA_TRY(cudaMemcpyAsync(trace_ + (size_t)i * d.max_tokens * W, x_, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, stream));
@@ -335,7 +367,7 @@ int Engine::plan_layers(int T) {
 int Engine::plan_head(const int32_t* rows, int n) {
     PlanState& p = *plan_;
     const int V = p.plan.vocab;
-    SP_LAUNCH(F_NORM, launch_row_norm(x_, rows, n, p.plan.width, p.final_norm, p.plan.form == FORM_PARALLEL, p.plan.eps, p.fin, p.wp, p.f32, stream));
+    SP_LAUNCH(F_NORM, launch_row_norm(x_, rows, n, p.plan.width, p.final_norm, p.plan.eps, p.fin, p.wp, p.f32, stream));
     if (p.plan.logit_scale == 1.f && p.plan.logit_softcap <= 0.f) {
         SP_TRY(plan_mat(p.head, p.fin, p.wp, n, logits_, V, true));
     } else {
@@ -343,7 +375,7 @@ int Engine::plan_head(const int32_t* rows, int n) {
         a.f32 = p.f32;
         a.nseg = a.n_outs = 1;
         a.m = n;
-        a.seg[0] = MatSeg{p.head.w, V, p.head.kp, 1, 0.f, 0.f, p.fin, p.wp, 0, nullptr, 0, 0};
+        a.seg[0] = MatSeg{p.head.w, V, p.head.kp, 1, MatUnit{}, p.fin, p.wp, 0, nullptr, 0, 0};
         a.outs[0] = MatOut{V, logits_, V, MAT_SOFTCAP, true, false};
         a.scale = p.plan.logit_scale;
         a.cap = p.plan.logit_softcap;

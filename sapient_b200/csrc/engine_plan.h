@@ -1,7 +1,7 @@
 // State of a plan-driven engine: the packed weights of every layer, the cache and state pools and the buffers of a step.
 // Owned by Engine, which keeps the sequence slots, the page tables, the step graphs and the host API. engine_plan.cu has
-// what every plan shares, engine_plan_latent.cu latent attention and experts, engine_plan_parallel.cu the parallel layer
-// form with grouped attention, state mixers and dense feed-forwards.
+// what every plan shares, engine_plan_post_norm.cu and engine_plan_parallel.cu the two layer forms (the first with experts, the
+// second with state mixers), engine_plan_latent.cu latent attention, engine_plan_grouped.cu grouped attention.
 #pragma once
 #include <algorithm>
 #include <map>
@@ -48,20 +48,24 @@ struct PlanLayer {
     PlanMat uv;                // per head: latent -> value
     PlanMat kv;                // per head key rows then value rows, each padded to 16: the expanded form
     PlanMat o;                 // output projection; parallel form: [W_o | W_down] over [mixer output | activation]
-    const float *norm1 = nullptr, *norm2 = nullptr, *dkv_norm = nullptr, *dwa = nullptr;
-    PlanMat router;            // experts rows, then the shared expert's gate row
+    RowGain norm1{}, norm2{};
+    const float *dkv_norm = nullptr, *dwa = nullptr;
+    PlanMat router;            // experts rows, then the shared expert's gate row where it has one
     const float* router_b = nullptr;
     PlanMat gu, down, shared_gu, shared_down;
+    PlanMat up;                // dense feed-forward of the post-norm form (down as above)
     LatentShape shape{};
     LatentCache cache{};       // the layer's own, or the one it borrows
     bool own = true, expand = false;
     const float2* cos_sin = nullptr;
-    // parallel form
-    int mix_rows = 0, silu_rows = 0, low_rows = 0, ff = 0;  // of proj: f32 rows, of which silu_rows come first, ...
-    int act_col = 0;           // first column of the activation in o's input
     GroupedShape grouped{};
     GroupedCache kv_cache{};
-    const float2 *cs_key = nullptr, *cs_val = nullptr;
+    GroupedInput grouped_in{};
+    GroupedTerms grouped_terms{};  // without the step's gate
+    int mix_rows = 0;          // of proj: f32 rows (grouped attention, state mixers)
+    // parallel form
+    int silu_rows = 0, low_rows = 0, ff = 0;  // of the mix_rows those that come first; rows of proj behind them
+    int act_col = 0;           // first column of the activation in o's input
     StateShape state_shape{};
     size_t state_at = 0;       // of a slot's floats
     PlanMat w2;
@@ -81,8 +85,8 @@ struct PlanState {
     bool f32 = false;
     int elem() const { return f32 ? 4 : 2; }
     std::vector<PlanLayer> layers;
-    PlanMat embed, head;
-    const float* final_norm = nullptr;
+    PlanMat embed, head, pos;  // pos: learned position vectors
+    RowGain final_norm{};
     int wp = 0;                // padded width
     size_t page_bytes = 0;     // all layers' rows of one page
     std::vector<size_t> cache_run, cache_base;  // per layer: bytes of a page (0: none of its own), offset of its slice
@@ -114,6 +118,12 @@ struct PlanState {
 
 size_t plan_latent_part_rows();  // engine_plan_latent.cu
 
+// A matrix that reads the mixer's input: tensor name behind "mix." and rows.
+struct MixPart {
+    std::string name;
+    int rows;
+};
+
 // Builds packed matrices out of the uploaded tensors.
 struct PlanPacker {
     Engine& e;
@@ -124,6 +134,9 @@ struct PlanPacker {
     const DevTensor* need(const std::string& name, int64_t rows, int64_t cols);
     int64_t rows_of(const std::string& name);            // first dimension of a tensor whose size only its shape tells
     const float* vec(const std::string& name, int64_t n);
+    RowGain gain(const std::string& name);               // of a norm of the stream (model_plan.h: NormGain)
+    std::vector<float> host(const std::string& name, int64_t rows, int64_t cols);
+    const float* upload(const std::vector<float>& v);
     bool alloc(PlanMat& m, int groups, int64_t rows, int k);
     // rows [r0, r0 + rows) of source tensor t to packed rows starting at `to` (counted over all groups), columns at c0
     bool put(PlanMat& m, int64_t to, const DevTensor* t, int64_t r0, int64_t rows, int k, bool transpose = false, int c0 = 0);
@@ -131,7 +144,11 @@ struct PlanPacker {
     const float2* angles(double base, int dims);
     void cache_slice(size_t page_bytes);                 // the next layer's share of the cache
     void latent_layer(int i);
+    // parts: the matrices that read the mixer's input, in the order of their output columns; out_cols: what W_o reads
+    void grouped_mixer(int i, std::vector<MixPart>& parts, int* out_cols);
+    const float* distance_bias(const std::string& name, int heads, int far, int* n_rel);
     void experts(int i);
+    void post_norm_layer(int i);
     void parallel_layer(int i);
 };
 

@@ -14,26 +14,13 @@ void PlanPacker::parallel_layer(int i) {
     PlanSizes& n = p.need;
     const std::string mx = lp.prefix + "mix.", ml = lp.prefix + "mlp.";
     const int W = p.plan.width;
-    l.norm1 = vec(lp.prefix + "norm1", W);
+    l.norm1 = gain(lp.prefix + "norm1");
     l.ff = lp.mlp == MLP_DENSE ? lp.dense.ff : 0;
-    // the matrices that read h, in the order of their output columns
-    struct Part { std::string name; int rows; };
-    std::vector<Part> parts;
+    std::vector<MixPart> parts;
     int out_cols = 0;
-    size_t page = 0;
     if (lp.mixer == MIX_GROUPED) {
-        const GroupedAttentionSpec& m = lp.grouped;
-        const int H = m.heads, G = m.kv_heads;
-        p.has_grouped = true;
-        l.grouped = GroupedShape{H, G, m.dim, m.vdim, m.rot.dims, m.window, m.scale};
-        parts = {{"q", H * m.dim}, {"k", G * m.dim}, {"v", G * m.vdim}};
-        out_cols = H * m.vdim;
-        l.kv_cache = GroupedCache{nullptr, e.kv_.page_table, e.kv_.max_pages, (m.dim + 15) & ~15, (m.vdim + 15) & ~15};
-        page = (size_t)G * KV_PAGE * (l.kv_cache.dim16 + l.kv_cache.vdim16) * p.elem();
-        l.cs_key = angles(m.rot.base, m.rot.dims);
-        if (m.rotate_values) l.cs_val = angles(m.rot.base, m.vdim);
-        PlanSizes::most(n.q, (size_t)H * l.kv_cache.dim16);
-        if (m.vdim > GROUPED_MAX_VDIM) { fail(SP_ERR_ARG, "attention values above " + std::to_string(GROUPED_MAX_VDIM) + " coordinates are not supported"); return; }
+        grouped_mixer(i, parts, &out_cols);
+        if (status != SP_OK) return;
     } else {
         const StateMixerSpec& m = lp.state;
         const int H = m.heads, hd = H * m.dim, hv = H * m.vdim;
@@ -63,12 +50,12 @@ void PlanPacker::parallel_layer(int i) {
             l.decay = (const float*)q;
         }
         PlanSizes::most(n.state_rec, state_record_floats(l.state_shape, p.f32));
+        cache_slice(0);
     }
-    cache_slice(page);
-    for (const Part& part : parts) l.mix_rows += part.rows;
+    for (const MixPart& part : parts) l.mix_rows += part.rows;
     if (!alloc(l.proj, 1, (int64_t)l.mix_rows + l.low_rows + l.ff, W)) return;
     int at = 0;
-    for (const Part& part : parts) {
+    for (const MixPart& part : parts) {
         put(l.proj, at, need(mx + part.name, part.rows, W), 0, part.rows, W);
         at += part.rows;
     }
@@ -80,20 +67,6 @@ void PlanPacker::parallel_layer(int i) {
     if (l.ff) put(l.o, 0, need(ml + "down", W, l.ff), 0, W, l.ff, false, l.act_col);
     PlanSizes::most(n.proj, (size_t)l.mix_rows);
     PlanSizes::most(n.mixed, (size_t)l.o.kp);
-}
-
-int Engine::plan_grouped(int li, int T) {
-    PlanState& p = *plan_;
-    PlanLayer& l = p.layers[(size_t)li];
-    const GroupedShape& s = l.grouped;
-    SP_LAUNCH(F_ROPE, launch_grouped_append(p.proj, l.mix_rows, s, l.kv_cache, l.cs_key, l.cs_val, d_tok_slot_, d_tok_pos_, p.q, p.f32, T, stream));
-    if (p.n_grouped > 0 && T > PLAN_ROWS && !graph_step_ && grouped_mma_supported(s)) {
-        SP_LAUNCH(F_ATTN, launch_grouped_prefill(p.q, s, l.kv_cache, l.cs_val, (const GroupedTile*)(p.dev_tiles + p.grouped_at), p.n_grouped, p.attn, l.o.kp, stream));
-        return SP_OK;
-    }
-    const int splits = T > PLAN_ROWS ? 1 : grouped_attention_splits(s, T, std::min(1 << plan_ctx_bucket(), s.window), p.f32);
-    SP_LAUNCH(F_ATTN, launch_grouped_attention(p.q, s, l.kv_cache, l.cs_val, d_tok_slot_, d_tok_pos_, p.attn, l.o.kp, splits, p.f32, T, stream));
-    return SP_OK;
 }
 
 int Engine::plan_state(int li, int T) {
@@ -132,12 +105,12 @@ int Engine::plan_layer_parallel(int i, int T) {
     PlanState& p = *plan_;
     PlanLayer& l = p.layers[(size_t)i];
     const int W = p.plan.width;
-    SP_LAUNCH(F_NORM, launch_row_norm(x_, nullptr, T, W, l.norm1, true, p.plan.eps, p.xb, p.wp, p.f32, stream));
+    SP_LAUNCH(F_NORM, launch_row_norm(x_, nullptr, T, W, l.norm1, p.plan.eps, p.xb, p.wp, p.f32, stream));
     MatArgs a{};
     a.f32 = p.f32;
     a.nseg = 1;
     a.m = T;
-    a.seg[0] = MatSeg{l.proj.w, l.proj.n, l.proj.kp, 1, 0.f, 0.f, p.xb, p.wp, 0, nullptr, 0, 0};
+    a.seg[0] = MatSeg{l.proj.w, l.proj.n, l.proj.kp, 1, MatUnit{}, p.xb, p.wp, 0, nullptr, 0, 0};
     int at = 0;
     auto rows_to = [&](int rows, void* y, int64_t ld, MatAct act, bool f32) {
         if (rows) a.outs[a.n_outs++] = MatOut{at += rows, y, ld, act, f32, false};
@@ -149,7 +122,7 @@ int Engine::plan_layer_parallel(int i, int T) {
     SP_TRY(plan_product(a, 0));
     SP_TRY(p.plan.layers[(size_t)i].mixer == MIX_GROUPED ? plan_grouped(i, T) : plan_state(i, T));
     a.n_outs = 1;
-    a.seg[0] = MatSeg{l.o.w, W, l.o.kp, 1, 0.f, 0.f, p.attn, l.o.kp, 0, nullptr, 0, 0};
+    a.seg[0] = MatSeg{l.o.w, W, l.o.kp, 1, MatUnit{}, p.attn, l.o.kp, 0, nullptr, 0, 0};
     a.outs[0] = MatOut{W, x_, W, MAT_ID, true, true};
     return plan_product(a, 0);
 }

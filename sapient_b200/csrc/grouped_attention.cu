@@ -1,6 +1,8 @@
-// Grouped-query attention over a paged cache of rotated keys and, where the design rotates them, rotated values
-// (plan_kernels.h). Keys and values may differ in size; scores, softmax and accumulation are f32, the softmax weights enter
-// the tensor cores as a leading bf16 part plus its remainder. A sliding window bounds the pages a block visits.
+// Grouped-query attention over a paged cache of keys and values, or of keys that are the values (plan_kernels.h). Keys and
+// values may differ in size; scores, softmax and accumulation are f32, the softmax weights enter the tensor cores as a leading
+// bf16 part plus its remainder. A sliding window bounds the pages a block visits. Distance biases, sinks and output gates are
+// uniform branches of the same kernels: a bias is read from a table by distance, in prompts through shared memory (a tile's
+// distances are one run of it), and is one constant for tiles that are far enough.
 #include <algorithm>
 
 #include "kernels.h"
@@ -16,77 +18,117 @@ cudaError_t count_launch_and_check();  // kernels.cu
 // ── rotation and cache append ──
 constexpr int GA_WARPS = 4;
 
-// dst[0 .. pad) = src[0 .. n) with coordinates i and i + dims / 2 turned by cs[i] for i < dims / 2; zeros past n.
-template <typename T>
-__device__ __forceinline__ void rotate_halves(const float* src, T* dst, const float2* cs, int dims, int n, int pad) {
+// dst[0 .. pad) = src(0 .. n) with coordinates i and i + dims / 2 turned by cs[i] for i < dims / 2; zeros past n.
+template <typename T, typename Src>
+__device__ __forceinline__ void rotate_halves(const Src& src, T* dst, const float2* cs, int dims, int n, int pad) {
     const int half = dims / 2, lane = threadIdx.x & 31;
     for (int i = lane; i < half; i += 32) {
-        const float u = src[i], v = src[i + half];
+        const float u = src(i), v = src(i + half);
         const float2 r = cs[i];
         dst[i] = from_f32<T>(u * r.x - v * r.y);
         dst[i + half] = from_f32<T>(v * r.x + u * r.y);
     }
-    for (int i = dims + lane; i < pad; i += 32) dst[i] = from_f32<T>(i < n ? src[i] : 0.f);
+    for (int i = dims + lane; i < pad; i += 32) dst[i] = from_f32<T>(i < n ? src(i) : 0.f);
 }
 
-// A warp per (token, part): the heads' queries, then the cached heads' keys and values.
+// A warp per (token, part): the heads' queries, then the cached heads' keys and values (shared: the keys alone).
 template <typename T>
 __global__ void __launch_bounds__(GA_WARPS * 32) grouped_append_kernel(const float* __restrict__ proj, int ldp, const GroupedShape s, const GroupedCache c,
-                                                                    const float2* __restrict__ cs_key, const float2* __restrict__ cs_val,
-                                                                    const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos, T* __restrict__ q) {
+                                                                    const GroupedInput in, const int32_t* __restrict__ tok_slot,
+                                                                    const int32_t* __restrict__ tok_pos, T* __restrict__ q) {
     pdl_wait();
     pdl_trigger();
-    const int t = blockIdx.x, part = blockIdx.y * GA_WARPS + (threadIdx.x >> 5), pos = tok_pos[t];
-    const float* pr = proj + (int64_t)t * ldp;
-    const float2* ck = cs_key + (int64_t)pos * (s.rot / 2);
-    if (part < s.heads) {
-        rotate_halves<T>(pr + (int64_t)part * s.dim, q + ((int64_t)t * s.heads + part) * c.dim16, ck, s.rot, s.dim, c.dim16);
+    const int t = blockIdx.x, part = blockIdx.y * GA_WARPS + (threadIdx.x >> 5), pos = tok_pos[t], lane = threadIdx.x & 31;
+    const bool query = part < s.heads;
+    const int per = c.shared ? 1 : 2, g = query ? 0 : (part - s.heads) / per;
+    if (g >= s.kv_heads) return;
+    const bool value = !query && (part - s.heads) % per == 1;
+    const int n = value ? s.vdim : s.dim;
+    const int64_t at = query ? (int64_t)part * s.dim : value ? (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)g * s.vdim : (int64_t)(s.heads + g) * s.dim;
+    const float* pr = proj + (int64_t)t * ldp + at;
+    const float* bias = in.bias ? in.bias + at : nullptr;
+    auto projected = [&](int i) { return bias ? pr[i] + bias[i] : pr[i]; };
+    float r = 1.f;
+    if (in.norm && !value) {
+        float ss = 0.f;
+        for (int i = lane; i < n; i += 32) {
+            const float v = projected(i);
+            ss = fmaf(v, v, ss);
+        }
+        r = rsqrtf(warp_sum(ss) / (float)n + in.eps);
+    }
+    const float2* ck = in.cs_key ? in.cs_key + (int64_t)pos * (s.rot / 2) : nullptr;
+    auto normed = [&](const float* gain, float mult) {
+        return [=](int i) { return gain ? projected(i) * mult * gain[i] : projected(i) * mult; };
+    };
+    if (query) {
+        if (in.temperature) r *= in.temperature[pos];
+        rotate_halves<T>(normed(in.q_gain, r), q + ((int64_t)t * s.heads + part) * c.dim16, ck, s.rot, s.dim, c.dim16);
         return;
     }
-    const int g = (part - s.heads) >> 1;
-    if (g >= s.kv_heads) return;
     const int page = c.page_table[(int64_t)tok_slot[t] * c.max_pages + pos / KV_PAGE];
-    T* row = reinterpret_cast<T*>(c.pool) + (((int64_t)page * s.kv_heads + g) * KV_PAGE + pos % KV_PAGE) * (c.dim16 + c.vdim16);
-    if (!((part - s.heads) & 1)) rotate_halves<T>(pr + (int64_t)s.heads * s.dim + (int64_t)g * s.dim, row, ck, s.rot, s.dim, c.dim16);
-    else
-        rotate_halves<T>(pr + (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)g * s.vdim, row + c.dim16, cs_val ? cs_val + (int64_t)pos * (s.vdim / 2) : nullptr,
-                         cs_val ? s.vdim : 0, s.vdim, c.vdim16);
+    T* row = reinterpret_cast<T*>(c.pool) + (((int64_t)page * s.kv_heads + g) * KV_PAGE + pos % KV_PAGE) * c.ld;
+    if (c.shared) {
+        rotate_halves<T>(projected, row, nullptr, 0, n, c.dim16);
+        if (lane == 0) *reinterpret_cast<float*>(row + c.dim16) = r;
+    } else if (value) {
+        rotate_halves<T>(projected, row + c.dim16, in.cs_val ? in.cs_val + (int64_t)pos * (s.vdim / 2) : nullptr, in.cs_val ? s.vdim : 0, n, c.vdim16);
+    } else {
+        rotate_halves<T>(normed(in.k_gain, r), row, ck, s.rot, n, c.dim16);
+    }
 }
 
-cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const float2* cs_key, const float2* cs_val,
+cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in,
                                   const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    const dim3 grid(n_tok, (s.heads + 2 * s.kv_heads + GA_WARPS - 1) / GA_WARPS), block(GA_WARPS * 32);
-    const cudaError_t le = f32 ? launch_pdl(grouped_append_kernel<float>, grid, block, 0, st, proj, ldp, s, c, cs_key, cs_val, tok_slot, tok_pos, (float*)q)
-                               : launch_pdl(grouped_append_kernel<bf16>, grid, block, 0, st, proj, ldp, s, c, cs_key, cs_val, tok_slot, tok_pos, (bf16*)q);
+    if (c.shared && (s.rot || in.cs_val || in.k_gain || s.dim != s.vdim)) return cudaErrorInvalidValue;
+    const dim3 grid(n_tok, (s.heads + (c.shared ? 1 : 2) * s.kv_heads + GA_WARPS - 1) / GA_WARPS), block(GA_WARPS * 32);
+    const cudaError_t le = f32 ? launch_pdl(grouped_append_kernel<float>, grid, block, 0, st, proj, ldp, s, c, in, tok_slot, tok_pos, (float*)q)
+                               : launch_pdl(grouped_append_kernel<bf16>, grid, block, 0, st, proj, ldp, s, c, in, tok_slot, tok_pos, (bf16*)q);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
-// Writes coordinates m and m + half of a head's mixture, turned back by the angles cs (null: as they are).
+// The f32 factor behind a shared row's key.
 template <typename T>
-__device__ __forceinline__ void store_turned(T* dst, int m, int half, float u, float v, const float2* cs) {
+__device__ __forceinline__ float row_factor(const T* row, int dim16) { return *reinterpret_cast<const float*>(row + dim16); }
+
+// Writes coordinates m and m + half of a head's mixture, turned back by the angles cs and gated (null: as they are).
+template <typename T>
+__device__ __forceinline__ void store_mixed(T* dst, int m, int half, float u, float v, const float2* cs, const float* gate) {
     if (cs) {
         const float2 r = cs[m];
         const float x = u * r.x + v * r.y;
         v = v * r.x - u * r.y;
         u = x;
     }
+    if (gate) {
+        u *= sigmoid_f32(gate[m]);
+        v *= sigmoid_f32(gate[m + half]);
+    }
     dst[m] = from_f32<T>(u);
     dst[m + half] = from_f32<T>(v);
+}
+
+template <typename T>
+__device__ __forceinline__ void store_one(T* dst, int m, float u, const float* gate) { dst[m] = from_f32<T>(gate ? u * sigmoid_f32(gate[m]) : u); }
+
+__device__ __forceinline__ const float* gate_row(const GroupedTerms& x, int64_t t, int h, int vdim) {
+    return x.gate ? x.gate + t * x.ldgate + (int64_t)h * vdim : nullptr;
 }
 
 // ── any compute type and sizes ──
 constexpr int GS_WARPS = 4, GS_PER_LANE = GROUPED_MAX_VDIM / 32;
 template <typename T>
 __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* __restrict__ q, const GroupedShape s, const GroupedCache c,
-                                                                    const float2* __restrict__ cs_val, const int32_t* __restrict__ tok_slot,
+                                                                    const GroupedTerms x, const int32_t* __restrict__ tok_slot,
                                                                     const int32_t* __restrict__ tok_pos, T* __restrict__ out, int ldo) {
     extern __shared__ float gs_smem[];  // query, then one output row per warp
     __shared__ float sm[GS_WARPS], sl[GS_WARPS];
     pdl_wait();
     pdl_trigger();
     const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = h / (s.heads / s.kv_heads);
-    const int ld = c.dim16 + c.vdim16, pos = tok_pos[t], lo = s.window > pos ? 0 : pos - s.window + 1;
+    const int pos = tok_pos[t], lo = s.window > pos ? 0 : pos - s.window + 1, val = c.shared ? 0 : c.dim16;
+    const float* rel = x.rel ? x.rel + (int64_t)h * x.n_rel : nullptr;
     float *qs = gs_smem, *os = gs_smem + c.dim16;
     for (int i = threadIdx.x; i < c.dim16; i += GS_WARPS * 32) qs[i] = to_f32(q[((int64_t)t * s.heads + h) * c.dim16 + i]);
     __syncthreads();
@@ -96,13 +138,16 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* 
     for (int i = 0; i < GS_PER_LANE; ++i) o[i] = 0.f;
     float m = -INFINITY, l = 0.f;
     for (int key = lo + warp; key <= pos; key += GS_WARPS) {
-        const T* row = reinterpret_cast<const T*>(c.pool) + (((int64_t)pt[key / KV_PAGE] * s.kv_heads + g) * KV_PAGE + key % KV_PAGE) * ld;
+        const T* row = reinterpret_cast<const T*>(c.pool) + (((int64_t)pt[key / KV_PAGE] * s.kv_heads + g) * KV_PAGE + key % KV_PAGE) * c.ld;
         float dot = 0.f;
         for (int i = lane; i < s.dim; i += 32) dot = fmaf(qs[i], to_f32(row[i]), dot);
-        const float sc = warp_sum(dot) * s.scale, mn = fmaxf(m, sc), corr = expf(m - mn), p = expf(sc - mn);
+        float sc = warp_sum(dot) * s.scale;
+        if (c.shared) sc *= row_factor(row, c.dim16);
+        if (rel) sc += rel[min(pos - key, x.n_rel - 1)];
+        const float mn = fmaxf(m, sc), corr = expf(m - mn), p = expf(sc - mn);
 #pragma unroll
         for (int i = 0; i < GS_PER_LANE; ++i)
-            if (lane + 32 * i < s.vdim) o[i] = fmaf(p, to_f32(row[c.dim16 + lane + 32 * i]), o[i] * corr);
+            if (lane + 32 * i < s.vdim) o[i] = fmaf(p, to_f32(row[val + lane + 32 * i]), o[i] * corr);
         l = fmaf(l, corr, p);
         m = mn;
     }
@@ -114,6 +159,10 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* 
     float M = -INFINITY, sum = 0.f, cw[GS_WARPS];
 #pragma unroll
     for (int w = 0; w < GS_WARPS; ++w) M = fmaxf(M, sm[w]);
+    if (x.sink) {
+        M = fmaxf(M, x.sink[h]);
+        sum = expf(x.sink[h] - M);
+    }
 #pragma unroll
     for (int w = 0; w < GS_WARPS; ++w) {
         cw[w] = sm[w] == -INFINITY ? 0.f : expf(sm[w] - M);
@@ -128,8 +177,10 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* 
     };
     T* d = out + (int64_t)t * ldo + (int64_t)h * s.vdim;
     const int half = s.vdim / 2;
-    for (int e = threadIdx.x; e < half; e += GS_WARPS * 32) store_turned<T>(d, e, half, mixed(e), mixed(e + half), cs_val ? cs_val + (int64_t)pos * half : nullptr);
-    if ((s.vdim & 1) && threadIdx.x == 0) d[s.vdim - 1] = from_f32<T>(mixed(s.vdim - 1));
+    const float* gate = gate_row(x, t, h, s.vdim);
+    for (int e = threadIdx.x; e < half; e += GS_WARPS * 32)
+        store_mixed<T>(d, e, half, mixed(e), mixed(e + half), x.cs_val ? x.cs_val + (int64_t)pos * half : nullptr, gate);
+    if ((s.vdim & 1) && threadIdx.x == 0) store_one<T>(d, s.vdim - 1, mixed(s.vdim - 1), gate);
 }
 
 // ── few rows, bf16 ──
@@ -137,15 +188,20 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_simple_kernel(const T* 
 // the four warps walks pages of 16 keys of its own with three stages of cp.async; with up to eight query heads the remainders
 // of the softmax weights fill the other eight rows of the tile, else they are a second product.
 constexpr int GD_WARPS = 4, GD_STAGES = 3, GD_MAX_SPLITS = 8;
-static size_t gd_smem(int dim16, int vdim16) { return (size_t)(GD_WARPS * GD_STAGES * KV_PAGE * (dim16 + vdim16 + 8) + 16 * (dim16 + 8)) * 2; }
+// Row stride of a page in shared memory: an odd number of 16-byte pieces where the sizes are multiples of 16.
+__host__ __device__ __forceinline__ int gd_row(const GroupedCache& c) { return c.shared ? c.ld : c.ld + 8; }
+static size_t gd_smem(const GroupedCache& c) {
+    const size_t ring = (size_t)(GD_WARPS * GD_STAGES * KV_PAGE * gd_row(c) + 16 * (c.dim16 + 8)) * 2, mixtures = (size_t)GD_WARPS * 16 * (c.vdim16 + 4) * 4;
+    return std::max(ring, mixtures);
+}
 
 template <int VT, bool PACKED>
 __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c,
-                                                                    const float2* __restrict__ cs_val, const int32_t* __restrict__ tok_slot,
+                                                                    const GroupedTerms x, const int32_t* __restrict__ tok_slot,
                                                                     const int32_t* __restrict__ tok_pos, bf16* __restrict__ out, int ldo, int n_splits) {
     extern __shared__ __align__(16) bf16 gd_sm[];
     __shared__ float m_s[GD_WARPS][16], l_s[GD_WARPS][16], bm_s[16], bl_s[16], share_s[16][GD_MAX_SPLITS];
-    const int ld = c.dim16 + c.vdim16, LD = ld + 8, LQ = c.dim16 + 8;
+    const int ld = c.ld, LD = gd_row(c), LQ = c.dim16 + 8, val = c.shared ? 0 : c.dim16;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int group = s.heads / s.kv_heads, tiles = (group + 15) / 16, kvh = blockIdx.x / tiles, h0 = kvh * group + (blockIdx.x % tiles) * 16;
     const int nq = min(16, (kvh + 1) * group - h0), t = blockIdx.y;
@@ -182,6 +238,10 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
     for (int i = 0; i < VT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const uint32_t qa = smem_addr(qs + (lane & 15) * LQ + (lane >> 4) * 8);
+    // this thread's heads' biases by distance (PACKED: one head), and the one for every key that is far
+    const float* rel0 = x.rel ? x.rel + (int64_t)(h0 + min(g, nq - 1)) * x.n_rel : nullptr;
+    const float* rel1 = x.rel ? x.rel + (int64_t)(h0 + min(g + 8, nq - 1)) * x.n_rel : nullptr;
+    const float far0 = rel0 ? rel0[x.n_rel - 1] : 0.f, far1 = rel1 ? rel1[x.n_rel - 1] : 0.f;
     for (int page = page0, st = 0; page <= page_end; page += stride, st = st + 1 == GD_STAGES ? 0 : st + 1) {
         cp_async_wait<GD_STAGES - 1>();
         __syncwarp();
@@ -197,14 +257,22 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
             mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
         }
         float x0 = m0, x1 = m1;
+        const bool near = x.rel && pos - (page * KV_PAGE + KV_PAGE - 1) < x.n_rel - 1;
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = page * KV_PAGE + 8 * j + 2 * tq + e;
                 const bool on = key >= lo && key <= pos;
-                sc[j][e] = on ? sc[j][e] * s.scale : -INFINITY;
-                sc[j][2 + e] = on ? sc[j][2 + e] * s.scale : -INFINITY;
+                float f = s.scale, b0 = far0, b1 = far1;
+                if (c.shared) f *= row_factor(kt + (8 * j + 2 * tq + e) * LD, c.dim16);
+                if (near) {
+                    const int dist = max(0, min(pos - key, x.n_rel - 1));
+                    b0 = rel0[dist];
+                    if (!PACKED) b1 = rel1[dist];
+                }
+                sc[j][e] = on ? fmaf(sc[j][e], f, b0) : -INFINITY;
+                sc[j][2 + e] = on ? fmaf(sc[j][2 + e], f, b1) : -INFINITY;
                 x0 = fmaxf(x0, sc[j][e]);
                 x1 = fmaxf(x1, sc[j][2 + e]);
             }
@@ -236,7 +304,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
         }
 #pragma unroll
         for (int i = 0; i < VT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
-        const uint32_t va = smem_addr(kt + (lane & 15) * LD + c.dim16 + (lane >> 4) * 8);
+        const uint32_t va = smem_addr(kt + (lane & 15) * LD + val + (lane >> 4) * 8);
 #pragma unroll
         for (int i = 0; i < VT; i += 2) {
             if (i * 8 < c.vdim16) {
@@ -312,15 +380,18 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
         float M = mp;
 #pragma unroll
         for (int off = GD_MAX_SPLITS / 2; off > 0; off >>= 1) M = fmaxf(M, __shfl_xor_sync(0xFFFFFFFFu, M, off));
+        const float sink = x.sink && r < nq ? x.sink[h0 + r] : -INFINITY;
+        M = fmaxf(M, sink);
         const float f = mp == -INFINITY ? 0.f : expf(mp - M);
         float L = f * lp;
 #pragma unroll
         for (int off = GD_MAX_SPLITS / 2; off > 0; off >>= 1) L += __shfl_xor_sync(0xFFFFFFFFu, L, off);
+        if (sink != -INFINITY) L += expf(sink - M);
         share_s[r][p] = f / L;
     }
     __syncthreads();
     const int half = (s.vdim + 1) / 2;
-    const float2* cs = cs_val ? cs_val + (int64_t)pos * half : nullptr;
+    const float2* cs = x.cs_val ? x.cs_val + (int64_t)pos * half : nullptr;
     for (int i = blockIdx.z * GD_WARPS * 32 + tid; i < nq * half; i += n_splits * GD_WARPS * 32) {
         const int r = i / half, e = i - r * half;
         const bool two = e + half < s.vdim;
@@ -338,8 +409,9 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
             }
         }
         bf16* d = out + (int64_t)t * ldo + (int64_t)(h0 + r) * s.vdim;
-        if (two) store_turned<bf16>(d, e, half, u, v, cs);
-        else d[e] = __float2bfloat16_rn(u);
+        const float* gate = gate_row(x, t, h0 + r, s.vdim);
+        if (two) store_mixed<bf16>(d, e, half, u, v, cs, gate);
+        else store_one<bf16>(d, e, u, gate);
     }
     if (n_splits > 1) cluster_sync();  // nobody leaves while its mixture is being read
 }
@@ -354,7 +426,7 @@ int grouped_attention_splits(const GroupedShape& s, int n_tok, int keys, bool f3
     return n;
 }
 
-cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const int32_t* tok_slot,
+cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const int32_t* tok_slot,
                                      const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
     if (n_splits < 1 || n_splits > GD_MAX_SPLITS || (n_splits & (n_splits - 1)) || s.vdim > GROUPED_MAX_VDIM) return cudaErrorInvalidValue;
@@ -373,13 +445,13 @@ cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const
     if (le != cudaSuccess) return le;
     const int group = s.heads / s.kv_heads;
     if (!f32 && grouped_mma_supported(s)) {
-        const size_t smem = gd_smem(c.dim16, c.vdim16);
+        const size_t smem = gd_smem(c);
         if (smem > CAP) return cudaErrorInvalidValue;
         const dim3 grid(s.kv_heads * ((group + 15) / 16), n_tok, n_splits), block(GD_WARPS * 32);
 #define SP_GD(VT)                                                                                                                                     \
-    le = group <= 8 ? launch_pdl_cluster(grouped_decode_kernel<VT, true>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, cs_val, tok_slot, tok_pos, \
+    le = group <= 8 ? launch_pdl_cluster(grouped_decode_kernel<VT, true>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, x, tok_slot, tok_pos, \
                                          (bf16*)out, ldo, n_splits)                                                                                   \
-                    : launch_pdl_cluster(grouped_decode_kernel<VT, false>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, cs_val, tok_slot, tok_pos, \
+                    : launch_pdl_cluster(grouped_decode_kernel<VT, false>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, x, tok_slot, tok_pos, \
                                          (bf16*)out, ldo, n_splits)
         if (c.vdim16 <= 32) SP_GD(4);
         else if (c.vdim16 <= 64) SP_GD(8);
@@ -391,25 +463,28 @@ cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const
     const dim3 grid(s.heads, n_tok), block(GS_WARPS * 32);
     const size_t smem = (size_t)(c.dim16 + GS_WARPS * s.vdim) * 4;
     if (n_splits != 1 || smem > 48 * 1024) return cudaErrorInvalidValue;
-    le = f32 ? launch_pdl(grouped_simple_kernel<float>, grid, block, smem, st, (const float*)q, s, c, cs_val, tok_slot, tok_pos, (float*)out, ldo)
-             : launch_pdl(grouped_simple_kernel<bf16>, grid, block, smem, st, (const bf16*)q, s, c, cs_val, tok_slot, tok_pos, (bf16*)out, ldo);
+    le = f32 ? launch_pdl(grouped_simple_kernel<float>, grid, block, smem, st, (const float*)q, s, c, x, tok_slot, tok_pos, (float*)out, ldo)
+             : launch_pdl(grouped_simple_kernel<bf16>, grid, block, smem, st, (const bf16*)q, s, c, x, tok_slot, tok_pos, (bf16*)out, ldo);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
 // ── many rows, bf16 ──
 // Block per (head, tile of 64 tokens), 4 warps x 16 query rows, key tiles of four pages double-buffered with cp.async.
 constexpr int GP_KEYS = 64, GP_WARPS = 4;
-static size_t gp_smem(int dim16, int vdim16) { return (size_t)(3 * 64 * (dim16 + 8) + 2 * GP_KEYS * (vdim16 + 8)) * 2; }
+static_assert(GROUPED_TAIL == 8, "a shared row's tail is the padding of its row in shared memory");
+static size_t gp_smem(const GroupedCache& c) { return (size_t)(3 * 64 * (c.dim16 + 8) + (c.shared ? 0 : 2 * GP_KEYS * (c.vdim16 + 8))) * 2; }
 
 template <int VT>
 __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c,
-                                                                     const float2* __restrict__ cs_val, const GroupedTile* __restrict__ tiles,
+                                                                     const GroupedTerms x, const GroupedTile* __restrict__ tiles,
                                                                      bf16* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) bf16 gp_sm[];
+    __shared__ float rel_s[2][GP_KEYS + 64];  // biases of a key tile: by 63 - (query row) + (key in the tile)
     pdl_wait();
     pdl_trigger();
-    const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, ld = c.dim16 + c.vdim16;
-    bf16 *qs = gp_sm, *ks = qs + 64 * LQ, *vs = ks + 2 * GP_KEYS * LQ;
+    const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, ld = c.ld;  // (shared: LV == LQ)
+    bf16 *qs = gp_sm, *ks = qs + 64 * LQ, *vs = c.shared ? ks : ks + 2 * GP_KEYS * LQ;
+    const int k_pieces = (c.shared ? c.ld : c.dim16) / 8, v_pieces = c.shared ? 0 : c.vdim16 / 8;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int h = blockIdx.x, kvh = h / (s.heads / s.kv_heads);
     const GroupedTile tl = tiles[blockIdx.y];
@@ -421,6 +496,8 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
         const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * c.dim16;
         for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
     }
+    const float* rel = x.rel ? x.rel + (int64_t)h * x.n_rel : nullptr;
+    const float far = rel ? rel[x.n_rel - 1] : 0.f;
     const int hi = tl.pos0 + tl.n - 1, lo = (s.window > tl.pos0 ? 0 : tl.pos0 - s.window + 1) / KV_PAGE * KV_PAGE;
     auto fetch = [&](int k0, int buf) {
         const int page = k0 / KV_PAGE + warp;
@@ -431,8 +508,12 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
         for (int i = 0; i < 4; ++i) {
             const int r = lr + 4 * i, bytes = k0 + r <= hi ? 16 : 0;  // keys past the newest: zeros
             const bf16* src = base + (r - warp * 16) * ld;
-            for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(kd + r * LQ + p * 8, src + p * 8, bytes);
-            for (int p = l8; p < c.vdim16 / 8; p += 8) cp_async16(vd + r * LV + p * 8, src + c.dim16 + p * 8, bytes);
+            for (int p = l8; p < k_pieces; p += 8) cp_async16(kd + r * LQ + p * 8, src + p * 8, bytes);
+            for (int p = l8; p < v_pieces; p += 8) cp_async16(vd + r * LV + p * 8, src + c.dim16 + p * 8, bytes);
+        }
+        if (rel && tid < GP_KEYS + 63) {  // (distances below zero are of keys that are not seen)
+            const int dist = max(0, min(tl.pos0 + 63 - k0 - tid, x.n_rel - 1));
+            cp_async4(&rel_s[buf][tid], rel + dist);
         }
     };
     fetch(lo, 0);
@@ -466,14 +547,22 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
             }
         }
         float x0 = m0, x1 = m1;
+        const bool near = rel && tl.pos0 - (k0 + GP_KEYS - 1) < x.n_rel - 1;
+        const float* rs = &rel_s[buf][63 - r0 + 2 * tq];  // of key 2 tq; the other row's stand eight before
         const bool edge = k0 + GP_KEYS - 1 > tl.pos0 || (int64_t)hi - k0 >= s.window;  // only the window's ends need the mask
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = k0 + 8 * j + 2 * tq + e;
-                sc[j][e] = (!edge || (key <= p0 && p0 - key < s.window)) ? sc[j][e] * s.scale : -INFINITY;
-                sc[j][2 + e] = (!edge || (key <= p1 && p1 - key < s.window)) ? sc[j][2 + e] * s.scale : -INFINITY;
+                float f = s.scale, b0 = far, b1 = far;
+                if (c.shared) f *= row_factor(kt + (8 * j + 2 * tq + e) * LQ, c.dim16);
+                if (near) {
+                    b0 = rs[8 * j + e];
+                    b1 = rs[8 * j + e - 8];
+                }
+                sc[j][e] = (!edge || (key <= p0 && p0 - key < s.window)) ? fmaf(sc[j][e], f, b0) : -INFINITY;
+                sc[j][2 + e] = (!edge || (key <= p1 && p1 - key < s.window)) ? fmaf(sc[j][2 + e], f, b1) : -INFINITY;
                 x0 = fmaxf(x0, sc[j][e]);
                 x1 = fmaxf(x1, sc[j][2 + e]);
             }
@@ -530,6 +619,12 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
         l0 += __shfl_xor_sync(0xFFFFFFFFu, l0, off);
         l1 += __shfl_xor_sync(0xFFFFFFFFu, l1, off);
     }
+    float f0 = 1.f / l0, f1 = 1.f / l1;
+    if (x.sink) {
+        const float sink = x.sink[h], M0 = fmaxf(m0, sink), M1 = fmaxf(m1, sink), e0 = expf(m0 - M0), e1 = expf(m1 - M1);
+        f0 = e0 / fmaf(l0, e0, expf(sink - M0));
+        f1 = e1 / fmaf(l1, e1, expf(sink - M1));
+    }
     // a coordinate's partner is half a head away: the warp's rows meet in shared memory, a column range at a time
     __syncthreads();
     const int LO = c.vdim16 + 4;
@@ -538,8 +633,8 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
     for (int i = 0; i < VT; ++i) {
         if (i * 8 < c.vdim16) {
             float* d = os + g * LO + i * 8 + 2 * tq;
-            *reinterpret_cast<float2*>(d) = make_float2(o[i][0] / l0, o[i][1] / l0);
-            *reinterpret_cast<float2*>(d + 8 * LO) = make_float2(o[i][2] / l1, o[i][3] / l1);
+            *reinterpret_cast<float2*>(d) = make_float2(o[i][0] * f0, o[i][1] * f0);
+            *reinterpret_cast<float2*>(d + 8 * LO) = make_float2(o[i][2] * f1, o[i][3] * f1);
         }
     }
     __syncwarp();
@@ -547,16 +642,17 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
     for (int r = 0; r < 16 && warp * 16 + r < tl.n; ++r) {
         const int row = warp * 16 + r;
         bf16* d = out + (int64_t)(tl.row0 + row) * ldo + (int64_t)h * s.vdim;
-        const float2* cs = cs_val ? cs_val + (int64_t)(tl.pos0 + row) * half : nullptr;
-        for (int e = lane; e < half; e += 32) store_turned<bf16>(d, e, half, os[r * LO + e], os[r * LO + e + half], cs);
-        if ((s.vdim & 1) && lane == 0) d[s.vdim - 1] = __float2bfloat16_rn(os[r * LO + s.vdim - 1]);
+        const float2* cs = x.cs_val ? x.cs_val + (int64_t)(tl.pos0 + row) * half : nullptr;
+        const float* gate = gate_row(x, tl.row0 + row, h, s.vdim);
+        for (int e = lane; e < half; e += 32) store_mixed<bf16>(d, e, half, os[r * LO + e], os[r * LO + e + half], cs, gate);
+        if ((s.vdim & 1) && lane == 0) store_one<bf16>(d, s.vdim - 1, os[r * LO + s.vdim - 1], gate);
     }
 }
 
-cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const GroupedTile* tiles,
+cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const GroupedTile* tiles,
                                    int n_tiles, void* out, int ldo, cudaStream_t st) {
     if (n_tiles == 0) return cudaSuccess;
-    const size_t smem = std::max(gp_smem(c.dim16, c.vdim16), (size_t)GP_WARPS * 16 * (c.vdim16 + 4) * 4);
+    const size_t smem = std::max(gp_smem(c), (size_t)GP_WARPS * 16 * (c.vdim16 + 4) * 4);
     constexpr int CAP = 200 * 1024;
     if (!grouped_mma_supported(s) || smem > CAP) return cudaErrorInvalidValue;
     static PerDeviceOnce once;
@@ -571,7 +667,7 @@ cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const G
     });
     if (le != cudaSuccess) return le;
     const dim3 grid(s.heads, n_tiles), block(GP_WARPS * 32);
-#define SP_GP(VT) le = launch_pdl(grouped_prefill_kernel<VT>, grid, block, smem, st, (const bf16*)q, s, c, cs_val, tiles, (bf16*)out, ldo)
+#define SP_GP(VT) le = launch_pdl(grouped_prefill_kernel<VT>, grid, block, smem, st, (const bf16*)q, s, c, x, tiles, (bf16*)out, ldo)
     if (c.vdim16 <= 32) SP_GP(4);
     else if (c.vdim16 <= 64) SP_GP(8);
     else if (c.vdim16 <= 128) SP_GP(16);

@@ -1,5 +1,5 @@
 // Matrix products on f32 weights (plan-driven models in f32): y[r, n] = sum_k x[r, k] W[n, k], dense, per head or grouped by
-// expert, plain or as the gate / up pair of a clamped gated unit. A block owns a 32 x 32 tile; plain fused multiply-adds.
+// expert, plain or as the gate / up pair of a gated unit. A block owns a 32 x 32 tile; plain fused multiply-adds.
 #include "kernels.h"
 #include "pdl.cuh"
 #include "plan_common.cuh"
@@ -92,7 +92,7 @@ __global__ void __launch_bounds__(256) mat_f32_kernel(const MatArgs a) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int c = c0 + tr + 8 * i;
-                if (c < w.cnt) mat_store(a, s, w, w.r_begin + c, n0 + tn, DUAL ? clamped_unit(acc[0][i], acc[D - 1][i], s.limit, s.alpha) : acc[0][i]);
+                if (c < w.cnt) mat_store(a, s, w, w.r_begin + c, n0 + tn, DUAL ? gated_unit(acc[0][i], acc[D - 1][i], s.unit) : acc[0][i]);
             }
     }
 }

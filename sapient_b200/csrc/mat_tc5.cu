@@ -1,5 +1,5 @@
 // Matrix products on bf16 weights with the 5th-generation tensor cores (tcgen05 + TMEM), for one row or thousands: dense,
-// per head or grouped by expert, plain or as the gate / up pair of a clamped gated unit.
+// per head or grouped by expert, plain or as the gate / up pair of a gated unit.
 //
 // y[r, n] = sum_k x[r, k] W[n, k]. A CTA owns 128 weight rows of one matrix (the MMA's M; for a gated unit 128 gate rows
 // and the 128 up rows that belong to them, two accumulators) x up to bn activation rows (the MMA's N), over all of K or a
@@ -42,7 +42,7 @@ struct MatTc5Seg {
     int64_t ygs;
     int xgs;              // elements between the inputs of consecutive groups
     int ldy, n, kp;
-    float limit, alpha;
+    MatUnit unit;
 };
 struct MatTc5Args {
     MatTc5Seg seg[2];
@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
         // gate: what the output gate's logit of (row, g) is; the callers load a batch of them before the first store
         auto gate_of = [&](int row) { return a.gate[(int64_t)row * a.ldgate + g]; };
         auto finish = [&](int row, float f, float up, float gate) {
-            if (DUAL) f = clamped_unit(f, up, s.limit, s.alpha);
+            if (DUAL) f = gated_unit(f, up, s.unit);
             if (a.gate) f *= sigmoid_f32(gate);
             yn[(int64_t)row * s.ldy] = from_f32<Out>(f);
         };
@@ -253,7 +253,7 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
 #pragma unroll
                         for (int j = 0; j < 16; ++j, d += s.ldy) {
                             float f = __uint_as_float(v[j]);
-                            if (DUAL) f = clamped_unit(f, __uint_as_float(up[j]), s.limit, s.alpha);
+                            if (DUAL) f = gated_unit(f, __uint_as_float(up[j]), s.unit);
                             *d = from_f32<Out>(f);
                         }
                     }
@@ -337,7 +337,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     for (int i = 0; i < a.nseg; ++i) {
         const MatSeg& s = a.seg[i];
         if (s.kp % MAT_KPAD != 0 || s.n <= 0 || s.ldx % 8 != 0 || s.xgs % 8 != 0 || (int64_t)s.groups * s.n * 2 >= (1ll << 31)) return cudaErrorInvalidValue;
-        k.seg[i] = MatTc5Seg{s.y, s.ygs, (int)s.xgs, s.ldy, s.n, s.kp, s.limit, s.alpha};
+        k.seg[i] = MatTc5Seg{s.y, s.ygs, (int)s.xgs, s.ldy, s.n, s.kp, s.unit};
         n_max = std::max(n_max, s.n);
         kp_max = std::max(kp_max, s.kp);
     }

@@ -36,10 +36,18 @@ struct Cfg {
     }
 };
 
-ClampedExpertSpec read_expert(const Cfg& c) {
-    ClampedExpertSpec e;
+GatedExpertSpec read_clamped_expert(const Cfg& c) {
+    GatedExpertSpec e;
     e.ff = c.size("ff");
     e.limit = (float)c.num("limit");
+    e.alpha = 1.702f;
+    e.shift = 1.f;
+    return e;
+}
+
+GatedExpertSpec read_silu_expert(const Cfg& c) {
+    GatedExpertSpec e;
+    e.ff = c.size("ff");
     return e;
 }
 
@@ -67,20 +75,34 @@ LatentAttentionSpec read_latent_attention(const Cfg& c, int layer, const ModelPl
     return m;
 }
 
-GroupedAttentionSpec read_grouped_attention(const Cfg& c, bool rotate_values) {
+// What every kind of grouped attention has.
+GroupedAttentionSpec read_heads(const Cfg& c) {
     GroupedAttentionSpec m;
     m.heads = c.size("heads");
     m.kv_heads = c.size("kv_heads");
     m.dim = c.size("dim");
     m.vdim = c.size("vdim");
     m.scale = (float)c.num("scale");
+    if (c.err->empty() && m.heads % m.kv_heads) c.fail("heads is no multiple of kv_heads");
+    return m;
+}
+
+TemperatureSpec read_temperature(const Cfg& c) {
+    TemperatureSpec t;
+    t.coef = c.num("coef");
+    t.every = c.num("every");
+    if (c.err->empty() && t.every <= 0) c.fail("every must be positive");
+    return t;
+}
+
+GroupedAttentionSpec read_rotated_attention(const Cfg& c, bool rotate_values) {
+    GroupedAttentionSpec m = read_heads(c);
     const Cfg rot = c.sub("rot");
     m.rot.base = rot.num("base");
     m.rot.dims = rot.has("dims") ? rot.size("dims", 0) : m.dim;
     m.rotate_values = rotate_values;
     if (c.has("mask") && c.sub("mask").has("size")) m.window = c.sub("mask").size("size");
     if (!c.err->empty()) return m;
-    if (m.heads % m.kv_heads) c.fail("heads is no multiple of kv_heads");
     if ((m.rot.dims & 1) || m.rot.dims > m.dim || m.rot.base <= 0) c.fail("rot does not fit dim");
     if (rotate_values && (m.vdim & 1)) c.fail("vdim must be even");
     return m;
@@ -123,6 +145,7 @@ int read_tedelix(const Json& cfg, ModelPlan* out) {
     p.width = c.size("width");
     p.eps = (float)c.sub("norm").num("eps");
     p.form = FORM_PARALLEL;
+    p.norm_gain = GAIN_COORD;
     p.tied_head = true;
     if (c.has("logit_scale")) p.logit_scale = (float)c.num("logit_scale");
     if (c.has("logit_softcap")) p.logit_softcap = (float)c.num("logit_softcap");
@@ -137,7 +160,7 @@ int read_tedelix(const Json& cfg, ModelPlan* out) {
         const std::string t = type ? type->str : "";
         if (t == "attention") {
             l.mixer = MIX_GROUPED;
-            l.grouped = read_grouped_attention(lc.sub("mixer"), true);
+            l.grouped = read_rotated_attention(lc.sub("mixer"), true);
         } else if (t == "lightning" || t == "general_delta") {
             l.mixer = MIX_STATE;
             l.state = read_state_mixer(lc.sub("mixer"), t == "lightning" ? STATE_DECAY : STATE_DELTA);
@@ -180,12 +203,92 @@ int read_lepalorn(const Json& cfg, ModelPlan* out) {
             l.mlp = MLP_MOE;
             l.moe.experts = m.sub("router").size("experts");
             l.moe.top = m.sub("router").size("top");
-            l.moe.expert = read_expert(m.sub("expert"));
+            l.moe.expert = read_clamped_expert(m.sub("expert"));
             if (m.has("shared")) {
-                l.moe.has_shared = true;
-                l.moe.shared = read_expert(m.sub("shared"));
+                l.moe.has_shared = l.moe.shared_gate = true;
+                l.moe.shared = read_clamped_expert(m.sub("shared"));
             }
             if (l.moe.top > l.moe.experts) m.fail("router.top exceeds router.experts");
+        }
+        p.layers.push_back(l);
+    }
+    if (!err.empty()) { set_error(err); return SP_ERR_ARG; }
+    *out = std::move(p);
+    return SP_OK;
+}
+
+// Fatilix's two kinds of attention: without rotation, queries with a temperature, a sink and an output gate; `shared`:
+// weighted norms and values that are the keys, else biases, unweighted norms and a distance bias.
+GroupedAttentionSpec read_sink_attention(const Cfg& c, bool shared) {
+    GroupedAttentionSpec m = read_heads(c);
+    m.sink = m.out_gate = true;
+    if (c.has("q_temp")) m.temperature = read_temperature(c.sub("q_temp"));
+    if (shared) {
+        m.shared_values = true;
+        m.qk_norm = QK_WEIGHTED;
+        if (c.err->empty() && m.vdim != m.dim) c.fail("vdim must be dim where the keys are the values");
+    } else {
+        m.biases = true;
+        m.qk_norm = QK_UNIT;
+        m.bias_max = c.size("bias_max");
+    }
+    return m;
+}
+
+MoeSpec read_grouped_choice(const Cfg& c) {
+    MoeSpec m;
+    const Cfg r = c.sub("router");
+    m.rule = ROUTE_ALL;
+    m.bias = "correction";
+    m.experts = r.size("experts");
+    m.top = r.size("top");
+    if (r.has("scale")) m.scale = (float)r.num("scale");
+    if (r.has("groups")) {
+        m.groups = r.sub("groups").size("count");
+        m.keep = r.sub("groups").size("keep");
+    }
+    m.expert = read_silu_expert(c.sub("expert"));
+    if (c.has("shared")) {
+        m.has_shared = true;
+        m.shared = read_silu_expert(c.sub("shared"));
+    }
+    if (!c.err->empty()) return m;
+    if (m.experts % m.groups) r.fail("groups.count does not divide experts");
+    else if (m.keep > m.groups) r.fail("groups.keep exceeds groups.count");
+    else if (m.top > m.experts / m.groups * m.keep) r.fail("top exceeds the experts of the groups kept");
+    return m;
+}
+
+int read_fatilix(const Json& cfg, ModelPlan* out) {
+    std::string err;
+    const Cfg c{&cfg, "", &err};
+    ModelPlan p;
+    p.name = "Fatilix";
+    p.vocab = c.size("vocab");
+    p.width = c.size("width");
+    p.max_positions = c.size("max_positions");
+    p.eps = (float)c.sub("norm").num("eps");
+    p.norm_gain = GAIN_OFFSET;
+    p.embed_scale = (float)c.sub("embedding").num("scale");
+    p.residual_mult = (float)c.num("residual_mult");
+    const Json* layers = cfg.get("layers");
+    if (!layers || layers->type != Json::ARR || layers->arr.empty()) c.fail("layers is missing or not a list");
+    for (size_t i = 0; err.empty() && i < layers->arr.size(); ++i) {
+        const std::string idx = std::to_string(i);
+        const Cfg lc{&layers->arr[i], "layers[" + idx + "].", &err};
+        LayerPlan l;
+        l.prefix = "l" + idx + ".";
+        const Json* type = lc.j->get("type");
+        const std::string t = type ? type->str : "";
+        if (t != "attention" && t != "attention_2") { lc.fail("type is not a mixer of this design"); break; }
+        l.mixer = MIX_GROUPED;
+        l.grouped = read_sink_attention(lc.sub("mixer"), t == "attention");
+        const Json* kind = lc.has("mlp") ? lc.sub("mlp").j->get("kind") : nullptr;
+        if (kind && kind->str == "moe") {
+            l.mlp = MLP_MOE;
+            l.moe = read_grouped_choice(lc.sub("mlp"));
+        } else {
+            read_dense(lc, &l);
         }
         p.layers.push_back(l);
     }
@@ -199,7 +302,7 @@ const ArchEntry ARCHS[] = {
     {"llama", ARCH_LLAMA, true, nullptr},   {"mistral", ARCH_LLAMA, true, nullptr}, {"qwen2", ARCH_LLAMA, true, nullptr},
     {"qwen3", ARCH_LLAMA, true, nullptr},   {"idefics3", ARCH_LLAMA, true, nullptr}, {"phi3", ARCH_LLAMA, true, nullptr},
     {"phi", ARCH_PHI2, true, nullptr},      {"phi2", ARCH_PHI2, true, nullptr},     {"Lepalorn", ARCH_PLAN, false, read_lepalorn},
-    {"Tedelix", ARCH_PLAN, false, read_tedelix},
+    {"Tedelix", ARCH_PLAN, false, read_tedelix}, {"Fatilix", ARCH_PLAN, false, read_fatilix},
 };
 
 }  // namespace

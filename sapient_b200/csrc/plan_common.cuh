@@ -19,10 +19,11 @@ template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __f
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-__device__ __forceinline__ float clamped_unit(float g, float u, float limit, float alpha) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g * sigmoid_f32(alpha * g) * (u + 1.0f);
+// The gated unit of plan_kernels.h: MatUnit.
+__device__ __forceinline__ float gated_unit(float g, float u, const MatUnit& p) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+    return g * sigmoid_f32(p.alpha * g) * (u + p.shift);
 }
 
 __device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
@@ -71,6 +72,9 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, int bytes
 }
 __device__ __forceinline__ void cp_async16_at(uint32_t dst, const void* src, int bytes) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_addr(dst)), "l"(src) : "memory");
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }

@@ -14,12 +14,17 @@ namespace sp {
 constexpr int MAT_KPAD = 64;
 inline int mat_kpad(int k) { return (k + MAT_KPAD - 1) / MAT_KPAD * MAT_KPAD; }
 
+// A gated unit: g = min(., limit), u = clamp(., +-limit), y = g sigmoid(alpha g) (u + shift).
+struct MatUnit {
+    float limit, alpha, shift;
+};
+
 // A family of equally shaped matrices [groups][rows][kp]. `dual`: rows = 2 n, the first n are the gate and the last n the
-// up-projection of a clamped gated unit, whose n activations are the output.
+// up-projection of a gated unit, whose n activations are the output.
 struct MatSeg {
     const void* w;
     int n, kp, groups;
-    float limit, alpha;        // dual: g = min(., limit), u = clamp(., +-limit), y = g sigmoid(alpha g) (u + 1)
+    MatUnit unit;              // dual
     const void* x;             // compute type
     int ldx;
     int64_t xgs;               // elements between the inputs of consecutive groups (per-head products)
@@ -93,15 +98,22 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st);
 int mat_tc5_take_timeout();    // as tc5_take_timeout (kernels.h)
 
 // ── the stream between the products ──
-// x0[t] = table[ids[t]] * scale (f32), xb (or null) = the same in the compute type (row stride ldb, padding zeroed).
-cudaError_t launch_embed_scaled(const void* table, int ldt, bool f32, const uint32_t* ids, int n_tok, int width, float scale, float* x0, void* xb,
-                                int ldb, cudaStream_t st);
-// x += rms_norm(y) * gain (one number), f32; xb as above.
-cudaError_t launch_norm_residual(const float* y, int ldy, const float* gain, float eps, const float* x, float* x_out, void* xb, int ldb, bool f32,
-                                 int n_tok, int width, cudaStream_t st);
+// x0[t] = table[ids[t]] * scale (+ pos_table[tok_pos[t]], or null) (f32), xb (or null) = the same in the compute type (row
+// stride ldb, padding zeroed). Both tables have rows of ldt.
+cudaError_t launch_embed_scaled(const void* table, const void* pos_table, int ldt, bool f32, const uint32_t* ids, const int32_t* tok_pos, int n_tok,
+                                int width, float scale, float* x0, void* xb, int ldb, cudaStream_t st);
+// The gain of a norm: one number, or one per coordinate.
+struct RowGain {
+    const float* g;
+    bool per_coord;
+};
+// x_out = x + mult * rms_norm(y) * gain, f32; xb as above.
+cudaError_t launch_norm_residual(const float* y, int ldy, const RowGain& gain, float eps, float mult, const float* x, float* x_out, void* xb, int ldb,
+                                 bool f32, int n_tok, int width, cudaStream_t st);
+// x_out = x + mult * rms_norm(mixture of expert outputs) * gain, then (dwa) the depth average.
 struct CombineArgs {
     const float* x;            // stream before the feed-forward
-    float* history;            // [depth + 1][rows_cap][width]: layer results, the embedding output first
+    float* history;            // [depth + 1][rows_cap][width]: layer results, the embedding output first (null: not kept)
     int64_t hist_stride;
     int depth;                 // this layer's result is history[depth]
     const float* dwa;          // [depth + 1] coefficients, null: no depth average
@@ -109,7 +121,8 @@ struct CombineArgs {
     void* xb;
     int ldb;
     bool f32;
-    // feed-forward (null y: none): sum over k of weight[t][k] * y[slot_of[t][k]] (+ sigmoid(shared_gate) * y_shared[t])
+    // feed-forward (null y: none): sum over k of weight[t][k] * y[slot_of[t][k]] (+ y_shared[t], times sigmoid(shared_gate)
+    // where that is given)
     const float* y;
     int ldy;
     const int32_t* slot_of;
@@ -118,22 +131,28 @@ struct CombineArgs {
     const float* y_shared;
     const float* shared_gate;
     int ld_gate;
-    const float* gain;
-    float eps;
+    RowGain gain;
+    float eps, mult;
 };
 cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStream_t st);
-// out (compute type) = rms_norm(x[rows[i] or i]) * gain; gain: one number, or one per coordinate (per_coord).
-cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, bool per_coord, float eps, void* out,
-                            int ldo, bool f32, cudaStream_t st);
+// out (compute type) = rms_norm(x[rows[i] or i]) * gain.
+cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const RowGain& gain, float eps, void* out, int ldo, bool f32,
+                            cudaStream_t st);
 
 // ── experts ──
-// Per token the `top` largest of logits[t][0..experts) + bias (ties: the lower index) with the softmax over the chosen ones
-// as weight[t][top], and the (token, choice) pairs sorted by expert: MoeRows tables and slot_of[t][k] = sorted row of a
-// pair. pick[t][top] is scratch.
+// How a token's experts follow from its logits (model_plan.h: RouteRule). Ties: the lower index.
+struct RouteShape {
+    int experts, top;
+    bool all;                  // ROUTE_ALL
+    int groups, keep;
+    float scale;
+};
+// Per token the chosen experts with their weights weight[t][top], and the (token, choice) pairs sorted by expert: MoeRows
+// tables and slot_of[t][k] = sorted row of a pair. pick[t][top] is scratch.
 struct MoeTables {
     int32_t *row_off, *row_src, *active, *n_active, *tile_group, *tile_row, *n_tiles, *slot_of;
 };
-cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
+cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, const RouteShape& r, int n_tok, int32_t* pick, float* weight,
                              const MoeTables& t, cudaStream_t st);
 // dst[i] = src[row_src[i]] for n rows of ld elements of the compute type (ld * element size a multiple of 16).
 cudaError_t launch_gather_act(const void* src, const int32_t* row_src, int n, int ld, bool f32, void* dst, cudaStream_t st);
@@ -184,30 +203,52 @@ cudaError_t launch_latent_expanded(const void* qf, const void* kv, const void* l
                                    const LatentTile* tiles, int n_tiles, const float* gate, int ldgate, void* out, int ldo, cudaStream_t st);
 
 // ── grouped attention ──
-// One layer's slice of the paged cache: [page][kv head][16 tokens][dim16 | vdim16] of the compute type, keys and values
-// rotated, padded with zeros to multiples of 16.
+// One layer's slice of the paged cache: [page][kv head][16 tokens][ld] of the compute type. A row is dim16 | vdim16: the
+// key and the value, rotated, padded with zeros to multiples of 16. Where the values are the keys (shared), a row is the key
+// as projected, once, and GROUPED_TAIL elements whose first four bytes are the f32 reciprocal of its root mean square (one
+// without a norm); scores take that factor, and the keys' norm weight is part of the queries.
+constexpr int GROUPED_TAIL = 8;
 struct GroupedCache {
     void* pool;
     const int32_t* page_table;
     int max_pages;
     int dim16, vdim16;
+    int ld;                    // shared ? dim16 + GROUPED_TAIL : dim16 + vdim16
+    bool shared;
 };
 struct GroupedShape {
     int heads, kv_heads, dim, vdim, rot;
     int window;
     float scale;
 };
-// proj[t] (f32, row stride ldp): queries head by head, keys, values. Rotates queries and keys by cs_key[pos][rot / 2] and,
-// where cs_val[pos][vdim / 2] is given, values; q[t][heads][dim16] in the compute type, keys and values to the cache.
-cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const float2* cs_key, const float2* cs_val,
+// What happens to queries, keys and values between the projection and the cache; null: nothing.
+struct GroupedInput {
+    const float* bias;         // [heads * dim | kv_heads * dim | kv_heads * vdim]
+    bool norm;                 // queries and keys over their root mean square ...
+    const float *q_gain, *k_gain;  // ... times [dim]
+    float eps;
+    const float* temperature;  // factor of the queries, by position
+    const float2 *cs_key, *cs_val;  // angles [pos][rot / 2] of queries and keys, [pos][vdim / 2] of values
+};
+// proj[t] (f32, row stride ldp): queries head by head, keys, values (not when shared). q[t][heads][dim16] in the compute type,
+// keys and values to the cache.
+cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in,
                                   const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st);
-// out[t][ldo] (compute type), head by head vdim values: the mixtures, turned back by cs_val (or null). Any sizes up to
-// GROUPED_MAX_VDIM. n_splits > 1 (bf16: grouped_attention_splits of the longest range to visit) splits the keys over the
-// blocks of a cluster.
+// What else enters the scores, the softmax and the output; null: nothing.
+struct GroupedTerms {
+    const float* rel;          // [heads][n_rel], added to the scaled score: by distance, the last one from there on
+    int n_rel;
+    const float* sink;         // [heads]: logit of one more term of the denominator
+    const float* gate;         // output times sigmoid(gate[t * ldgate + head * vdim + coordinate])
+    int64_t ldgate;
+    const float2* cs_val;      // mixtures are turned back by these angles
+};
+// out[t][ldo] (compute type), head by head vdim values: the mixtures. Any sizes up to GROUPED_MAX_VDIM. n_splits > 1 (bf16:
+// grouped_attention_splits of the longest range to visit) splits the keys over the blocks of a cluster.
 constexpr int GROUPED_MAX_VDIM = 1024;
 bool grouped_mma_supported(const GroupedShape& s);
 int grouped_attention_splits(const GroupedShape& s, int n_tok, int keys, bool f32);
-cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const int32_t* tok_slot,
+cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const int32_t* tok_slot,
                                      const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st);
 // bf16, many rows: tiles of up to GROUPED_Q_TILE consecutive tokens of one sequence.
 struct GroupedTile {
@@ -216,7 +257,7 @@ struct GroupedTile {
     int32_t slot;
 };
 constexpr int GROUPED_Q_TILE = 64;
-cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const float2* cs_val, const GroupedTile* tiles,
+cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const GroupedTile* tiles,
                                    int n_tiles, void* out, int ldo, cudaStream_t st);
 
 // ── mixers with a state matrix (model_plan.h: StateMixerSpec) ──

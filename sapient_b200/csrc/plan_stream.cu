@@ -31,71 +31,78 @@ template <> struct Row<4> {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __restrict__ table, int ldt, const uint32_t* __restrict__ ids, int width,
-                                                                  float scale, float* __restrict__ x0, T* __restrict__ xb, int ldb) {
+__global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __restrict__ table, const T* __restrict__ pos_table, int ldt,
+                                                                  const uint32_t* __restrict__ ids, const int32_t* __restrict__ tok_pos, int width, float scale,
+                                                                  float* __restrict__ x0, T* __restrict__ xb, int ldb) {
     pdl_wait();
     pdl_trigger();
     const int t = blockIdx.x;
     const T* row = table + (int64_t)ids[t] * ldt;
+    const T* prow = pos_table ? pos_table + (int64_t)tok_pos[t] * ldt : nullptr;
     for (int c = threadIdx.x; c < ldb; c += ST_THREADS) {
-        const float v = c < width ? to_f32(row[c]) * scale : 0.f;
+        float v = c < width ? to_f32(row[c]) * scale : 0.f;
+        if (prow && c < width) v += to_f32(prow[c]);
         if (c < width) x0[(int64_t)t * width + c] = v;
         if (xb) xb[(int64_t)t * ldb + c] = from_f32<T>(v);
     }
 }
 
-cudaError_t launch_embed_scaled(const void* table, int ldt, bool f32, const uint32_t* ids, int n_tok, int width, float scale, float* x0, void* xb,
-                                int ldb, cudaStream_t st) {
+cudaError_t launch_embed_scaled(const void* table, const void* pos_table, int ldt, bool f32, const uint32_t* ids, const int32_t* tok_pos, int n_tok,
+                                int width, float scale, float* x0, void* xb, int ldb, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    cudaError_t le = f32 ? launch_pdl(embed_scaled_kernel<float>, dim3(n_tok), dim3(ST_THREADS), 0, st, (const float*)table, ldt, ids, width, scale, x0, (float*)xb, ldb)
-                         : launch_pdl(embed_scaled_kernel<bf16>, dim3(n_tok), dim3(ST_THREADS), 0, st, (const bf16*)table, ldt, ids, width, scale, x0, (bf16*)xb, ldb);
+    const dim3 grid(n_tok), block(ST_THREADS);
+#define SP_EM(T) launch_pdl(embed_scaled_kernel<T>, grid, block, 0, st, (const T*)table, (const T*)pos_table, ldt, ids, tok_pos, width, scale, x0, (T*)xb, ldb)
+    const cudaError_t le = f32 ? SP_EM(float) : SP_EM(bf16);
+#undef SP_EM
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(ST_THREADS) norm_residual_kernel(const float* __restrict__ y, int ldy, const float* __restrict__ gain, float eps,
+__global__ void __launch_bounds__(ST_THREADS) norm_residual_kernel(const float* __restrict__ y, int ldy, const RowGain gain, float eps, float mult,
                                                                    const float* x, float* x_out, T* __restrict__ xb, int ldb, int width) {
     __shared__ float sh[ST_WARPS];
     pdl_wait();
     pdl_trigger();
     const int64_t t = blockIdx.x;
     const float* yr = y + t * ldy;
-    const float g = *gain;
-    float ss = 0.f, v[V], o[V];
+    const float g0 = gain.per_coord ? 1.f : *gain.g;
+    float ss = 0.f, v[V], o[V], g[V];
     for (int c = V * threadIdx.x; c < width; c += V * ST_THREADS) {
         Row<V>::load(yr + c, v);
 #pragma unroll
         for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
     }
-    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps) * g;
+    const float r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + eps) * g0 * mult;
+#pragma unroll
+    for (int i = 0; i < V; ++i) g[i] = 1.f;
     for (int c = V * threadIdx.x; c < ldb; c += V * ST_THREADS) {
 #pragma unroll
         for (int i = 0; i < V; ++i) o[i] = 0.f;
         if (c < width) {
             Row<V>::load(yr + c, v);
             Row<V>::load(x + t * width + c, o);
+            if (gain.per_coord) Row<V>::load(gain.g + c, g);
 #pragma unroll
-            for (int i = 0; i < V; ++i) o[i] = fmaf(v[i], r, o[i]);
+            for (int i = 0; i < V; ++i) o[i] = fmaf(v[i] * g[i], r, o[i]);
             Row<V>::store(x_out + t * width + c, o);
         }
         Row<V>::store(xb + t * ldb + c, o);
     }
 }
 
-template <typename T>
-static cudaError_t norm_residual_by_width(const float* y, int ldy, const float* gain, float eps, const float* x, float* x_out, void* xb, int ldb,
-                                          int n_tok, int width, cudaStream_t st) {
-    return width % 4 == 0 && ldy % 4 == 0
-               ? launch_pdl(norm_residual_kernel<T, 4>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (T*)xb, ldb, width)
-               : launch_pdl(norm_residual_kernel<T, 1>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, x, x_out, (T*)xb, ldb, width);
+// Four coordinates at a time: rows and gains start on 16-byte boundaries.
+static bool wide_rows(int width, int ld, const RowGain& gain) {
+    return width % 4 == 0 && ld % 4 == 0 && (!gain.per_coord || (reinterpret_cast<uintptr_t>(gain.g) & 15) == 0);
 }
 
-cudaError_t launch_norm_residual(const float* y, int ldy, const float* gain, float eps, const float* x, float* x_out, void* xb, int ldb, bool f32,
-                                 int n_tok, int width, cudaStream_t st) {
+cudaError_t launch_norm_residual(const float* y, int ldy, const RowGain& gain, float eps, float mult, const float* x, float* x_out, void* xb, int ldb,
+                                 bool f32, int n_tok, int width, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
-    cudaError_t le = f32 ? norm_residual_by_width<float>(y, ldy, gain, eps, x, x_out, xb, ldb, n_tok, width, st)
-                         : norm_residual_by_width<bf16>(y, ldy, gain, eps, x, x_out, xb, ldb, n_tok, width, st);
+    const bool wide = wide_rows(width, ldy, gain);
+#define SP_NR(T, V) launch_pdl(norm_residual_kernel<T, V>, dim3(n_tok), dim3(ST_THREADS), 0, st, y, ldy, gain, eps, mult, x, x_out, (T*)xb, ldb, width)
+    const cudaError_t le = f32 ? (wide ? SP_NR(float, 4) : SP_NR(float, 1)) : (wide ? SP_NR(bf16, 4) : SP_NR(bf16, 1));
+#undef SP_NR
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
 }
@@ -118,11 +125,11 @@ __global__ void __launch_bounds__(ST_THREADS) combine_kernel(const CombineArgs a
     }
     if (a.dwa)
         for (int j = threadIdx.x; j <= a.depth; j += ST_THREADS) dwa_s[j] = a.dwa[j];
-    const float sg = a.shared_gate ? sigmoid_f32(a.shared_gate[t * a.ld_gate]) : 0.f;
+    const float sg = a.shared_gate ? sigmoid_f32(a.shared_gate[t * a.ld_gate]) : 1.f;
     __syncthreads();
     float r = 0.f;
     if (a.y) {
-        const float gain = *a.gain;
+        const float gain = a.gain.per_coord ? 1.f : *a.gain.g;
         float ss = 0.f;
         for (int c = V * threadIdx.x; c < width; c += V * ST_THREADS) {
             float s[V], q[V];
@@ -143,9 +150,9 @@ __global__ void __launch_bounds__(ST_THREADS) combine_kernel(const CombineArgs a
 #pragma unroll
             for (int i = 0; i < V; ++i) ss = fmaf(s[i], s[i], ss);
         }
-        r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + a.eps) * gain;
+        r = rsqrtf(block_sum<ST_WARPS>(ss, sh) / (float)width + a.eps) * gain * a.mult;
     }
-    float* mine = a.history + (int64_t)a.depth * a.hist_stride + t * width;
+    float* mine = a.history ? a.history + (int64_t)a.depth * a.hist_stride + t * width : nullptr;
     for (int c = V * threadIdx.x; c < a.ldb; c += V * ST_THREADS) {
         float v[V], q[V];
 #pragma unroll
@@ -154,10 +161,16 @@ __global__ void __launch_bounds__(ST_THREADS) combine_kernel(const CombineArgs a
             Row<V>::load(a.x + t * width + c, v);
             if (a.y) {
                 Row<V>::load(ff + c, q);  // written above by this same thread
+                if (a.gain.per_coord) {
+                    float g[V];
+                    Row<V>::load(a.gain.g + c, g);
+#pragma unroll
+                    for (int i = 0; i < V; ++i) q[i] *= g[i];
+                }
 #pragma unroll
                 for (int i = 0; i < V; ++i) v[i] = fmaf(q[i], r, v[i]);
             }
-            Row<V>::store(mine + c, v);
+            if (mine) Row<V>::store(mine + c, v);
             if (a.dwa) {
                 const float* h = a.history + t * width + c;
                 float s[V];
@@ -195,7 +208,7 @@ cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStrea
     });
     if (le != cudaSuccess) return le;
     const dim3 grid(n_tok), block(ST_THREADS);
-    if (width % 4 == 0) le = a.f32 ? launch_pdl(combine_kernel<float, 4>, grid, block, smem, st, a, width) : launch_pdl(combine_kernel<bf16, 4>, grid, block, smem, st, a, width);
+    if (wide_rows(width, a.y ? a.ldy : width, a.gain)) le = a.f32 ? launch_pdl(combine_kernel<float, 4>, grid, block, smem, st, a, width) : launch_pdl(combine_kernel<bf16, 4>, grid, block, smem, st, a, width);
     else le = a.f32 ? launch_pdl(combine_kernel<float, 1>, grid, block, smem, st, a, width) : launch_pdl(combine_kernel<bf16, 1>, grid, block, smem, st, a, width);
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
@@ -203,7 +216,7 @@ cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStrea
 
 template <typename T, int V>
 __global__ void __launch_bounds__(ST_THREADS) row_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, int width,
-                                                              const float* __restrict__ gain, bool per_coord, float eps, T* __restrict__ out, int ldo) {
+                                                              const RowGain gain, float eps, T* __restrict__ out, int ldo) {
     __shared__ float sh[ST_WARPS];
     pdl_wait();
     pdl_trigger();
@@ -220,20 +233,20 @@ __global__ void __launch_bounds__(ST_THREADS) row_norm_kernel(const float* __res
         for (int i = 0; i < V; ++i) v[i] = 0.f;
         if (c < width) {
             Row<V>::load(xr + c, v);
-            if (per_coord) Row<V>::load(gain + c, g);
+            if (gain.per_coord) Row<V>::load(gain.g + c, g);
 #pragma unroll
-            for (int i = 0; i < V; ++i) v[i] = v[i] * r * (per_coord ? g[i] : *gain);
+            for (int i = 0; i < V; ++i) v[i] = v[i] * r * (gain.per_coord ? g[i] : *gain.g);
         }
         Row<V>::store(out + (int64_t)blockIdx.x * ldo + c, v);
     }
 }
 
-cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const float* gain, bool per_coord, float eps, void* out,
-                            int ldo, bool f32, cudaStream_t st) {
+cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const RowGain& gain, float eps, void* out, int ldo, bool f32,
+                            cudaStream_t st) {
     if (n_rows == 0) return cudaSuccess;
-    const bool wide = width % 4 == 0 && ldo % 4 == 0 && (!per_coord || (reinterpret_cast<uintptr_t>(gain) & 15) == 0);
+    const bool wide = wide_rows(width, ldo, gain);
     const dim3 grid(n_rows), block(ST_THREADS);
-#define SP_RN(T, V) launch_pdl(row_norm_kernel<T, V>, grid, block, 0, st, x, rows, width, gain, per_coord, eps, (T*)out, ldo)
+#define SP_RN(T, V) launch_pdl(row_norm_kernel<T, V>, grid, block, 0, st, x, rows, width, gain, eps, (T*)out, ldo)
     const cudaError_t le = f32 ? (wide ? SP_RN(float, 4) : SP_RN(float, 1)) : (wide ? SP_RN(bf16, 4) : SP_RN(bf16, 1));
 #undef SP_RN
     if (le != cudaSuccess) return le;
@@ -241,28 +254,67 @@ cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int
 }
 
 // ── experts ──
-// One warp's choice for token t: its logits wait in shared memory (z, `experts` floats) and a chosen one is struck out.
-__device__ __forceinline__ void choose_experts(const float* __restrict__ logits, const float* __restrict__ bias, int experts, int top, float* z,
+// Index of the largest of z[0 .. n) that is below `below`, the lower index first; *value is it. Past n: none (or only NaN).
+__device__ __forceinline__ int warp_argmax(const float* z, int n, float below, float* value) {
+    float v = -INFINITY;
+    int at = 0x7FFFFFFF;
+    for (int e = threadIdx.x & 31; e < n; e += 32)
+        if (z[e] < below && (z[e] > v || (z[e] == v && e < at))) { v = z[e]; at = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xFFFFFFFFu, v, o);
+        const int oa = __shfl_xor_sync(0xFFFFFFFFu, at, o);
+        if (ov > v || (ov == v && oa < at)) { v = ov; at = oa; }
+    }
+    *value = v;
+    return at;
+}
+
+__host__ __device__ __forceinline__ int route_floats(const RouteShape& r) { return r.experts + (r.keep < r.groups ? r.groups : 0); }
+
+// One warp's choice for a token: its logits (ROUTE_ALL: probabilities) plus bias wait in shared memory (z, route_floats) and a
+// chosen one is struck out.
+__device__ __forceinline__ void choose_experts(const float* __restrict__ logits, const float* __restrict__ bias, const RouteShape& r, float* z,
                                                int32_t* pick, float* weight) {
-    const int lane = threadIdx.x & 31;
-    for (int e = lane; e < experts; e += 32) z[e] = logits[e] + (bias ? bias[e] : 0.f);
+    const int lane = threadIdx.x & 31, experts = r.experts, top = r.top;
+    float best = -INFINITY, all = 0.f;
+    if (r.all) {
+        for (int e = lane; e < experts; e += 32) best = fmaxf(best, logits[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) best = fmaxf(best, __shfl_xor_sync(0xFFFFFFFFu, best, o));
+        for (int e = lane; e < experts; e += 32) all += expf(logits[e] - best);
+        all = warp_sum(all);
+    }
+    for (int e = lane; e < experts; e += 32) z[e] = (r.all ? expf(logits[e] - best) / all : logits[e]) + (bias ? bias[e] : 0.f);
     __syncwarp();
+    float v;
+    if (r.keep < r.groups) {  // a kept group is marked by an infinite score, the experts of the others are struck out
+        const int run = experts / r.groups;
+        float* gs = z + experts;
+        for (int g = lane; g < r.groups; g += 32) {
+            float m = -INFINITY;
+            for (int e = g * run; e < (g + 1) * run; ++e) m = fmaxf(m, z[e]);
+            gs[g] = m;
+        }
+        __syncwarp();
+        for (int k = 0; k < r.keep; ++k) {
+            const int at = warp_argmax(gs, r.groups, INFINITY, &v);
+            __syncwarp();
+            if (lane == 0 && at < r.groups) gs[at] = INFINITY;
+            __syncwarp();
+        }
+        for (int e = lane; e < experts; e += 32)
+            if (gs[e / run] != INFINITY) z[e] = -INFINITY;
+        __syncwarp();
+    }
     float best0 = 0.f, sum = 0.f;
     for (int k = 0; k < top; ++k) {
-        float v = -INFINITY;
-        int at = 0x7FFFFFFF;
-        for (int e = lane; e < experts; e += 32)
-            if (z[e] > v || (z[e] == v && e < at)) { v = z[e]; at = e; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xFFFFFFFFu, v, o);
-            const int oa = __shfl_xor_sync(0xFFFFFFFFu, at, o);
-            if (ov > v || (ov == v && oa < at)) { v = ov; at = oa; }
-        }
+        int at = warp_argmax(z, experts, INFINITY, &v);
         if (at >= experts) at = k;  // logits that compare with nothing (NaN) still name a valid expert
         if (k == 0) best0 = v;
-        const float ex = expf(v - best0);
+        const float ex = r.all ? expf(logits[at] - best) / all : expf(v - best0);
         sum += ex;
+        __syncwarp();
         if (lane == 0) {
             pick[k] = at;
             weight[k] = ex;
@@ -270,18 +322,19 @@ __device__ __forceinline__ void choose_experts(const float* __restrict__ logits,
         }
         __syncwarp();
     }
-    for (int k = lane; k < top; k += 32) weight[k] /= sum;
+    const float norm = r.all ? r.scale / (sum + 1e-20f) : 1.f / sum;
+    for (int k = lane; k < top; k += 32) weight[k] *= norm;
 }
 
 constexpr int TK_WARPS = 4;
 __global__ void __launch_bounds__(TK_WARPS * 32) moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok,
-                                                                 int experts, int top, int32_t* __restrict__ pick, float* __restrict__ weight) {
+                                                                 const RouteShape r, int32_t* __restrict__ pick, float* __restrict__ weight) {
     extern __shared__ float tk_smem[];
     pdl_wait();
     pdl_trigger();
     const int warp = threadIdx.x >> 5, t = blockIdx.x * TK_WARPS + warp;
     if (t >= n_tok) return;
-    choose_experts(logits + (int64_t)t * ld, bias, experts, top, tk_smem + warp * experts, pick + (int64_t)t * top, weight + (int64_t)t * top);
+    choose_experts(logits + (int64_t)t * ld, bias, r, tk_smem + warp * route_floats(r), pick + (int64_t)t * r.top, weight + (int64_t)t * r.top);
 }
 
 // One block: counts per expert, prefix sums, the tables. Within an expert the rows come in no particular order (every row
@@ -341,32 +394,34 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int32_t* __restri
 }
 
 // Choice and grouping of up to 8 tokens in one block, a warp per token.
-__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok, int experts,
-                                                         int top, float* __restrict__ weight, const MoeTables t) {
+__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int n_tok,
+                                                         const RouteShape r, float* __restrict__ weight, const MoeTables t) {
     extern __shared__ int mr_smem[];  // counts and offsets, the choices, a row of logits per warp
     pdl_wait();
     pdl_trigger();
-    int* pick = mr_smem + 2 * experts;
-    float* z = reinterpret_cast<float*>(pick + n_tok * top);
+    int* pick = mr_smem + 2 * r.experts;
+    float* z = reinterpret_cast<float*>(pick + n_tok * r.top);
     const int warp = threadIdx.x >> 5;
-    if (warp < n_tok) choose_experts(logits + (int64_t)warp * ld, bias, experts, top, z + warp * experts, pick + warp * top, weight + (int64_t)warp * top);
+    if (warp < n_tok) choose_experts(logits + (int64_t)warp * ld, bias, r, z + warp * route_floats(r), pick + warp * r.top, weight + (int64_t)warp * r.top);
     __syncthreads();
-    group_rows(pick, n_tok * top, experts, top, t, mr_smem);
+    group_rows(pick, n_tok * r.top, r.experts, r.top, t, mr_smem);
 }
 
-cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, int n_tok, int experts, int top, int32_t* pick, float* weight,
+cudaError_t launch_moe_route(const float* logits, int ld, const float* bias, const RouteShape& r, int n_tok, int32_t* pick, float* weight,
                              const MoeTables& t, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
+    if (r.groups < 1 || r.keep < 1 || r.keep > r.groups || r.experts % r.groups || r.top > r.experts / r.groups * r.keep) return cudaErrorInvalidValue;
     constexpr size_t CAP = 48 * 1024;
-    const size_t small = ((size_t)(2 + n_tok) * experts + (size_t)n_tok * top) * 4;
+    const int experts = r.experts, top = r.top, z = route_floats(r);
+    const size_t small = ((size_t)2 * experts + (size_t)n_tok * (z + top)) * 4;
     if (n_tok <= 8 && small <= CAP) {
-        const cudaError_t le = launch_pdl(moe_route_kernel, dim3(1), dim3(256), small, st, logits, ld, bias, n_tok, experts, top, weight, t);
+        const cudaError_t le = launch_pdl(moe_route_kernel, dim3(1), dim3(256), small, st, logits, ld, bias, n_tok, r, weight, t);
         return le != cudaSuccess ? le : count_launch_and_check();
     }
-    const size_t rows = (size_t)TK_WARPS * experts * 4, counts = (size_t)experts * 8;
+    const size_t rows = (size_t)TK_WARPS * z * 4, counts = (size_t)experts * 8;
     if (rows > CAP || counts > CAP) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(moe_topk_kernel, dim3((n_tok + TK_WARPS - 1) / TK_WARPS), dim3(TK_WARPS * 32), rows, st, logits, ld, bias, n_tok, experts, top,
-                                pick, weight);
+    cudaError_t le = launch_pdl(moe_topk_kernel, dim3((n_tok + TK_WARPS - 1) / TK_WARPS), dim3(TK_WARPS * 32), rows, st, logits, ld, bias, n_tok, r, pick,
+                                weight);
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     le = launch_pdl(moe_group_kernel, dim3(1), dim3(1024), counts, st, (const int32_t*)pick, n_tok * top, experts, top, t);
