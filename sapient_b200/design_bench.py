@@ -28,6 +28,13 @@ TEDELIX = {
     "8b": dict(layers=_PATTERN, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, state_heads=64, state_dim=64, state_vdim=64, window=2048, ff=12288, vocab=32768),
 }
 TEDELIX_RANK = 64  # of the decay logits
+# dense and active expert feed-forwards of a size have equal weights
+FATILIX = {
+    "2b": dict(layers=["attention_2", "attention"] * 3, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=9216, experts=64, top=8, groups=8, keep=4,
+               expert_ff=512, shared_ff=2048, vocab=32768, max_positions=4096, bias_max=512),
+    "8b": dict(layers=["attention_2", "attention"] * 2, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=18432, experts=32, top=4, groups=4, keep=2,
+               expert_ff=2048, shared_ff=4096, vocab=32768, max_positions=4096, bias_max=512),
+}
 
 
 def lepalorn_llama(s: dict) -> dict:
@@ -38,6 +45,11 @@ def lepalorn_llama(s: dict) -> dict:
 def tedelix_llama(s: dict) -> dict:
     """Same width, heads, layers and feed-forward weights (three matrices for two)."""
     return _llama(s, len(s["layers"]), s["kv_heads"], 2 * s["ff"] // 3)
+
+
+def fatilix_llama(s: dict) -> dict:
+    """Same width, heads, layers and active feed-forward weights."""
+    return _llama(s, len(s["layers"]), s["kv_heads"], s["top"] * s["expert_ff"] + s["shared_ff"])
 
 
 def _llama(s: dict, layers: int, kv_heads: int, ffn: int) -> dict:
@@ -53,6 +65,11 @@ def lepalorn_model(s: dict):
 def tedelix_model(s: dict):
     cfg = synth.tedelix_config(**s)
     return cfg, synth.tedelix_weights(cfg, seed=11, rank=TEDELIX_RANK, device="cuda")
+
+
+def fatilix_model(s: dict):
+    cfg = synth.fatilix_config(**s)
+    return cfg, synth.fatilix_weights(cfg, seed=11, device="cuda")
 
 
 def design_engine(cfg: dict, W: dict, **kw):
@@ -124,6 +141,22 @@ def tedelix_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
             "norm": (rows * W * 6 * L, 0), "rope_kv": (rows * n["attention"] * 6 * (H * D + G * (D + V)), 0)}
 
 
+def fatilix_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    """The same. Cached rows are read once: keys and values, or keys that are the values with their f32 factor; queries, mixtures
+    and gate logits move once per token."""
+    W, H, G, D, V, E, top = (s[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "experts", "top"))
+    n = {t: s["layers"].count(t) for t in ("attention", "attention_2")}
+    L = len(s["layers"])
+    mats = L * (H * (D + 2 * V) + G * D) * W + n["attention_2"] * (G * V + 2 * s["ff"]) * W + n["attention"] * (E + 3 * s["shared_ff"]) * W
+    active, used, head = n["attention"] * 3 * s["expert_ff"] * W, _distinct(E, top, rows), s["vocab"] * W
+    keys = _pairs(rows, 1 << 30) if prefill else rows * ctx
+    cached = G * (n["attention"] * (2 * D + 4) + n["attention_2"] * 2 * (D + V))
+    return {"gemv": (2 * (mats + active * used + head), 2 * rows * (mats + active * top) + 2 * head * (1 if prefill else rows)),
+            "attention": (cached * (rows if prefill else keys) + L * rows * H * (2 * D + 6 * V), L * 2 * H * (D + V) * keys),
+            "norm": (rows * W * (14 * L + n["attention_2"] * 14 + n["attention"] * (14 + 4 * top)), 0),
+            "rope_kv": (rows * (L * 6 * H * D + G * (n["attention"] * (6 * D + 4) + n["attention_2"] * 6 * (D + V))), 0)}
+
+
 def llama_work(c: dict, rows: int, ctx: int, prefill: bool) -> dict:
     q, kv = c["n_heads"] * c["head_dim"], c["n_kv_heads"] * c["head_dim"]
     mats = c["n_layers"] * (2 * (q + kv) * c["hidden"] + 3 * c["ffn"] * c["hidden"])
@@ -136,7 +169,8 @@ def llama_work(c: dict, rows: int, ctx: int, prefill: bool) -> dict:
 
 # design -> (sizes, model of a size, its work, the Llama block of equal size)
 DESIGNS = {"lepalorn": ("Lepalorn", LEPALORN, lepalorn_model, lepalorn_work, lepalorn_llama),
-           "tedelix": ("Tedelix", TEDELIX, tedelix_model, tedelix_work, tedelix_llama)}
+           "tedelix": ("Tedelix", TEDELIX, tedelix_model, tedelix_work, tedelix_llama),
+           "fatilix": ("Fatilix", FATILIX, fatilix_model, fatilix_work, fatilix_llama)}
 
 
 def _families(ms: dict, work: dict, peaks: dict) -> dict:

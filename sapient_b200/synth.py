@@ -502,6 +502,71 @@ def tedelix_weights(cfg: dict, seed: int, rank: int = 64, device: str = "cpu") -
     return W
 
 
+def fatilix_config(layers, width: int, heads: int, kv_heads: int, dim: int, vdim: int, ff: int, experts: int, top: int, groups: int, keep: int,
+                   expert_ff: int, shared_ff: int, vocab: int, max_positions: int, bias_max: int, temp_every: int = 256, dense_types=("attention_2",)) -> dict:
+    """layers: the types in order; layers of one type are equal. Layers of `dense_types` have a dense feed-forward, the others
+    experts. Values of `attention` are its keys, so their size is dim."""
+    temp = {"coef": 0.3, "every": temp_every}
+    mixers = {"attention": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": temp},
+              "attention_2": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "q_temp": temp, "bias_max": bias_max}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 2.0}, "expert": {"ff": expert_ff}}
+    if shared_ff:
+        moe["shared"] = {"ff": shared_ff}
+    return {"architecture": "Fatilix", "vocab": vocab, "width": width, "max_positions": max_positions, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "residual_mult": 0.5, "layers": [{"type": t, "mixer": dict(mixers[t]), "mlp": {"kind": "dense", "ff": ff} if t in dense_types else dict(moe)} for t in layers]}
+
+
+def fatilix_weights(cfg: dict, seed: int, bias_rows: int = 32, device: str = "cpu") -> dict:
+    """Random bf16 weights, rows scaled so that activations keep their magnitude. bias_rows: of the distance bias tables."""
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W: dict = {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = (torch.randn(n, k, generator=g, device=device, dtype=torch.float32) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(name, n, mean=0.0, spread=0.1):
+        W[name] = (mean + spread * torch.randn(n, generator=g, device=device)).to(torch.bfloat16)
+
+    w = cfg["width"]
+    mat("embed", cfg["vocab"], w, w ** 0.5)
+    mat("pos", cfg["max_positions"], w, 0.3 * w ** 0.5)
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp, p = layer["mixer"], layer.get("mlp"), f"l{i}."
+        H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        shared = layer["type"] == "attention"
+        vec(p + "norm1", w)
+        for n, rows in (("q", H * D), ("k", G * D)) + (() if shared else (("v", G * V),)):
+            mat(p + "mix." + n, rows, w)
+            if not shared:
+                vec(p + f"mix.{n}.b", rows)
+        if shared:
+            vec(p + "mix.q.norm", D, 1.0)
+            vec(p + "mix.k.norm", D, 1.0)
+        else:
+            mat(p + "mix.rel", bias_rows, H, H ** 0.5)
+        vec(p + "mix.sink", H, 0.0, 1.0)
+        mat(p + "mix.g", H * V, w)
+        mat(p + "mix.o", w, H * V)
+        if not mlp:
+            continue
+        vec(p + "norm2", w)
+        if mlp["kind"] == "dense":
+            mat(p + "mlp.up", mlp["ff"], w)
+            mat(p + "mlp.down", w, mlp["ff"])
+            continue
+        E = mlp["router"]["experts"]
+        mat(p + "mlp.router", E, w)
+        vec(p + "mlp.correction", E, 0.0, 0.5 / E)
+        for tag, ff in [(f"mlp.e{e}.", mlp["expert"]["ff"]) for e in range(E)] + ([("mlp.shared.", mlp["shared"]["ff"])] if mlp.get("shared") else []):
+            mat(p + tag + "gate", ff, w)
+            mat(p + tag + "up", ff, w)
+            mat(p + tag + "down", w, ff)
+    vec("final.norm", w)
+    mat("head", cfg["vocab"], w)
+    return W
+
+
 def write_safetensors(path: str, cfg: dict, W: dict) -> None:
     """A model directory: config.json and model.safetensors (bf16 tensors)."""
     import json
