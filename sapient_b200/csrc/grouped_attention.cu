@@ -195,13 +195,14 @@ static size_t gd_smem(const GroupedCache& c) {
     return std::max(ring, mixtures);
 }
 
-template <int VT, bool PACKED>
+// REL: a distance bias, SHARED: keys that are the values.
+template <int VT, bool PACKED, bool REL, bool SHARED>
 __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c,
                                                                     const GroupedTerms x, const int32_t* __restrict__ tok_slot,
                                                                     const int32_t* __restrict__ tok_pos, bf16* __restrict__ out, int ldo, int n_splits) {
     extern __shared__ __align__(16) bf16 gd_sm[];
     __shared__ float m_s[GD_WARPS][16], l_s[GD_WARPS][16], bm_s[16], bl_s[16], share_s[16][GD_MAX_SPLITS];
-    const int ld = c.ld, LD = gd_row(c), LQ = c.dim16 + 8, val = c.shared ? 0 : c.dim16;
+    const int ld = c.ld, LD = gd_row(c), LQ = c.dim16 + 8, val = SHARED ? 0 : c.dim16;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int group = s.heads / s.kv_heads, tiles = (group + 15) / 16, kvh = blockIdx.x / tiles, h0 = kvh * group + (blockIdx.x % tiles) * 16;
     const int nq = min(16, (kvh + 1) * group - h0), t = blockIdx.y;
@@ -239,10 +240,22 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const uint32_t qa = smem_addr(qs + (lane & 15) * LQ + (lane >> 4) * 8);
     // this thread's heads' biases by distance (PACKED: one head), and the one for every key that is far
-    const float* rel0 = x.rel ? x.rel + (int64_t)(h0 + min(g, nq - 1)) * x.n_rel : nullptr;
-    const float* rel1 = x.rel ? x.rel + (int64_t)(h0 + min(g + 8, nq - 1)) * x.n_rel : nullptr;
-    const float far0 = rel0 ? rel0[x.n_rel - 1] : 0.f, far1 = rel1 ? rel1[x.n_rel - 1] : 0.f;
+    const float* rel0 = REL ? x.rel + (int64_t)(h0 + min(g, nq - 1)) * x.n_rel : nullptr;
+    const float* rel1 = REL && !PACKED ? x.rel + (int64_t)(h0 + min(g + 8, nq - 1)) * x.n_rel : nullptr;
+    const float far0 = REL ? rel0[x.n_rel - 1] : 0.f, far1 = REL && !PACKED ? rel1[x.n_rel - 1] : 0.f;
     for (int page = page0, st = 0; page <= page_end; page += stride, st = st + 1 == GD_STAGES ? 0 : st + 1) {
+        float b0[2][2], b1[2][2];
+        if (REL) {
+            const bool near = pos - (page * KV_PAGE + KV_PAGE - 1) < x.n_rel - 1;
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int dist = max(0, min(pos - (page * KV_PAGE + 8 * j + 2 * tq + e), x.n_rel - 1));
+                    b0[j][e] = near ? rel0[dist] : far0;
+                    b1[j][e] = PACKED ? 0.f : near ? rel1[dist] : far1;
+                }
+        }
         cp_async_wait<GD_STAGES - 1>();
         __syncwarp();
         const bf16* kt = ring + st * KV_PAGE * LD;
@@ -257,22 +270,16 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const bf1
             mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
         }
         float x0 = m0, x1 = m1;
-        const bool near = x.rel && pos - (page * KV_PAGE + KV_PAGE - 1) < x.n_rel - 1;
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = page * KV_PAGE + 8 * j + 2 * tq + e;
                 const bool on = key >= lo && key <= pos;
-                float f = s.scale, b0 = far0, b1 = far1;
-                if (c.shared) f *= row_factor(kt + (8 * j + 2 * tq + e) * LD, c.dim16);
-                if (near) {
-                    const int dist = max(0, min(pos - key, x.n_rel - 1));
-                    b0 = rel0[dist];
-                    if (!PACKED) b1 = rel1[dist];
-                }
-                sc[j][e] = on ? fmaf(sc[j][e], f, b0) : -INFINITY;
-                sc[j][2 + e] = on ? fmaf(sc[j][2 + e], f, b1) : -INFINITY;
+                float f = s.scale;
+                if (SHARED) f *= row_factor(kt + (8 * j + 2 * tq + e) * LD, c.dim16);
+                sc[j][e] = on ? (REL ? fmaf(sc[j][e], f, b0[j][e]) : sc[j][e] * f) : -INFINITY;
+                sc[j][2 + e] = on ? (REL ? fmaf(sc[j][2 + e], f, b1[j][e]) : sc[j][2 + e] * f) : -INFINITY;
                 x0 = fmaxf(x0, sc[j][e]);
                 x1 = fmaxf(x1, sc[j][2 + e]);
             }
@@ -426,38 +433,41 @@ int grouped_attention_splits(const GroupedShape& s, int n_tok, int keys, bool f3
     return n;
 }
 
+using GroupedDecodeFn = void (*)(const bf16*, GroupedShape, GroupedCache, GroupedTerms, const int32_t*, const int32_t*, bf16*, int, int);
+template <int VT>
+static GroupedDecodeFn gd_kernel(bool packed, bool rel, bool shared) {
+    if (packed) return rel ? (shared ? grouped_decode_kernel<VT, true, true, true> : grouped_decode_kernel<VT, true, true, false>)
+                           : (shared ? grouped_decode_kernel<VT, true, false, true> : grouped_decode_kernel<VT, true, false, false>);
+    return rel ? (shared ? grouped_decode_kernel<VT, false, true, true> : grouped_decode_kernel<VT, false, true, false>)
+               : (shared ? grouped_decode_kernel<VT, false, false, true> : grouped_decode_kernel<VT, false, false, false>);
+}
+static GroupedDecodeFn gd_kernel(int vdim16, bool packed, bool rel, bool shared) {
+    return vdim16 <= 32 ? gd_kernel<4>(packed, rel, shared) : vdim16 <= 64 ? gd_kernel<8>(packed, rel, shared)
+                      : vdim16 <= 128 ? gd_kernel<16>(packed, rel, shared) : gd_kernel<32>(packed, rel, shared);
+}
+
 cudaError_t launch_grouped_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const int32_t* tok_slot,
                                      const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
     if (n_splits < 1 || n_splits > GD_MAX_SPLITS || (n_splits & (n_splits - 1)) || s.vdim > GROUPED_MAX_VDIM) return cudaErrorInvalidValue;
-    constexpr int CAP = 220 * 1024;
-    static PerDeviceOnce once;
-    cudaError_t le = once.run([] {
-        const void* fns[] = {(const void*)grouped_decode_kernel<4, true>, (const void*)grouped_decode_kernel<8, true>, (const void*)grouped_decode_kernel<16, true>,
-                             (const void*)grouped_decode_kernel<32, true>, (const void*)grouped_decode_kernel<4, false>, (const void*)grouped_decode_kernel<8, false>,
-                             (const void*)grouped_decode_kernel<16, false>, (const void*)grouped_decode_kernel<32, false>};
-        for (const void* f : fns) {
-            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
-            if (e != cudaSuccess) return e;
-        }
-        return cudaSuccess;
-    });
-    if (le != cudaSuccess) return le;
-    const int group = s.heads / s.kv_heads;
+    cudaError_t le;
     if (!f32 && grouped_mma_supported(s)) {
+        constexpr int CAP = 220 * 1024;
+        static PerDeviceOnce once;
+        le = once.run([] {
+            for (int i = 0; i < 32; ++i) {
+                const cudaError_t e = cudaFuncSetAttribute((const void*)gd_kernel(32 << (i >> 3), i & 1, i & 2, i & 4), cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+                if (e != cudaSuccess) return e;
+            }
+            return cudaSuccess;
+        });
+        if (le != cudaSuccess) return le;
+        const int group = s.heads / s.kv_heads;
         const size_t smem = gd_smem(c);
         if (smem > CAP) return cudaErrorInvalidValue;
         const dim3 grid(s.kv_heads * ((group + 15) / 16), n_tok, n_splits), block(GD_WARPS * 32);
-#define SP_GD(VT)                                                                                                                                     \
-    le = group <= 8 ? launch_pdl_cluster(grouped_decode_kernel<VT, true>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, x, tok_slot, tok_pos, \
-                                         (bf16*)out, ldo, n_splits)                                                                                   \
-                    : launch_pdl_cluster(grouped_decode_kernel<VT, false>, grid, block, smem, st, n_splits, (const bf16*)q, s, c, x, tok_slot, tok_pos, \
-                                         (bf16*)out, ldo, n_splits)
-        if (c.vdim16 <= 32) SP_GD(4);
-        else if (c.vdim16 <= 64) SP_GD(8);
-        else if (c.vdim16 <= 128) SP_GD(16);
-        else SP_GD(32);
-#undef SP_GD
+        le = launch_pdl_cluster(gd_kernel(c.vdim16, group <= 8, x.rel, c.shared), grid, block, smem, st, n_splits, (const bf16*)q, s, c, x, tok_slot, tok_pos,
+                                (bf16*)out, ldo, n_splits);
         return le != cudaSuccess ? le : count_launch_and_check();
     }
     const dim3 grid(s.heads, n_tok), block(GS_WARPS * 32);
@@ -474,17 +484,17 @@ constexpr int GP_KEYS = 64, GP_WARPS = 4;
 static_assert(GROUPED_TAIL == 8, "a shared row's tail is the padding of its row in shared memory");
 static size_t gp_smem(const GroupedCache& c) { return (size_t)(3 * 64 * (c.dim16 + 8) + (c.shared ? 0 : 2 * GP_KEYS * (c.vdim16 + 8))) * 2; }
 
-template <int VT>
+template <int VT, bool REL, bool SHARED>
 __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c,
                                                                      const GroupedTerms x, const GroupedTile* __restrict__ tiles,
                                                                      bf16* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) bf16 gp_sm[];
-    __shared__ float rel_s[2][GP_KEYS + 64];  // biases of a key tile: by 63 - (query row) + (key in the tile)
+    __shared__ float rel_s[2][REL ? GP_KEYS + 64 : 1];  // biases of a key tile: by 63 - (query row) + (key in the tile)
     pdl_wait();
     pdl_trigger();
     const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, ld = c.ld;  // (shared: LV == LQ)
-    bf16 *qs = gp_sm, *ks = qs + 64 * LQ, *vs = c.shared ? ks : ks + 2 * GP_KEYS * LQ;
-    const int k_pieces = (c.shared ? c.ld : c.dim16) / 8, v_pieces = c.shared ? 0 : c.vdim16 / 8;
+    bf16 *qs = gp_sm, *ks = qs + 64 * LQ, *vs = SHARED ? ks : ks + 2 * GP_KEYS * LQ;
+    const int k_pieces = (SHARED ? c.ld : c.dim16) / 8, v_pieces = SHARED ? 0 : c.vdim16 / 8;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int h = blockIdx.x, kvh = h / (s.heads / s.kv_heads);
     const GroupedTile tl = tiles[blockIdx.y];
@@ -496,8 +506,8 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
         const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * c.dim16;
         for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
     }
-    const float* rel = x.rel ? x.rel + (int64_t)h * x.n_rel : nullptr;
-    const float far = rel ? rel[x.n_rel - 1] : 0.f;
+    const float* rel = REL ? x.rel + (int64_t)h * x.n_rel : nullptr;
+    const float far = REL ? rel[x.n_rel - 1] : 0.f;
     const int hi = tl.pos0 + tl.n - 1, lo = (s.window > tl.pos0 ? 0 : tl.pos0 - s.window + 1) / KV_PAGE * KV_PAGE;
     auto fetch = [&](int k0, int buf) {
         const int page = k0 / KV_PAGE + warp;
@@ -511,7 +521,7 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
             for (int p = l8; p < k_pieces; p += 8) cp_async16(kd + r * LQ + p * 8, src + p * 8, bytes);
             for (int p = l8; p < v_pieces; p += 8) cp_async16(vd + r * LV + p * 8, src + c.dim16 + p * 8, bytes);
         }
-        if (rel && tid < GP_KEYS + 63) {  // (distances below zero are of keys that are not seen)
+        if (REL && tid < GP_KEYS + 63) {  // (distances below zero are of keys that are not seen)
             const int dist = max(0, min(tl.pos0 + 63 - k0 - tid, x.n_rel - 1));
             cp_async4(&rel_s[buf][tid], rel + dist);
         }
@@ -547,8 +557,8 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
             }
         }
         float x0 = m0, x1 = m1;
-        const bool near = rel && tl.pos0 - (k0 + GP_KEYS - 1) < x.n_rel - 1;
-        const float* rs = &rel_s[buf][63 - r0 + 2 * tq];  // of key 2 tq; the other row's stand eight before
+        const bool near = REL && tl.pos0 - (k0 + GP_KEYS - 1) < x.n_rel - 1;
+        const float* rs = REL ? &rel_s[buf][63 - r0 + 2 * tq] : nullptr;  // of key 2 tq; the other row's stand eight before
         const bool edge = k0 + GP_KEYS - 1 > tl.pos0 || (int64_t)hi - k0 >= s.window;  // only the window's ends need the mask
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -556,13 +566,13 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
             for (int e = 0; e < 2; ++e) {
                 const int key = k0 + 8 * j + 2 * tq + e;
                 float f = s.scale, b0 = far, b1 = far;
-                if (c.shared) f *= row_factor(kt + (8 * j + 2 * tq + e) * LQ, c.dim16);
+                if (SHARED) f *= row_factor(kt + (8 * j + 2 * tq + e) * LQ, c.dim16);
                 if (near) {
                     b0 = rs[8 * j + e];
                     b1 = rs[8 * j + e - 8];
                 }
-                sc[j][e] = (!edge || (key <= p0 && p0 - key < s.window)) ? fmaf(sc[j][e], f, b0) : -INFINITY;
-                sc[j][2 + e] = (!edge || (key <= p1 && p1 - key < s.window)) ? fmaf(sc[j][2 + e], f, b1) : -INFINITY;
+                sc[j][e] = (!edge || (key <= p0 && p0 - key < s.window)) ? (REL ? fmaf(sc[j][e], f, b0) : sc[j][e] * f) : -INFINITY;
+                sc[j][2 + e] = (!edge || (key <= p1 && p1 - key < s.window)) ? (REL ? fmaf(sc[j][2 + e], f, b1) : sc[j][2 + e] * f) : -INFINITY;
                 x0 = fmaxf(x0, sc[j][e]);
                 x1 = fmaxf(x1, sc[j][2 + e]);
             }
@@ -649,6 +659,17 @@ __global__ void __launch_bounds__(GP_WARPS * 32) grouped_prefill_kernel(const bf
     }
 }
 
+using GroupedPrefillFn = void (*)(const bf16*, GroupedShape, GroupedCache, GroupedTerms, const GroupedTile*, bf16*, int);
+template <int VT>
+static GroupedPrefillFn gp_kernel(bool rel, bool shared) {
+    return rel ? (shared ? grouped_prefill_kernel<VT, true, true> : grouped_prefill_kernel<VT, true, false>)
+               : (shared ? grouped_prefill_kernel<VT, false, true> : grouped_prefill_kernel<VT, false, false>);
+}
+static GroupedPrefillFn gp_kernel(int vdim16, bool rel, bool shared) {
+    return vdim16 <= 32 ? gp_kernel<4>(rel, shared) : vdim16 <= 64 ? gp_kernel<8>(rel, shared)
+                      : vdim16 <= 128 ? gp_kernel<16>(rel, shared) : gp_kernel<32>(rel, shared);
+}
+
 cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const GroupedTile* tiles,
                                    int n_tiles, void* out, int ldo, cudaStream_t st) {
     if (n_tiles == 0) return cudaSuccess;
@@ -657,22 +678,15 @@ cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const G
     if (!grouped_mma_supported(s) || smem > CAP) return cudaErrorInvalidValue;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
-        const void* fns[] = {(const void*)grouped_prefill_kernel<4>, (const void*)grouped_prefill_kernel<8>, (const void*)grouped_prefill_kernel<16>,
-                             (const void*)grouped_prefill_kernel<32>};
-        for (const void* f : fns) {
-            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+        for (int i = 0; i < 16; ++i) {
+            const cudaError_t e = cudaFuncSetAttribute((const void*)gp_kernel(32 << (i >> 2), i & 1, i & 2), cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
             if (e != cudaSuccess) return e;
         }
         return cudaSuccess;
     });
     if (le != cudaSuccess) return le;
     const dim3 grid(s.heads, n_tiles), block(GP_WARPS * 32);
-#define SP_GP(VT) le = launch_pdl(grouped_prefill_kernel<VT>, grid, block, smem, st, (const bf16*)q, s, c, x, tiles, (bf16*)out, ldo)
-    if (c.vdim16 <= 32) SP_GP(4);
-    else if (c.vdim16 <= 64) SP_GP(8);
-    else if (c.vdim16 <= 128) SP_GP(16);
-    else SP_GP(32);
-#undef SP_GP
+    le = launch_pdl(gp_kernel(c.vdim16, x.rel, c.shared), grid, block, smem, st, (const bf16*)q, s, c, x, tiles, (bf16*)out, ldo);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
