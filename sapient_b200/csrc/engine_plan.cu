@@ -313,6 +313,8 @@ int Engine::plan_stage(int T) {
             for (int t = 0; t < n; t += GROUPED_Q_TILE) tiles[p.n_grouped++] = GroupedTile{i + t, std::min(GROUPED_Q_TILE, n - t), p_pos_[i] + t, p_slot_[i]};
             i += n;
         }
+        // the longest ranges of keys first: the blocks that start last are short
+        std::stable_sort(tiles, tiles + p.n_grouped, [](const GroupedTile& a, const GroupedTile& b) { return a.pos0 > b.pos0; });
     }
     if (p.has_state) {
         StateSegment* seg = reinterpret_cast<StateSegment*>(p.host_tiles + p.seg_at);
