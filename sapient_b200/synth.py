@@ -503,20 +503,20 @@ def tedelix_weights(cfg: dict, seed: int, rank: int = 64, device: str = "cpu") -
 
 
 def fatilix_config(layers, width: int, heads: int, kv_heads: int, dim: int, vdim: int, ff: int, experts: int, top: int, groups: int, keep: int,
-                   expert_ff: int, shared_ff: int, vocab: int, max_positions: int, bias_max: int, temp_every: int = 256, dense_types=("attention_2",)) -> dict:
+                   expert_ff: int, shared_ff: int, vocab: int, max_positions: int, bias_max: int, temp_every: int = 500, dense_types=("attention_2",)) -> dict:
     """layers: the types in order; layers of one type are equal. Layers of `dense_types` have a dense feed-forward, the others
     experts. Values of `attention` are its keys, so their size is dim."""
-    temp = {"coef": 0.3, "every": temp_every}
+    temp = {"coef": 0.2, "every": temp_every}
     mixers = {"attention": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": temp},
               "attention_2": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "q_temp": temp, "bias_max": bias_max}}
-    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 2.0}, "expert": {"ff": expert_ff}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 1.5}, "expert": {"ff": expert_ff}}
     if shared_ff:
         moe["shared"] = {"ff": shared_ff}
     return {"architecture": "Fatilix", "vocab": vocab, "width": width, "max_positions": max_positions, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
             "residual_mult": 0.5, "layers": [{"type": t, "mixer": dict(mixers[t]), "mlp": {"kind": "dense", "ff": ff} if t in dense_types else dict(moe)} for t in layers]}
 
 
-def fatilix_weights(cfg: dict, seed: int, bias_rows: int = 32, device: str = "cpu") -> dict:
+def fatilix_weights(cfg: dict, seed: int, bias_rows: int = 48, device: str = "cpu") -> dict:
     """Random bf16 weights, rows scaled so that activations keep their magnitude. bias_rows: of the distance bias tables."""
     g = torch.Generator(device=device)
     g.manual_seed(seed)
