@@ -67,11 +67,11 @@ Engine::Engine(const SpModelDesc& desc, const ModelPlan& plan, bool f32) : Engin
     if (plan.max_positions > 0) r.max_ctx = std::min(r.max_ctx, plan.max_positions);
     // informative only: a plan's layers have sizes of their own
     const LayerPlan& l = plan.layers[0];
-    r.n_heads = l.mixer == MIX_LATENT ? l.latent.heads : l.mixer == MIX_GROUPED ? l.grouped.heads : l.state.heads;
-    r.n_kv_heads = l.mixer == MIX_LATENT ? 1 : l.mixer == MIX_GROUPED ? l.grouped.kv_heads : l.state.heads;
-    r.head_dim = l.mixer == MIX_LATENT ? l.latent.dim + l.latent.rot_dim : l.mixer == MIX_GROUPED ? l.grouped.dim : l.state.dim;
-    r.rotary_dim = l.mixer == MIX_LATENT ? l.latent.rot_dim : l.mixer == MIX_GROUPED ? l.grouped.rot.dims : 0;
-    r.rope_theta = l.mixer == MIX_LATENT ? (float)l.latent.rot.base : l.mixer == MIX_GROUPED ? (float)l.grouped.rot.base : 0.f;
+    r.n_heads = l.mixer == MIX_LATENT ? l.latent.heads : l.has_grouped() ? l.grouped.heads : l.state.heads;
+    r.n_kv_heads = l.mixer == MIX_LATENT ? 1 : l.has_grouped() ? l.grouped.kv_heads : l.state.heads;
+    r.head_dim = l.mixer == MIX_LATENT ? l.latent.dim + l.latent.rot_dim : l.has_grouped() ? l.grouped.dim : l.state.dim;
+    r.rotary_dim = l.mixer == MIX_LATENT ? l.latent.rot_dim : l.has_grouped() ? l.grouped.rot.dims : l.state.rot.dims;
+    r.rope_theta = l.mixer == MIX_LATENT ? (float)l.latent.rot.base : l.has_grouped() ? (float)l.grouped.rot.base : l.state.rot.dims ? (float)l.state.rot.base : 0.f;
     r.ffn = l.mlp == MLP_MOE ? l.moe.expert.ff : l.mlp == MLP_DENSE ? l.dense.ff : 0;
     return r;
 }()) {

@@ -247,9 +247,12 @@ class Engine {
     void plan_stage_latent(int T);
     int plan_layer_post_norm(int layer, int T);
     int plan_layer_parallel(int layer, int T);
+    int plan_layer_pre_norm(int layer, int T);
     int plan_latent(int layer, int T);
     int plan_grouped(int layer, int T);
     int plan_state(int layer, int T);
+    int plan_mixer_in(int layer, int T, MatArgs& a);
+    int plan_mixers(int layer, int T);
     int plan_experts(int layer, int T);
     int plan_dense(int layer, int T);
     int plan_rollback(int slot, int n, int* kept);

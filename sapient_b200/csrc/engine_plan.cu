@@ -1,6 +1,6 @@
 // Plan-driven models (model_plan.h) on the resident engine: what every plan shares — weights packed once into the shapes
 // the kernels read, a paged cache behind the same page pool, state pools, the buffers and tables of a step, the output head.
-// The layers themselves are in engine_plan_post_norm.cu and engine_plan_parallel.cu. bf16 products run on the tcgen05 kernel
+// The layers themselves are in engine_plan_post_norm.cu, engine_plan_parallel.cu and engine_plan_pre_norm.cu. bf16 products run on the tcgen05 kernel
 // (mat_tc5.cu) at every row count, f32 ones on mat_f32.cu. Steps of up to PLAN_ROWS rows can be captured as a graph.
 #include "engine_plan.h"
 
@@ -63,6 +63,11 @@ RowGain PlanPacker::gain(const std::string& name) {
     return RowGain{upload(g), true};
 }
 
+TanhNorm PlanPacker::tanh_norm(const std::string& name) {
+    const std::vector<float> alpha = host(name + ".alpha", 1, 1);
+    return TanhNorm{alpha.empty() ? 0.f : alpha[0], vec(name, p.plan.width), vec(name + ".b", p.plan.width)};
+}
+
 std::vector<float> PlanPacker::host(const std::string& name, int64_t rows, int64_t cols) {
     const DevTensor* t = need(name, rows, cols);
     const int64_t n = rows * cols;
@@ -118,15 +123,29 @@ int64_t PlanPacker::rows_of(const std::string& name) {
     return t->dims[0];
 }
 
-const float2* PlanPacker::angles(double base, int dims) {
+const float2* PlanPacker::angles(const RotarySpec& rot) {
+    const int dims = rot.dims;
     if (dims == 0) return nullptr;
-    const float2*& tab = p.angles[{base, dims}];
+    const float2*& tab = p.angles[{rot.base, (double)dims, rot.factor, rot.original, rot.fast, rot.slow}];
     if (tab) return tab;
     const int half = dims / 2, ctx = e.d.max_ctx;
+    const bool stretched = rot.factor > 0;
+    double lo = 0, hi = 0, grow = 1;
+    if (stretched) {
+        // the pair that turns this often within the original length
+        auto pair = [&](double turns) { return dims * std::log(rot.original / (2 * 3.14159265358979323846 * turns)) / (2 * std::log(rot.base)); };
+        lo = std::max(std::floor(pair(rot.fast)), 0.0);
+        hi = std::min(std::ceil(pair(rot.slow)), dims - 1.0);
+        grow = 0.1 * std::log(rot.factor) + 1.0;
+    }
     std::vector<float2> cs((size_t)ctx * half);
     for (int i = 0; i < half; ++i) {
-        const double f = std::pow(base, -2.0 * i / dims);
-        for (int pos = 0; pos < ctx; ++pos) cs[(size_t)pos * half + i] = make_float2((float)std::cos(pos * f), (float)std::sin(pos * f));
+        double f = std::pow(rot.base, -2.0 * i / dims);
+        if (stretched) {
+            const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            f = f / rot.factor * ramp + f * (1 - ramp);
+        }
+        for (int pos = 0; pos < ctx; ++pos) cs[(size_t)pos * half + i] = make_float2((float)(std::cos(pos * f) * grow), (float)(std::sin(pos * f) * grow));
     }
     void* q = nullptr;
     if (cudaMalloc(&q, cs.size() * sizeof(float2)) != cudaSuccess) { fail(SP_ERR_OOM, "cannot allocate the angle tables"); return nullptr; }
@@ -164,7 +183,8 @@ int Engine::finalize_plan() {
     if (mp.tied_head) p.head = p.embed;
     else if (pk.alloc(p.head, 1, mp.vocab, W)) pk.put(p.head, 0, pk.need("head", mp.vocab, W), 0, mp.vocab, W);
     if (mp.max_positions > 0 && pk.alloc(p.pos, 1, mp.max_positions, W)) pk.put(p.pos, 0, pk.need("pos", mp.max_positions, W), 0, mp.max_positions, W);
-    p.final_norm = pk.gain("final.norm");
+    if (mp.norm == NORM_TANH) p.final_tanh = pk.tanh_norm("final.norm");
+    else p.final_norm = pk.gain("final.norm");
     // pages first: the layers' cache slices are laid out one after another
     const int pages_per_seq = (d.max_ctx + KV_PAGE - 1) / KV_PAGE;
     const int64_t n_pages = d.kv_pages > 0 ? d.kv_pages : (int64_t)d.max_batch * pages_per_seq;
@@ -176,6 +196,7 @@ int Engine::finalize_plan() {
     kv_.page_table = d_page_table_;
     for (int i = 0; i < L && pk.status == SP_OK; ++i) {
         if (mp.form == FORM_PARALLEL) pk.parallel_layer(i);
+        else if (mp.form == FORM_PRE_NORM) pk.pre_norm_layer(i);
         else pk.post_norm_layer(i);
     }
     if (pk.status != SP_OK) return pk.status;
@@ -192,7 +213,7 @@ int Engine::finalize_plan() {
     SP_CUDA_TRY(cudaMalloc(&p.cache, p.cache_bytes + 1024));
     SP_CUDA_TRY(cudaMemset(p.cache, 0, p.cache_bytes + 1024));
     const size_t state_bytes = p.slot_state * (size_t)d.max_batch * 4;
-    if (p.has_state) {
+    if (p.slot_state > 0) {
         SP_CUDA_TRY(cudaMalloc((void**)&p.states, state_bytes));
         SP_CUDA_TRY(cudaMemset(p.states, 0, state_bytes));
         p.checkpoint_len.assign((size_t)d.max_batch, -1);
@@ -204,7 +225,7 @@ int Engine::finalize_plan() {
         const int from = lp.mixer == MIX_LATENT ? lp.latent.kv_from : -1;
         void* slice = (uint8_t*)p.cache + p.cache_base[(size_t)(from >= 0 ? from : i)];
         if (lp.mixer == MIX_LATENT) l.cache.pool = slice;
-        else if (lp.mixer == MIX_GROUPED) l.kv_cache.pool = slice;
+        else if (lp.has_grouped()) l.kv_cache.pool = slice;
     }
     // buffers of a step
     const size_t T = (size_t)d.max_tokens;
@@ -232,6 +253,9 @@ int Engine::finalize_plan() {
         p.part = (float*)take(plan_latent_part_rows() * n.part * 4);
     }
     p.q = take(T * n.q * el);
+    p.stat = (float2*)take(T * n.stat * sizeof(float2));
+    p.score = (float*)take(n.score * 4);
+    p.score_part = (float2*)take(PLAN_ROWS * n.stat * MIXED_SPLITS * sizeof(float2));
     p.low = take(T * n.low * el);
     if (mp.form == FORM_POST_NORM) {
         p.y = (float*)take(T * W * 4);
@@ -272,7 +296,10 @@ int Engine::finalize_plan() {
     if (long_steps) {
         p.keys_at = p.has_latent ? T * (sizeof(LatentTile) / 4) : 0;
         p.grouped_at = p.keys_at + 2 * (size_t)p.keys_cap;
-        p.seg_at = p.grouped_at + (p.has_grouped ? T * (sizeof(GroupedTile) / 4) : 0);
+        p.narrow_at = p.grouped_at + (p.has_grouped ? T * (sizeof(GroupedTile) / 4) : 0);
+        p.back_at = p.narrow_at + (p.has_mixed ? T * (sizeof(GroupedTile) / 4) : 0);
+        p.ends_at = p.back_at + (p.has_conv ? T : 0);
+        p.seg_at = p.ends_at + (p.has_conv ? (size_t)d.max_batch : 0);
         p.groups_at = (p.seg_at + (p.has_state ? (size_t)d.max_batch * (sizeof(StateSegment) / 4) : 0) + 3) / 4 * 4;
         p.table_ints = p.groups_at + p.groups_cap * state_group(p.f32);
         p.dev_tiles = (int32_t*)take(p.table_ints * 4);
@@ -302,19 +329,32 @@ int Engine::plan_ctx_bucket() const {
 // Tables of the staged tokens, for steps longer than PLAN_ROWS. Host data only: called outside graphs.
 int Engine::plan_stage(int T) {
     PlanState& p = *plan_;
-    p.n_tiles = p.n_keys = p.n_grouped = p.n_seg = p.n_groups = 0;
+    p.n_tiles = p.n_keys = p.n_grouped = p.n_narrow = p.n_ends = p.n_seg = p.n_groups = 0;
     if (T <= PLAN_ROWS) return SP_OK;
     if (p.has_latent && !p.f32) plan_stage_latent(T);
     if (p.has_grouped && !p.f32) {
-        GroupedTile* tiles = reinterpret_cast<GroupedTile*>(p.host_tiles + p.grouped_at);
+        GroupedTile *tiles = reinterpret_cast<GroupedTile*>(p.host_tiles + p.grouped_at), *narrow = reinterpret_cast<GroupedTile*>(p.host_tiles + p.narrow_at);
         for (int i = 0; i < T;) {
             int n = 1;
             while (i + n < T && p_slot_[i + n] == p_slot_[i] && p_pos_[i + n] == p_pos_[i] + n) ++n;
             for (int t = 0; t < n; t += GROUPED_Q_TILE) tiles[p.n_grouped++] = GroupedTile{i + t, std::min(GROUPED_Q_TILE, n - t), p_pos_[i] + t, p_slot_[i]};
+            if (p.has_mixed)
+                for (int t = 0; t < n; t += MIXED_Q_TILE) narrow[p.n_narrow++] = GroupedTile{i + t, std::min(MIXED_Q_TILE, n - t), p_pos_[i] + t, p_slot_[i]};
             i += n;
         }
         // the longest ranges of keys first: the blocks that start last are short
-        std::stable_sort(tiles, tiles + p.n_grouped, [](const GroupedTile& a, const GroupedTile& b) { return a.pos0 > b.pos0; });
+        auto later = [](const GroupedTile& a, const GroupedTile& b) { return a.pos0 > b.pos0; };
+        std::stable_sort(tiles, tiles + p.n_grouped, later);
+        std::stable_sort(narrow, narrow + p.n_narrow, later);
+    }
+    if (p.has_conv) {
+        std::vector<int> last((size_t)d.max_batch, -1);
+        for (int i = 0; i < T; ++i) {
+            p.host_tiles[p.back_at + i] = last[p_slot_[i]];
+            last[p_slot_[i]] = i;
+        }
+        for (int s = 0; s < d.max_batch; ++s)
+            if (last[s] >= 0) p.host_tiles[p.ends_at + p.n_ends++] = last[s];
     }
     if (p.has_state) {
         StateSegment* seg = reinterpret_cast<StateSegment*>(p.host_tiles + p.seg_at);
@@ -354,11 +394,12 @@ int Engine::plan_mat(const PlanMat& w, const void* x, int ldx, int m, void* y, i
 int Engine::plan_layers(int T) {
     PlanState& p = *plan_;
     const int W = p.plan.width, L = (int)p.layers.size();
-    const bool parallel = p.plan.form == FORM_PARALLEL;
-    SP_LAUNCH(F_EMBED, launch_embed_scaled(p.embed.w, p.pos.w, p.embed.kp, p.f32, d_ids_, d_tok_pos_, T, W, p.plan.embed_scale, p.history ? p.history : x_,
-                                           parallel ? nullptr : p.xb, p.wp, stream));
+    const LayerForm form = p.plan.form;
+    const TanhNorm first = p.plan.norm == NORM_TANH ? p.layers[0].tanh1 : TanhNorm{};
+    SP_LAUNCH(F_EMBED, launch_embed_scaled(p.embed.w, p.pos.w, p.embed.kp, p.f32, d_ids_, d_tok_pos_, T, W, p.plan.embed_scale, first, p.history ? p.history : x_,
+                                           form == FORM_POST_NORM || first.w ? p.xb : nullptr, p.wp, stream));
     for (int i = 0; i < L; ++i) {
-        SP_TRY(parallel ? plan_layer_parallel(i, T) : plan_layer_post_norm(i, T));
+        SP_TRY(form == FORM_PARALLEL ? plan_layer_parallel(i, T) : form == FORM_PRE_NORM ? plan_layer_pre_norm(i, T) : plan_layer_post_norm(i, T));
         if (trace_on) SP_CUDA_TRY(cudaMemcpyAsync(trace_ + (size_t)i * d.max_tokens * W, x_, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, stream));
     }
     trace_tokens_ = T;
@@ -369,7 +410,8 @@ int Engine::plan_layers(int T) {
 int Engine::plan_head(const int32_t* rows, int n) {
     PlanState& p = *plan_;
     const int V = p.plan.vocab;
-    SP_LAUNCH(F_NORM, launch_row_norm(x_, rows, n, p.plan.width, p.final_norm, p.plan.eps, p.fin, p.wp, p.f32, stream));
+    if (p.plan.norm == NORM_TANH) SP_LAUNCH(F_NORM, launch_tanh_norm(x_, rows, n, p.plan.width, p.final_tanh, p.fin, p.wp, p.f32, stream));
+    else SP_LAUNCH(F_NORM, launch_row_norm(x_, rows, n, p.plan.width, p.final_norm, p.plan.eps, p.fin, p.wp, p.f32, stream));
     if (p.plan.logit_scale == 1.f && p.plan.logit_softcap <= 0.f) {
         SP_TRY(plan_mat(p.head, p.fin, p.wp, n, logits_, V, true));
     } else {
@@ -379,8 +421,8 @@ int Engine::plan_head(const int32_t* rows, int n) {
         a.m = n;
         a.seg[0] = MatSeg{p.head.w, V, p.head.kp, 1, MatUnit{}, p.fin, p.wp, 0, nullptr, 0, 0};
         a.outs[0] = MatOut{V, logits_, V, MAT_SOFTCAP, true, false};
-        a.scale = p.plan.logit_scale;
-        a.cap = p.plan.logit_softcap;
+        a.arg[0] = p.plan.logit_scale;
+        a.arg[1] = p.plan.logit_softcap;
         SP_TRY(plan_product(a, 0));
     }
     SP_LAUNCH(F_ARGMAX, launch_argmax(logits_, n, V, V, d_argmax_, stream, argmax_scratch_));
@@ -388,7 +430,7 @@ int Engine::plan_head(const int32_t* rows, int n) {
 }
 
 // ── rollback of sequences with a state ──
-bool Engine::keeps_state() const { return plan_ && plan_->has_state; }
+bool Engine::keeps_state() const { return plan_ && plan_->slot_state > 0; }
 
 int Engine::checkpoint(int slot) {
     if (slot < 0 || slot >= d.max_batch) { set_error("slot out of range"); return SP_ERR_ARG; }

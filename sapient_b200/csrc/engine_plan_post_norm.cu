@@ -17,20 +17,10 @@ void PlanPacker::post_norm_layer(int i) {
         latent_layer(i);
     } else {
         std::vector<MixPart> parts;
-        int out_cols = 0;
-        grouped_mixer(i, parts, &out_cols);
-        if (status != SP_OK) return;
-        for (const MixPart& part : parts) l.mix_rows += part.rows;
-        if (!alloc(l.proj, 1, l.mix_rows, W)) return;
-        int at = 0;
-        for (const MixPart& part : parts) {
-            put(l.proj, at, need(lp.prefix + "mix." + part.name, part.rows, W), 0, part.rows, W);
-            at += part.rows;
-        }
-        if (!alloc(l.o, 1, W, out_cols)) return;
-        put(l.o, 0, need(lp.prefix + "mix.o", W, out_cols), 0, W, out_cols);
-        PlanSizes::most(p.need.proj, (size_t)l.mix_rows);
-        PlanSizes::most(p.need.mixed, (size_t)l.o.kp);
+        const int out_cols = mixers(i, parts);
+        if (status != SP_OK || !alloc(l.proj, 1, l.mix_rows, W) || !alloc(l.o, 1, W, out_cols)) return;
+        put_mixer_rows(i, parts);
+        put_mixer_out(i);
     }
     if (p.plan.depth_average) l.dwa = vec(lp.prefix + "dwa", i + 2);
     if (status != SP_OK || lp.mlp == MLP_NONE) return;

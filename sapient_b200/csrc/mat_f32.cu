@@ -44,8 +44,10 @@ __device__ __forceinline__ void mat_store(const MatArgs& a, const MatSeg& s, con
         int i = 0;
         while (n >= a.outs[i].n_end) ++i;
         float* y = reinterpret_cast<float*>(a.outs[i].y) + row * a.outs[i].ldy + n - (i ? a.outs[i - 1].n_end : 0);
-        v = mat_act(a.outs[i].act, v, a.scale, a.cap);
-        *y = a.outs[i].add ? *y + v : v;
+        v = mat_act(a.outs[i].act, v, a.arg);
+        if (a.outs[i].add) v += *y;
+        *y = v;
+        if (a.norm.fn.w) reinterpret_cast<float*>(a.norm.y)[row * a.norm.ldy + n] = tanh_norm(a.norm.fn, v, n);
         return;
     }
     if (a.gate) v *= sigmoid_f32(a.gate[(int64_t)row * a.ldgate + w.g]);

@@ -57,11 +57,13 @@ struct MatTc5Args {
     int ldgate;
     int n_outs;
     MatOut outs[MAT_MAX_OUTS];
-    float scale, cap;
+    float arg[2];
+    MatNorm norm;
 };
 
-// OUTS: a plain product whose weight rows go where a.outs says (OUT_F32 then has no meaning).
-template <bool DUAL, bool OUT_F32, bool OUTS = false>
+// OUTS: a plain product whose weight rows go where a.outs says (OUT_F32 then has no meaning). NORM: it adds into the stream and
+// leaves the norm of the sums, too.
+template <bool DUAL, bool OUT_F32, bool OUTS = false, bool NORM = false>
 __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args a, const __grid_constant__ CUtensorMap map_w0,
                                                              const __grid_constant__ CUtensorMap map_x0, const __grid_constant__ CUtensorMap map_w1,
                                                              const __grid_constant__ CUtensorMap map_x1) {
@@ -205,9 +207,22 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
             if (a.outs[i].f32) of = reinterpret_cast<float*>(a.outs[i].y) + col;
             else ob = reinterpret_cast<bf16*>(a.outs[i].y) + col;
         }
+        float norm_w = 0.f, norm_b = 0.f;
+        bf16* on = nullptr;
+        if (NORM && n < s.n) {
+            norm_w = a.norm.fn.w[n];
+            norm_b = a.norm.fn.b[n];
+            on = reinterpret_cast<bf16*>(a.norm.y) + n;
+        }
         auto held = [&](int row) { return add ? of[row * oldd] : 0.f; };
         auto put = [&](int row, float f, float before) {
-            f = mat_act(act, f, a.scale, a.cap);
+            f = mat_act(act, f, a.arg);
+            if (NORM) {
+                f += before;
+                of[row * oldd] = f;
+                on[row * a.norm.ldy] = __float2bfloat16_rn(fmaf(tanh_by_exp(a.norm.fn.alpha * f), norm_w, norm_b));
+                return;
+            }
             if (of) of[row * oldd] = add ? before + f : f;
             else ob[row * oldd] = __float2bfloat16_rn(f);
         };
@@ -353,7 +368,8 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     k.slots0 = a.moe ? max_tiles : groups * k.row_tiles;
     const int slots = k.slots0 + (a.nseg == 2 ? k.row_tiles : 0);
     k.moe = a.moe; k.gather = a.gather; k.rows = a.rows; k.gate = a.gate; k.ldgate = a.ldgate;
-    k.n_outs = a.n_outs; k.scale = a.scale; k.cap = a.cap;
+    k.n_outs = a.n_outs; k.norm = a.norm;
+    std::copy(a.arg, a.arg + 2, k.arg);
     std::copy(a.outs, a.outs + MAT_MAX_OUTS, k.outs);
     const int acc = a.dual ? 2 : 1;
     k.stage_bytes = acc * MT_A_BYTES + bn * MT_BK * 2;
@@ -375,7 +391,7 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
         const void* fns[] = {(const void*)mat_tc5_kernel<false, false>, (const void*)mat_tc5_kernel<false, true>, (const void*)mat_tc5_kernel<true, false>,
-                             (const void*)mat_tc5_kernel<true, true>, (const void*)mat_tc5_kernel<false, true, true>};
+                             (const void*)mat_tc5_kernel<true, true>, (const void*)mat_tc5_kernel<false, true, true>, (const void*)mat_tc5_kernel<false, true, true, true>};
         for (const void* f : fns) {
             const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, MT_SMEM + 1024);
             if (e != cudaSuccess) return e;
@@ -387,7 +403,8 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st) {
     const dim3 grid((unsigned)row_blocks, (unsigned)slots, (unsigned)k.parts), block(MT_THREADS);
     const size_t smem = (size_t)(k.stages * k.stage_bytes + 1024);
 #define SP_MT(DUAL, F32) le = launch_pdl_cluster(mat_tc5_kernel<DUAL, F32>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1])
-    if (a.n_outs) le = launch_pdl_cluster(mat_tc5_kernel<false, true, true>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1]);
+    if (a.n_outs && a.norm.fn.w) le = launch_pdl_cluster(mat_tc5_kernel<false, true, true, true>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1]);
+    else if (a.n_outs) le = launch_pdl_cluster(mat_tc5_kernel<false, true, true>, grid, block, smem, st, k.parts, k, mw[0], mx[0], mw[1], mx[1]);
     else if (a.dual) { if (a.out_f32) SP_MT(true, true); else SP_MT(true, false); }
     else { if (a.out_f32) SP_MT(false, true); else SP_MT(false, false); }
 #undef SP_MT

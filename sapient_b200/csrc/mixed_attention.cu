@@ -1,0 +1,813 @@
+// Grouped attention whose heads' softmax weights are mixed before they meet the values (plan_kernels.h). A head's mixture needs the
+// normalised weights of all heads, so scores and denominators come first, weights and values second:
+//   few rows    scores_kernel leaves scores and, per split of the keys, maximum and sum; mix_kernel makes the weights of all heads
+//               where it needs them, mixes them as a small product (16 output heads x heads x keys) whose accumulators are the A
+//               operand of the product with the values, and adds the splits' shares over a cluster.
+//   many rows   stats_kernel walks the keys of 64 query rows per head; prefill_kernel has 16 query rows of all heads (a cluster
+//               where one block cannot hold them): every warp makes its heads' weights for a page of keys, all read all of them.
+//   any sizes   simple_scores_kernel, simple_mix_kernel: plain arithmetic, rows in batches that the scratch holds.
+// The products' bf16 operands that stand for weights are a leading part plus its remainder; everything else is f32. Pages that hold
+// kept first keys and pages of the window are one run of visited pages.
+#include <algorithm>
+#include <climits>
+
+#include "kernels.h"
+#include "pdl.cuh"
+#include "plan_common.cuh"
+#include "plan_kernels.h"
+#include "sp_common.cuh"
+
+namespace sp {
+
+cudaError_t count_launch_and_check();  // kernels.cu
+
+// Pages visited by queries at positions p0 .. p1: `kept` pages from the first, then those from page `first` to the one of p1.
+struct Visit {
+    int kept, first, pages;
+    __device__ __forceinline__ Visit(const GroupedShape& s, int p0, int p1) {
+        first = (s.window > p0 ? 0 : p0 - s.window + 1) / KV_PAGE;
+        kept = min((s.keep + KV_PAGE - 1) / KV_PAGE, first);
+        pages = kept + p1 / KV_PAGE - first + 1;
+    }
+    __device__ __forceinline__ int page(int v) const { return v < kept ? v : first + v - kept; }
+};
+__device__ __forceinline__ bool visible(const GroupedShape& s, int key, int pos) { return key <= pos && (pos - key < s.window || key < s.keep); }
+
+int mixed_span(const GroupedShape& s, int max_ctx) {
+    const int64_t window = (int64_t)s.window + 2 * KV_PAGE + (s.keep + KV_PAGE - 1) / KV_PAGE * KV_PAGE;
+    return (int)((std::min<int64_t>(window, max_ctx) + KV_PAGE - 1) / KV_PAGE * KV_PAGE);
+}
+
+// The scaled and capped score of a dot product, and the tensor-core kernels' version: tanh z = 1 - 2 / (e^(2 z) + 1), whose error
+// is absolute, as softmax needs it.
+__device__ __forceinline__ float score_of(const GroupedShape& s, float dot) {
+    const float z = dot * s.scale;
+    return s.softcap > 0.f ? s.softcap * tanhf(z / s.softcap) : z;
+}
+struct FastScore {
+    float scale, cap;
+    __device__ __forceinline__ explicit FastScore(const GroupedShape& s) : scale(s.softcap > 0.f ? 2.f * s.scale / s.softcap : s.scale), cap(s.softcap) {}
+    __device__ __forceinline__ float operator()(float dot) const {
+        const float z = dot * scale;
+        return cap > 0.f ? fmaf(-2.f * cap, __fdividef(1.f, __expf(z) + 1.f), cap) : z;
+    }
+};
+
+__device__ __forceinline__ float2 stat_of(float m, float l, const float* sink, int h) {  // maximum, 1 / denominator
+    if (sink) {
+        const float M = fmaxf(m, sink[h]);
+        l = l * expf(m - M) + expf(sink[h] - M);
+        m = M;
+    }
+    return make_float2(m, 1.f / l);
+}
+
+// ── any sizes ──
+constexpr int MS_WARPS = 4, MS_PER_LANE = GROUPED_MAX_VDIM / 32;
+template <typename T>
+__global__ void __launch_bounds__(MS_WARPS * 32) simple_scores_kernel(const T* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
+                                                                   const MixedScratch m, const int32_t* __restrict__ tok_slot,
+                                                                   const int32_t* __restrict__ tok_pos, int t0) {
+    extern __shared__ float ms_q[];
+    __shared__ float sm[MS_WARPS], sl[MS_WARPS];
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.x, t = t0 + blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = h / (s.heads / s.kv_heads), pos = tok_pos[t];
+    for (int i = threadIdx.x; i < s.dim; i += MS_WARPS * 32) ms_q[i] = to_f32(q[((int64_t)t * s.heads + h) * c.dim16 + i]);
+    __syncthreads();
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    const Visit vis(s, pos, pos);
+    float* out = m.score + ((int64_t)blockIdx.y * s.heads + h) * m.span;
+    float mx = -INFINITY, l = 0.f;
+    for (int i = warp; i < vis.pages * KV_PAGE; i += MS_WARPS) {
+        const int page = vis.page(i / KV_PAGE), key = page * KV_PAGE + i % KV_PAGE;
+        float sc = -INFINITY;
+        if (visible(s, key, pos)) {
+            const T* row = reinterpret_cast<const T*>(c.pool) + (((int64_t)pt[page] * s.kv_heads + g) * KV_PAGE + i % KV_PAGE) * c.ld;
+            float dot = 0.f;
+            for (int e = lane; e < s.dim; e += 32) dot = fmaf(ms_q[e], to_f32(row[e]), dot);
+            sc = score_of(s, warp_sum(dot));
+            const float mn = fmaxf(mx, sc);
+            l = fmaf(l, expf(mx - mn), expf(sc - mn));
+            mx = mn;
+        }
+        if (lane == 0) out[i] = sc;
+    }
+    if (lane == 0) { sm[warp] = mx; sl[warp] = l; }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        float M = -INFINITY, L = 0.f;
+        for (int w = 0; w < MS_WARPS; ++w) M = fmaxf(M, sm[w]);
+        for (int w = 0; w < MS_WARPS; ++w) L += sm[w] == -INFINITY ? 0.f : sl[w] * expf(sm[w] - M);
+        m.stat[(int64_t)t * s.heads + h] = stat_of(M, L, x.sink, h);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(MS_WARPS * 32) simple_mix_kernel(const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
+                                                                const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos, int t0,
+                                                                T* __restrict__ out, int ldo) {
+    extern __shared__ float ms_o[];  // an output row per warp
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.x, t = t0 + blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = h / (s.heads / s.kv_heads), pos = tok_pos[t];
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    const Visit vis(s, pos, pos);
+    const float* score = m.score + (int64_t)blockIdx.y * s.heads * m.span;
+    const float2* stat = m.stat + (int64_t)t * s.heads;
+    float o[MS_PER_LANE];
+#pragma unroll
+    for (int i = 0; i < MS_PER_LANE; ++i) o[i] = 0.f;
+    for (int i = warp; i < vis.pages * KV_PAGE; i += MS_WARPS) {
+        const int page = vis.page(i / KV_PAGE);
+        if (!visible(s, page * KV_PAGE + i % KV_PAGE, pos)) continue;
+        float p = 0.f;
+        for (int e = lane; e < s.heads; e += 32) p = fmaf(x.mix[(int64_t)h * s.heads + e], expf(score[(int64_t)e * m.span + i] - stat[e].x) * stat[e].y, p);
+        p = warp_sum(p);
+        const T* row = reinterpret_cast<const T*>(c.pool) + (((int64_t)pt[page] * s.kv_heads + g) * KV_PAGE + i % KV_PAGE) * c.ld + c.dim16;
+#pragma unroll
+        for (int j = 0; j < MS_PER_LANE; ++j)
+            if (lane + 32 * j < s.vdim) o[j] = fmaf(p, to_f32(row[lane + 32 * j]), o[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < MS_PER_LANE; ++j)
+        if (lane + 32 * j < s.vdim) ms_o[warp * s.vdim + lane + 32 * j] = o[j];
+    __syncthreads();
+    for (int e = threadIdx.x; e < s.vdim; e += MS_WARPS * 32) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < MS_WARPS; ++w) v += ms_o[w * s.vdim + e];
+        out[(int64_t)t * ldo + (int64_t)h * s.vdim + e] = from_f32<T>(v);
+    }
+}
+
+template <typename T>
+static cudaError_t simple_launch(const T* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m, const int32_t* tok_slot,
+                                 const int32_t* tok_pos, T* out, int ldo, int n_tok, cudaStream_t st) {
+    for (int t0 = 0; t0 < n_tok; t0 += m.rows) {
+        const dim3 grid(s.heads, std::min(m.rows, n_tok - t0)), block(MS_WARPS * 32);
+        cudaError_t le = launch_pdl(simple_scores_kernel<T>, grid, block, (size_t)s.dim * 4, st, q, s, c, x, m, tok_slot, tok_pos, t0);
+        if (le == cudaSuccess) le = count_launch_and_check();
+        if (le == cudaSuccess) le = launch_pdl(simple_mix_kernel<T>, grid, block, (size_t)MS_WARPS * s.vdim * 4, st, s, c, x, m, tok_slot, tok_pos, t0, out, ldo);
+        if (le == cudaSuccess) le = count_launch_and_check();
+        if (le != cudaSuccess) return le;
+    }
+    return cudaSuccess;
+}
+
+// ── few rows ──
+// Blocks as in grouped_attention.cu: (cached head, 16 of its query heads; token; split of the keys), four warps that walk pages of
+// their own with three stages of cp.async.
+constexpr int MD_WARPS = 4, MD_STAGES = 3;
+
+// `width` elements (a multiple of 8) of each row of a page, at column `col`, to rows of ld_s elements.
+__device__ __forceinline__ void fetch_page(const GroupedCache& c, int kv_heads, int kvh, int page_id, int live, int col, int width, uint32_t dst, int ld_s, int lane, int lanes) {
+    const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)page_id * kv_heads + kvh) * KV_PAGE * c.ld + col;
+    const int pieces = width / 8;
+    int r = lane / pieces, p = lane - r * pieces;
+    for (int i = lane; i < KV_PAGE * pieces; i += lanes) {
+        cp_async16_at(dst + (uint32_t)(r * ld_s + p * 8) * 2, src + (int64_t)r * c.ld + p * 8, r < live ? 16 : 0);
+        p += lanes;
+        while (p >= pieces) { p -= pieces; ++r; }
+    }
+}
+
+__global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedScratch m,
+                                                                  const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos, int n_splits) {
+    extern __shared__ __align__(16) bf16 md_sm[];
+    __shared__ float m_s[MD_WARPS][16], l_s[MD_WARPS][16];
+    const int LD = c.dim16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int group = s.heads / s.kv_heads, tiles = (group + 15) / 16, kvh = blockIdx.x / tiles, h0 = kvh * group + (blockIdx.x % tiles) * 16;
+    const int nq = min(16, (kvh + 1) * group - h0), t = blockIdx.y;
+    bf16 *qs = md_sm, *ring = md_sm + 16 * LD + warp * MD_STAGES * KV_PAGE * LD;
+    pdl_wait();
+    pdl_trigger();
+    const int pos = tok_pos[t], stride = MD_WARPS * n_splits;
+    const Visit vis(s, pos, pos);
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    for (int i = tid; i < 16 * (c.dim16 / 8); i += MD_WARPS * 32) {
+        const int r = i / (c.dim16 / 8), p = i - r * (c.dim16 / 8);
+        *reinterpret_cast<uint4*>(qs + r * LD + p * 8) =
+            r < nq ? *reinterpret_cast<const uint4*>(q + ((int64_t)t * s.heads + h0 + r) * c.dim16 + p * 8) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    auto fetch = [&](int v, int st) {
+        if (v < vis.pages) {
+            const int page = vis.page(v);
+            fetch_page(c, s.kv_heads, kvh, pt[page], pos - page * KV_PAGE + 1, 0, c.dim16, smem_addr(ring + st * KV_PAGE * LD), LD, lane, 32);
+        }
+        cp_async_commit();
+    };
+    const int v0 = blockIdx.z * MD_WARPS + warp;
+#pragma unroll
+    for (int i = 0; i < MD_STAGES; ++i) fetch(v0 + i * stride, i);
+    __syncthreads();
+    const FastScore score(s);
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const uint32_t qa = smem_addr(qs + (lane & 15) * LD + (lane >> 4) * 8);
+    float* const out = m.score + ((int64_t)t * s.heads + h0) * m.span;
+    for (int v = v0, st = 0; v < vis.pages; v += stride, st = st + 1 == MD_STAGES ? 0 : st + 1) {
+        cp_async_wait<MD_STAGES - 1>();
+        __syncwarp();
+        const bf16* kt = ring + st * KV_PAGE * LD;
+        float sc[2][4] = {};
+        const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8);
+#pragma unroll 4
+        for (int k = 0; k < c.dim16; k += 16) {
+            uint32_t a[4], b[4];
+            ldsm_x4(a, qa + 2 * k);
+            ldsm_x4(b, ka + 2 * k);
+            mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+            mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        }
+        const int key0 = vis.page(v) * KV_PAGE;
+        float x0 = m0, x1 = m1;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const bool on = visible(s, key0 + 8 * j + 2 * tq + e, pos);
+                sc[j][e] = on ? score(sc[j][e]) : -INFINITY;
+                sc[j][2 + e] = on ? score(sc[j][2 + e]) : -INFINITY;
+                x0 = fmaxf(x0, sc[j][e]);
+                x1 = fmaxf(x1, sc[j][2 + e]);
+            }
+            float* d = out + v * KV_PAGE + 8 * j + 2 * tq;
+            if (g < nq) *reinterpret_cast<float2*>(d + (int64_t)g * m.span) = make_float2(sc[j][0], sc[j][1]);
+            if (g + 8 < nq) *reinterpret_cast<float2*>(d + (int64_t)(g + 8) * m.span) = make_float2(sc[j][2], sc[j][3]);
+        }
+        // (a thread's own maxima: its quad meets at the end; kept pages may show a thread nothing)
+        const float b0 = x0 == -INFINITY ? 0.f : x0, b1 = x1 == -INFINITY ? 0.f : x1;
+        l0 = l0 * expf(m0 - b0) + expf(sc[0][0] - b0) + expf(sc[0][1] - b0) + expf(sc[1][0] - b0) + expf(sc[1][1] - b0);
+        l1 = l1 * expf(m1 - b1) + expf(sc[0][2] - b1) + expf(sc[0][3] - b1) + expf(sc[1][2] - b1) + expf(sc[1][3] - b1);
+        m0 = x0;
+        m1 = x1;
+        __syncwarp();  // the stage has been read
+        fetch(v + MD_STAGES * stride, st);
+    }
+    cp_async_wait<0>();
+    auto meet = [](float& a, float& b, float om, float ol) {  // (maximum, sum) of two parts
+        const float M = fmaxf(a, om), base = M == -INFINITY ? 0.f : M;
+        b = b * expf(a - base) + ol * expf(om - base);
+        a = M;
+    };
+#pragma unroll
+    for (int off = 1; off < 4; off <<= 1) {
+        meet(m0, l0, __shfl_xor_sync(0xFFFFFFFFu, m0, off), __shfl_xor_sync(0xFFFFFFFFu, l0, off));
+        meet(m1, l1, __shfl_xor_sync(0xFFFFFFFFu, m1, off), __shfl_xor_sync(0xFFFFFFFFu, l1, off));
+    }
+    if (tq == 0) {
+        m_s[warp][g] = m0;
+        l_s[warp][g] = l0;
+        m_s[warp][g + 8] = m1;
+        l_s[warp][g + 8] = l1;
+    }
+    __syncthreads();
+    if (tid < nq) {
+        float M = m_s[0][tid], L = l_s[0][tid];
+#pragma unroll
+        for (int w = 1; w < MD_WARPS; ++w) meet(M, L, m_s[w][tid], l_s[w][tid]);
+        m.part[((int64_t)t * s.heads + h0 + tid) * MIXED_SPLITS + blockIdx.z] = make_float2(M, L);
+    }
+}
+
+// The splits of a token and cached head are a cluster. Shared memory: maxima and reciprocal denominators of all heads, the block's
+// rows of the mixing matrix (leading part, remainder), the ring of values, where the shares meet at the end.
+__host__ __device__ __forceinline__ int md_heads16(const GroupedShape& s) { return (s.heads + 15) & ~15; }
+static size_t md_mix_smem(const GroupedShape& s, const GroupedCache& c) {
+    const size_t head = (size_t)md_heads16(s) * 8 + (size_t)2 * 16 * (md_heads16(s) + 8) * 2;
+    return head + std::max((size_t)MD_WARPS * MD_STAGES * KV_PAGE * (c.vdim16 + 8) * 2, (size_t)MD_WARPS * 16 * (c.vdim16 + 4) * 4);
+}
+
+template <int VT, bool PACKED>
+__global__ void __launch_bounds__(MD_WARPS * 32) mixed_mix_kernel(const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
+                                                               const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
+                                                               bf16* __restrict__ out, int ldo, int n_splits) {
+    extern __shared__ __align__(16) uint8_t mm_sm[];
+    const int H16 = md_heads16(s), LT = H16 + 8, LV = c.vdim16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int group = s.heads / s.kv_heads, tiles = (group + 15) / 16, kvh = blockIdx.x / tiles, h0 = kvh * group + (blockIdx.x % tiles) * 16;
+    const int nq = min(16, (kvh + 1) * group - h0), t = blockIdx.y;
+    float2* const stat = reinterpret_cast<float2*>(mm_sm);
+    bf16 *t_hi = reinterpret_cast<bf16*>(stat + H16), *t_lo = t_hi + 16 * LT, *rings = t_lo + 16 * LT, *ring = rings + warp * MD_STAGES * KV_PAGE * LV;
+    for (int i = tid; i < 16 * H16; i += MD_WARPS * 32) {  // (no kernel writes the mixing matrix)
+        const int r = i / H16, e = i - r * H16;
+        const float v = r < nq && e < s.heads ? x.mix[(int64_t)(h0 + r) * s.heads + e] : 0.f;
+        const bf16 hi = __float2bfloat16_rn(v);
+        t_hi[r * LT + e] = hi;
+        t_lo[r * LT + e] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+    pdl_wait();
+    pdl_trigger();
+    const int pos = tok_pos[t], stride = MD_WARPS * n_splits;
+    const Visit vis(s, pos, pos);
+    const int32_t* pt = c.page_table + (int64_t)tok_slot[t] * c.max_pages;
+    auto fetch = [&](int v, int st) {
+        if (v < vis.pages) {
+            const int page = vis.page(v);
+            fetch_page(c, s.kv_heads, kvh, pt[page], pos - page * KV_PAGE + 1, c.dim16, c.vdim16, smem_addr(ring + st * KV_PAGE * LV), LV, lane, 32);
+        }
+        cp_async_commit();
+    };
+    const int v0 = blockIdx.z * MD_WARPS + warp;
+#pragma unroll
+    for (int i = 0; i < MD_STAGES; ++i) fetch(v0 + i * stride, i);
+    for (int h = tid; h < H16; h += MD_WARPS * 32) {
+        float2 r = make_float2(INFINITY, 0.f);  // heads that do not exist weigh nothing
+        if (h < s.heads) {
+            const float2* p = m.part + ((int64_t)t * s.heads + h) * MIXED_SPLITS;
+            float M = -INFINITY, L = 0.f;
+            for (int i = 0; i < n_splits; ++i) M = fmaxf(M, p[i].x);
+            for (int i = 0; i < n_splits; ++i) L += p[i].x == -INFINITY ? 0.f : p[i].y * expf(p[i].x - M);
+            r = stat_of(M, L, x.sink, h);
+        }
+        stat[h] = r;
+    }
+    __syncthreads();
+    float o[VT][4];
+#pragma unroll
+    for (int i = 0; i < VT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    const uint32_t ta = smem_addr(t_hi + (lane & 15) * LT + (lane >> 4) * 8), lo_off = 2u * 16 * LT;
+    const float* const score = m.score + (int64_t)t * s.heads * m.span;
+    for (int v = v0, st = 0; v < vis.pages; v += stride, st = st + 1 == MD_STAGES ? 0 : st + 1) {
+        float p[2][4] = {};  // mixed weights: rows g and g + 8 (heads), keys 8 j + 2 tq and the next
+        for (int k = 0; k < H16; k += 16) {
+            uint32_t hi[2][2], lw[2][2], a[4], r[4];
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int e0 = k + 8 * i + 2 * tq, e1 = min(e0 + 1, s.heads - 1);
+                    const float* d = score + v * KV_PAGE + 8 * j + g;
+                    const float2 s0 = stat[e0], s1 = stat[e0 + 1];
+                    const float w0 = expf(d[(int64_t)min(e0, s.heads - 1) * m.span] - s0.x) * s0.y, w1 = expf(d[(int64_t)e1 * m.span] - s1.x) * s1.y;
+                    hi[j][i] = pack_bf16(w0, w1);
+                    const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi[j][i]));
+                    lw[j][i] = pack_bf16(w0 - back.x, w1 - back.y);
+                }
+            ldsm_x4(a, ta + 2 * k);
+            ldsm_x4(r, ta + lo_off + 2 * k);
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                mma_bf16(p[j], a[0], a[1], a[2], a[3], hi[j][0], hi[j][1]);
+                mma_bf16(p[j], a[0], a[1], a[2], a[3], lw[j][0], lw[j][1]);
+                mma_bf16(p[j], r[0], r[1], r[2], r[3], hi[j][0], hi[j][1]);
+            }
+        }
+        uint32_t hi[4], lw[4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int r2 = 0; r2 < 2; ++r2) {
+                hi[2 * j + r2] = pack_bf16(p[j][2 * r2], p[j][2 * r2 + 1]);
+                const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi[2 * j + r2]));
+                lw[2 * j + r2] = pack_bf16(p[j][2 * r2] - back.x, p[j][2 * r2 + 1] - back.y);
+            }
+        if (PACKED) {  // row g + 8: the remainders of row g
+            hi[1] = lw[0];
+            hi[3] = lw[2];
+        }
+        cp_async_wait<MD_STAGES - 1>();
+        __syncwarp();
+        const uint32_t va = smem_addr(ring + st * KV_PAGE * LV + (lane & 15) * LV + (lane >> 4) * 8);
+#pragma unroll
+        for (int i = 0; i < VT; i += 2) {
+            if (i * 8 < c.vdim16) {
+                uint32_t b[4];
+                ldsm_x4_t(b, va + 2 * (i * 8));
+                mma_bf16(o[i], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+                mma_bf16(o[i + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+                if (!PACKED) {
+                    mma_bf16(o[i], lw[0], lw[1], lw[2], lw[3], b[0], b[1]);
+                    mma_bf16(o[i + 1], lw[0], lw[1], lw[2], lw[3], b[2], b[3]);
+                }
+            }
+        }
+        __syncwarp();  // the stage has been read
+        fetch(v + MD_STAGES * stride, st);
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    const int LO = c.vdim16 + 4, rows = PACKED ? 8 : 16;
+    float* const os = reinterpret_cast<float*>(rings);
+#pragma unroll
+    for (int i = 0; i < VT; ++i) {
+        if (i * 8 < c.vdim16) {
+            float* d = os + (warp * rows + g) * LO + i * 8 + 2 * tq;
+            if (PACKED) *reinterpret_cast<float2*>(d) = make_float2(o[i][0] + o[i][2], o[i][1] + o[i][3]);
+            else {
+                *reinterpret_cast<float2*>(d) = make_float2(o[i][0], o[i][1]);
+                *reinterpret_cast<float2*>(d + 8 * LO) = make_float2(o[i][2], o[i][3]);
+            }
+        }
+    }
+    __syncthreads();
+    bf16* const d = out + (int64_t)t * ldo + (int64_t)h0 * s.vdim;
+    auto share = [&](int r, int e) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < MD_WARPS; ++w) v += os[(w * rows + r) * LO + e];
+        return v;
+    };
+    if (n_splits == 1) {
+        for (int i = tid; i < nq * s.vdim; i += MD_WARPS * 32) d[i] = __float2bfloat16_rn(share(i / s.vdim, i % s.vdim));
+        return;
+    }
+    for (int i = tid; i < nq * s.vdim; i += MD_WARPS * 32) os[(i / s.vdim) * LO + i % s.vdim] = share(i / s.vdim, i % s.vdim);  // in the first warp's place
+    cluster_sync();
+    for (int i = blockIdx.z * MD_WARPS * 32 + tid; i < nq * s.vdim; i += n_splits * MD_WARPS * 32) {
+        const uint32_t a = smem_addr(os + (i / s.vdim) * LO + i % s.vdim);
+        float v = 0.f;
+        for (int p = 0; p < n_splits; ++p) v += ld_peer(peer_smem(a, p));
+        d[i] = __float2bfloat16_rn(v);
+    }
+    cluster_sync();  // nobody leaves while its share is being read
+}
+
+int mixed_attention_splits(const GroupedShape& s, int n_tok, int keys) {
+    const int group = s.heads / s.kv_heads, blocks = s.kv_heads * ((group + 15) / 16) * n_tok, slots = 2 * device_sm_count();
+    int n = 1;
+    while (n < MIXED_SPLITS && blocks * 2 * n <= slots && keys >= 128 * 2 * n) n <<= 1;
+    return n;
+}
+
+using MixedMixFn = void (*)(GroupedShape, GroupedCache, MixedTerms, MixedScratch, const int32_t*, const int32_t*, bf16*, int, int);
+static MixedMixFn mm_kernel(int vdim16, bool packed) {
+    if (vdim16 <= 32) return packed ? mixed_mix_kernel<4, true> : mixed_mix_kernel<4, false>;
+    if (vdim16 <= 64) return packed ? mixed_mix_kernel<8, true> : mixed_mix_kernel<8, false>;
+    if (vdim16 <= 128) return packed ? mixed_mix_kernel<16, true> : mixed_mix_kernel<16, false>;
+    return packed ? mixed_mix_kernel<32, true> : mixed_mix_kernel<32, false>;
+}
+constexpr int MD_CAP = 220 * 1024;
+
+cudaError_t launch_mixed_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
+                                   const int32_t* tok_slot, const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st) {
+    if (n_tok == 0) return cudaSuccess;
+    if (s.vdim > GROUPED_MAX_VDIM || c.shared || m.rows < 1) return cudaErrorInvalidValue;
+    if (f32) return simple_launch<float>((const float*)q, s, c, x, m, tok_slot, tok_pos, (float*)out, ldo, n_tok, st);
+    if (!mixed_mma_supported(s, c) || n_tok > m.rows) return simple_launch<bf16>((const bf16*)q, s, c, x, m, tok_slot, tok_pos, (bf16*)out, ldo, n_tok, st);
+    if (n_splits < 1 || n_splits > MIXED_SPLITS || (n_splits & (n_splits - 1))) return cudaErrorInvalidValue;
+    static PerDeviceOnce once;
+    cudaError_t le = once.run([] {
+        for (int i = 0; i < 8; ++i) {
+            const cudaError_t e = cudaFuncSetAttribute((const void*)mm_kernel(32 << (i >> 1), i & 1), cudaFuncAttributeMaxDynamicSharedMemorySize, MD_CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaFuncSetAttribute(mixed_scores_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MD_CAP);
+    });
+    if (le != cudaSuccess) return le;
+    const int group = s.heads / s.kv_heads;
+    const dim3 grid(s.kv_heads * ((group + 15) / 16), n_tok, n_splits), block(MD_WARPS * 32);
+    const size_t smem = (size_t)(16 + MD_WARPS * MD_STAGES * KV_PAGE) * (c.dim16 + 8) * 2;
+    le = launch_pdl(mixed_scores_kernel, grid, block, smem, st, (const bf16*)q, s, c, m, tok_slot, tok_pos, n_splits);
+    if (le == cudaSuccess) le = count_launch_and_check();
+    if (le != cudaSuccess) return le;
+    le = launch_pdl_cluster(mm_kernel(c.vdim16, group <= 8), grid, block, md_mix_smem(s, c), st, n_splits, s, c, x, m, tok_slot, tok_pos, (bf16*)out, ldo, n_splits);
+    return le != cudaSuccess ? le : count_launch_and_check();
+}
+
+// ── many rows: denominators ──
+// Block per (head, tile of 64 tokens), 4 warps x 16 query rows, key tiles of four visited pages, double-buffered.
+constexpr int MT_KEYS = 64, MT_WARPS = 4;
+__global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
+                                                                 const MixedScratch m, const GroupedTile* __restrict__ tiles) {
+    extern __shared__ __align__(16) bf16 mt_sm[];
+    pdl_wait();
+    pdl_trigger();
+    const int LQ = c.dim16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    bf16 *qs = mt_sm, *ks = qs + 64 * LQ;
+    const int h = blockIdx.x, kvh = h / (s.heads / s.kv_heads);
+    const GroupedTile tl = tiles[blockIdx.y];
+    const int hi = tl.pos0 + tl.n - 1;
+    const Visit vis(s, tl.pos0, hi);
+    const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages;
+    const int l8 = lane & 7, lr = warp * 16 + (lane >> 3);  // copies: eight lanes per row, a page per warp
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int r = lr + 4 * i;
+        const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * c.dim16;
+        for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
+    }
+    auto fetch = [&](int v0, int buf) {
+        const int v = v0 + warp, page = vis.page(min(v, vis.pages - 1));
+        const bf16* base = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[page] * s.kv_heads + kvh) * KV_PAGE * c.ld;
+        bf16* kd = ks + buf * MT_KEYS * LQ;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = lr + 4 * i, in = r - warp * 16, bytes = v < vis.pages && page * KV_PAGE + in <= hi ? 16 : 0;
+            for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(kd + r * LQ + p * 8, base + in * c.ld + p * 8, bytes);
+        }
+    };
+    fetch(0, 0);
+    cp_async_commit();
+    const FastScore score(s);
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const int r0 = warp * 16 + g, r1 = r0 + 8, p0 = tl.pos0 + min(r0, tl.n - 1), p1 = tl.pos0 + min(r1, tl.n - 1);
+    for (int v0 = 0, buf = 0; v0 < vis.pages; v0 += MT_KEYS / KV_PAGE, buf ^= 1) {
+        cp_async_wait<0>();
+        __syncthreads();
+        if (v0 + MT_KEYS / KV_PAGE < vis.pages) fetch(v0 + MT_KEYS / KV_PAGE, buf ^ 1);
+        cp_async_commit();
+        const bf16* kt = ks + buf * MT_KEYS * LQ;
+        float sc[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+        const uint32_t qa = smem_addr(qs + (warp * 16 + (lane & 15)) * LQ + (lane >> 4) * 8);
+        const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8);
+        for (int k = 0; k < c.dim16; k += 16) {
+            uint32_t a[4];
+            ldsm_x4(a, qa + 2 * k);
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                uint32_t b[4];
+                ldsm_x4(b, ka + 2 * (8 * j * LQ + k));
+                mma_bf16(sc[j], a[0], a[1], a[2], a[3], b[0], b[1]);
+                mma_bf16(sc[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+            }
+        }
+        float x0 = m0, x1 = m1;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int v = v0 + j / 2, key0 = vis.page(min(v, vis.pages - 1)) * KV_PAGE + 8 * (j & 1) + 2 * tq;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                sc[j][e] = v < vis.pages && visible(s, key0 + e, p0) ? score(sc[j][e]) : -INFINITY;
+                sc[j][2 + e] = v < vis.pages && visible(s, key0 + e, p1) ? score(sc[j][2 + e]) : -INFINITY;
+                x0 = fmaxf(x0, sc[j][e]);
+                x1 = fmaxf(x1, sc[j][2 + e]);
+            }
+        }
+#pragma unroll
+        for (int off = 1; off < 4; off <<= 1) {
+            x0 = fmaxf(x0, __shfl_xor_sync(0xFFFFFFFFu, x0, off));
+            x1 = fmaxf(x1, __shfl_xor_sync(0xFFFFFFFFu, x1, off));
+        }
+        const float b0 = x0 == -INFINITY ? 0.f : x0, b1 = x1 == -INFINITY ? 0.f : x1;
+        float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            s0 += __expf(sc[j][0] - b0) + __expf(sc[j][1] - b0);
+            s1 += __expf(sc[j][2] - b1) + __expf(sc[j][3] - b1);
+        }
+        l0 = fmaf(l0, expf(m0 - b0), s0);
+        l1 = fmaf(l1, expf(m1 - b1), s1);
+        m0 = x0;
+        m1 = x1;
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int off = 1; off < 4; off <<= 1) {
+        l0 += __shfl_xor_sync(0xFFFFFFFFu, l0, off);
+        l1 += __shfl_xor_sync(0xFFFFFFFFu, l1, off);
+    }
+    if (tq == 0) {
+        if (r0 < tl.n) m.stat[(int64_t)(tl.row0 + r0) * s.heads + h] = stat_of(m0, l0, x.sink, h);
+        if (r1 < tl.n) m.stat[(int64_t)(tl.row0 + r1) * s.heads + h] = stat_of(m1, l1, x.sink, h);
+    }
+}
+
+// ── many rows: weights and values ──
+// Block (cluster rank: a run of 8 HPW heads, tile of 16 tokens), a warp per HPW heads. Per page of keys: weights of the block's
+// heads into every block's shared memory, one barrier, then each warp mixes for its heads and multiplies with the values. Keys are
+// two stages ahead of the barrier, values one; weights alternate between two buffers. A thread's four keys of the A operand are
+// neighbours, so that it reads a head's weights as one float4; the values' rows are numbered the same way.
+constexpr int MP_WARPS = 8, MP_MAX_CLUSTER = 8, MP_CAP = 224 * 1024;
+struct MixedTiling {
+    int heads, kv, cluster;    // heads of a block, cached heads they touch at most, blocks
+    int q, k, v, w, mix;       // offsets in shared memory (bytes)
+    size_t smem;
+};
+__host__ __device__ __forceinline__ MixedTiling mp_tiling(const GroupedShape& s, const GroupedCache& c, int hpw) {
+    MixedTiling t;
+    const int group = s.heads / s.kv_heads;
+    t.heads = MP_WARPS * hpw < s.heads ? MP_WARPS * hpw : s.heads;
+    t.cluster = (s.heads + t.heads - 1) / t.heads;
+    const int touched = (t.heads + group - 2) / group + 1;  // a run may begin inside a group
+    t.kv = t.heads % group == 0 || group % t.heads == 0 ? (t.heads + group - 1) / group : touched < s.kv_heads ? touched : s.kv_heads;
+    int cl = 1;
+    while (cl < t.cluster) cl <<= 1;
+    t.cluster = cl;
+    t.q = 0;
+    t.k = t.q + MP_WARPS * hpw * 16 * (c.dim16 + 8) * 2;
+    t.v = t.k + 2 * t.kv * KV_PAGE * (c.dim16 + 8) * 2;
+    t.w = t.v + 2 * t.kv * KV_PAGE * (c.vdim16 + 8) * 2;
+    t.mix = t.w + 2 * s.heads * 16 * KV_PAGE * 4;
+    t.smem = (size_t)t.mix + (size_t)MP_WARPS * hpw * s.heads * 4;
+    return t;
+}
+static int mp_heads_per_warp(const GroupedShape& s, const GroupedCache& c) {  // 0: not covered
+    if (s.dim > 256 || s.vdim > 256) return 0;
+    for (int hpw = c.vdim16 <= 128 && s.heads > MP_WARPS ? 2 : 1; hpw > 0; --hpw) {
+        const MixedTiling t = mp_tiling(s, c, hpw);
+        if (t.cluster <= MP_MAX_CLUSTER && t.smem <= MP_CAP) return hpw;
+    }
+    return 0;
+}
+
+__device__ __forceinline__ void st_peer(uint32_t addr, float a, float b) {
+    asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};\n" ::"r"(addr), "f"(a), "f"(b) : "memory");
+}
+
+template <int VT, int HPW>
+__global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
+                                                                      const MixedScratch m, const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) uint8_t mp_sm[];
+    const MixedTiling tg = mp_tiling(s, c, HPW);
+    const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, H = s.heads, group = H / s.kv_heads;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
+    const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
+    const uint32_t sm = smem_addr(mp_sm);
+    float* const ws = reinterpret_cast<float*>(mp_sm + tg.w);    // [2][head][16 rows][16 keys]
+    float* const mix = reinterpret_cast<float*>(mp_sm + tg.mix); // [warp][head][HPW]
+    for (int i = tid; i < MP_WARPS * HPW * H; i += MP_WARPS * 32) {
+        const int hh = i % HPW, e = i / HPW % H, h = i / HPW / H * HPW + hh;
+        mix[i] = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
+    }
+    pdl_wait();
+    pdl_trigger();
+    const GroupedTile tl = tiles[blockIdx.y];
+    const int hi = tl.pos0 + tl.n - 1;
+    const Visit vis(s, tl.pos0, hi);
+    const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages;
+    auto fetch = [&](int v, int stage, int col, int width, int base, int ld) {
+        if (v < vis.pages)
+            for (int i = warp; i < nkv; i += MP_WARPS) {
+                const int page = vis.page(v);
+                fetch_page(c, s.kv_heads, kv0 + i, pt[page], hi - page * KV_PAGE + 1, col, width, sm + (uint32_t)(base + ((stage * tg.kv + i) * KV_PAGE * ld) * 2), ld, lane, 32);
+            }
+    };
+    auto fetch_k = [&](int v) { fetch(v, v & 1, 0, c.dim16, tg.k, LQ); };
+    auto fetch_v = [&](int v) { fetch(v, v & 1, c.dim16, c.vdim16, tg.v, LV); };
+    for (int i = warp; i < nh * 16; i += MP_WARPS) {
+        const int h = i / 16, r = i % 16;
+        const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * H + h0 + h) * c.dim16;
+        for (int p = lane; p < c.dim16 / 8; p += 32) cp_async16_at(sm + (uint32_t)(tg.q + (i * LQ + p * 8) * 2), src + p * 8, 16);
+    }
+    fetch_k(0);
+    cp_async_commit();
+    const int ra = min(g, tl.n - 1), rb = min(g + 8, tl.n - 1), pa = tl.pos0 + ra, pb = tl.pos0 + rb;
+    float2 sa[HPW], sb[HPW];
+#pragma unroll
+    for (int j = 0; j < HPW; ++j) {
+        const int h = min(h0 + warp * HPW + j, H - 1);
+        sa[j] = m.stat[(int64_t)(tl.row0 + ra) * H + h];
+        sb[j] = m.stat[(int64_t)(tl.row0 + rb) * H + h];
+    }
+    cp_async_wait<0>();
+    if (tg.cluster == 1) __syncthreads();
+    else cluster_sync();  // (also: every peer has started)
+    fetch_k(1);
+    fetch_v(0);
+    cp_async_commit();
+    const FastScore score(s);
+    float o[HPW][VT][4];
+#pragma unroll
+    for (int j = 0; j < HPW; ++j)
+#pragma unroll
+        for (int i = 0; i < VT; ++i) o[j][i][0] = o[j][i][1] = o[j][i][2] = o[j][i][3] = 0.f;
+    const int vrow = lane & 7, v_key = 4 * (vrow >> 1) + (vrow & 1) + 2 * ((lane >> 3) & 1);  // the key of the operand's row lane & 15
+    for (int v = 0; v < vis.pages; ++v) {
+        const int key0 = vis.page(v) * KV_PAGE;
+#pragma unroll
+        for (int j = 0; j < HPW; ++j) {
+            const int h = warp * HPW + j;
+            if (h >= nh) continue;
+            const uint32_t qa = sm + (uint32_t)(tg.q + ((h * 16 + (lane & 15)) * LQ + (lane >> 4) * 8) * 2);
+            const uint32_t ka = sm + (uint32_t)(tg.k + ((((v & 1) * tg.kv + (h0 + h) / group - kv0) * KV_PAGE + (lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8) * 2);
+            float sc[2][4] = {};
+#pragma unroll 4
+            for (int k = 0; k < c.dim16; k += 16) {
+                uint32_t a[4], b[4];
+                ldsm_x4(a, qa + 2 * k);
+                ldsm_x4(b, ka + 2 * k);
+                mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+            }
+            const uint32_t wd = sm + (uint32_t)(tg.w + ((((v & 1) * H + h0 + h) * 16 + g) * KV_PAGE + 2 * tq) * 4);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const int key = key0 + 8 * n + 2 * tq;
+                float w[4];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    w[e] = visible(s, key + e, pa) ? __expf(score(sc[n][e]) - sa[j].x) * sa[j].y : 0.f;
+                    w[2 + e] = visible(s, key + e, pb) ? __expf(score(sc[n][2 + e]) - sb[j].x) * sb[j].y : 0.f;
+                }
+                if (tg.cluster == 1) {
+                    float* d = ws + ((((v & 1) * H + h0 + h) * 16 + g) * KV_PAGE + 8 * n + 2 * tq);
+                    *reinterpret_cast<float2*>(d) = make_float2(w[0], w[1]);
+                    *reinterpret_cast<float2*>(d + 8 * KV_PAGE) = make_float2(w[2], w[3]);
+                } else {
+                    for (int p = 0; p < tg.cluster; ++p) {
+                        const uint32_t a = peer_smem(wd + 32u * n, p);
+                        st_peer(a, w[0], w[1]);
+                        st_peer(a + 8 * KV_PAGE * 4, w[2], w[3]);
+                    }
+                }
+            }
+        }
+        cp_async_wait<0>();
+        if (tg.cluster == 1) __syncthreads();
+        else cluster_sync();
+        fetch_k(v + 2);
+        fetch_v(v + 1);
+        cp_async_commit();
+        if (warp * HPW >= nh) continue;
+        float p[HPW][8];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8
+#pragma unroll
+        for (int j = 0; j < HPW; ++j)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) p[j][i] = 0.f;
+        const float* wr = ws + ((v & 1) * H * 16 + g) * KV_PAGE + 4 * tq;
+        const float* mr = mix + warp * H * HPW;
+#pragma unroll 4
+        for (int e = 0; e < H; ++e) {
+            const float4 a = *reinterpret_cast<const float4*>(wr + e * 16 * KV_PAGE), b = *reinterpret_cast<const float4*>(wr + (e * 16 + 8) * KV_PAGE);
+            const float w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int j = 0; j < HPW; ++j) {
+                const float f = mr[e * HPW + j];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) p[j][i] = fmaf(f, w[i], p[j][i]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < HPW; ++j) {
+            const int h = warp * HPW + j;
+            if (h >= nh) continue;
+            uint32_t a[4], r[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {  // operand registers: (row g, keys 0 1), (row g + 8, keys 0 1), (row g, keys 2 3), (row g + 8, keys 2 3)
+                const float u = p[j][4 * (i & 1) + 2 * (i >> 1)], w = p[j][4 * (i & 1) + 2 * (i >> 1) + 1];
+                a[i] = pack_bf16(u, w);
+                const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[i]));
+                r[i] = pack_bf16(u - back.x, w - back.y);
+            }
+            const uint32_t va = sm + (uint32_t)(tg.v + ((((v & 1) * tg.kv + (h0 + h) / group - kv0) * KV_PAGE + v_key) * LV + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int i = 0; i < VT; i += 2) {
+                if (i * 8 < c.vdim16) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, va + 2 * (i * 8));
+                    mma_bf16(o[j][i], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(o[j][i + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    mma_bf16(o[j][i], r[0], r[1], r[2], r[3], b[0], b[1]);
+                    mma_bf16(o[j][i + 1], r[0], r[1], r[2], r[3], b[2], b[3]);
+                }
+            }
+        }
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int j = 0; j < HPW; ++j) {
+        const int h = warp * HPW + j;
+        if (h >= nh) continue;
+        bf16* d = out + (int64_t)tl.row0 * ldo + (int64_t)(h0 + h) * s.vdim;
+#pragma unroll
+        for (int i = 0; i < VT; ++i) {
+            const int col = i * 8 + 2 * tq;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                if (col + e >= s.vdim) continue;
+                if (g < tl.n) d[(int64_t)g * ldo + col + e] = __float2bfloat16_rn(o[j][i][e]);
+                if (g + 8 < tl.n) d[(int64_t)(g + 8) * ldo + col + e] = __float2bfloat16_rn(o[j][i][2 + e]);
+            }
+        }
+    }
+    if (tg.cluster > 1) cluster_sync();  // nobody leaves while a peer may still write here
+}
+
+bool mixed_mma_supported(const GroupedShape& s, const GroupedCache& c) {
+    return mp_heads_per_warp(s, c) > 0 && md_mix_smem(s, c) <= MD_CAP && (size_t)(16 + MD_WARPS * MD_STAGES * KV_PAGE) * (c.dim16 + 8) * 2 <= MD_CAP;
+}
+
+using MixedPrefillFn = void (*)(const bf16*, GroupedShape, GroupedCache, MixedTerms, MixedScratch, const GroupedTile*, bf16*, int);
+static MixedPrefillFn mp_kernel(int vdim16, int hpw) {
+    if (vdim16 <= 32) return hpw == 2 ? mixed_prefill_kernel<4, 2> : mixed_prefill_kernel<4, 1>;
+    if (vdim16 <= 64) return hpw == 2 ? mixed_prefill_kernel<8, 2> : mixed_prefill_kernel<8, 1>;
+    if (vdim16 <= 128) return hpw == 2 ? mixed_prefill_kernel<16, 2> : mixed_prefill_kernel<16, 1>;
+    return mixed_prefill_kernel<32, 1>;
+}
+
+cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
+                                 const GroupedTile* wide, int n_wide, const GroupedTile* narrow, int n_narrow, void* out, int ldo, cudaStream_t st) {
+    if (n_wide == 0 || n_narrow == 0) return cudaSuccess;
+    const int hpw = mp_heads_per_warp(s, c);
+    if (!hpw) return cudaErrorInvalidValue;
+    static PerDeviceOnce once;
+    cudaError_t le = once.run([] {
+        for (int i = 0; i < 7; ++i) {
+            const cudaError_t e = cudaFuncSetAttribute((const void*)mp_kernel(32 << (i >> 1), 2 - (i & 1)), cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaFuncSetAttribute(mixed_stats_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+    });
+    if (le != cudaSuccess) return le;
+    le = launch_pdl(mixed_stats_kernel, dim3(s.heads, n_wide), dim3(MT_WARPS * 32), (size_t)3 * 64 * (c.dim16 + 8) * 2, st, (const bf16*)q, s, c, x, m, wide);
+    if (le == cudaSuccess) le = count_launch_and_check();
+    if (le != cudaSuccess) return le;
+    const MixedTiling t = mp_tiling(s, c, hpw);
+    le = launch_pdl_cluster(mp_kernel(c.vdim16, hpw), dim3(1, n_narrow, t.cluster), dim3(MP_WARPS * 32), t.smem, st, t.cluster, (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
+    return le != cudaSuccess ? le : count_launch_and_check();
+}
+
+}  // namespace sp

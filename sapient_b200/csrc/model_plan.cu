@@ -95,19 +95,35 @@ TemperatureSpec read_temperature(const Cfg& c) {
     return t;
 }
 
+// The entry "rot" of a mixer whose heads have `dim` coordinates.
+RotarySpec read_rotary(const Cfg& c, int dim) {
+    RotarySpec r;
+    const Cfg rot = c.sub("rot");
+    r.base = rot.num("base");
+    r.dims = rot.has("dims") ? rot.size("dims", 0) : dim;
+    if (c.err->empty() && ((r.dims & 1) || r.dims > dim || r.base <= 0)) c.fail("rot does not fit dim");
+    if (rot.has("scaling")) {
+        const Cfg s = rot.sub("scaling");
+        r.factor = s.num("factor");
+        r.original = s.num("original");
+        r.fast = s.num("fast");
+        r.slow = s.num("slow");
+        if (c.err->empty() && (r.factor <= 0 || r.original <= 0 || r.fast <= 0 || r.slow <= 0 || r.base == 1.0)) s.fail("its numbers must be positive, and rot.base not one");
+    }
+    return r;
+}
+
 GroupedAttentionSpec read_rotated_attention(const Cfg& c, bool rotate_values) {
     GroupedAttentionSpec m = read_heads(c);
-    const Cfg rot = c.sub("rot");
-    m.rot.base = rot.num("base");
-    m.rot.dims = rot.has("dims") ? rot.size("dims", 0) : m.dim;
+    m.rot = read_rotary(c, m.dim);
     m.rotate_values = rotate_values;
     if (c.has("mask") && c.sub("mask").has("size")) m.window = c.sub("mask").size("size");
     if (!c.err->empty()) return m;
-    if ((m.rot.dims & 1) || m.rot.dims > m.dim || m.rot.base <= 0) c.fail("rot does not fit dim");
     if (rotate_values && (m.vdim & 1)) c.fail("vdim must be even");
     return m;
 }
 
+// The sizes of a mixer with a state, and its decays where the rule has them.
 StateMixerSpec read_state_mixer(const Cfg& c, StateRule rule) {
     StateMixerSpec m;
     m.rule = rule;
@@ -164,6 +180,7 @@ int read_tedelix(const Json& cfg, ModelPlan* out) {
         } else if (t == "lightning" || t == "general_delta") {
             l.mixer = MIX_STATE;
             l.state = read_state_mixer(lc.sub("mixer"), t == "lightning" ? STATE_DECAY : STATE_DELTA);
+            l.state.silu_inputs = l.state.norm_all = t == "lightning";
         } else {
             lc.fail("type is not a mixer of this design");
             break;
@@ -297,12 +314,86 @@ int read_fatilix(const Json& cfg, ModelPlan* out) {
     return SP_OK;
 }
 
+// Decaying sum over rotated queries and scaled, rotated keys.
+StateMixerSpec read_retention(const Cfg& c) {
+    StateMixerSpec m = read_state_mixer(c, STATE_DECAY);
+    m.rot = read_rotary(c, m.dim);
+    m.key_scale = 1.f / std::sqrt((float)m.dim);
+    m.gain = STATE_GAIN_NONE;
+    m.gate = STATE_GATE_SILU;
+    return m;
+}
+
+// Attention over convolved, biased projections whose heads' weights are mixed.
+GroupedAttentionSpec read_talking_attention(const Cfg& c) {
+    GroupedAttentionSpec m = read_heads(c);
+    m.rot = read_rotary(c, m.dim);
+    m.rot.neighbours = true;
+    m.biases = m.sink = m.talk = true;
+    m.conv = c.size("conv");
+    m.score_softcap = (float)c.num("softcap");
+    m.window = c.sub("mask").size("size");
+    m.keep_first = c.sub("mask").size("keep_first", 0);
+    if (c.err->empty() && m.conv > CONV_MAX_TAPS) c.fail("conv is above " + std::to_string(CONV_MAX_TAPS));
+    if (c.err->empty() && m.score_softcap <= 0) c.fail("softcap must be positive");
+    return m;
+}
+
+int read_revelix(const Json& cfg, ModelPlan* out) {
+    std::string err;
+    const Cfg c{&cfg, "", &err};
+    ModelPlan p;
+    p.name = "Revelix";
+    p.vocab = c.size("vocab");
+    p.width = c.size("width");
+    p.eps = (float)c.sub("norm").num("eps");
+    p.form = FORM_PRE_NORM;
+    p.norm = NORM_TANH;
+    p.tied_head = true;
+    if (c.has("logit_scale")) p.logit_scale = (float)c.num("logit_scale");
+    const Json* layers = cfg.get("layers");
+    if (!layers || layers->type != Json::ARR || layers->arr.empty()) c.fail("layers is missing or not a list");
+    for (size_t i = 0; err.empty() && i < layers->arr.size(); ++i) {
+        const std::string idx = std::to_string(i);
+        const Cfg lc{&layers->arr[i], "layers[" + idx + "].", &err};
+        LayerPlan l;
+        l.prefix = "l" + idx + ".";
+        const Json* type = lc.j->get("type");
+        const std::string t = type ? type->str : "";
+        if (t == "retention") {
+            l.mixer = MIX_STATE;
+            l.state = read_retention(lc.sub("mixer"));
+        } else if (t == "parallel") {
+            const Cfg m = lc.sub("mixer");
+            l.mixer = MIX_BOTH;
+            l.grouped = read_talking_attention(m.sub("left"));
+            l.grouped.at = "mix.left.";
+            l.grouped.out_scale = (float)m.num("left_scale");
+            l.state = read_state_mixer(m.sub("right"), STATE_FORGET);
+            l.state.gain = STATE_GAIN_HEAD;
+            l.state.gate = STATE_GATE_NONE;
+            l.state.at = "mix.right.";
+            l.state.out_scale = (float)m.num("right_scale");
+        } else {
+            lc.fail("type is not a mixer of this design");
+            break;
+        }
+        read_dense(lc, &l);
+        l.dense.act = DENSE_XIELU;
+        p.layers.push_back(l);
+    }
+    if (!err.empty()) { set_error(err); return SP_ERR_ARG; }
+    *out = std::move(p);
+    return SP_OK;
+}
+
 // GGUF names: crates/sapient-models/src/forward/mod.rs:223-316 (family dispatch of the reference's loader).
 const ArchEntry ARCHS[] = {
     {"llama", ARCH_LLAMA, true, nullptr},   {"mistral", ARCH_LLAMA, true, nullptr}, {"qwen2", ARCH_LLAMA, true, nullptr},
     {"qwen3", ARCH_LLAMA, true, nullptr},   {"idefics3", ARCH_LLAMA, true, nullptr}, {"phi3", ARCH_LLAMA, true, nullptr},
     {"phi", ARCH_PHI2, true, nullptr},      {"phi2", ARCH_PHI2, true, nullptr},     {"Lepalorn", ARCH_PLAN, false, read_lepalorn},
     {"Tedelix", ARCH_PLAN, false, read_tedelix}, {"Fatilix", ARCH_PLAN, false, read_fatilix},
+    {"Revelix", ARCH_PLAN, false, read_revelix},
 };
 
 }  // namespace

@@ -21,10 +21,14 @@ namespace sp {
 enum ArchBlock : int { ARCH_LLAMA = 0, ARCH_PHI2 = 1, ARCH_PLAN = 2 };
 
 // Rotary position embedding over `dims` coordinates, angle position * base^(-2 i / dims) for pair i. Pairs are neighbours
-// (2 i, 2 i + 1) in latent attention and halves (i, i + dims / 2) in grouped attention.
+// (2 i, 2 i + 1) in latent attention and where `neighbours` is set, else halves (i, i + dims / 2). With factor > 0 frequencies are
+// stretched for contexts beyond `original`: pairs that turn more than `fast` times within it keep theirs, pairs that turn less than
+// `slow` times have it divided by factor, with a linear ramp over the pairs between; sines and cosines grow by 0.1 ln(factor) + 1.
 struct RotarySpec {
     double base = 10000.0;
     int dims = 0;
+    bool neighbours = false;
+    double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;
 };
 
 // Latent attention: per token only a normed latent of kv_rank values and one rotated key part of rot_dim values shared by
@@ -52,6 +56,10 @@ struct TemperatureSpec {
 // mixture is turned back by the query's. A distance bias adds table[bucket(i - j)][head] to the scaled score: a bucket per
 // distance up to half of the table's rows, then logarithmic ones up to bias_max. A sink is one more term exp(sink[head]) in
 // the softmax's denominator. An output gate multiplies the mixtures, coordinate by coordinate, by sigmoid(W_g h).
+// A short convolution over time (conv taps per channel, the last one on the token itself) comes between bias and norm; the
+// taps - 1 values before a token are state of its sequence. keep_first: the sequence's first keys stay visible behind the window.
+// score_softcap: s <- cap tanh(s / cap) on the scaled score. talk: the heads' softmax weights are mixed, w_h <- sum_g T[h][g] w_g
+// (without the sink's share), before they meet the values of h's cached head. Outputs are multiplied by out_scale.
 struct GroupedAttentionSpec {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
     int window = 0x7FFFFFFF;  // as above
@@ -64,19 +72,40 @@ struct GroupedAttentionSpec {
     TemperatureSpec temperature;
     int bias_max = 0;            // 0: no distance bias
     bool sink = false, out_gate = false;
+    int conv = 0;                // 0: no convolution
+    int keep_first = 0;
+    float score_softcap = 0.f;   // 0: no cap
+    bool talk = false;
+    float out_scale = 1.f;
+    std::string at = "mix.";     // tensor names behind the layer's prefix
 };
+constexpr int CONV_MAX_TAPS = 32;
 
 // A mixer whose memory is one matrix S [dim][vdim] per head and sequence, in f32, zero at the start; o = S^T q.
-//   STATE_DECAY  S <- decay_h S + k v^T; q, k, v through silu; the heads' outputs are normed together.
-//   STATE_DELTA  S <- diag(w) S - (a u)(u^T S) + k v^T with the unit key u = k / |k|, w = exp(-e^(-1/2) sigmoid(low-rank
-//                logit)) and a = sigmoid(projection) per head and key channel; each head's output is normed by itself.
-// Both then take a gain per coordinate and a sigmoid gate.
+//   STATE_DECAY   S <- decay_h S + k v^T.
+//   STATE_DELTA   S <- diag(w) S - (a u)(u^T S) + k v^T with the unit key u = k / |k|, w = exp(-e^(-1/2) sigmoid(low-rank
+//                 logit)) and a = sigmoid(projection) per head and key channel.
+//   STATE_FORGET  S <- diag(f) S + (1 - f) v^T, f = l + (1 - l) sigmoid(projection + bias) per head and key channel, between the
+//                 learned bound l and one. q through silu.
+// The decaying sum may take q, k and v through silu, or rotate q and k by position, and scales its keys. Outputs are divided by
+// their root mean square, head by head or all heads of a token together, then take a gain and a gate by a projection of h.
 constexpr int STATE_MAX_DIM = 512;  // key channels the kernels cover
-enum StateRule : int { STATE_DECAY = 0, STATE_DELTA = 1 };
+enum StateRule : int { STATE_DECAY = 0, STATE_DELTA = 1, STATE_FORGET = 2 };
+enum StateGate : int { STATE_GATE_NONE = 0, STATE_GATE_SIGMOID = 1, STATE_GATE_SILU = 2 };
+// The gain after the norm: none, one number per coordinate, or per coordinate of a head and the same for all heads.
+enum StateGain : int { STATE_GAIN_NONE = 0, STATE_GAIN_COORD = 1, STATE_GAIN_HEAD = 2 };
 struct StateMixerSpec {
     StateRule rule = STATE_DECAY;
     int heads = 0, dim = 0, vdim = 0;
-    std::vector<float> decay;  // STATE_DECAY: per head
+    std::vector<float> decay;   // STATE_DECAY: per head
+    bool silu_inputs = false;   // STATE_DECAY
+    RotarySpec rot;             // STATE_DECAY
+    float key_scale = 1.f;      // STATE_DECAY
+    bool norm_all = false;      // STATE_DECAY
+    StateGain gain = STATE_GAIN_COORD;
+    StateGate gate = STATE_GATE_SIGMOID;
+    float out_scale = 1.f;
+    std::string at = "mix.";    // tensor names behind the layer's prefix
 };
 
 // Gated expert: g = min(W_gate x, limit), u = clamp(W_up x, +-limit), y = W_down (g sigmoid(alpha g) (u + shift)). As it
@@ -105,12 +134,17 @@ struct MoeSpec {
     GatedExpertSpec shared;
 };
 
-enum MixerKind : int { MIX_LATENT = 0, MIX_GROUPED = 1, MIX_STATE = 2 };
+// MIX_BOTH: grouped attention and a state mixer side by side; both read the same input, their outputs are added.
+enum MixerKind : int { MIX_LATENT = 0, MIX_GROUPED = 1, MIX_STATE = 2, MIX_BOTH = 3 };
 enum MlpKind : int { MLP_NONE = 0, MLP_MOE = 1, MLP_DENSE = 2 };
 
-// W_down act(W_up h), act = the square of relu.
+// W_down act(W_up h).
+//   DENSE_RELU2  the square of relu
+//   DENSE_XIELU  z / 2 + softplus(p) z^2 right of zero, z / 2 + (1/2 + softplus(q)) (e^z - 1 - z) left of it, with learned p, q
+enum DenseAct : int { DENSE_RELU2 = 0, DENSE_XIELU = 1 };
 struct DenseSpec {
     int ff = 0;
+    DenseAct act = DENSE_RELU2;
 };
 
 struct LayerPlan {
@@ -122,12 +156,18 @@ struct LayerPlan {
     MlpKind mlp = MLP_NONE;
     MoeSpec moe;
     DenseSpec dense;
+    bool has_grouped() const { return mixer == MIX_GROUPED || mixer == MIX_BOTH; }
+    bool has_state() const { return mixer == MIX_STATE || mixer == MIX_BOTH; }
 };
 
 // What happens to the residual stream x in a layer.
 //   FORM_POST_NORM  x <- x + m norm(mixer(x)), then x <- x + m norm(ff(x)), m = residual_mult.
 //   FORM_PARALLEL   x <- x + mixer(h) + ff(h) with h = norm(x). Both sublayers are one product in and one product out.
-enum LayerForm : int { FORM_POST_NORM = 0, FORM_PARALLEL = 1 };
+//   FORM_PRE_NORM   x <- x + mixer(norm(x)), then x <- x + ff(norm(x)).
+enum LayerForm : int { FORM_POST_NORM = 0, FORM_PARALLEL = 1, FORM_PRE_NORM = 2 };
+
+// The stream's norm: by the root mean square, or tanh(alpha x) w + b with a learned number alpha and vectors w, b.
+enum NormKind : int { NORM_RMS = 0, NORM_TANH = 1 };
 
 // The gain of the stream's norms: one number, one per coordinate, or one per coordinate stored as its distance from one.
 enum NormGain : int { GAIN_SCALAR = 0, GAIN_COORD = 1, GAIN_OFFSET = 2 };
@@ -139,16 +179,12 @@ struct ModelPlan {
     int max_positions = 0;       // rows of a table of learned position vectors, added to the embedding (0: none)
     float residual_mult = 1.f;
     LayerForm form = FORM_POST_NORM;
+    NormKind norm = NORM_RMS;
     NormGain norm_gain = GAIN_SCALAR;
     bool depth_average = false;  // after each layer the stream becomes a learned combination of every layer result so far
     bool tied_head = false;      // logits from the embedding table
     float logit_scale = 1.f, logit_softcap = 0.f;  // z <- z * scale, then cap * tanh(z / cap) (0: no cap)
     std::vector<LayerPlan> layers;
-    bool recurrent() const {     // some layer keeps a state that cannot be rolled back
-        for (const LayerPlan& l : layers)
-            if (l.mixer == MIX_STATE) return true;
-        return false;
-    }
 };
 
 struct ArchEntry {

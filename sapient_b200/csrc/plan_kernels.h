@@ -35,7 +35,9 @@ struct MatSeg {
 
 // Where a range of a matrix's rows goes: output elements [previous n_end, n_end) of every activation row to y (column 0 is
 // the range's first), through an activation, as f32 or in the compute type; `add`: y (f32) += instead of =.
-enum MatAct : int { MAT_ID = 0, MAT_RELU2, MAT_TANH, MAT_SILU, MAT_SOFTCAP };  // softcap: cap * tanh(scale * z / cap)
+//   MAT_SOFTCAP  arg[1] * tanh(arg[0] * z / arg[1])
+//   MAT_XIELU    z / 2 + arg[0] z^2 right of zero, z / 2 + arg[1] (e^z - 1 - z) left of it
+enum MatAct : int { MAT_ID = 0, MAT_RELU2, MAT_TANH, MAT_SILU, MAT_SOFTCAP, MAT_XIELU };
 struct MatOut {
     int n_end;
     void* y;
@@ -44,6 +46,18 @@ struct MatOut {
     bool f32, add;
 };
 constexpr int MAT_MAX_OUTS = 4;
+
+// A norm without statistics: tanh(alpha x) w[c] + b[c] (null w: none).
+struct TanhNorm {
+    float alpha;
+    const float *w, *b;
+};
+// What a product that adds into the stream leaves beside it: the norm of the sums in the compute type.
+struct MatNorm {
+    TanhNorm fn;
+    void* y;
+    int64_t ldy;
+};
 
 // Rows of a step sorted by expert, made on the device by launch_moe_route.
 struct MoeRows {
@@ -71,7 +85,8 @@ struct MatArgs {
     int ldgate;
     int n_outs;                // > 0: one plain product whose rows go where outs[] says (seg[0].y is not used)
     MatOut outs[MAT_MAX_OUTS];
-    float scale, cap;          // of MAT_SOFTCAP
+    float arg[2];              // of the activation
+    MatNorm norm;              // null w: none; else one range that adds
 };
 
 // The ranges cover the matrix, and the product is a plain one.
@@ -83,7 +98,7 @@ inline bool mat_outs_valid(const MatArgs& a) {
         if (a.outs[i].n_end <= n || !a.outs[i].y || (a.outs[i].add && !a.outs[i].f32 && !a.f32)) return false;
         n = a.outs[i].n_end;
     }
-    return n == a.seg[0].n;
+    return n == a.seg[0].n && (!a.norm.fn.w || (a.n_outs == 1 && a.outs[0].add));
 }
 
 // f32: plain fused multiply-adds on 32 x 32 tiles, any shape and row count.
@@ -98,10 +113,10 @@ cudaError_t launch_mat_tc5(const MatArgs& a, int max_tiles, cudaStream_t st);
 int mat_tc5_take_timeout();    // as tc5_take_timeout (kernels.h)
 
 // ── the stream between the products ──
-// x0[t] = table[ids[t]] * scale (+ pos_table[tok_pos[t]], or null) (f32), xb (or null) = the same in the compute type (row
-// stride ldb, padding zeroed). Both tables have rows of ldt.
+// x0[t] = table[ids[t]] * scale (+ pos_table[tok_pos[t]], or null) (f32), xb (or null) = the same, or its norm (norm.w), in the
+// compute type (row stride ldb, padding zeroed). Both tables have rows of ldt.
 cudaError_t launch_embed_scaled(const void* table, const void* pos_table, int ldt, bool f32, const uint32_t* ids, const int32_t* tok_pos, int n_tok,
-                                int width, float scale, float* x0, void* xb, int ldb, cudaStream_t st);
+                                int width, float scale, const TanhNorm& norm, float* x0, void* xb, int ldb, cudaStream_t st);
 // The gain of a norm: one number, or one per coordinate.
 struct RowGain {
     const float* g;
@@ -138,6 +153,8 @@ cudaError_t launch_combine(const CombineArgs& a, int n_tok, int width, cudaStrea
 // out (compute type) = rms_norm(x[rows[i] or i]) * gain.
 cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int width, const RowGain& gain, float eps, void* out, int ldo, bool f32,
                             cudaStream_t st);
+// out (compute type) = tanh norm of x[rows[i] or i].
+cudaError_t launch_tanh_norm(const float* x, const int32_t* rows, int n_rows, int width, const TanhNorm& norm, void* out, int ldo, bool f32, cudaStream_t st);
 
 // ── experts ──
 // How a token's experts follow from its logits (model_plan.h: RouteRule). Ties: the lower index.
@@ -220,6 +237,9 @@ struct GroupedShape {
     int heads, kv_heads, dim, vdim, rot;
     int window;
     float scale;
+    bool neighbours;           // rotation of pairs (2 i, 2 i + 1), else (i, i + rot / 2)
+    int keep;                  // attention with mixed heads: first keys that stay visible behind the window
+    float softcap;             // attention with mixed heads: of the scaled scores (0: none)
 };
 // What happens to queries, keys and values between the projection and the cache; null: nothing.
 struct GroupedInput {
@@ -229,11 +249,22 @@ struct GroupedInput {
     float eps;
     const float* temperature;  // factor of the queries, by position
     const float2 *cs_key, *cs_val;  // angles [pos][rot / 2] of queries and keys, [pos][vdim / 2] of values
+    // Convolution over time behind the bias: [channels][taps], the last tap on the token itself. The taps - 1 values before a
+    // slot's next token are at tail + slot * tail_stride, [taps - 1][channels], the oldest first; what stands for tokens before
+    // the sequence's start is not read. Rows of a slot may stand anywhere in a step.
+    const float* conv;
+    int taps;
+    float* tail;
+    int64_t tail_stride;
+    const int32_t* back;       // row of the slot's token before this one, -1: in an earlier step. Null (up to 32 rows): found out
 };
 // proj[t] (f32, row stride ldp): queries head by head, keys, values (not when shared). q[t][heads][dim16] in the compute type,
 // keys and values to the cache.
 cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in,
                                   const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st);
+// Steps with a table `back`: brings the tails up to date once the rows have been appended. ends[i]: a slot's last row in the step.
+cudaError_t launch_conv_tails(const float* proj, int ldp, const GroupedShape& s, const GroupedInput& in, const int32_t* tok_slot, const int32_t* ends,
+                              int n_ends, cudaStream_t st);
 // What else enters the scores, the softmax and the output; null: nothing.
 struct GroupedTerms {
     const float* rel;          // [heads][n_rel], added to the scaled score: by distance, the last one from there on
@@ -260,6 +291,33 @@ constexpr int GROUPED_Q_TILE = 64;
 cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const GroupedTile* tiles,
                                    int n_tiles, void* out, int ldo, cudaStream_t st);
 
+// ── grouped attention whose heads' softmax weights are mixed ──
+// w_h <- sum_g mix[h][g] w_g over all query heads, then head h takes the values of its own cached head. Needs every head's weights
+// where one head's mixture is made, so there are two passes: scores and softmax denominators, then weights and values. Windows may
+// keep a sequence's first keys, scores may be capped, denominators may have a sink. Kept pages and the window's pages are visited
+// as one run: a row's i-th visited key is at score[row][head][i].
+struct MixedTerms {
+    const float* mix;          // [heads][heads]
+    const float* sink;         // [heads] or null
+};
+struct MixedScratch {
+    float* score;              // [rows][heads][span]
+    int rows, span;            // span: mixed_span()
+    float2* part;              // [rows][heads][MIXED_SPLITS]: maximum and sum of a split of the keys
+    float2* stat;              // [tokens of a step][heads]: maximum and reciprocal of the denominator
+};
+constexpr int MIXED_SPLITS = 8;
+int mixed_span(const GroupedShape& s, int max_ctx);       // most keys a token visits, whole pages
+bool mixed_mma_supported(const GroupedShape& s, const GroupedCache& c);
+int mixed_attention_splits(const GroupedShape& s, int n_tok, int keys);
+// Few rows (bf16), or any sizes and rows in plain arithmetic (f32, and sizes the tensor-core kernels do not cover; n_splits 1).
+cudaError_t launch_mixed_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
+                                   const int32_t* tok_slot, const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st);
+// bf16, many rows: the step's tokens as tiles of GROUPED_Q_TILE (first pass) and of MIXED_Q_TILE (second).
+constexpr int MIXED_Q_TILE = 16;
+cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
+                                 const GroupedTile* wide, int n_wide, const GroupedTile* narrow, int n_narrow, void* out, int ldo, cudaStream_t st);
+
 // ── mixers with a state matrix (model_plan.h: StateMixerSpec) ──
 // State of a slot: [heads][vdim][dim_pad] f32, slots slot_stride floats apart (a value column's keys are contiguous). A sequence's first token (position 0)
 // starts from zeros, whatever the slot held.
@@ -268,6 +326,10 @@ struct StateShape {
     int rule;                  // StateRule
     int dim_pad;               // state_dim_pad(dim)
     float eps;
+    bool norm_all;             // STATE_DECAY: all heads of a token are normed together
+    int gate;                  // StateGate
+    int rot;                   // STATE_DECAY: coordinates of queries and keys that are rotated, in halves
+    float key_scale;           // STATE_DECAY
 };
 int state_dim_pad(int dim);
 struct StateArgs {
@@ -275,17 +337,20 @@ struct StateArgs {
     float* state;
     int64_t slot_stride;
     const float* decay;        // STATE_DECAY: [heads]
-    // STATE_DECAY: proj[t] = q | k | v (silu applied) | gate logits. STATE_DELTA: r | k | v | removal logits | gate logits.
+    // STATE_DECAY: proj[t] = q | k | v (silu applied where the mixer has it) | gate logits. STATE_DELTA: r | k | v | removal logits |
+    // gate logits. STATE_FORGET: q (silu applied) | forget logits | v. No gate: no logits.
     const float* proj;
     int ldp;
-    const float* a_bias;       // STATE_DELTA: [heads * dim]
+    const float* a_bias;       // STATE_DELTA: of the removal logits, STATE_FORGET: of the forget logits, [heads * dim]
+    const float* lower;        // STATE_FORGET: [heads * dim]
+    const float2* cs;          // STATE_DECAY: angles [pos][rot / 2]
     const float* w0;           // STATE_DELTA: decay logit = w0 + W2 low[t]
     const void* w2;            // compute type, [heads * dim][ldlow]
     const void* low;           // compute type, [t][ldlow]
     int ldlow;
     const float* wlogit;       // many rows: W2 low[t] (f32, [t][heads * dim])
     float* rec;                // many rows: scratch, state_record_floats per group
-    const float* gain;         // [heads * vdim]
+    const float* gain;         // [heads * vdim] or null
     const int32_t *tok_slot, *tok_pos;
     void* out;                 // compute type, [t][ldo]
     int ldo;

@@ -33,7 +33,7 @@ template <> struct Row<4> {
 template <typename T>
 __global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __restrict__ table, const T* __restrict__ pos_table, int ldt,
                                                                   const uint32_t* __restrict__ ids, const int32_t* __restrict__ tok_pos, int width, float scale,
-                                                                  float* __restrict__ x0, T* __restrict__ xb, int ldb) {
+                                                                  const TanhNorm norm, float* __restrict__ x0, T* __restrict__ xb, int ldb) {
     pdl_wait();
     pdl_trigger();
     const int t = blockIdx.x;
@@ -43,15 +43,16 @@ __global__ void __launch_bounds__(ST_THREADS) embed_scaled_kernel(const T* __res
         float v = c < width ? to_f32(row[c]) * scale : 0.f;
         if (prow && c < width) v += to_f32(prow[c]);
         if (c < width) x0[(int64_t)t * width + c] = v;
+        if (norm.w && c < width) v = tanh_norm(norm, v, c);
         if (xb) xb[(int64_t)t * ldb + c] = from_f32<T>(v);
     }
 }
 
 cudaError_t launch_embed_scaled(const void* table, const void* pos_table, int ldt, bool f32, const uint32_t* ids, const int32_t* tok_pos, int n_tok,
-                                int width, float scale, float* x0, void* xb, int ldb, cudaStream_t st) {
+                                int width, float scale, const TanhNorm& norm, float* x0, void* xb, int ldb, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
     const dim3 grid(n_tok), block(ST_THREADS);
-#define SP_EM(T) launch_pdl(embed_scaled_kernel<T>, grid, block, 0, st, (const T*)table, (const T*)pos_table, ldt, ids, tok_pos, width, scale, x0, (T*)xb, ldb)
+#define SP_EM(T) launch_pdl(embed_scaled_kernel<T>, grid, block, 0, st, (const T*)table, (const T*)pos_table, ldt, ids, tok_pos, width, scale, norm, x0, (T*)xb, ldb)
     const cudaError_t le = f32 ? SP_EM(float) : SP_EM(bf16);
 #undef SP_EM
     if (le != cudaSuccess) return le;
@@ -251,6 +252,23 @@ cudaError_t launch_row_norm(const float* x, const int32_t* rows, int n_rows, int
 #undef SP_RN
     if (le != cudaSuccess) return le;
     return count_launch_and_check();
+}
+
+template <typename T>
+__global__ void __launch_bounds__(ST_THREADS) tanh_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, int width, const TanhNorm norm,
+                                                               T* __restrict__ out, int ldo) {
+    pdl_wait();
+    pdl_trigger();
+    const float* xr = x + (int64_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * width;
+    for (int c = threadIdx.x; c < ldo; c += ST_THREADS) out[(int64_t)blockIdx.x * ldo + c] = from_f32<T>(c < width ? tanh_norm(norm, xr[c], c) : 0.f);
+}
+
+cudaError_t launch_tanh_norm(const float* x, const int32_t* rows, int n_rows, int width, const TanhNorm& norm, void* out, int ldo, bool f32, cudaStream_t st) {
+    if (n_rows == 0) return cudaSuccess;
+    const dim3 grid(n_rows), block(ST_THREADS);
+    const cudaError_t le = f32 ? launch_pdl(tanh_norm_kernel<float>, grid, block, 0, st, x, rows, width, norm, (float*)out, ldo)
+                               : launch_pdl(tanh_norm_kernel<bf16>, grid, block, 0, st, x, rows, width, norm, (bf16*)out, ldo);
+    return le != cudaSuccess ? le : count_launch_and_check();
 }
 
 // ── experts ──

@@ -7,7 +7,8 @@
 //   (I + L) D = U~ S + A V,  O = R~ S + Ark V - Arb D,  S <- g_16 (S + K~^T V - B~^T D)
 // with D the values found under the unit keys and L, A, Arb, Ark the lower triangles of U~ B~^T, U~ K~^T (strict), R~ B~^T, R~ K~^T.
 // A kernel that is parallel over chunks and heads solves for U = (I + L)^-1 U~, P = (I + L)^-1 A, R = R~ - Arb U, Q = Ark - Arb P,
-// which leaves the scan D = U S + P V, O = R S + Q V and the update. The decaying sum has R, Q and K only.
+// which leaves the scan D = U S + P V, O = R S + Q V and the update. The decaying sum and the forget gate have R, Q and K only; a
+// gate may forget everything at once, so its products of decays are made without a division, one for each pair of tokens.
 #include <algorithm>
 
 #include "kernels.h"
@@ -52,10 +53,12 @@ StateRecordView state_chunk_view(const StateShape& s) {
 
 // ── what a chunk owes to itself ──
 constexpr int CP_THREADS = 128;
-static size_t cp_smem(const StateShape& s) { return ((size_t)(s.rule == STATE_DELTA ? 4 : 2) * CH * (s.dim_pad + 4) + 4 * CH * CH) * 4; }
+__host__ __device__ constexpr int cp_rows(int rule) { return rule == STATE_DELTA ? 4 : rule == STATE_FORGET ? 3 : 2; }
+static size_t cp_smem(const StateShape& s) { return ((size_t)cp_rows(s.rule) * CH * (s.dim_pad + 4) + 4 * CH * CH) * 4; }
 
-template <bool DELTA>
+template <int RULE>
 __global__ void __launch_bounds__(CP_THREADS, 6) chunk_prepare_kernel(const StateArgs a, const int32_t* __restrict__ groups) {
+    constexpr bool DELTA = RULE == STATE_DELTA, FORGET = RULE == STATE_FORGET;
     extern __shared__ __align__(16) float cp_sm[];
     __shared__ float inv_s[CH], pow_s[CH + 1];
     __shared__ int row_s[CH];
@@ -66,7 +69,7 @@ __global__ void __launch_bounds__(CP_THREADS, 6) chunk_prepare_kernel(const Stat
     const ChunkRecord rec = chunk_record(a.s);
     float* out = a.rec + ((int64_t)blockIdx.x * H + h) * rec.floats;
     float *rs = cp_sm, *ks = rs + CH * LD, *us = ks + CH * LD, *bs = us + CH * LD;
-    float* tri = cp_sm + (DELTA ? 4 : 2) * CH * LD;  // Ark, Arb, A, L [CH][CH]
+    float* tri = cp_sm + cp_rows(RULE) * CH * LD;  // Ark, Arb, A, L [CH][CH]
     if (tid < CH) row_s[tid] = groups[(int64_t)blockIdx.x * CH + tid];
     __syncthreads();
     int n = 0;  // tokens of the chunk
@@ -77,9 +80,10 @@ __global__ void __launch_bounds__(CP_THREADS, 6) chunk_prepare_kernel(const Stat
     for (int t = warp; t < CH; t += CP_THREADS / 32) {
         const int64_t row = max(row_s[t], 0);
         const float* pr = a.proj + row * a.ldp + h * D;
-        const float* src[4] = {pr + co.r, pr + co.k, DELTA ? a.wlogit + (row * H + h) * D : nullptr, pr + co.a};
+        const float* src[4] = {pr + co.r, pr + co.k, DELTA ? a.wlogit + (row * H + h) * D : pr + co.a, pr + co.a};
 #pragma unroll
-        for (int q = 0; q < (DELTA ? 4 : 2); ++q) {
+        for (int q = 0; q < cp_rows(RULE); ++q) {
+            if (FORGET && q == 1) continue;  // the keys follow from the forget logits
             float* d = cp_sm + (q * CH + t) * LD;
             if (wide)
                 for (int c = 4 * lane; c < DP; c += 128) cp_async16(d + c, src[q] + min(c, D - 4), t < n && c < D ? 16 : 0);
@@ -100,13 +104,92 @@ __global__ void __launch_bounds__(CP_THREADS, 6) chunk_prepare_kernel(const Stat
             out[rec.v + i] = t < n && c < V ? a.proj[(int64_t)row_s[t] * a.ldp + co.v + h * V + c] : 0.f;
         }
     }
-    const float decay = DELTA ? 0.f : a.decay[h];
-    if (!DELTA && tid == 0) {
+    const float decay = RULE == STATE_DECAY ? a.decay[h] : 0.f;
+    if (RULE == STATE_DECAY && tid == 0) {
         pow_s[0] = 1.f;
         for (int i = 0; i < CH; ++i) pow_s[i + 1] = pow_s[i] * decay;
     }
     cp_async_wait<0>();
     __syncthreads();
+    if (RULE == STATE_DECAY && (a.s.rot || a.s.key_scale != 1.f)) {
+        const int half = a.s.rot / 2, parts = DP - half;  // pairs, then single coordinates
+        for (int i = tid; i < CH * parts; i += CP_THREADS) {
+            const int t = i / parts, c = i - t * parts;
+            float *r = rs + t * LD, *k = ks + t * LD;
+            if (t >= n) continue;
+            if (c < half) {
+                const float2 w = a.cs[(int64_t)a.tok_pos[row_s[t]] * half + c];
+                const float ru = r[c], rv = r[c + half], ku = k[c], kv = k[c + half];
+                r[c] = ru * w.x - rv * w.y;
+                r[c + half] = rv * w.x + ru * w.y;
+                k[c] = (ku * w.x - kv * w.y) * a.s.key_scale;
+                k[c + half] = (kv * w.x + ku * w.y) * a.s.key_scale;
+            } else {
+                k[c + half] *= a.s.key_scale;
+            }
+        }
+        __syncthreads();
+    }
+    if (FORGET) {
+        for (int c = tid; c < DP; c += CP_THREADS) {
+            const bool on = c < D;
+            const int hc = h * D + min(c, D - 1);
+            const float bias = a.a_bias[hc], lower = a.lower[hc];
+            float g = 1.f;
+#pragma unroll 4
+            for (int t = 0; t < CH; ++t) {
+                const float2 f = on && t < n ? forget_gate(us[t * LD + c] + bias, lower) : make_float2(1.f, 0.f);
+                us[t * LD + c] = f.x;
+                ks[t * LD + c] = f.y;
+                g *= f.x;
+                out[rec.r + t * rec.row + c] = rs[t * LD + c] * g;
+            }
+            out[rec.g + c] = g;
+            float after = 1.f;
+#pragma unroll
+            for (int t = CH - 4; t >= 0; t -= 4) {
+                float k[4];
+#pragma unroll
+                for (int i = 3; i >= 0; --i) {
+                    k[i] = ks[(t + i) * LD + c] * after;
+                    after *= us[(t + i) * LD + c];
+                }
+                *reinterpret_cast<float4*>(out + rec.k + c * TS + t) = make_float4(k[0], k[1], k[2], k[3]);
+            }
+        }
+        __syncthreads();
+        // thread (s, eighth of the channels): token s's key on its way through the later tokens
+        const int s = tid >> 3, c8 = tid & 7;
+        float acc[CH];
+#pragma unroll
+        for (int t = 0; t < CH; ++t) acc[t] = 0.f;
+        for (int c = 4 * c8; c < DP; c += 32) {
+            float4 p = *reinterpret_cast<const float4*>(ks + s * LD + c);
+#pragma unroll
+            for (int t = 0; t < CH; ++t) {
+                if (t < s) continue;
+                if (t > s) {
+                    const float4 f = *reinterpret_cast<const float4*>(us + t * LD + c);
+                    p.x *= f.x; p.y *= f.y; p.z *= f.z; p.w *= f.w;
+                }
+                const float4 r = *reinterpret_cast<const float4*>(rs + t * LD + c);
+                acc[t] = fmaf(r.x, p.x, fmaf(r.y, p.y, fmaf(r.z, p.z, fmaf(r.w, p.w, acc[t]))));
+            }
+        }
+        // the eight lanes share out the sixteen sums while they make them
+#pragma unroll
+        for (int m = 4; m > 0; m >>= 1) {
+            const bool up = c8 & m;
+#pragma unroll
+            for (int i = 0; i < 2 * m; ++i) {
+                const float send = up ? acc[i] : acc[i + 2 * m], keep = up ? acc[i + 2 * m] : acc[i];
+                acc[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, m);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) out[rec.q + (2 * c8 + i) * TS + s] = acc[i];
+        return;
+    }
     if (DELTA) {
         for (int t = warp; t < CH; t += CP_THREADS / 32) {
             float ss = 0.f;
@@ -447,15 +530,19 @@ cudaError_t launch_state_chunks(const StateArgs& a, const StateSegment* seg, int
     const bool delta = a.s.rule == STATE_DELTA;
     constexpr int CAP = 160 * 1024;
     static PerDeviceOnce once;
+    const auto prepare = a.s.rule == STATE_DELTA ? chunk_prepare_kernel<STATE_DELTA> : a.s.rule == STATE_FORGET ? chunk_prepare_kernel<STATE_FORGET> : chunk_prepare_kernel<STATE_DECAY>;
     cudaError_t le = once.run([] {
-        const cudaError_t e = cudaFuncSetAttribute(chunk_prepare_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
-        return e != cudaSuccess ? e : cudaFuncSetAttribute(chunk_prepare_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+        for (const auto f : {chunk_prepare_kernel<STATE_DELTA>, chunk_prepare_kernel<STATE_FORGET>, chunk_prepare_kernel<STATE_DECAY>}) {
+            const cudaError_t e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
     });
     if (le != cudaSuccess) return le;
     const size_t smem = cp_smem(a.s);
     if (smem > CAP) return cudaErrorInvalidValue;
     const dim3 grid(n_groups, a.s.heads), block(CP_THREADS);
-    le = delta ? launch_pdl(chunk_prepare_kernel<true>, grid, block, smem, st, a, groups) : launch_pdl(chunk_prepare_kernel<false>, grid, block, smem, st, a, groups);
+    le = launch_pdl(prepare, grid, block, smem, st, a, groups);
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     le = cudaErrorInvalidValue;

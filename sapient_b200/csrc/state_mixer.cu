@@ -1,7 +1,7 @@
 // Mixers whose memory is a state matrix per head and sequence (plan_kernels.h, model_plan.h: StateMixerSpec).
 //
 // A value column j of S never meets another one: S[:, j] <- w . S[:, j] + k (v_j - a (u.S[:, j]) |k|^-1) in the delta rule,
-// S[:, j] <- decay S[:, j] + k v_j in the decaying sum, o_j = r . S[:, j]. So L lanes share a column, 4 R keys each in
+// S[:, j] <- decay S[:, j] + k v_j in the decaying sum, S[:, j] <- f . S[:, j] + (1 - f) v_j with a forget gate, o_j = r . S[:, j]. So L lanes share a column, 4 R keys each in
 // registers, and columns spread over warps and blocks. Everything is f32.
 //   Step (few rows): a block has a whole head, so gates, recurrence, norm and output gate are one launch; where the norm runs
 //   over all heads the blocks of a row are a cluster and exchange their sums of squares. The state is requested before the
@@ -41,12 +41,12 @@ __device__ __forceinline__ void dot4(const float4& a, const float4& b, float4& a
 
 // One token of one column: updates the lane's keys and returns the column's output (the same in its L lanes). Vectors are in
 // shared memory, dim_pad floats each.
-template <int L, int R, bool DELTA>
+template <int L, int R, int RULE>
 __device__ __forceinline__ float state_token(float4 (&st)[R], const float* kv, const float* rv, const float* wv, const float* av, float decay, float v, int l) {
     float4 k[R];
 #pragma unroll
     for (int i = 0; i < R; ++i) k[i] = *reinterpret_cast<const float4*>(kv + 4 * (l + L * i));
-    if (DELTA) {
+    if (RULE == STATE_DELTA) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < R; ++i) dot4(k[i], st[i], acc);
@@ -62,10 +62,12 @@ __device__ __forceinline__ float state_token(float4 (&st)[R], const float* kv, c
     } else {
 #pragma unroll
         for (int i = 0; i < R; ++i) {
-            st[i].x = fmaf(k[i].x, v, decay * st[i].x);
-            st[i].y = fmaf(k[i].y, v, decay * st[i].y);
-            st[i].z = fmaf(k[i].z, v, decay * st[i].z);
-            st[i].w = fmaf(k[i].w, v, decay * st[i].w);
+            float4 w = make_float4(decay, decay, decay, decay);
+            if (RULE == STATE_FORGET) w = *reinterpret_cast<const float4*>(wv + 4 * (l + L * i));
+            st[i].x = fmaf(k[i].x, v, w.x * st[i].x);
+            st[i].y = fmaf(k[i].y, v, w.y * st[i].y);
+            st[i].z = fmaf(k[i].z, v, w.z * st[i].z);
+            st[i].w = fmaf(k[i].w, v, w.w * st[i].w);
         }
     }
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -97,14 +99,16 @@ __device__ __forceinline__ float dot_low(const bf16* w, const bf16* x, int n, in
 }
 
 // ── few rows ──
-// Block (row, group of hp heads); the groups of a row form a cluster of `cl` where the norm runs over all heads.
-template <typename T, int L, int R, bool DELTA>
+// Block (row, group of hp heads); the groups of a row form a cluster of `cl` where the norm runs over all heads, else hp is one.
+__host__ __device__ constexpr int step_vectors(int rule) { return rule == STATE_DELTA ? 4 : rule == STATE_FORGET ? 3 : 2; }
+template <typename T, int L, int R, int RULE>
 __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int n_tok, int hp, int cl) {
     extern __shared__ __align__(16) float ss_smem[];
     __shared__ float cl_sum;
     constexpr int DP = 4 * L * R;
+    constexpr bool DELTA = RULE == STATE_DELTA;
     const int tid = threadIdx.x, lane = tid & 31, t = blockIdx.x, l = tid % L, H = a.s.heads, D = a.s.dim, V = a.s.vdim;
-    float *kv = ss_smem, *rv = kv + DP, *wv = rv + DP, *av = wv + DP, *os = DELTA ? av + DP : wv;
+    float *kv = ss_smem, *rv = kv + DP, *wv = rv + DP, *av = wv + DP, *os = ss_smem + step_vectors(RULE) * DP;
     const int mine = lane < n_tok ? a.tok_slot[lane] : -1, slot = __shfl_sync(0xFFFFFFFFu, mine, t);
     uint32_t rows = __ballot_sync(0xFFFFFFFFu, mine == slot);
     if (rows & ((1u << t) - 1)) return;  // an earlier row of this slot has a block that takes this one too
@@ -154,19 +158,28 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
                         av[c] = on ? sigmoid_f32(pr[co.a + hc] + a.a_bias[hc]) * inv : 0.f;
                     }
                 }
-            } else {
+            } else if (RULE == STATE_FORGET) {
                 for (int c = tid; c < DP; c += blockDim.x) {
-                    kv[c] = c < D ? pr[co.k + h * D + c] : 0.f;
-                    rv[c] = c < D ? pr[co.r + h * D + c] : 0.f;
+                    const int hc = h * D + c;
+                    const float2 f = c < D ? forget_gate(pr[co.a + hc] + a.a_bias[hc], a.lower[hc]) : make_float2(0.f, 0.f);
+                    wv[c] = f.x;
+                    kv[c] = f.y;
+                    rv[c] = c < D ? pr[co.r + hc] : 0.f;
+                }
+            } else {
+                const float2* cs = a.s.rot ? a.cs + (int64_t)a.tok_pos[row] * (a.s.rot / 2) : nullptr;
+                for (int c = tid; c < DP; c += blockDim.x) {
+                    kv[c] = c < D ? rotated(pr + co.k + h * D, c, a.s.rot, cs) * a.s.key_scale : 0.f;
+                    rv[c] = c < D ? rotated(pr + co.r + h * D, c, a.s.rot, cs) : 0.f;
                 }
             }
             __syncthreads();
-            const float decay = DELTA ? 0.f : a.decay[h];
+            const float decay = RULE == STATE_DECAY ? a.decay[h] : 0.f;
             for (int c0 = 0; c0 < V; c0 += per_pass) {
                 const int col = c0 + tid / L;
                 if (!ready) load(h, col);
                 ready = keep;
-                const float o = state_token<L, R, DELTA>(st, kv, rv, wv, av, decay, col < V ? pr[co.v + h * V + col] : 0.f, l);
+                const float o = state_token<L, R, RULE>(st, kv, rv, wv, av, decay, col < V ? pr[co.v + h * V + col] : 0.f, l);
                 if (col < V) {
                     float* p = at(h, col);
 #pragma unroll
@@ -182,7 +195,7 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
         for (int i = lane; i < n; i += 32) ss = fmaf(os[i], os[i], ss);
         ss = warp_sum(ss);
         int count = n;
-        if (!DELTA) {
+        if (RULE == STATE_DECAY && a.s.norm_all) {
             count = H * V;
             if (cl > 1) {
                 if (tid == 0) cl_sum = ss;
@@ -194,7 +207,7 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
         }
         const float r = rsqrtf(ss / (float)count + a.s.eps);
         T* out = reinterpret_cast<T*>(a.out) + row * a.ldo + (int64_t)h0 * V;
-        for (int i = tid; i < n; i += blockDim.x) out[i] = from_f32<T>(os[i] * r * a.gain[h0 * V + i] * sigmoid_f32(pr[co.g + h0 * V + i]));
+        for (int i = tid; i < n; i += blockDim.x) out[i] = from_f32<T>(os[i] * r * state_factor(a, pr + co.g, h0 * V + i));
         __syncthreads();
         fresh = false;
     }
@@ -202,31 +215,33 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
 
 constexpr int SS_MAX_CLUSTER = 8;
 
-template <typename T, int L, int R, bool DELTA>
+template <typename T, int L, int R, int RULE>
 static cudaError_t state_step_launch(const StateArgs& a, int n_tok, cudaStream_t st) {
     int hp = 1, cl = 1;
-    if (!DELTA) {
+    const bool all_heads = RULE == STATE_DECAY && a.s.norm_all;
+    if (all_heads) {
         hp = (a.s.heads + SS_MAX_CLUSTER - 1) / SS_MAX_CLUSTER;
         while (cl < SS_MAX_CLUSTER && cl * hp < a.s.heads) cl <<= 1;
     }
     const int all = L * a.s.vdim, threads = all <= 1024 ? (all + 31) / 32 * 32 : 512;
-    const size_t smem = ((size_t)(DELTA ? 4 : 2) * 4 * L * R + (size_t)hp * a.s.vdim) * 4;
+    const size_t smem = ((size_t)step_vectors(RULE) * 4 * L * R + (size_t)hp * a.s.vdim) * 4;
     constexpr int CAP = 200 * 1024;
     if (smem > CAP) return cudaErrorInvalidValue;
     static PerDeviceOnce once;
-    const cudaError_t le = once.run([] { return cudaFuncSetAttribute(state_step_kernel<T, L, R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP); });
+    const cudaError_t le = once.run([] { return cudaFuncSetAttribute(state_step_kernel<T, L, R, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP); });
     if (le != cudaSuccess) return le;
-    return launch_pdl_cluster(state_step_kernel<T, L, R, DELTA>, dim3(n_tok, 1, DELTA ? a.s.heads : cl), dim3(threads), smem, st, cl, a, n_tok, hp, cl);
+    return launch_pdl_cluster(state_step_kernel<T, L, R, RULE>, dim3(n_tok, 1, all_heads ? cl : a.s.heads), dim3(threads), smem, st, cl, a, n_tok, hp, cl);
 }
 
 cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st) {
     if (n_tok == 0) return cudaSuccess;
     if (n_tok > STATE_STEP_ROWS || a.s.dim > STATE_MAX_DIM || a.s.dim_pad != state_dim_pad(a.s.dim)) return cudaErrorInvalidValue;
-    const bool delta = a.s.rule == STATE_DELTA;
+    const int rule = a.s.rule;
     cudaError_t le = cudaErrorInvalidValue;
-#define SP_SS(L, R)                                                                                                                    \
-    le = a.f32 ? (delta ? state_step_launch<float, L, R, true>(a, n_tok, st) : state_step_launch<float, L, R, false>(a, n_tok, st))       \
-               : (delta ? state_step_launch<bf16, L, R, true>(a, n_tok, st) : state_step_launch<bf16, L, R, false>(a, n_tok, st))
+#define SP_SR(T, L, R)                                                                                                                     \
+    (rule == STATE_DELTA ? state_step_launch<T, L, R, STATE_DELTA>(a, n_tok, st) : rule == STATE_FORGET ? state_step_launch<T, L, R, STATE_FORGET>(a, n_tok, st) \
+                                                                                                : state_step_launch<T, L, R, STATE_DECAY>(a, n_tok, st))
+#define SP_SS(L, R) le = a.f32 ? SP_SR(float, L, R) : SP_SR(bf16, L, R)
     switch (a.s.dim_pad) {
         case 16: SP_SS(4, 1); break;
         case 32: SP_SS(4, 2); break;
@@ -236,6 +251,7 @@ cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st) {
         case 512: SP_SS(32, 4); break;
     }
 #undef SP_SS
+#undef SP_SR
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
@@ -249,8 +265,8 @@ cudaError_t launch_state_step(const StateArgs& a, int n_tok, cudaStream_t st) {
 // Auk = u_t c(s, t - 1) k_s, Aub = u_t c(s, t - 1) a_s u_s, Ark = r_t c(s, t) k_s, Arb = r_t c(s, t) a_s u_s. So the scan's
 // chain of reductions has a link per group, not per token. Everything but d, o and S is made by a kernel that is parallel
 // over groups and heads; a sequence's last group is filled up with tokens that change nothing (k = r = a = 0, decay 1).
-// Per (group, head) a record: U | R | K | B as [4][dim_pad] each, c(0, 4) (delta; the decaying sum has R | K only), the
-// coefficients, and the values [4][v_pad], where the scan leaves the outputs.
+// Per (group, head) a record: U | R | K | B as [4][dim_pad] each (R | K without the delta rule), c(0, 4) by channel (not in the
+// decaying sum), the coefficients, and the values [4][v_pad], where the scan leaves the outputs.
 constexpr int SGRP = STATE_GROUP_F32, A_UB = 8, A_RK = 16, A_RB = 32, A_FLOATS = 48;  // Auk at 0: (t, s < t) in order of t
 struct StateRecord {
     int k, b, c, a, v, v_pad, floats;  // offsets of U (or R) = 0, ...
@@ -264,7 +280,7 @@ __host__ __device__ __forceinline__ StateRecord state_record(const StateShape& s
     r.k = r.r + m;
     r.b = r.k + m;
     r.c = delta ? r.b + m : r.b;
-    r.a = delta ? r.c + s.dim_pad : r.c;
+    r.a = s.rule == STATE_DECAY ? r.c : r.c + s.dim_pad;
     r.v = r.a + A_FLOATS;
     r.v_pad = (s.vdim + 3) & ~3;
     r.floats = r.v + SGRP * r.v_pad;
@@ -293,8 +309,9 @@ __device__ __forceinline__ float warp_sums(float (&p)[32]) {
 
 // A warp per (group, head).
 constexpr int SG_WARPS = 4;
-template <bool DELTA>
+template <int RULE>
 __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const StateArgs a, const int4* __restrict__ groups) {
+    constexpr bool DELTA = RULE == STATE_DELTA;
     pdl_wait();
     pdl_trigger();
     const int h = blockIdx.y * SG_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = a.s.dim, DP = a.s.dim_pad, V = a.s.vdim, H = a.s.heads;
@@ -318,7 +335,7 @@ __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const Stat
 #pragma unroll
         for (int t = 0; t < SGRP; ++t) inv[t] = 1.0f / sqrtf(warp_sum(inv[t]) + 1e-6f);
     }
-    const float decay = DELTA ? 0.f : a.decay[h];
+    const float decay = RULE == STATE_DECAY ? a.decay[h] : 1.f;
     float p[32];  // Auk, Aub (t, s < t), then Ark, Arb (t, s <= t); the decaying sum: Ark alone
 #pragma unroll
     for (int i = 0; i < 32; ++i) p[i] = 0.f;
@@ -330,9 +347,20 @@ __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const Stat
 #pragma unroll
         for (int t = 0; t < SGRP; ++t) {
             const bool live = on && row[t] >= 0;
-            k[t] = live ? pr[t][co.k + hc] : 0.f;
-            r[t] = live ? pr[t][co.r + hc] : 0.f;
             w[t] = row[t] < 0 ? 1.f : decay;
+            if (RULE == STATE_DECAY) {
+                const float2* cs = live && a.s.rot ? a.cs + (int64_t)a.tok_pos[row[t]] * (a.s.rot / 2) : nullptr;
+                k[t] = live ? rotated(pr[t] + co.k + h * D, c, a.s.rot, cs) * a.s.key_scale : 0.f;
+                r[t] = live ? rotated(pr[t] + co.r + h * D, c, a.s.rot, cs) : 0.f;
+            } else {
+                k[t] = live ? pr[t][co.k + hc] : 0.f;
+                r[t] = live ? pr[t][co.r + hc] : 0.f;
+            }
+            if (RULE == STATE_FORGET) {
+                const float2 f = live ? forget_gate(pr[t][co.a + hc] + a.a_bias[hc], a.lower[hc]) : make_float2(1.f, 0.f);
+                w[t] = f.x;
+                k[t] = f.y;
+            }
             if (DELTA) {
                 w[t] = live ? channel_decay(a.wlogit[(int64_t)row[t] * H * D + hc] + a.w0[hc]) : 1.f;
                 u[t] = k[t] * inv[t];
@@ -376,7 +404,7 @@ __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const Stat
             if (DELTA) out[rec.b + t * DP + c] = after * b[t];
             after *= w[t];
         }
-        if (DELTA) out[rec.c + c] = before;
+        if (RULE != STATE_DECAY) out[rec.c + c] = before;
         whole = before;
     }
     const float sum = warp_sums(p);
@@ -390,7 +418,7 @@ __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const Stat
         const int i = lane - first, q = i % 10, t = q >= 6 ? 3 : q >= 3 ? 2 : q >= 1 ? 1 : 0;
         A[(i >= 10 ? A_RB : A_RK) + 4 * t + q - t * (t + 1) / 2] = sum;
     }
-    if (!DELTA && lane == 0) A[0] = whole;
+    if (RULE == STATE_DECAY && lane == 0) A[0] = whole;
     for (int c = lane; c < rec.v_pad; c += 32)
 #pragma unroll
         for (int t = 0; t < SGRP; ++t) out[rec.v + t * rec.v_pad + c] = c < V && row[t] >= 0 ? pr[t][co.v + h * V + c] : 0.f;
@@ -398,10 +426,11 @@ __global__ void __launch_bounds__(SG_WARPS * 32) state_prepare_kernel(const Stat
 
 // Block (SC_COLS columns, head, segment); records arrive in tiles of tg groups, two stages of cp.async.
 constexpr int SC_COLS = 16;
-template <int L, int R, bool DELTA>
+template <int L, int R, int RULE>
 __global__ void __launch_bounds__(SC_COLS * L) state_scan_kernel(const StateArgs a, const StateSegment* __restrict__ segs, int tg) {
     extern __shared__ __align__(16) float sc_smem[];
     constexpr int DP = 4 * L * R, THREADS = SC_COLS * L;
+    constexpr bool DELTA = RULE == STATE_DELTA;
     const int tid = threadIdx.x, l = tid % L, cl = tid / L, H = a.s.heads, V = a.s.vdim, h = blockIdx.y, col0 = blockIdx.x * SC_COLS, col = col0 + cl;
     const StateRecord rec = state_record(a.s);
     const int stage = rec.v + SGRP * SC_COLS;  // floats of a group in shared memory: the record with this block's values only
@@ -462,12 +491,12 @@ __global__ void __launch_bounds__(SC_COLS * L) state_scan_kernel(const StateArgs
                 e[2] = fmaf(k0.y, v[0], fmaf(k0.z, v[1], fmaf(-b0.y, e[0], fmaf(-b0.z, e[1], e[2]))));
                 e[3] = fmaf(k0.w, v[0], fmaf(k1.x, v[1], fmaf(k1.y, v[2], fmaf(-b0.w, e[0], fmaf(-b1.x, e[1], fmaf(-b1.y, e[2], e[3]))))));
             }
-            const float whole = DELTA ? 0.f : A[0];
+            const float whole = RULE == STATE_DECAY ? A[0] : 0.f;
 #pragma unroll
             for (int i = 0; i < R; ++i) {
                 const int at = 4 * (l + L * i);
                 float4 c = make_float4(whole, whole, whole, whole);
-                if (DELTA) c = *reinterpret_cast<const float4*>(d + rec.c + at);
+                if (RULE != STATE_DECAY) c = *reinterpret_cast<const float4*>(d + rec.c + at);
                 st[i].x *= c.x; st[i].y *= c.y; st[i].z *= c.z; st[i].w *= c.w;
 #pragma unroll
                 for (int t = 0; t < SGRP; ++t) {
@@ -510,9 +539,9 @@ __global__ void __launch_bounds__(SC_COLS * L) state_scan_kernel(const StateArgs
         for (int i = 0; i < R; ++i) *reinterpret_cast<float4*>(state + 4 * L * i) = st[i];
 }
 
-// Norms of the scan's outputs, gain, gate. Delta: a warp per (token, head); else a block per token, for the norm is over all heads.
+// Norms of the scan's outputs, gain, gate. EACH: a warp per (token, head); else a block per token, for the norm is over all heads.
 constexpr int SN_WARPS = 8, SN_KEEP = 4;  // values a lane keeps in registers
-template <typename T, bool DELTA>
+template <typename T, bool EACH>
 __global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateArgs a, const StateRecordView rec, const int32_t* __restrict__ groups, int group) {
     __shared__ float sh[SN_WARPS];
     pdl_wait();
@@ -522,8 +551,8 @@ __global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateAr
     if (row < 0) return;
     const float *o = a.rec + (int64_t)(blockIdx.x / group) * H * rec.floats + rec.v + t * rec.v_pad, *g = a.proj + row * a.ldp + state_cols(a.s).g;
     T* out = reinterpret_cast<T*>(a.out) + row * a.ldo;
-    auto finish = [&](int h, int i, float v, float r) { out[h * V + i] = from_f32<T>(v * r * a.gain[h * V + i] * sigmoid_f32(g[h * V + i])); };
-    if (DELTA) {
+    auto finish = [&](int h, int i, float v, float r) { out[h * V + i] = from_f32<T>(v * r * state_factor(a, g, h * V + i)); };
+    if (EACH) {
         const int h = blockIdx.y * SN_WARPS + warp;
         if (h >= H) return;
         const float* oh = o + (int64_t)h * rec.floats;
@@ -532,7 +561,7 @@ __global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateAr
         for (int j = 0; j < SN_KEEP; ++j) {
             const int i = lane + 32 * j;
             v[j] = i < V ? oh[i] : 0.f;
-            f[j] = i < V ? a.gain[h * V + i] * sigmoid_f32(g[h * V + i]) : 0.f;
+            f[j] = i < V ? state_factor(a, g, h * V + i) : 0.f;
             ss = fmaf(v[j], v[j], ss);
         }
         for (int i = lane + 32 * SN_KEEP; i < V; i += 32) ss = fmaf(oh[i], oh[i], ss);
@@ -552,26 +581,29 @@ __global__ void __launch_bounds__(SN_WARPS * 32) state_norm_kernel(const StateAr
     for (int i = threadIdx.x; i < H * V; i += SN_WARPS * 32) finish(i / V, i % V, o[(int64_t)(i / V) * rec.floats + i % V], r);
 }
 
-template <int L, int R, bool DELTA>
+template <int L, int R, int RULE>
 static cudaError_t state_scan_launch(const StateArgs& a, const StateSegment* seg, int n_seg, cudaStream_t st) {
     constexpr int CAP = 96 * 1024;
     const size_t group = (size_t)(state_record(a.s).v + SGRP * SC_COLS) * 4;
     int tg = 4;
     while (tg > 1 && 2 * tg * group > CAP) tg >>= 1;
     static PerDeviceOnce once;
-    const cudaError_t le = once.run([] { return cudaFuncSetAttribute(state_scan_kernel<L, R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP); });
+    const cudaError_t le = once.run([] { return cudaFuncSetAttribute(state_scan_kernel<L, R, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, CAP); });
     if (le != cudaSuccess) return le;
-    return launch_pdl(state_scan_kernel<L, R, DELTA>, dim3((a.s.vdim + SC_COLS - 1) / SC_COLS, a.s.heads, n_seg), dim3(SC_COLS * L), 2 * tg * group, st, a, seg, tg);
+    return launch_pdl(state_scan_kernel<L, R, RULE>, dim3((a.s.vdim + SC_COLS - 1) / SC_COLS, a.s.heads, n_seg), dim3(SC_COLS * L), 2 * tg * group, st, a, seg, tg);
 }
 
 static cudaError_t launch_state_groups(const StateArgs& a, const StateSegment* seg, int n_seg, const int4* groups, int n_groups, cudaStream_t st) {
-    const bool delta = a.s.rule == STATE_DELTA;
+    const int rule = a.s.rule;
     const dim3 pg(n_groups, (a.s.heads + SG_WARPS - 1) / SG_WARPS);
-    cudaError_t le = delta ? launch_pdl(state_prepare_kernel<true>, pg, dim3(SG_WARPS * 32), 0, st, a, groups) : launch_pdl(state_prepare_kernel<false>, pg, dim3(SG_WARPS * 32), 0, st, a, groups);
+    const auto prepare = rule == STATE_DELTA ? state_prepare_kernel<STATE_DELTA> : rule == STATE_FORGET ? state_prepare_kernel<STATE_FORGET> : state_prepare_kernel<STATE_DECAY>;
+    cudaError_t le = launch_pdl(prepare, pg, dim3(SG_WARPS * 32), 0, st, a, groups);
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     le = cudaErrorInvalidValue;
-#define SP_SC(L, R) le = delta ? state_scan_launch<L, R, true>(a, seg, n_seg, st) : state_scan_launch<L, R, false>(a, seg, n_seg, st)
+#define SP_SC(L, R)                                                                                                                            \
+    le = rule == STATE_DELTA ? state_scan_launch<L, R, STATE_DELTA>(a, seg, n_seg, st) : rule == STATE_FORGET ? state_scan_launch<L, R, STATE_FORGET>(a, seg, n_seg, st) \
+                                                                                                      : state_scan_launch<L, R, STATE_DECAY>(a, seg, n_seg, st)
     switch (a.s.dim_pad) {
         case 16: SP_SC(4, 1); break;
         case 32: SP_SC(8, 1); break;
@@ -589,12 +621,12 @@ cudaError_t launch_state_scan(const StateArgs& a, const StateSegment* seg, int n
     if (a.s.dim > STATE_MAX_DIM || a.s.dim_pad != state_dim_pad(a.s.dim)) return cudaErrorInvalidValue;
     cudaError_t le = a.f32 ? launch_state_groups(a, seg, n_seg, reinterpret_cast<const int4*>(groups), n_groups, st) : launch_state_chunks(a, seg, n_seg, groups, n_groups, st);
     if (le != cudaSuccess) return le;
-    const bool delta = a.s.rule == STATE_DELTA;
+    const bool each = !a.s.norm_all;
     const int group = state_group(a.f32);
-    const dim3 grid(n_groups * group, delta ? (a.s.heads + SN_WARPS - 1) / SN_WARPS : 1), block(SN_WARPS * 32);
+    const dim3 grid(n_groups * group, each ? (a.s.heads + SN_WARPS - 1) / SN_WARPS : 1), block(SN_WARPS * 32);
     const StateRecordView rec = state_view(a.s, a.f32);
 #define SP_SN(T, D) launch_pdl(state_norm_kernel<T, D>, grid, block, 0, st, a, rec, groups, group)
-    le = a.f32 ? (delta ? SP_SN(float, true) : SP_SN(float, false)) : (delta ? SP_SN(bf16, true) : SP_SN(bf16, false));
+    le = a.f32 ? (each ? SP_SN(float, true) : SP_SN(float, false)) : (each ? SP_SN(bf16, true) : SP_SN(bf16, false));
 #undef SP_SN
     return le != cudaSuccess ? le : count_launch_and_check();
 }
