@@ -284,7 +284,7 @@ def main() -> None:
     ap.add_argument("--no-batch32", action="store_true", help="skip the 32-sequence decode section")
     ap.add_argument("--no-sweep", action="store_true", help="skip the operator sweep section")
     ap.add_argument("--design", default=None, help="instead of the default workload: prefill and decode throughput of a layer-plan design "
-                    "(Lepalorn, Tedelix, Fatilix) beside the Llama block at equal size, one JSON line per size")
+                    "(Lepalorn, Tedelix, Fatilix, Revelix) beside the Llama block at equal size, one JSON line per size")
     ap.add_argument("--design-size", default=None, help="only this size")
     ap.add_argument("--design-only", action="store_true", help="without the Llama block")
     args = ap.parse_args()

@@ -35,6 +35,13 @@ FATILIX = {
     "8b": dict(layers=["attention_2", "attention"] * 2, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=18432, experts=32, top=4, groups=4, keep=2,
                expert_ff=2048, shared_ff=4096, vocab=32768, max_positions=4096, bias_max=512),
 }
+_ATTENTION = dict(conv=4, keep_first=4, vocab=32768)
+REVELIX = {
+    "2b": dict(layers=["retention", "parallel", "parallel"] * 2, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, state_heads=16, state_dim=64, state_vdim=64,
+               retention_heads=16, retention_dim=128, retention_vdim=128, window=1024, ff=6144, **_ATTENTION),
+    "8b": dict(layers=["retention", "parallel", "parallel", "retention"], width=4096, heads=32, kv_heads=8, dim=128, vdim=128, state_heads=32, state_dim=64, state_vdim=64,
+               retention_heads=32, retention_dim=128, retention_vdim=128, window=2048, ff=12288, **_ATTENTION),
+}
 
 
 def lepalorn_llama(s: dict) -> dict:
@@ -50,6 +57,12 @@ def tedelix_llama(s: dict) -> dict:
 def fatilix_llama(s: dict) -> dict:
     """Same width, heads, layers and active feed-forward weights."""
     return _llama(s, len(s["layers"]), s["kv_heads"], s["top"] * s["expert_ff"] + s["shared_ff"])
+
+
+def revelix_llama(s: dict) -> dict:
+    """Same width, heads, layers and, over all layers, feed-forward weights."""
+    ff = 2 * s["ff"] * s["layers"].count("parallel") / (3 * len(s["layers"]))
+    return _llama(s, len(s["layers"]), s["kv_heads"], round(ff / 256) * 256)
 
 
 def _llama(s: dict, layers: int, kv_heads: int, ffn: int) -> dict:
@@ -70,6 +83,11 @@ def tedelix_model(s: dict):
 def fatilix_model(s: dict):
     cfg = synth.fatilix_config(**s)
     return cfg, synth.fatilix_weights(cfg, seed=11, device="cuda")
+
+
+def revelix_model(s: dict):
+    cfg = synth.revelix_config(**s)
+    return cfg, synth.revelix_weights(cfg, seed=11, device="cuda")
 
 
 def design_engine(cfg: dict, W: dict, **kw):
@@ -157,6 +175,25 @@ def fatilix_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
             "rope_kv": (rows * (L * 6 * H * D + G * (n["attention"] * (6 * D + 4) + n["attention_2"] * 6 * (D + V))), 0)}
 
 
+def revelix_work(s: dict, rows: int, ctx: int, prefill: bool) -> dict:
+    """The same. Attention: scores, mixed weights and mixtures; states as for Tedelix; the stream's norms are part of the products."""
+    W, H, G, D, V, F = (s[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "ff"))
+    P, R = s["layers"].count("parallel"), s["layers"].count("retention")
+    hd, hv, rd, rv = (s[a] * s[b] for a, b in (("state_heads", "state_dim"), ("state_heads", "state_vdim"), ("retention_heads", "retention_dim"),
+                                               ("retention_heads", "retention_vdim")))
+    qkv = H * D + G * (D + V)
+    mats = P * (qkv + H * V + 2 * hd + 2 * hv + 2 * F) * W + R * (2 * rd + 3 * rv) * W
+    head = s["vocab"] * W
+    span = s["window"] + s["keep_first"]
+    keys = _pairs(rows, span) if prefill else rows * min(ctx, span)
+    seqs = 1 if prefill else rows
+    states = 8 * seqs * (P * hd * s["state_vdim"] + R * rd * s["retention_vdim"])
+    return {"gemv": (2 * (mats + head), 2 * rows * mats + 2 * head * (1 if prefill else rows)),
+            "attention": (P * 2 * (G * (D + V) * (rows if prefill else keys) + rows * H * (D + V)), P * 2 * H * (D + V + H) * keys),
+            "state": (states + rows * (P * (4 * (2 * hd + hv) + 2 * hv) + R * (4 * (2 * rd + 2 * rv) + 2 * rv)), 0),
+            "norm": ((1 if prefill else rows) * W * 6, 0), "rope_kv": (rows * P * 6 * qkv, 0)}
+
+
 def llama_work(c: dict, rows: int, ctx: int, prefill: bool) -> dict:
     q, kv = c["n_heads"] * c["head_dim"], c["n_kv_heads"] * c["head_dim"]
     mats = c["n_layers"] * (2 * (q + kv) * c["hidden"] + 3 * c["ffn"] * c["hidden"])
@@ -170,7 +207,8 @@ def llama_work(c: dict, rows: int, ctx: int, prefill: bool) -> dict:
 # design -> (sizes, model of a size, its work, the Llama block of equal size)
 DESIGNS = {"lepalorn": ("Lepalorn", LEPALORN, lepalorn_model, lepalorn_work, lepalorn_llama),
            "tedelix": ("Tedelix", TEDELIX, tedelix_model, tedelix_work, tedelix_llama),
-           "fatilix": ("Fatilix", FATILIX, fatilix_model, fatilix_work, fatilix_llama)}
+           "fatilix": ("Fatilix", FATILIX, fatilix_model, fatilix_work, fatilix_llama),
+           "revelix": ("Revelix", REVELIX, revelix_model, revelix_work, revelix_llama)}
 
 
 def _families(ms: dict, work: dict, peaks: dict) -> dict:

@@ -567,6 +567,75 @@ def fatilix_weights(cfg: dict, seed: int, bias_rows: int = 48, device: str = "cp
     return W
 
 
+def revelix_config(layers, width: int, heads: int, kv_heads: int, dim: int, vdim: int, state_heads: int, state_dim: int, state_vdim: int, retention_heads: int,
+                   retention_dim: int, retention_vdim: int, window: int, keep_first: int, ff: int, vocab: int, rot: int | None = None, conv: int = 4) -> dict:
+    """layers: the types in order; layers of one type are equal. Retention layers have no feed-forward."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "softcap": 50.0, "conv": conv,
+            "mask": {"size": window, "keep_first": keep_first},
+            "rot": {"base": 10000.0, "dims": dim if rot is None else rot, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mixers = {
+        "retention": {"heads": retention_heads, "dim": retention_dim, "vdim": retention_vdim, "rot": {"base": 10000.0, "dims": retention_dim},
+                      "decay": [1.0 - 2.0 ** (-5 - 5.0 * i / max(1, retention_heads - 1)) for i in range(retention_heads)]},
+        "parallel": {"left": left, "right": {"heads": state_heads, "dim": state_dim, "vdim": state_vdim}, "left_scale": 0.75, "right_scale": 0.9},
+    }
+    return {"architecture": "Revelix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "layers": [{"type": t, "mixer": dict(mixers[t]), "mlp": {"kind": "dense", "ff": ff} if t == "parallel" else None} for t in layers]}
+
+
+def revelix_weights(cfg: dict, seed: int, device: str = "cpu") -> dict:
+    """Random bf16 weights, rows scaled so that activations keep their magnitude."""
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W: dict = {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = (torch.randn(n, k, generator=g, device=device, dtype=torch.float32) * (gain * k ** -0.5)).to(torch.bfloat16)
+
+    def vec(name, n, mean=0.0, spread=0.1):
+        W[name] = (mean + spread * torch.randn(n, generator=g, device=device)).to(torch.bfloat16)
+
+    def norm(name):
+        vec(name, w, 1.0)
+        vec(name + ".b", w)
+        W[name + ".alpha"] = torch.tensor([0.5], device=device, dtype=torch.bfloat16)
+
+    w = cfg["width"]
+    mat("embed", cfg["vocab"], w, w ** 0.5)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        norm(p + "norm1")
+        if layer["type"] == "retention":
+            H, D, V = m["heads"], m["dim"], m["vdim"]
+            for n, rows in (("q", H * D), ("k", H * D), ("v", H * V), ("g", H * V)):
+                mat(p + "mix." + n, rows, w)
+            mat(p + "mix.o", w, H * V, 0.5)
+        else:
+            a, b, left, right = m["left"], m["right"], p + "mix.left.", p + "mix.right."
+            H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * V)):
+                mat(left + n, rows, w)
+                vec(left + n + ".b", rows)
+                W[left + n + ".conv"] = torch.cat([0.2 * torch.randn(rows, a["conv"] - 1, generator=g, device=device), torch.ones(rows, 1, device=device)], 1).to(torch.bfloat16)
+            W[left + "talk"] = (torch.eye(H, device=device) + 0.1 * torch.randn(H, H, generator=g, device=device)).to(torch.bfloat16)
+            vec(left + "sink", H, 0.0, 1.0)
+            mat(left + "o", w, H * V, 0.5)
+            H, D, V = b["heads"], b["dim"], b["vdim"]
+            mat(right + "q", H * D, w)
+            mat(right + "f", H * D, w)
+            vec(right + "f.b", H * D, 3.0, 1.0)
+            W[right + "lower"] = (0.9 * torch.rand(H * D, generator=g, device=device)).to(torch.bfloat16)
+            mat(right + "v", H * V, w)
+            vec(right + "norm", V, 1.0)
+            mat(right + "o", w, H * V, 0.5)
+        if layer.get("mlp"):
+            norm(p + "norm2")
+            mat(p + "mlp.up", layer["mlp"]["ff"], w)
+            mat(p + "mlp.down", w, layer["mlp"]["ff"], 0.5)
+            vec(p + "mlp.act", 2)
+    norm("final.norm")
+    return W
+
+
 def write_safetensors(path: str, cfg: dict, W: dict) -> None:
     """A model directory: config.json and model.safetensors (bf16 tensors)."""
     import json
