@@ -18,7 +18,7 @@ SOURCES = ["kernels.cu", "attention.cu", "engine.cu", "engine_forward.cu", "engi
            "attention_static.cu", "tp.cu", "gemm_tc5.cu", "gemv_ring.cu", "spec.cu", "batcher.cu", "nccl_arm.cu", "gemv_rows.cu",
            "model_plan.cu", "safetensors.cu", "engine_plan.cu", "engine_plan_post_norm.cu", "engine_plan_parallel.cu", "engine_plan_pre_norm.cu", "engine_plan_state.cu",
            "engine_plan_latent.cu", "engine_plan_grouped.cu", "mat_f32.cu", "mat_tc5.cu",
-           "plan_stream.cu", "latent_attention.cu", "grouped_attention.cu", "mixed_attention.cu", "state_mixer.cu", "state_chunk.cu"]
+           "plan_stream.cu", "latent_attention.cu", "grouped_attention.cu", "mixed_attention.cu", "grouped_conv.cu", "state_mixer.cu", "state_chunk.cu"]
 FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "--shared",

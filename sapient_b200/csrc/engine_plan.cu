@@ -297,7 +297,7 @@ int Engine::finalize_plan() {
         p.keys_at = p.has_latent ? T * (sizeof(LatentTile) / 4) : 0;
         p.grouped_at = p.keys_at + 2 * (size_t)p.keys_cap;
         p.narrow_at = p.grouped_at + (p.has_grouped ? T * (sizeof(GroupedTile) / 4) : 0);
-        p.back_at = p.narrow_at + (p.has_mixed ? T * (sizeof(GroupedTile) / 4) : 0);
+        p.back_at = p.narrow_at + (p.has_mixed || p.has_conv ? T * (sizeof(GroupedTile) / 4) : 0);
         p.ends_at = p.back_at + (p.has_conv ? T : 0);
         p.seg_at = p.ends_at + (p.has_conv ? (size_t)d.max_batch : 0);
         p.groups_at = (p.seg_at + (p.has_state ? (size_t)d.max_batch * (sizeof(StateSegment) / 4) : 0) + 3) / 4 * 4;
@@ -332,21 +332,19 @@ int Engine::plan_stage(int T) {
     p.n_tiles = p.n_keys = p.n_grouped = p.n_narrow = p.n_ends = p.n_seg = p.n_groups = 0;
     if (T <= PLAN_ROWS) return SP_OK;
     if (p.has_latent && !p.f32) plan_stage_latent(T);
-    if (p.has_grouped && !p.f32) {
-        GroupedTile *tiles = reinterpret_cast<GroupedTile*>(p.host_tiles + p.grouped_at), *narrow = reinterpret_cast<GroupedTile*>(p.host_tiles + p.narrow_at);
+    // tiles of consecutive tokens of a sequence; the longest ranges of keys first: the blocks that start last are short
+    auto tile_rows = [&](size_t at, int rows, int& count) {
+        GroupedTile* tiles = reinterpret_cast<GroupedTile*>(p.host_tiles + at);
         for (int i = 0; i < T;) {
             int n = 1;
             while (i + n < T && p_slot_[i + n] == p_slot_[i] && p_pos_[i + n] == p_pos_[i] + n) ++n;
-            for (int t = 0; t < n; t += GROUPED_Q_TILE) tiles[p.n_grouped++] = GroupedTile{i + t, std::min(GROUPED_Q_TILE, n - t), p_pos_[i] + t, p_slot_[i]};
-            if (p.has_mixed)
-                for (int t = 0; t < n; t += MIXED_Q_TILE) narrow[p.n_narrow++] = GroupedTile{i + t, std::min(MIXED_Q_TILE, n - t), p_pos_[i] + t, p_slot_[i]};
+            for (int t = 0; t < n; t += rows) tiles[count++] = GroupedTile{i + t, std::min(rows, n - t), p_pos_[i] + t, p_slot_[i]};
             i += n;
         }
-        // the longest ranges of keys first: the blocks that start last are short
-        auto later = [](const GroupedTile& a, const GroupedTile& b) { return a.pos0 > b.pos0; };
-        std::stable_sort(tiles, tiles + p.n_grouped, later);
-        std::stable_sort(narrow, narrow + p.n_narrow, later);
-    }
+        std::stable_sort(tiles, tiles + count, [](const GroupedTile& a, const GroupedTile& b) { return a.pos0 > b.pos0; });
+    };
+    if (p.has_grouped && !p.f32) tile_rows(p.grouped_at, GROUPED_Q_TILE, p.n_grouped);
+    if (p.has_conv || (p.has_mixed && !p.f32)) tile_rows(p.narrow_at, MIXED_Q_TILE, p.n_narrow);
     if (p.has_conv) {
         std::vector<int> last((size_t)d.max_batch, -1);
         for (int i = 0; i < T; ++i) {

@@ -43,6 +43,10 @@ int PlanPacker::grouped_mixer(int i, std::vector<MixPart>& all_parts) {
     l.mixed = m.talk || m.keep_first > 0 || m.score_softcap > 0 || m.out_scale != 1.f;
     if (m.vdim > GROUPED_MAX_VDIM) { fail(SP_ERR_ARG, "attention values above " + std::to_string(GROUPED_MAX_VDIM) + " coordinates are not supported"); return 0; }
     if (m.shared_values && (m.rot.dims || m.rotate_values || m.vdim != m.dim || m.conv)) { fail(SP_ERR_ARG, "keys that are the values cannot be rotated or convolved"); return 0; }
+    if (m.conv && (m.qk_norm != QK_NONE || m.temperature.coef != 0.0 || m.rotate_values)) {
+        fail(SP_ERR_ARG, "convolutions do not go with norms or temperatures of queries and keys, or with rotated values");
+        return 0;
+    }
     if (l.mixed && (m.shared_values || m.rotate_values || m.bias_max > 0 || m.out_gate)) {
         fail(SP_ERR_ARG, "mixed heads, kept first keys and capped scores do not go with distance biases, output gates or values that are rotated or the keys");
         return 0;
@@ -76,7 +80,10 @@ int PlanPacker::grouped_mixer(int i, std::vector<MixPart>& all_parts) {
             channels += (size_t)part.rows;
         }
         if (status != SP_OK) return 0;
-        in.conv = upload(all);
+        std::vector<float> by_tap(all.size());
+        for (size_t ch = 0; ch < channels; ++ch)
+            for (int j = 0; j < m.conv; ++j) by_tap[(size_t)j * channels + ch] = all[ch * (size_t)m.conv + j];
+        in.conv = upload(by_tap);
         in.taps = m.conv;
         l.tail_at = slot_floats((size_t)(m.conv - 1) * channels);
         p.has_conv = true;
@@ -143,11 +150,16 @@ int Engine::plan_grouped(int li, int T) {
         in.tail_stride = (int64_t)p.slot_state;
         in.back = T > PLAN_ROWS ? p.dev_tiles + p.back_at : nullptr;
     }
-    SP_LAUNCH(F_ROPE, launch_grouped_append(proj, l.mix_rows, s, l.kv_cache, in, d_tok_slot_, d_tok_pos_, p.q, p.f32, T, stream));
-    if (in.back) SP_LAUNCH(F_ROPE, launch_conv_tails(proj, l.mix_rows, s, in, d_tok_slot_, p.dev_tiles + p.ends_at, p.n_ends, stream));
+    if (in.conv) {
+        const GroupedTile* tiles = in.back ? (const GroupedTile*)(p.dev_tiles + p.narrow_at) : nullptr;
+        SP_LAUNCH(F_ROPE, launch_conv_append(proj, l.mix_rows, s, l.kv_cache, in, tiles, p.n_narrow, d_tok_slot_, d_tok_pos_, p.q, p.f32, T, stream));
+        if (in.back) SP_LAUNCH(F_ROPE, launch_conv_tails(proj, l.mix_rows, s, in, d_tok_slot_, p.dev_tiles + p.ends_at, p.n_ends, stream));
+    } else {
+        SP_LAUNCH(F_ROPE, launch_grouped_append(proj, l.mix_rows, s, l.kv_cache, in, d_tok_slot_, d_tok_pos_, p.q, p.f32, T, stream));
+    }
     if (l.mixed) {
-        const MixedScratch m{p.score, l.mixed_rows, l.mixed_span, p.score_part, p.stat};
-        if (p.n_narrow > 0 && T > PLAN_ROWS && !graph_step_ && mixed_mma_supported(s, l.kv_cache)) {
+        const MixedScratch m{p.score, l.mixed_rows, l.mixed_span, p.score_part, p.stat, (float*)p.stat};  // (a step uses one of the last two)
+        if (p.n_grouped > 0 && T > PLAN_ROWS && !graph_step_ && mixed_mma_supported(s, l.kv_cache)) {
             SP_LAUNCH(F_ATTN, launch_mixed_prefill(p.q, s, l.kv_cache, l.mixed_terms, m, (const GroupedTile*)(p.dev_tiles + p.grouped_at), p.n_grouped,
                                                    (const GroupedTile*)(p.dev_tiles + p.narrow_at), p.n_narrow, p.attn, l.o.kp, stream));
             return SP_OK;

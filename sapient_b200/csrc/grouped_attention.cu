@@ -4,10 +4,8 @@
 // uniform branches of the same kernels: a bias is read from a table by distance, in prompts through shared memory (a tile's
 // distances are one run of it), and is one constant for tiles that are far enough.
 #include <algorithm>
-#include <climits>
 
 #include "kernels.h"
-#include "model_plan.h"
 #include "pdl.cuh"
 #include "plan_common.cuh"
 #include "plan_kernels.h"
@@ -35,147 +33,51 @@ __device__ __forceinline__ void rotate_pairs(const Src& src, T* dst, const float
     for (int i = dims + lane; i < pad; i += 32) dst[i] = from_f32<T>(i < n ? src(i) : 0.f);
 }
 
-// A warp per (token, part): the heads' queries, then the cached heads' keys and values (shared: the keys alone). CONV: without a
-// table `back` the warp of a slot's first row takes all of the slot's rows in order and then moves the tail.
-template <typename T, bool CONV>
+// A warp per (token, part): the heads' queries, then the cached heads' keys and values (shared: the keys alone).
+template <typename T>
 __global__ void __launch_bounds__(GA_WARPS * 32) grouped_append_kernel(const float* __restrict__ proj, int ldp, const GroupedShape s, const GroupedCache c,
                                                                     const GroupedInput in, const int32_t* __restrict__ tok_slot,
                                                                     const int32_t* __restrict__ tok_pos, T* __restrict__ q) {
-    __shared__ int from_s[GA_WARPS][CONV ? CONV_MAX_TAPS : 1];
     pdl_wait();
     pdl_trigger();
-    const int part = blockIdx.y * GA_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int t = blockIdx.x, part = blockIdx.y * GA_WARPS + (threadIdx.x >> 5), pos = tok_pos[t], lane = threadIdx.x & 31;
     const bool query = part < s.heads;
     const int per = c.shared ? 1 : 2, g = query ? 0 : (part - s.heads) / per;
     if (g >= s.kv_heads) return;
     const bool value = !query && (part - s.heads) % per == 1;
     const int n = value ? s.vdim : s.dim;
     const int64_t at = query ? (int64_t)part * s.dim : value ? (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)g * s.vdim : (int64_t)(s.heads + g) * s.dim;
+    const float* pr = proj + (int64_t)t * ldp + at;
     const float* bias = in.bias ? in.bias + at : nullptr;
-    const int slot = tok_slot[blockIdx.x];
-    auto biased = [&](int row, int i) {
-        const float v = proj[(int64_t)row * ldp + at + i];
-        return bias ? v + bias[i] : v;
+    auto projected = [&](int i) { return bias ? pr[i] + bias[i] : pr[i]; };
+    float r = 1.f;
+    if (in.norm && !value) {
+        float ss = 0.f;
+        for (int i = lane; i < n; i += 32) {
+            const float v = projected(i);
+            ss = fmaf(v, v, ss);
+        }
+        r = rsqrtf(warp_sum(ss) / (float)n + in.eps);
+    }
+    const float2* ck = in.cs_key ? in.cs_key + (int64_t)pos * (s.rot / 2) : nullptr;
+    auto normed = [&](const float* gain, float mult) {
+        return [=](int i) { return gain ? projected(i) * mult * gain[i] : projected(i) * mult; };
     };
-    // CONV: where the value d tokens back is: a row, -1 - (place in the tail), or nowhere
-    constexpr int NOWHERE = INT_MIN;
-    int* const from = from_s[threadIdx.x >> 5];
-    float* const tail = CONV ? in.tail + slot * in.tail_stride + at : nullptr;
-    const int channels = (s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim;
-    auto earlier = [&](int r, int i) { return r >= 0 ? biased(r, i) : tail[(int64_t)(-1 - r) * channels + i]; };
-
-    // row t; `before`: rows of its slot that come before it (without a table)
-    auto append = [&](int t, uint32_t before) {
-        const int pos = tok_pos[t];
-        if (CONV) {
-            __syncwarp();
-            if (lane == 0) {
-                int k = __popc(before), r = t;  // rows of the slot before this one
-                if (in.back)
-                    for (int b = in.back[t]; b >= 0 && k < in.taps; b = in.back[b]) ++k;
-                for (int d = 0; d < in.taps; ++d) {
-                    from[d] = pos < d ? NOWHERE : d <= k ? r : -1 - (in.taps - 1 + k - d);
-                    if (d >= k) continue;
-                    r = in.back ? in.back[r] : 31 - __clz(before);
-                    before &= ~(1u << (r & 31));
-                }
-            }
-            __syncwarp();
-        }
-        auto projected = [&](int i) {
-            if (!CONV) return biased(t, i);
-            const float* w = in.conv + (at + i) * in.taps + in.taps - 1;
-            float v = 0.f;
-            for (int d = in.taps - 1; d >= 0; --d)
-                if (from[d] != NOWHERE) v = fmaf(w[-d], earlier(from[d], i), v);
-            return v;
-        };
-        float r = 1.f;
-        if (in.norm && !value) {
-            float ss = 0.f;
-            for (int i = lane; i < n; i += 32) {
-                const float v = projected(i);
-                ss = fmaf(v, v, ss);
-            }
-            r = rsqrtf(warp_sum(ss) / (float)n + in.eps);
-        }
-        const float2* ck = in.cs_key ? in.cs_key + (int64_t)pos * (s.rot / 2) : nullptr;
-        auto normed = [&](const float* gain, float mult) {
-            return [=](int i) { return gain ? projected(i) * mult * gain[i] : projected(i) * mult; };
-        };
-        if (query) {
-            if (in.temperature) r *= in.temperature[pos];
-            rotate_pairs<T>(normed(in.q_gain, r), q + ((int64_t)t * s.heads + part) * c.dim16, ck, s.rot, s.neighbours, s.dim, c.dim16);
-            return;
-        }
-        const int page = c.page_table[(int64_t)slot * c.max_pages + pos / KV_PAGE];
-        T* row = reinterpret_cast<T*>(c.pool) + (((int64_t)page * s.kv_heads + g) * KV_PAGE + pos % KV_PAGE) * c.ld;
-        if (c.shared) {
-            rotate_pairs<T>(projected, row, nullptr, 0, false, n, c.dim16);
-            if (lane == 0) *reinterpret_cast<float*>(row + c.dim16) = r;
-        } else if (value) {
-            rotate_pairs<T>(projected, row + c.dim16, in.cs_val ? in.cs_val + (int64_t)pos * (s.vdim / 2) : nullptr, in.cs_val ? s.vdim : 0, false, n, c.vdim16);
-        } else {
-            rotate_pairs<T>(normed(in.k_gain, r), row, ck, s.rot, s.neighbours, n, c.dim16);
-        }
-    };
-    if (!CONV || in.back) {
-        append(blockIdx.x, 0u);
+    if (query) {
+        if (in.temperature) r *= in.temperature[pos];
+        rotate_pairs<T>(normed(in.q_gain, r), q + ((int64_t)t * s.heads + part) * c.dim16, ck, s.rot, s.neighbours, s.dim, c.dim16);
         return;
     }
-    const uint32_t rows = __ballot_sync(0xFFFFFFFFu, lane < (int)gridDim.x && tok_slot[min(lane, (int)gridDim.x - 1)] == slot);
-    if (rows & ((1u << blockIdx.x) - 1)) return;
-    for (uint32_t left = rows; left; left &= left - 1) {
-        const int t = __ffs(left) - 1;
-        append(t, rows & ((1u << t) - 1));
+    const int page = c.page_table[(int64_t)tok_slot[t] * c.max_pages + pos / KV_PAGE];
+    T* row = reinterpret_cast<T*>(c.pool) + (((int64_t)page * s.kv_heads + g) * KV_PAGE + pos % KV_PAGE) * c.ld;
+    if (c.shared) {
+        rotate_pairs<T>(projected, row, nullptr, 0, false, n, c.dim16);
+        if (lane == 0) *reinterpret_cast<float*>(row + c.dim16) = r;
+    } else if (value) {
+        rotate_pairs<T>(projected, row + c.dim16, in.cs_val ? in.cs_val + (int64_t)pos * (s.vdim / 2) : nullptr, in.cs_val ? s.vdim : 0, false, n, c.vdim16);
+    } else {
+        rotate_pairs<T>(normed(in.k_gain, r), row, ck, s.rot, s.neighbours, n, c.dim16);
     }
-    // every lane moves its channels, the oldest place first: what it reads stands behind what it writes
-    __syncwarp();
-    for (int i = lane; i < n; i += 32)
-        for (int j = 0; j < in.taps - 1; ++j) {
-            const int r = from[in.taps - 2 - j];  // as the last row saw them
-            if (r != NOWHERE) tail[(int64_t)j * channels + i] = earlier(r, i);
-        }
-}
-
-// A thread per channel of a slot whose last row in the step is ends[blockIdx.y].
-constexpr int CT_THREADS = 128;
-__global__ void __launch_bounds__(CT_THREADS) conv_tails_kernel(const float* __restrict__ proj, int ldp, int channels, const GroupedInput in,
-                                                             const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ ends) {
-    __shared__ int rows[CONV_MAX_TAPS];  // the slot's last rows, the newest first
-    pdl_wait();
-    pdl_trigger();
-    const int end = ends[blockIdx.y], i = blockIdx.x * CT_THREADS + threadIdx.x, keep = in.taps - 1;
-    if (threadIdx.x == 0)
-        for (int d = 0, r = end; d < keep; ++d) {
-            rows[d] = r;
-            if (r >= 0) r = in.back[r];
-        }
-    __syncthreads();
-    if (i >= channels) return;
-    int n = 0;
-    while (n < keep && rows[n] >= 0) ++n;
-    float* const tail = in.tail + tok_slot[end] * in.tail_stride + i;
-    for (int j = 0; j < keep; ++j) {
-        const int d = keep - 1 - j;
-        float v;
-        if (d < n) {
-            v = proj[(int64_t)rows[d] * ldp + i];
-            if (in.bias) v += in.bias[i];
-        } else {
-            v = tail[(int64_t)(j + n) * channels];
-        }
-        tail[(int64_t)j * channels] = v;
-    }
-}
-
-cudaError_t launch_conv_tails(const float* proj, int ldp, const GroupedShape& s, const GroupedInput& in, const int32_t* tok_slot, const int32_t* ends,
-                              int n_ends, cudaStream_t st) {
-    if (n_ends == 0 || in.taps <= 1) return cudaSuccess;
-    if (!in.conv || in.taps > CONV_MAX_TAPS || !in.back) return cudaErrorInvalidValue;
-    const int channels = (s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim;
-    const cudaError_t le = launch_pdl(conv_tails_kernel, dim3((channels + CT_THREADS - 1) / CT_THREADS, n_ends), dim3(CT_THREADS), 0, st, proj, ldp, channels, in, tok_slot, ends);
-    return le != cudaSuccess ? le : count_launch_and_check();
 }
 
 cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in,
@@ -183,10 +85,9 @@ cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape
     if (n_tok == 0) return cudaSuccess;
     if (c.shared && (s.rot || in.cs_val || in.k_gain || s.dim != s.vdim)) return cudaErrorInvalidValue;
     const dim3 grid(n_tok, (s.heads + (c.shared ? 1 : 2) * s.kv_heads + GA_WARPS - 1) / GA_WARPS), block(GA_WARPS * 32);
-    if (in.conv && (c.shared || in.taps < 1 || in.taps > CONV_MAX_TAPS || (!in.back && n_tok > 32))) return cudaErrorInvalidValue;
-#define SP_GA(T, CONV) launch_pdl(grouped_append_kernel<T, CONV>, grid, block, 0, st, proj, ldp, s, c, in, tok_slot, tok_pos, (T*)q)
-    const cudaError_t le = f32 ? (in.conv ? SP_GA(float, true) : SP_GA(float, false)) : (in.conv ? SP_GA(bf16, true) : SP_GA(bf16, false));
-#undef SP_GA
+    if (in.conv) return cudaErrorInvalidValue;
+    const cudaError_t le = f32 ? launch_pdl(grouped_append_kernel<float>, grid, block, 0, st, proj, ldp, s, c, in, tok_slot, tok_pos, (float*)q)
+                               : launch_pdl(grouped_append_kernel<bf16>, grid, block, 0, st, proj, ldp, s, c, in, tok_slot, tok_pos, (bf16*)q);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 

@@ -215,8 +215,7 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
             on = reinterpret_cast<bf16*>(a.norm.y) + n;
         }
         auto held = [&](int row) { return add ? of[row * oldd] : 0.f; };
-        auto put = [&](int row, float f, float before) {
-            f = mat_act(act, f, a.arg);
+        auto put = [&](int row, float f, float before) {  // (f has been through the activation)
             if (NORM) {
                 f += before;
                 of[row * oldd] = f;
@@ -244,12 +243,16 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
                     }
                 } else if (OUTS) {
                     if (n < s.n) {
-                        float before[16];
+                        float before[16], f[16];
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) before[j] = c + j < cols ? held(r0 + c + j) : 0.f;
+                        for (int j = 0; j < 16; ++j) {
+                            before[j] = c + j < cols ? held(r0 + c + j) : 0.f;
+                            f[j] = __uint_as_float(v[j]);
+                        }
+                        if (!NORM) mat_act_fast(act, f, a.arg);
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
-                            if (c + j < cols) put(r0 + c + j, __uint_as_float(v[j]), before[j]);
+                            if (c + j < cols) put(r0 + c + j, f[j], before[j]);
                     }
                 } else if (n < s.n) {
                     if (by_index || a.gate || c + 16 > cols) {
@@ -302,6 +305,7 @@ __global__ void __launch_bounds__(MT_THREADS, 2) mat_tc5_kernel(const MatTc5Args
                             if (DUAL) up[j] += ld_peer(peer + (uint32_t)(a.bn + c) * MT_BM * 4);
                         }
                     }
+                    if (OUTS && !NORM) mat_act_fast(act, f, a.arg);
 #pragma unroll
                     for (int j = 0; j < NC; ++j)
                         if (row[j] >= 0) {

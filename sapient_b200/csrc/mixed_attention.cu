@@ -1,6 +1,6 @@
 // Grouped attention whose heads' softmax weights are mixed before they meet the values (plan_kernels.h). A head's mixture needs the
 // normalised weights of all heads, so scores and denominators come first, weights and values second:
-//   few rows    scores_kernel leaves scores and, per split of the keys, maximum and sum; mix_kernel makes the weights of all heads
+//   few rows    scores_kernel leaves scores (in powers of two, below their cap) and, per split of the keys, maximum and sum; mix_kernel makes the weights of all heads
 //               where it needs them, mixes them as a small product (16 output heads x heads x keys) whose accumulators are the A
 //               operand of the product with the values, and adds the splits' shares over a cluster.
 //   many rows   stats_kernel walks the keys of 64 query rows per head; prefill_kernel has 16 query rows of all heads (a cluster
@@ -38,20 +38,41 @@ int mixed_span(const GroupedShape& s, int max_ctx) {
     return (int)((std::min<int64_t>(window, max_ctx) + KV_PAGE - 1) / KV_PAGE * KV_PAGE);
 }
 
-// The scaled and capped score of a dot product, and the tensor-core kernels' version: tanh z = 1 - 2 / (e^(2 z) + 1), whose error
-// is absolute, as softmax needs it.
+// The scaled and capped score of a dot product.
 __device__ __forceinline__ float score_of(const GroupedShape& s, float dot) {
     const float z = dot * s.scale;
     return s.softcap > 0.f ? s.softcap * tanhf(z / s.softcap) : z;
 }
-struct FastScore {
-    float scale, cap;
-    __device__ __forceinline__ explicit FastScore(const GroupedShape& s) : scale(s.softcap > 0.f ? 2.f * s.scale / s.softcap : s.scale), cap(s.softcap) {}
-    __device__ __forceinline__ float operator()(float dot) const {
-        const float z = dot * scale;
-        return cap > 0.f ? fmaf(-2.f * cap, __fdividef(1.f, __expf(z) + 1.f), cap) : z;
+// The tensor-core kernels' version, in powers of two: log2 e^(score - top), where top is the cap (no cap: 0). tanh z = 1 - 2 / (e^(2 z) + 1)
+// has an absolute error, as softmax needs it.
+constexpr float LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+struct Log2Score {
+    float a, b, top;
+    bool cap;
+    __device__ __forceinline__ explicit Log2Score(const GroupedShape& s) : cap(s.softcap > 0.f) {
+        a = cap ? 2.f * s.scale / s.softcap * LOG2E : s.scale * LOG2E;
+        b = -2.f * s.softcap * LOG2E;
+        top = cap ? s.softcap : 0.f;
+    }
+    __device__ __forceinline__ float operator()(float dot, float more) const {  // ... plus `more`
+        return cap ? fmaf(b, rcp_fast(exp2_fast(dot * a) + 1.f), more) : fmaf(dot, a, more);
     }
 };
+// What to add to a log2 score for its normalised weight: maximum and sum of the keys, and the sink.
+__device__ __forceinline__ float log2_norm(float m, float l, float sink) {
+    const float M = fmaxf(m, sink);
+    return -M - log2f(l * exp2f(m - M) + exp2f(sink - M));
+}
 
 __device__ __forceinline__ float2 stat_of(float m, float l, const float* sink, int h) {  // maximum, 1 / denominator
     if (sink) {
@@ -201,8 +222,8 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16*
 #pragma unroll
     for (int i = 0; i < MD_STAGES; ++i) fetch(v0 + i * stride, i);
     __syncthreads();
-    const FastScore score(s);
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const Log2Score score(s);
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // maxima in powers of two, from the top
     const uint32_t qa = smem_addr(qs + (lane & 15) * LD + (lane >> 4) * 8);
     float* const out = m.score + ((int64_t)t * s.heads + h0) * m.span;
     for (int v = v0, st = 0; v < vis.pages; v += stride, st = st + 1 == MD_STAGES ? 0 : st + 1) {
@@ -226,8 +247,8 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16*
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const bool on = visible(s, key0 + 8 * j + 2 * tq + e, pos);
-                sc[j][e] = on ? score(sc[j][e]) : -INFINITY;
-                sc[j][2 + e] = on ? score(sc[j][2 + e]) : -INFINITY;
+                sc[j][e] = on ? score(sc[j][e], 0.f) : -INFINITY;
+                sc[j][2 + e] = on ? score(sc[j][2 + e], 0.f) : -INFINITY;
                 x0 = fmaxf(x0, sc[j][e]);
                 x1 = fmaxf(x1, sc[j][2 + e]);
             }
@@ -237,8 +258,8 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16*
         }
         // (a thread's own maxima: its quad meets at the end; kept pages may show a thread nothing)
         const float b0 = x0 == -INFINITY ? 0.f : x0, b1 = x1 == -INFINITY ? 0.f : x1;
-        l0 = l0 * expf(m0 - b0) + expf(sc[0][0] - b0) + expf(sc[0][1] - b0) + expf(sc[1][0] - b0) + expf(sc[1][1] - b0);
-        l1 = l1 * expf(m1 - b1) + expf(sc[0][2] - b1) + expf(sc[0][3] - b1) + expf(sc[1][2] - b1) + expf(sc[1][3] - b1);
+        l0 = l0 * exp2_fast(m0 - b0) + exp2_fast(sc[0][0] - b0) + exp2_fast(sc[0][1] - b0) + exp2_fast(sc[1][0] - b0) + exp2_fast(sc[1][1] - b0);
+        l1 = l1 * exp2_fast(m1 - b1) + exp2_fast(sc[0][2] - b1) + exp2_fast(sc[0][3] - b1) + exp2_fast(sc[1][2] - b1) + exp2_fast(sc[1][3] - b1);
         m0 = x0;
         m1 = x1;
         __syncwarp();  // the stage has been read
@@ -247,7 +268,7 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16*
     cp_async_wait<0>();
     auto meet = [](float& a, float& b, float om, float ol) {  // (maximum, sum) of two parts
         const float M = fmaxf(a, om), base = M == -INFINITY ? 0.f : M;
-        b = b * expf(a - base) + ol * expf(om - base);
+        b = b * exp2_fast(a - base) + ol * exp2_fast(om - base);
         a = M;
     };
 #pragma unroll
@@ -274,7 +295,7 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_scores_kernel(const bf16*
 // rows of the mixing matrix (leading part, remainder), the ring of values, where the shares meet at the end.
 __host__ __device__ __forceinline__ int md_heads16(const GroupedShape& s) { return (s.heads + 15) & ~15; }
 static size_t md_mix_smem(const GroupedShape& s, const GroupedCache& c) {
-    const size_t head = (size_t)md_heads16(s) * 8 + (size_t)2 * 16 * (md_heads16(s) + 8) * 2;
+    const size_t head = (size_t)md_heads16(s) * 4 + (size_t)2 * 16 * (md_heads16(s) + 8) * 2;
     return head + std::max((size_t)MD_WARPS * MD_STAGES * KV_PAGE * (c.vdim16 + 8) * 2, (size_t)MD_WARPS * 16 * (c.vdim16 + 4) * 4);
 }
 
@@ -286,8 +307,8 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_mix_kernel(const GroupedS
     const int H16 = md_heads16(s), LT = H16 + 8, LV = c.vdim16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int group = s.heads / s.kv_heads, tiles = (group + 15) / 16, kvh = blockIdx.x / tiles, h0 = kvh * group + (blockIdx.x % tiles) * 16;
     const int nq = min(16, (kvh + 1) * group - h0), t = blockIdx.y;
-    float2* const stat = reinterpret_cast<float2*>(mm_sm);
-    bf16 *t_hi = reinterpret_cast<bf16*>(stat + H16), *t_lo = t_hi + 16 * LT, *rings = t_lo + 16 * LT, *ring = rings + warp * MD_STAGES * KV_PAGE * LV;
+    float* const norm = reinterpret_cast<float*>(mm_sm);  // what makes a head's score its weight, in powers of two
+    bf16 *t_hi = reinterpret_cast<bf16*>(norm + H16), *t_lo = t_hi + 16 * LT, *rings = t_lo + 16 * LT, *ring = rings + warp * MD_STAGES * KV_PAGE * LV;
     for (int i = tid; i < 16 * H16; i += MD_WARPS * 32) {  // (no kernel writes the mixing matrix)
         const int r = i / H16, e = i - r * H16;
         const float v = r < nq && e < s.heads ? x.mix[(int64_t)(h0 + r) * s.heads + e] : 0.f;
@@ -311,15 +332,15 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_mix_kernel(const GroupedS
 #pragma unroll
     for (int i = 0; i < MD_STAGES; ++i) fetch(v0 + i * stride, i);
     for (int h = tid; h < H16; h += MD_WARPS * 32) {
-        float2 r = make_float2(INFINITY, 0.f);  // heads that do not exist weigh nothing
+        float r = -INFINITY;  // heads that do not exist weigh nothing
         if (h < s.heads) {
             const float2* p = m.part + ((int64_t)t * s.heads + h) * MIXED_SPLITS;
             float M = -INFINITY, L = 0.f;
             for (int i = 0; i < n_splits; ++i) M = fmaxf(M, p[i].x);
-            for (int i = 0; i < n_splits; ++i) L += p[i].x == -INFINITY ? 0.f : p[i].y * expf(p[i].x - M);
-            r = stat_of(M, L, x.sink, h);
+            for (int i = 0; i < n_splits; ++i) L += p[i].x == -INFINITY ? 0.f : p[i].y * exp2f(p[i].x - M);
+            r = log2_norm(M, L, x.sink ? (x.sink[h] - Log2Score(s).top) * LOG2E : -INFINITY);
         }
-        stat[h] = r;
+        norm[h] = r;
     }
     __syncthreads();
     float o[VT][4];
@@ -335,10 +356,10 @@ __global__ void __launch_bounds__(MD_WARPS * 32) mixed_mix_kernel(const GroupedS
             for (int j = 0; j < 2; ++j)
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
-                    const int e0 = k + 8 * i + 2 * tq, e1 = min(e0 + 1, s.heads - 1);
+                    const int e0 = k + 8 * i + 2 * tq;
                     const float* d = score + v * KV_PAGE + 8 * j + g;
-                    const float2 s0 = stat[e0], s1 = stat[e0 + 1];
-                    const float w0 = expf(d[(int64_t)min(e0, s.heads - 1) * m.span] - s0.x) * s0.y, w1 = expf(d[(int64_t)e1 * m.span] - s1.x) * s1.y;
+                    const float w0 = exp2_fast(d[(int64_t)min(e0, s.heads - 1) * m.span] + norm[e0]);
+                    const float w1 = exp2_fast(d[(int64_t)min(e0 + 1, s.heads - 1) * m.span] + norm[e0 + 1]);
                     hi[j][i] = pack_bf16(w0, w1);
                     const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi[j][i]));
                     lw[j][i] = pack_bf16(w0 - back.x, w1 - back.y);
@@ -466,7 +487,10 @@ cudaError_t launch_mixed_attention(const void* q, const GroupedShape& s, const G
 
 // ── many rows: denominators ──
 // Block per (head, tile of 64 tokens), 4 warps x 16 query rows, key tiles of four visited pages, double-buffered.
+// CAPPED: the cap is low enough to stand for the maximum.
 constexpr int MT_KEYS = 64, MT_WARPS = 4;
+constexpr float MT_CAP = 40.f;  // e^(-2 * 40) is a normal float
+template <bool CAPPED>
 __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
                                                                  const MixedScratch m, const GroupedTile* __restrict__ tiles) {
     extern __shared__ __align__(16) bf16 mt_sm[];
@@ -498,8 +522,8 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
     };
     fetch(0, 0);
     cp_async_commit();
-    const FastScore score(s);
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const Log2Score score(s);
+    float m0 = CAPPED ? 0.f : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
     const int r0 = warp * 16 + g, r1 = r0 + 8, p0 = tl.pos0 + min(r0, tl.n - 1), p1 = tl.pos0 + min(r1, tl.n - 1);
     for (int v0 = 0, buf = 0; v0 < vis.pages; v0 += MT_KEYS / KV_PAGE, buf ^= 1) {
         cp_async_wait<0>();
@@ -523,34 +547,52 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
                 mma_bf16(sc[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
         }
-        float x0 = m0, x1 = m1;
+        // a run of pages that all rows see whole needs no mask
+        const int first = vis.page(v0) * KV_PAGE, last = vis.page(min(v0 + MT_KEYS / KV_PAGE, vis.pages) - 1) * KV_PAGE + KV_PAGE - 1;
+        const bool whole = v0 + MT_KEYS / KV_PAGE <= vis.pages && last <= tl.pos0 && (hi - first < s.window || last < s.keep);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const int v = v0 + j / 2, key0 = vis.page(min(v, vis.pages - 1)) * KV_PAGE + 8 * (j & 1) + 2 * tq;
+        for (int j = 0; j < 8; ++j)
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                sc[j][e] = v < vis.pages && visible(s, key0 + e, p0) ? score(sc[j][e]) : -INFINITY;
-                sc[j][2 + e] = v < vis.pages && visible(s, key0 + e, p1) ? score(sc[j][2 + e]) : -INFINITY;
-                x0 = fmaxf(x0, sc[j][e]);
-                x1 = fmaxf(x1, sc[j][2 + e]);
+            for (int e = 0; e < 4; ++e) sc[j][e] = score(sc[j][e], 0.f);
+        if (!whole) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const int v = v0 + j / 2, key0 = vis.page(min(v, vis.pages - 1)) * KV_PAGE + 8 * (j & 1) + 2 * tq;
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    if (v >= vis.pages || !visible(s, key0 + e, p0)) sc[j][e] = -INFINITY;
+                    if (v >= vis.pages || !visible(s, key0 + e, p1)) sc[j][2 + e] = -INFINITY;
+                }
             }
         }
+        float b0 = 0.f, b1 = 0.f;
+        if (!CAPPED) {
+            float x0 = m0, x1 = m1;
 #pragma unroll
-        for (int off = 1; off < 4; off <<= 1) {
-            x0 = fmaxf(x0, __shfl_xor_sync(0xFFFFFFFFu, x0, off));
-            x1 = fmaxf(x1, __shfl_xor_sync(0xFFFFFFFFu, x1, off));
+            for (int j = 0; j < 8; ++j) {
+                x0 = fmaxf(x0, fmaxf(sc[j][0], sc[j][1]));
+                x1 = fmaxf(x1, fmaxf(sc[j][2], sc[j][3]));
+            }
+#pragma unroll
+            for (int off = 1; off < 4; off <<= 1) {
+                x0 = fmaxf(x0, __shfl_xor_sync(0xFFFFFFFFu, x0, off));
+                x1 = fmaxf(x1, __shfl_xor_sync(0xFFFFFFFFu, x1, off));
+            }
+            b0 = x0 == -INFINITY ? 0.f : x0;
+            b1 = x1 == -INFINITY ? 0.f : x1;
+            l0 *= exp2_fast(m0 - b0);
+            l1 *= exp2_fast(m1 - b1);
+            m0 = x0;
+            m1 = x1;
         }
-        const float b0 = x0 == -INFINITY ? 0.f : x0, b1 = x1 == -INFINITY ? 0.f : x1;
         float s0 = 0.f, s1 = 0.f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            s0 += __expf(sc[j][0] - b0) + __expf(sc[j][1] - b0);
-            s1 += __expf(sc[j][2] - b1) + __expf(sc[j][3] - b1);
+            s0 += exp2_fast(sc[j][0] - b0) + exp2_fast(sc[j][1] - b0);
+            s1 += exp2_fast(sc[j][2] - b1) + exp2_fast(sc[j][3] - b1);
         }
-        l0 = fmaf(l0, expf(m0 - b0), s0);
-        l1 = fmaf(l1, expf(m1 - b1), s1);
-        m0 = x0;
-        m1 = x1;
+        l0 += s0;
+        l1 += s1;
     }
     cp_async_wait<0>();
 #pragma unroll
@@ -559,8 +601,9 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
         l1 += __shfl_xor_sync(0xFFFFFFFFu, l1, off);
     }
     if (tq == 0) {
-        if (r0 < tl.n) m.stat[(int64_t)(tl.row0 + r0) * s.heads + h] = stat_of(m0, l0, x.sink, h);
-        if (r1 < tl.n) m.stat[(int64_t)(tl.row0 + r1) * s.heads + h] = stat_of(m1, l1, x.sink, h);
+        const float sink = x.sink ? (x.sink[h] - score.top) * LOG2E : -INFINITY;
+        if (r0 < tl.n) m.norm[(int64_t)(tl.row0 + r0) * s.heads + h] = log2_norm(m0, l0, sink);
+        if (r1 < tl.n) m.norm[(int64_t)(tl.row0 + r1) * s.heads + h] = log2_norm(m1, l1, sink);
     }
 }
 
@@ -568,7 +611,7 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 // Block (cluster rank: a run of 8 HPW heads, tile of 16 tokens), a warp per HPW heads. Per page of keys: weights of the block's
 // heads into every block's shared memory, one barrier, then each warp mixes for its heads and multiplies with the values. Keys are
 // two stages ahead of the barrier, values one; weights alternate between two buffers. A thread's four keys of the A operand are
-// neighbours, so that it reads a head's weights as one float4; the values' rows are numbered the same way.
+// neighbours, so that it reads a head's weights as one vector; the values' rows are numbered the same way.
 constexpr int MP_WARPS = 8, MP_MAX_CLUSTER = 8, MP_CAP = 224 * 1024;
 struct MixedTiling {
     int heads, kv, cluster;    // heads of a block, cached heads they touch at most, blocks
@@ -579,23 +622,21 @@ __host__ __device__ __forceinline__ MixedTiling mp_tiling(const GroupedShape& s,
     MixedTiling t;
     const int group = s.heads / s.kv_heads;
     t.heads = MP_WARPS * hpw < s.heads ? MP_WARPS * hpw : s.heads;
-    t.cluster = (s.heads + t.heads - 1) / t.heads;
+    t.cluster = 1;
+    while (t.cluster * t.heads < s.heads) t.cluster <<= 1;
     const int touched = (t.heads + group - 2) / group + 1;  // a run may begin inside a group
     t.kv = t.heads % group == 0 || group % t.heads == 0 ? (t.heads + group - 1) / group : touched < s.kv_heads ? touched : s.kv_heads;
-    int cl = 1;
-    while (cl < t.cluster) cl <<= 1;
-    t.cluster = cl;
     t.q = 0;
     t.k = t.q + MP_WARPS * hpw * 16 * (c.dim16 + 8) * 2;
     t.v = t.k + 2 * t.kv * KV_PAGE * (c.dim16 + 8) * 2;
     t.w = t.v + 2 * t.kv * KV_PAGE * (c.vdim16 + 8) * 2;
     t.mix = t.w + 2 * s.heads * 16 * KV_PAGE * 4;
-    t.smem = (size_t)t.mix + (size_t)MP_WARPS * hpw * s.heads * 4;
+    t.smem = (size_t)t.mix + (size_t)MP_WARPS * hpw * s.heads * 8;
     return t;
 }
 static int mp_heads_per_warp(const GroupedShape& s, const GroupedCache& c) {  // 0: not covered
     if (s.dim > 256 || s.vdim > 256) return 0;
-    for (int hpw = c.vdim16 <= 128 && s.heads > MP_WARPS ? 2 : 1; hpw > 0; --hpw) {
+    for (int hpw = 1; hpw <= (c.vdim16 <= 128 ? 2 : 1); ++hpw) {
         const MixedTiling t = mp_tiling(s, c, hpw);
         if (t.cluster <= MP_MAX_CLUSTER && t.smem <= MP_CAP) return hpw;
     }
@@ -605,10 +646,16 @@ static int mp_heads_per_warp(const GroupedShape& s, const GroupedCache& c) {  //
 __device__ __forceinline__ void st_peer(uint32_t addr, float a, float b) {
     asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};\n" ::"r"(addr), "f"(a), "f"(b) : "memory");
 }
+// Two floats in a register pair: d += a * b.
+__device__ __forceinline__ void fma_pair(unsigned long long& d, unsigned long long a, unsigned long long b) {
+    asm("fma.rn.f32x2 %0, %1, %2, %0;\n" : "+l"(d) : "l"(a), "l"(b));
+}
+__device__ __forceinline__ float2 pair_of(unsigned long long v) { return make_float2(__uint_as_float((uint32_t)v), __uint_as_float((uint32_t)(v >> 32))); }
 
 template <int VT, int HPW>
-__global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
-                                                                      const MixedScratch m, const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
+__global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
+    mixed_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
+                         const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) uint8_t mp_sm[];
     const MixedTiling tg = mp_tiling(s, c, HPW);
     const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, H = s.heads, group = H / s.kv_heads;
@@ -616,11 +663,11 @@ __global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const b
     const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
     const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
     const uint32_t sm = smem_addr(mp_sm);
-    float* const ws = reinterpret_cast<float*>(mp_sm + tg.w);    // [2][head][16 rows][16 keys]
-    float* const mix = reinterpret_cast<float*>(mp_sm + tg.mix); // [warp][head][HPW]
+    float2* const mix = reinterpret_cast<float2*>(mp_sm + tg.mix);  // [warp][head][HPW], twice side by side
     for (int i = tid; i < MP_WARPS * HPW * H; i += MP_WARPS * 32) {
         const int hh = i % HPW, e = i / HPW % H, h = i / HPW / H * HPW + hh;
-        mix[i] = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
+        const float f = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
+        mix[i] = make_float2(f, f);
     }
     pdl_wait();
     pdl_trigger();
@@ -628,15 +675,18 @@ __global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const b
     const int hi = tl.pos0 + tl.n - 1;
     const Visit vis(s, tl.pos0, hi);
     const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages;
-    auto fetch = [&](int v, int stage, int col, int width, int base, int ld) {
-        if (v < vis.pages)
-            for (int i = warp; i < nkv; i += MP_WARPS) {
-                const int page = vis.page(v);
-                fetch_page(c, s.kv_heads, kv0 + i, pt[page], hi - page * KV_PAGE + 1, col, width, sm + (uint32_t)(base + ((stage * tg.kv + i) * KV_PAGE * ld) * 2), ld, lane, 32);
-            }
+    // half a warp per row, the rows of all cached heads spread over the block
+    auto fetch = [&](int v, int col, int width, int base, int ld) {
+        if (v >= vis.pages) return;
+        const int page = vis.page(v), live = hi - page * KV_PAGE + 1, half = tid >> 4, l16 = tid & 15;
+        const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[page] * s.kv_heads + kv0) * KV_PAGE * c.ld + col;
+        const uint32_t dst = sm + (uint32_t)(base + (v & 1) * tg.kv * KV_PAGE * ld * 2);
+        for (int row = half; row < nkv * KV_PAGE; row += MP_WARPS * 2)
+            for (int p = l16; p < width / 8; p += 16)
+                cp_async16_at(dst + (uint32_t)(row * ld + p * 8) * 2, src + (int64_t)row * c.ld + p * 8, row % KV_PAGE < live ? 16 : 0);
     };
-    auto fetch_k = [&](int v) { fetch(v, v & 1, 0, c.dim16, tg.k, LQ); };
-    auto fetch_v = [&](int v) { fetch(v, v & 1, c.dim16, c.vdim16, tg.v, LV); };
+    auto fetch_k = [&](int v) { fetch(v, 0, c.dim16, tg.k, LQ); };
+    auto fetch_v = [&](int v) { fetch(v, c.dim16, c.vdim16, tg.v, LV); };
     for (int i = warp; i < nh * 16; i += MP_WARPS) {
         const int h = i / 16, r = i % 16;
         const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * H + h0 + h) * c.dim16;
@@ -645,12 +695,12 @@ __global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const b
     fetch_k(0);
     cp_async_commit();
     const int ra = min(g, tl.n - 1), rb = min(g + 8, tl.n - 1), pa = tl.pos0 + ra, pb = tl.pos0 + rb;
-    float2 sa[HPW], sb[HPW];
+    float na[HPW], nb[HPW];  // of the two rows: what makes a score a weight
 #pragma unroll
     for (int j = 0; j < HPW; ++j) {
         const int h = min(h0 + warp * HPW + j, H - 1);
-        sa[j] = m.stat[(int64_t)(tl.row0 + ra) * H + h];
-        sb[j] = m.stat[(int64_t)(tl.row0 + rb) * H + h];
+        na[j] = m.norm[(int64_t)(tl.row0 + ra) * H + h];
+        nb[j] = m.norm[(int64_t)(tl.row0 + rb) * H + h];
     }
     cp_async_wait<0>();
     if (tg.cluster == 1) __syncthreads();
@@ -658,47 +708,61 @@ __global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const b
     fetch_k(1);
     fetch_v(0);
     cp_async_commit();
-    const FastScore score(s);
+    const Log2Score score(s);
     float o[HPW][VT][4];
 #pragma unroll
     for (int j = 0; j < HPW; ++j)
 #pragma unroll
         for (int i = 0; i < VT; ++i) o[j][i][0] = o[j][i][1] = o[j][i][2] = o[j][i][3] = 0.f;
-    const int vrow = lane & 7, v_key = 4 * (vrow >> 1) + (vrow & 1) + 2 * ((lane >> 3) & 1);  // the key of the operand's row lane & 15
+    // this thread's places in shared memory, stage 0 of each
+    uint32_t qa[HPW], ka[HPW], va[HPW], wd[HPW];
+    const int v_key = 4 * ((lane & 7) >> 1) + (lane & 1) + 2 * ((lane >> 3) & 1);  // the key of the operand's row lane & 15
+#pragma unroll
+    for (int j = 0; j < HPW; ++j) {
+        const int h = min(warp * HPW + j, max(nh - 1, 0)), kv = (h0 + h) / group - kv0;
+        qa[j] = sm + (uint32_t)(tg.q + ((h * 16 + (lane & 15)) * LQ + (lane >> 4) * 8) * 2);
+        ka[j] = sm + (uint32_t)(tg.k + ((kv * KV_PAGE + (lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8) * 2);
+        va[j] = sm + (uint32_t)(tg.v + ((kv * KV_PAGE + v_key) * LV + (lane >> 4) * 8) * 2);
+        wd[j] = sm + (uint32_t)(tg.w + (((h0 + h) * 16 + g) * KV_PAGE + 2 * tq) * 4);
+    }
+    const uint32_t k_stage = (uint32_t)(tg.kv * KV_PAGE * LQ * 2), v_stage = (uint32_t)(tg.kv * KV_PAGE * LV * 2), w_stage = (uint32_t)(H * 16 * KV_PAGE * 4);
+    const uint8_t* const wr0 = mp_sm + tg.w + (g * KV_PAGE + 4 * tq) * 4;
+    const float2* const mr = mix + warp * H * HPW;
     for (int v = 0; v < vis.pages; ++v) {
         const int key0 = vis.page(v) * KV_PAGE;
+        const uint32_t odd = v & 1;
+        const bool whole = key0 + KV_PAGE - 1 <= tl.pos0 && (hi - key0 < s.window || key0 + KV_PAGE <= s.keep);  // every row sees the page
 #pragma unroll
         for (int j = 0; j < HPW; ++j) {
-            const int h = warp * HPW + j;
-            if (h >= nh) continue;
-            const uint32_t qa = sm + (uint32_t)(tg.q + ((h * 16 + (lane & 15)) * LQ + (lane >> 4) * 8) * 2);
-            const uint32_t ka = sm + (uint32_t)(tg.k + ((((v & 1) * tg.kv + (h0 + h) / group - kv0) * KV_PAGE + (lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8) * 2);
+            if (warp * HPW + j >= nh) continue;
             float sc[2][4] = {};
+            const uint32_t kp = ka[j] + odd * k_stage;
 #pragma unroll 4
             for (int k = 0; k < c.dim16; k += 16) {
                 uint32_t a[4], b[4];
-                ldsm_x4(a, qa + 2 * k);
-                ldsm_x4(b, ka + 2 * k);
+                ldsm_x4(a, qa[j] + 2 * k);
+                ldsm_x4(b, kp + 2 * k);
                 mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
                 mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
-            const uint32_t wd = sm + (uint32_t)(tg.w + ((((v & 1) * H + h0 + h) * 16 + g) * KV_PAGE + 2 * tq) * 4);
+            const uint32_t wp = wd[j] + odd * w_stage;
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                const int key = key0 + 8 * n + 2 * tq;
                 float w[4];
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    w[e] = visible(s, key + e, pa) ? __expf(score(sc[n][e]) - sa[j].x) * sa[j].y : 0.f;
-                    w[2 + e] = visible(s, key + e, pb) ? __expf(score(sc[n][2 + e]) - sb[j].x) * sb[j].y : 0.f;
+                for (int e = 0; e < 4; ++e) w[e] = exp2_fast(score(sc[n][e], e < 2 ? na[j] : nb[j]));
+                if (!whole) {
+                    const int key = key0 + 8 * n + 2 * tq;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) w[e] = visible(s, key + (e & 1), e < 2 ? pa : pb) ? w[e] : 0.f;
                 }
                 if (tg.cluster == 1) {
-                    float* d = ws + ((((v & 1) * H + h0 + h) * 16 + g) * KV_PAGE + 8 * n + 2 * tq);
+                    float* d = reinterpret_cast<float*>(mp_sm + (wp - sm)) + 8 * n;
                     *reinterpret_cast<float2*>(d) = make_float2(w[0], w[1]);
                     *reinterpret_cast<float2*>(d + 8 * KV_PAGE) = make_float2(w[2], w[3]);
                 } else {
                     for (int p = 0; p < tg.cluster; ++p) {
-                        const uint32_t a = peer_smem(wd + 32u * n, p);
+                        const uint32_t a = peer_smem(wp + 32u * n, p);
                         st_peer(a, w[0], w[1]);
                         st_peer(a + 8 * KV_PAGE * 4, w[2], w[3]);
                     }
@@ -712,42 +776,46 @@ __global__ void __launch_bounds__(MP_WARPS * 32, 1) mixed_prefill_kernel(const b
         fetch_v(v + 1);
         cp_async_commit();
         if (warp * HPW >= nh) continue;
-        float p[HPW][8];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8
+        unsigned long long p[HPW][4];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8, in pairs
 #pragma unroll
         for (int j = 0; j < HPW; ++j)
 #pragma unroll
-            for (int i = 0; i < 8; ++i) p[j][i] = 0.f;
-        const float* wr = ws + ((v & 1) * H * 16 + g) * KV_PAGE + 4 * tq;
-        const float* mr = mix + warp * H * HPW;
+            for (int i = 0; i < 4; ++i) p[j][i] = 0ull;
+        const uint8_t* wr = wr0 + odd * w_stage;
 #pragma unroll 4
         for (int e = 0; e < H; ++e) {
-            const float4 a = *reinterpret_cast<const float4*>(wr + e * 16 * KV_PAGE), b = *reinterpret_cast<const float4*>(wr + (e * 16 + 8) * KV_PAGE);
-            const float w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
-#pragma unroll
-            for (int j = 0; j < HPW; ++j) {
-                const float f = mr[e * HPW + j];
-#pragma unroll
-                for (int i = 0; i < 8; ++i) p[j][i] = fmaf(f, w[i], p[j][i]);
+            const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(wr + e * 16 * KV_PAGE * 4), b = *reinterpret_cast<const ulonglong2*>(wr + (e * 16 + 8) * KV_PAGE * 4);
+            const unsigned long long w[4] = {a.x, a.y, b.x, b.y};
+            unsigned long long f[HPW];
+            if (HPW == 2) {
+                const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(mr + e * 2);
+                f[0] = t.x;
+                f[HPW - 1] = t.y;
+            } else {
+                f[0] = *reinterpret_cast<const unsigned long long*>(mr + e);
             }
+#pragma unroll
+            for (int j = 0; j < HPW; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) fma_pair(p[j][i], f[j], w[i]);
         }
 #pragma unroll
         for (int j = 0; j < HPW; ++j) {
-            const int h = warp * HPW + j;
-            if (h >= nh) continue;
+            if (warp * HPW + j >= nh) continue;
             uint32_t a[4], r[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {  // operand registers: (row g, keys 0 1), (row g + 8, keys 0 1), (row g, keys 2 3), (row g + 8, keys 2 3)
-                const float u = p[j][4 * (i & 1) + 2 * (i >> 1)], w = p[j][4 * (i & 1) + 2 * (i >> 1) + 1];
-                a[i] = pack_bf16(u, w);
+                const float2 u = pair_of(p[j][2 * (i & 1) + (i >> 1)]);
+                a[i] = pack_bf16(u.x, u.y);
                 const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[i]));
-                r[i] = pack_bf16(u - back.x, w - back.y);
+                r[i] = pack_bf16(u.x - back.x, u.y - back.y);
             }
-            const uint32_t va = sm + (uint32_t)(tg.v + ((((v & 1) * tg.kv + (h0 + h) / group - kv0) * KV_PAGE + v_key) * LV + (lane >> 4) * 8) * 2);
+            const uint32_t vp = va[j] + odd * v_stage;
 #pragma unroll
             for (int i = 0; i < VT; i += 2) {
                 if (i * 8 < c.vdim16) {
                     uint32_t b[4];
-                    ldsm_x4_t(b, va + 2 * (i * 8));
+                    ldsm_x4_t(b, vp + 2 * (i * 8));
                     mma_bf16(o[j][i], a[0], a[1], a[2], a[3], b[0], b[1]);
                     mma_bf16(o[j][i + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
                     mma_bf16(o[j][i], r[0], r[1], r[2], r[3], b[0], b[1]);
@@ -799,10 +867,11 @@ cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const Gro
             const cudaError_t e = cudaFuncSetAttribute((const void*)mp_kernel(32 << (i >> 1), 2 - (i & 1)), cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
             if (e != cudaSuccess) return e;
         }
-        return cudaFuncSetAttribute(mixed_stats_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+        const cudaError_t e = cudaFuncSetAttribute(mixed_stats_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+        return e != cudaSuccess ? e : cudaFuncSetAttribute(mixed_stats_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
     });
     if (le != cudaSuccess) return le;
-    le = launch_pdl(mixed_stats_kernel, dim3(s.heads, n_wide), dim3(MT_WARPS * 32), (size_t)3 * 64 * (c.dim16 + 8) * 2, st, (const bf16*)q, s, c, x, m, wide);
+    le = launch_pdl(s.softcap > 0.f && s.softcap <= MT_CAP ? mixed_stats_kernel<true> : mixed_stats_kernel<false>, dim3(s.heads, n_wide), dim3(MT_WARPS * 32), (size_t)3 * 64 * (c.dim16 + 8) * 2, st, (const bf16*)q, s, c, x, m, wide);
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     const MixedTiling t = mp_tiling(s, c, hpw);

@@ -98,7 +98,7 @@ inline bool mat_outs_valid(const MatArgs& a) {
         if (a.outs[i].n_end <= n || !a.outs[i].y || (a.outs[i].add && !a.outs[i].f32 && !a.f32)) return false;
         n = a.outs[i].n_end;
     }
-    return n == a.seg[0].n && (!a.norm.fn.w || (a.n_outs == 1 && a.outs[0].add));
+    return n == a.seg[0].n && (!a.norm.fn.w || (a.n_outs == 1 && a.outs[0].add && a.outs[0].act == MAT_ID));
 }
 
 // f32: plain fused multiply-adds on 32 x 32 tiles, any shape and row count.
@@ -249,22 +249,19 @@ struct GroupedInput {
     float eps;
     const float* temperature;  // factor of the queries, by position
     const float2 *cs_key, *cs_val;  // angles [pos][rot / 2] of queries and keys, [pos][vdim / 2] of values
-    // Convolution over time behind the bias: [channels][taps], the last tap on the token itself. The taps - 1 values before a
-    // slot's next token are at tail + slot * tail_stride, [taps - 1][channels], the oldest first; what stands for tokens before
-    // the sequence's start is not read. Rows of a slot may stand anywhere in a step.
+    // Convolution over time behind the bias (launch_conv_append): [taps][channels], the last tap on the token itself. The taps - 1
+    // values before a slot's next token are at tail + slot * tail_stride, [taps - 1][channels], the oldest first; what stands for
+    // tokens before the sequence's start is not read. Rows of a slot may stand anywhere in a step.
     const float* conv;
     int taps;
     float* tail;
     int64_t tail_stride;
-    const int32_t* back;       // row of the slot's token before this one, -1: in an earlier step. Null (up to 32 rows): found out
+    const int32_t* back;       // many rows: row of the slot's token before this one, -1: in an earlier step
 };
 // proj[t] (f32, row stride ldp): queries head by head, keys, values (not when shared). q[t][heads][dim16] in the compute type,
 // keys and values to the cache.
 cudaError_t launch_grouped_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in,
                                   const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st);
-// Steps with a table `back`: brings the tails up to date once the rows have been appended. ends[i]: a slot's last row in the step.
-cudaError_t launch_conv_tails(const float* proj, int ldp, const GroupedShape& s, const GroupedInput& in, const int32_t* tok_slot, const int32_t* ends,
-                              int n_ends, cudaStream_t st);
 // What else enters the scores, the softmax and the output; null: nothing.
 struct GroupedTerms {
     const float* rel;          // [heads][n_rel], added to the scaled score: by distance, the last one from there on
@@ -291,6 +288,15 @@ constexpr int GROUPED_Q_TILE = 64;
 cudaError_t launch_grouped_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const GroupedTerms& x, const GroupedTile* tiles,
                                    int n_tiles, void* out, int ldo, cudaStream_t st);
 
+// launch_grouped_append with a convolution (without norms, temperature and rotated values). Up to 32 rows: tiles null; the tails
+// are brought up to date. More: tiles of up to MIXED_Q_TILE tokens that cover the step, and launch_conv_tails behind it with every
+// slot's last row in the step.
+constexpr int MIXED_Q_TILE = 16;
+cudaError_t launch_conv_append(const float* proj, int ldp, const GroupedShape& s, const GroupedCache& c, const GroupedInput& in, const GroupedTile* tiles,
+                               int n_tiles, const int32_t* tok_slot, const int32_t* tok_pos, void* q, bool f32, int n_tok, cudaStream_t st);
+cudaError_t launch_conv_tails(const float* proj, int ldp, const GroupedShape& s, const GroupedInput& in, const int32_t* tok_slot, const int32_t* ends,
+                              int n_ends, cudaStream_t st);
+
 // ── grouped attention whose heads' softmax weights are mixed ──
 // w_h <- sum_g mix[h][g] w_g over all query heads, then head h takes the values of its own cached head. Needs every head's weights
 // where one head's mixture is made, so there are two passes: scores and softmax denominators, then weights and values. Windows may
@@ -304,7 +310,8 @@ struct MixedScratch {
     float* score;              // [rows][heads][span]
     int rows, span;            // span: mixed_span()
     float2* part;              // [rows][heads][MIXED_SPLITS]: maximum and sum of a split of the keys
-    float2* stat;              // [tokens of a step][heads]: maximum and reciprocal of the denominator
+    float2* stat;              // plain arithmetic: [tokens of a step][heads], maximum and reciprocal of the denominator
+    float* norm;               // many rows: [tokens of a step][heads], what makes a log2 score a weight
 };
 constexpr int MIXED_SPLITS = 8;
 int mixed_span(const GroupedShape& s, int max_ctx);       // most keys a token visits, whole pages
@@ -314,7 +321,6 @@ int mixed_attention_splits(const GroupedShape& s, int n_tok, int keys);
 cudaError_t launch_mixed_attention(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
                                    const int32_t* tok_slot, const int32_t* tok_pos, void* out, int ldo, int n_splits, bool f32, int n_tok, cudaStream_t st);
 // bf16, many rows: the step's tokens as tiles of GROUPED_Q_TILE (first pass) and of MIXED_Q_TILE (second).
-constexpr int MIXED_Q_TILE = 16;
 cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
                                  const GroupedTile* wide, int n_wide, const GroupedTile* narrow, int n_narrow, void* out, int ldo, cudaStream_t st);
 

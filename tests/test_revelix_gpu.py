@@ -163,7 +163,7 @@ def test_activation_far_from_zero(dtype):
 @BOTH
 def test_varied_layers_prompt_and_decode(dtype):
     cfg = M.varied()
-    W = M.weights(cfg, seed=1)
+    W = M.weights(cfg, seed=4)
     ids = M.tokens(cfg, 150)
     want, _ = L.forward(cfg, W, ids)
     eng = engine(cfg, W, dtype)
