@@ -487,16 +487,16 @@ cudaError_t launch_mixed_attention(const void* q, const GroupedShape& s, const G
 
 // ── many rows: denominators ──
 // Block per (head, tile of 64 tokens), 4 warps x 16 query rows, key tiles of four visited pages, double-buffered.
-// CAPPED: the cap is low enough to stand for the maximum.
+// CAPPED: the cap is low enough for sums of e^score as they are.
 constexpr int MT_KEYS = 64, MT_WARPS = 4;
-constexpr float MT_CAP = 40.f;  // e^(-2 * 40) is a normal float
-template <bool CAPPED>
+constexpr float MT_CAP = 70.f;
+template <bool CAPPED, int DIM>  // DIM: of the keys, padded (0: any)
 __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x,
                                                                  const MixedScratch m, const GroupedTile* __restrict__ tiles) {
     extern __shared__ __align__(16) bf16 mt_sm[];
     pdl_wait();
     pdl_trigger();
-    const int LQ = c.dim16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int D16 = DIM ? DIM : c.dim16, LQ = D16 + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     bf16 *qs = mt_sm, *ks = qs + 64 * LQ;
     const int h = blockIdx.x, kvh = h / (s.heads / s.kv_heads);
     const GroupedTile tl = tiles[blockIdx.y];
@@ -507,8 +507,8 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int r = lr + 4 * i;
-        const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * c.dim16;
-        for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
+        const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * s.heads + h) * D16;
+        for (int p = l8; p < D16 / 8; p += 8) cp_async16(qs + r * LQ + p * 8, src + p * 8, 16);
     }
     auto fetch = [&](int v0, int buf) {
         const int v = v0 + warp, page = vis.page(min(v, vis.pages - 1));
@@ -517,13 +517,14 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const int r = lr + 4 * i, in = r - warp * 16, bytes = v < vis.pages && page * KV_PAGE + in <= hi ? 16 : 0;
-            for (int p = l8; p < c.dim16 / 8; p += 8) cp_async16(kd + r * LQ + p * 8, base + in * c.ld + p * 8, bytes);
+            for (int p = l8; p < D16 / 8; p += 8) cp_async16(kd + r * LQ + p * 8, base + in * c.ld + p * 8, bytes);
         }
     };
     fetch(0, 0);
     cp_async_commit();
     const Log2Score score(s);
-    float m0 = CAPPED ? 0.f : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
+    const float mid = CAPPED ? score.top * LOG2E : 0.f;
+    float m0 = CAPPED ? -mid : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
     const int r0 = warp * 16 + g, r1 = r0 + 8, p0 = tl.pos0 + min(r0, tl.n - 1), p1 = tl.pos0 + min(r1, tl.n - 1);
     for (int v0 = 0, buf = 0; v0 < vis.pages; v0 += MT_KEYS / KV_PAGE, buf ^= 1) {
         cp_async_wait<0>();
@@ -536,7 +537,8 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
         for (int j = 0; j < 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
         const uint32_t qa = smem_addr(qs + (warp * 16 + (lane & 15)) * LQ + (lane >> 4) * 8);
         const uint32_t ka = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * LQ + ((lane >> 3) & 1) * 8);
-        for (int k = 0; k < c.dim16; k += 16) {
+#pragma unroll(DIM ? DIM / 16 : 1)
+        for (int k = 0; k < D16; k += 16) {
             uint32_t a[4];
             ldsm_x4(a, qa + 2 * k);
 #pragma unroll
@@ -553,7 +555,7 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 #pragma unroll
         for (int j = 0; j < 8; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) sc[j][e] = score(sc[j][e], 0.f);
+            for (int e = 0; e < 4; ++e) sc[j][e] = score(sc[j][e], mid);
         if (!whole) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
@@ -611,7 +613,8 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 // Block (cluster rank: a run of 8 HPW heads, tile of 16 tokens), a warp per HPW heads. Per page of keys: weights of the block's
 // heads into every block's shared memory, one barrier, then each warp mixes for its heads and multiplies with the values. Keys are
 // two stages ahead of the barrier, values one; weights alternate between two buffers. A thread's four keys of the A operand are
-// neighbours, so that it reads a head's weights as one vector; the values' rows are numbered the same way.
+// neighbours, so that it reads a head's weights as one vector; the values' rows are numbered the same way. FULL: sizes at compile
+// time (keys and values of 8 VT coordinates), a warp's heads have the same cached head and share its fragments.
 constexpr int MP_WARPS = 8, MP_MAX_CLUSTER = 8, MP_CAP = 224 * 1024;
 struct MixedTiling {
     int heads, kv, cluster;    // heads of a block, cached heads they touch at most, blocks
@@ -636,7 +639,7 @@ __host__ __device__ __forceinline__ MixedTiling mp_tiling(const GroupedShape& s,
 }
 static int mp_heads_per_warp(const GroupedShape& s, const GroupedCache& c) {  // 0: not covered
     if (s.dim > 256 || s.vdim > 256) return 0;
-    for (int hpw = 1; hpw <= (c.vdim16 <= 128 ? 2 : 1); ++hpw) {
+    for (int hpw = c.vdim16 <= 128 && s.heads > MP_WARPS ? 2 : 1; hpw > 0; --hpw) {
         const MixedTiling t = mp_tiling(s, c, hpw);
         if (t.cluster <= MP_MAX_CLUSTER && t.smem <= MP_CAP) return hpw;
     }
@@ -652,13 +655,13 @@ __device__ __forceinline__ void fma_pair(unsigned long long& d, unsigned long lo
 }
 __device__ __forceinline__ float2 pair_of(unsigned long long v) { return make_float2(__uint_as_float((uint32_t)v), __uint_as_float((uint32_t)(v >> 32))); }
 
-template <int VT, int HPW>
+template <int VT, int HPW, bool FULL>
 __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
     mixed_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
                          const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) uint8_t mp_sm[];
     const MixedTiling tg = mp_tiling(s, c, HPW);
-    const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, H = s.heads, group = H / s.kv_heads;
+    const int D16 = FULL ? 8 * VT : c.dim16, V16 = FULL ? 8 * VT : c.vdim16, LQ = D16 + 8, LV = V16 + 8, H = s.heads, group = H / s.kv_heads;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
     const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
@@ -675,24 +678,27 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
     const int hi = tl.pos0 + tl.n - 1;
     const Visit vis(s, tl.pos0, hi);
     const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages;
-    // half a warp per row, the rows of all cached heads spread over the block
-    auto fetch = [&](int v, int col, int width, int base, int ld) {
+    auto id = [&](int v) { return v < vis.pages ? pt[vis.page(v)] : 0; };
+    // page v, whose place in the pool is `page`: half a warp per row, the rows of all cached heads spread over the block
+    auto fetch = [&](int v, int page, int col, int width, int base, int ld) {
         if (v >= vis.pages) return;
-        const int page = vis.page(v), live = hi - page * KV_PAGE + 1, half = tid >> 4, l16 = tid & 15;
-        const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)pt[page] * s.kv_heads + kv0) * KV_PAGE * c.ld + col;
+        const int live = hi - vis.page(v) * KV_PAGE + 1, half = tid >> 4, l16 = tid & 15;
+        const bf16* src = reinterpret_cast<const bf16*>(c.pool) + ((int64_t)page * s.kv_heads + kv0) * KV_PAGE * c.ld + col;
         const uint32_t dst = sm + (uint32_t)(base + (v & 1) * tg.kv * KV_PAGE * ld * 2);
         for (int row = half; row < nkv * KV_PAGE; row += MP_WARPS * 2)
             for (int p = l16; p < width / 8; p += 16)
                 cp_async16_at(dst + (uint32_t)(row * ld + p * 8) * 2, src + (int64_t)row * c.ld + p * 8, row % KV_PAGE < live ? 16 : 0);
     };
-    auto fetch_k = [&](int v) { fetch(v, 0, c.dim16, tg.k, LQ); };
-    auto fetch_v = [&](int v) { fetch(v, c.dim16, c.vdim16, tg.v, LV); };
+    auto fetch_k = [&](int v, int page) { fetch(v, page, 0, D16, tg.k, LQ); };
+    auto fetch_v = [&](int v, int page) { fetch(v, page, D16, V16, tg.v, LV); };
+    int next = id(1), after = id(2);  // places of pages v + 1 and v + 2
     for (int i = warp; i < nh * 16; i += MP_WARPS) {
         const int h = i / 16, r = i % 16;
         const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * H + h0 + h) * c.dim16;
-        for (int p = lane; p < c.dim16 / 8; p += 32) cp_async16_at(sm + (uint32_t)(tg.q + (i * LQ + p * 8) * 2), src + p * 8, 16);
+        for (int p = lane; p < D16 / 8; p += 32) cp_async16_at(sm + (uint32_t)(tg.q + (i * LQ + p * 8) * 2), src + p * 8, 16);
     }
-    fetch_k(0);
+    const int page0 = id(0);
+    fetch_k(0, page0);
     cp_async_commit();
     const int ra = min(g, tl.n - 1), rb = min(g + 8, tl.n - 1), pa = tl.pos0 + ra, pb = tl.pos0 + rb;
     float na[HPW], nb[HPW];  // of the two rows: what makes a score a weight
@@ -705,8 +711,8 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
     cp_async_wait<0>();
     if (tg.cluster == 1) __syncthreads();
     else cluster_sync();  // (also: every peer has started)
-    fetch_k(1);
-    fetch_v(0);
+    fetch_k(1, next);
+    fetch_v(0, page0);
     cp_async_commit();
     const Log2Score score(s);
     float o[HPW][VT][4];
@@ -732,25 +738,51 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
         const int key0 = vis.page(v) * KV_PAGE;
         const uint32_t odd = v & 1;
         const bool whole = key0 + KV_PAGE - 1 <= tl.pos0 && (hi - key0 < s.window || key0 + KV_PAGE <= s.keep);  // every row sees the page
+        float sc[HPW][2][4];
+#pragma unroll
+        for (int j = 0; j < HPW; ++j)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) sc[j][e >> 2][e & 3] = 0.f;
+        if (FULL) {
+            if (warp * HPW < nh) {
+                const uint32_t kp = ka[0] + odd * k_stage;
+#pragma unroll
+                for (int k = 0; k < 8 * VT; k += 16) {
+                    uint32_t b[4];
+                    ldsm_x4(b, kp + 2 * k);
+#pragma unroll
+                    for (int j = 0; j < HPW; ++j) {
+                        uint32_t a[4];
+                        ldsm_x4(a, qa[j] + 2 * k);
+                        mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                        mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    }
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < HPW; ++j) {
+                if (warp * HPW + j >= nh) continue;
+                const uint32_t kp = ka[j] + odd * k_stage;
+#pragma unroll 4
+                for (int k = 0; k < c.dim16; k += 16) {
+                    uint32_t a[4], b[4];
+                    ldsm_x4(a, qa[j] + 2 * k);
+                    ldsm_x4(b, kp + 2 * k);
+                    mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
+            }
+        }
 #pragma unroll
         for (int j = 0; j < HPW; ++j) {
             if (warp * HPW + j >= nh) continue;
-            float sc[2][4] = {};
-            const uint32_t kp = ka[j] + odd * k_stage;
-#pragma unroll 4
-            for (int k = 0; k < c.dim16; k += 16) {
-                uint32_t a[4], b[4];
-                ldsm_x4(a, qa[j] + 2 * k);
-                ldsm_x4(b, kp + 2 * k);
-                mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
-            }
             const uint32_t wp = wd[j] + odd * w_stage;
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 float w[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) w[e] = exp2_fast(score(sc[n][e], e < 2 ? na[j] : nb[j]));
+                for (int e = 0; e < 4; ++e) w[e] = exp2_fast(score(sc[j][n][e], e < 2 ? na[j] : nb[j]));
                 if (!whole) {
                     const int key = key0 + 8 * n + 2 * tq;
 #pragma unroll
@@ -772,9 +804,11 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
         cp_async_wait<0>();
         if (tg.cluster == 1) __syncthreads();
         else cluster_sync();
-        fetch_k(v + 2);
-        fetch_v(v + 1);
+        fetch_k(v + 2, after);
+        fetch_v(v + 1, next);
         cp_async_commit();
+        next = after;
+        after = id(v + 3);
         if (warp * HPW >= nh) continue;
         unsigned long long p[HPW][4];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8, in pairs
 #pragma unroll
@@ -799,27 +833,48 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
 #pragma unroll
                 for (int i = 0; i < 4; ++i) fma_pair(p[j][i], f[j], w[i]);
         }
+        uint32_t a[HPW][4], r[HPW][4];
 #pragma unroll
-        for (int j = 0; j < HPW; ++j) {
-            if (warp * HPW + j >= nh) continue;
-            uint32_t a[4], r[4];
+        for (int j = 0; j < HPW; ++j)
 #pragma unroll
             for (int i = 0; i < 4; ++i) {  // operand registers: (row g, keys 0 1), (row g + 8, keys 0 1), (row g, keys 2 3), (row g + 8, keys 2 3)
                 const float2 u = pair_of(p[j][2 * (i & 1) + (i >> 1)]);
-                a[i] = pack_bf16(u.x, u.y);
-                const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[i]));
-                r[i] = pack_bf16(u.x - back.x, u.y - back.y);
+                a[j][i] = pack_bf16(u.x, u.y);
+                const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[j][i]));
+                r[j][i] = pack_bf16(u.x - back.x, u.y - back.y);
             }
-            const uint32_t vp = va[j] + odd * v_stage;
+        if (FULL) {
+            const uint32_t vp = va[0] + odd * v_stage;
 #pragma unroll
             for (int i = 0; i < VT; i += 2) {
-                if (i * 8 < c.vdim16) {
-                    uint32_t b[4];
-                    ldsm_x4_t(b, vp + 2 * (i * 8));
-                    mma_bf16(o[j][i], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    mma_bf16(o[j][i + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                    mma_bf16(o[j][i], r[0], r[1], r[2], r[3], b[0], b[1]);
-                    mma_bf16(o[j][i + 1], r[0], r[1], r[2], r[3], b[2], b[3]);
+                uint32_t b[4];
+                ldsm_x4_t(b, vp + 2 * (i * 8));
+#pragma unroll
+                for (int j = 0; j < HPW; ++j) {
+                    mma_bf16(o[j][i], a[j][0], a[j][1], a[j][2], a[j][3], b[0], b[1]);
+                    mma_bf16(o[j][i + 1], a[j][0], a[j][1], a[j][2], a[j][3], b[2], b[3]);
+                }
+#pragma unroll
+                for (int j = 0; j < HPW; ++j) {
+                    mma_bf16(o[j][i], r[j][0], r[j][1], r[j][2], r[j][3], b[0], b[1]);
+                    mma_bf16(o[j][i + 1], r[j][0], r[j][1], r[j][2], r[j][3], b[2], b[3]);
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < HPW; ++j) {
+                if (warp * HPW + j >= nh) continue;
+                const uint32_t vp = va[j] + odd * v_stage;
+#pragma unroll
+                for (int i = 0; i < VT; i += 2) {
+                    if (i * 8 < c.vdim16) {
+                        uint32_t b[4];
+                        ldsm_x4_t(b, vp + 2 * (i * 8));
+                        mma_bf16(o[j][i], a[j][0], a[j][1], a[j][2], a[j][3], b[0], b[1]);
+                        mma_bf16(o[j][i + 1], a[j][0], a[j][1], a[j][2], a[j][3], b[2], b[3]);
+                        mma_bf16(o[j][i], r[j][0], r[j][1], r[j][2], r[j][3], b[0], b[1]);
+                        mma_bf16(o[j][i + 1], r[j][0], r[j][1], r[j][2], r[j][3], b[2], b[3]);
+                    }
                 }
             }
         }
@@ -849,11 +904,22 @@ bool mixed_mma_supported(const GroupedShape& s, const GroupedCache& c) {
 }
 
 using MixedPrefillFn = void (*)(const bf16*, GroupedShape, GroupedCache, MixedTerms, MixedScratch, const GroupedTile*, bf16*, int);
-static MixedPrefillFn mp_kernel(int vdim16, int hpw) {
-    if (vdim16 <= 32) return hpw == 2 ? mixed_prefill_kernel<4, 2> : mixed_prefill_kernel<4, 1>;
-    if (vdim16 <= 64) return hpw == 2 ? mixed_prefill_kernel<8, 2> : mixed_prefill_kernel<8, 1>;
-    if (vdim16 <= 128) return hpw == 2 ? mixed_prefill_kernel<16, 2> : mixed_prefill_kernel<16, 1>;
-    return mixed_prefill_kernel<32, 1>;
+static MixedPrefillFn mp_kernel(int vdim16, int hpw, bool full) {
+    if (full) return vdim16 == 64 ? mixed_prefill_kernel<8, 2, true> : mixed_prefill_kernel<16, 2, true>;
+    if (vdim16 <= 32) return hpw == 2 ? mixed_prefill_kernel<4, 2, false> : mixed_prefill_kernel<4, 1, false>;
+    if (vdim16 <= 64) return hpw == 2 ? mixed_prefill_kernel<8, 2, false> : mixed_prefill_kernel<8, 1, false>;
+    if (vdim16 <= 128) return hpw == 2 ? mixed_prefill_kernel<16, 2, false> : mixed_prefill_kernel<16, 1, false>;
+    return mixed_prefill_kernel<32, 1, false>;
+}
+using MixedStatsFn = void (*)(const bf16*, GroupedShape, GroupedCache, MixedTerms, MixedScratch, const GroupedTile*);
+static MixedStatsFn mt_kernel(bool capped, int dim16) {
+    if (dim16 == 64) return capped ? mixed_stats_kernel<true, 64> : mixed_stats_kernel<false, 64>;
+    if (dim16 == 128) return capped ? mixed_stats_kernel<true, 128> : mixed_stats_kernel<false, 128>;
+    return capped ? mixed_stats_kernel<true, 0> : mixed_stats_kernel<false, 0>;
+}
+// The variant with sizes at compile time: two heads per warp that have the same cached head, all of them there.
+static bool mp_full(const GroupedShape& s, const GroupedCache& c, int hpw) {
+    return hpw == 2 && (s.heads / s.kv_heads) % 2 == 0 && c.dim16 == c.vdim16 && (c.dim16 == 64 || c.dim16 == 128);
 }
 
 cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
@@ -863,19 +929,23 @@ cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const Gro
     if (!hpw) return cudaErrorInvalidValue;
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
-        for (int i = 0; i < 7; ++i) {
-            const cudaError_t e = cudaFuncSetAttribute((const void*)mp_kernel(32 << (i >> 1), 2 - (i & 1)), cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+        for (int i = 0; i < 9; ++i) {
+            const MixedPrefillFn f = i < 7 ? mp_kernel(32 << (i >> 1), 2 - (i & 1), false) : mp_kernel(64 << (i - 7), 2, true);
+            const cudaError_t e = cudaFuncSetAttribute((const void*)f, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
             if (e != cudaSuccess) return e;
         }
-        const cudaError_t e = cudaFuncSetAttribute(mixed_stats_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
-        return e != cudaSuccess ? e : cudaFuncSetAttribute(mixed_stats_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+        for (int i = 0; i < 6; ++i) {
+            const cudaError_t e = cudaFuncSetAttribute((const void*)mt_kernel(i & 1, 64 * (i >> 1)), cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
+            if (e != cudaSuccess) return e;
+        }
+        return cudaSuccess;
     });
     if (le != cudaSuccess) return le;
-    le = launch_pdl(s.softcap > 0.f && s.softcap <= MT_CAP ? mixed_stats_kernel<true> : mixed_stats_kernel<false>, dim3(s.heads, n_wide), dim3(MT_WARPS * 32), (size_t)3 * 64 * (c.dim16 + 8) * 2, st, (const bf16*)q, s, c, x, m, wide);
+    le = launch_pdl(mt_kernel(s.softcap > 0.f && s.softcap <= MT_CAP, c.dim16), dim3(s.heads, n_wide), dim3(MT_WARPS * 32), (size_t)3 * 64 * (c.dim16 + 8) * 2, st, (const bf16*)q, s, c, x, m, wide);
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     const MixedTiling t = mp_tiling(s, c, hpw);
-    le = launch_pdl_cluster(mp_kernel(c.vdim16, hpw), dim3(1, n_narrow, t.cluster), dim3(MP_WARPS * 32), t.smem, st, t.cluster, (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
+    le = launch_pdl_cluster(mp_kernel(c.vdim16, hpw, mp_full(s, c, hpw)), dim3(1, n_narrow, t.cluster), dim3(MP_WARPS * 32), t.smem, st, t.cluster, (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
