@@ -9,6 +9,7 @@
 // The products' bf16 operands that stand for weights are a leading part plus its remainder; everything else is f32. Pages that hold
 // kept first keys and pages of the window are one run of visited pages.
 #include <algorithm>
+#include <atomic>
 #include <climits>
 
 #include "kernels.h"
@@ -613,8 +614,7 @@ __global__ void __launch_bounds__(MT_WARPS * 32) mixed_stats_kernel(const bf16* 
 // Block (cluster rank: a run of 8 HPW heads, tile of 16 tokens), a warp per HPW heads. Per page of keys: weights of the block's
 // heads into every block's shared memory, one barrier, then each warp mixes for its heads and multiplies with the values. Keys are
 // two stages ahead of the barrier, values one; weights alternate between two buffers. A thread's four keys of the A operand are
-// neighbours, so that it reads a head's weights as one vector; the values' rows are numbered the same way. FULL: sizes at compile
-// time (keys and values of 8 VT coordinates), a warp's heads have the same cached head and share its fragments.
+// neighbours, so that it reads a head's weights as one vector; the values' rows are numbered the same way.
 constexpr int MP_WARPS = 8, MP_MAX_CLUSTER = 8, MP_CAP = 224 * 1024;
 struct MixedTiling {
     int heads, kv, cluster;    // heads of a block, cached heads they touch at most, blocks
@@ -655,13 +655,13 @@ __device__ __forceinline__ void fma_pair(unsigned long long& d, unsigned long lo
 }
 __device__ __forceinline__ float2 pair_of(unsigned long long v) { return make_float2(__uint_as_float((uint32_t)v), __uint_as_float((uint32_t)(v >> 32))); }
 
-template <int VT, int HPW, bool FULL>
+template <int VT, int HPW>
 __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
     mixed_prefill_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
                          const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) uint8_t mp_sm[];
     const MixedTiling tg = mp_tiling(s, c, HPW);
-    const int D16 = FULL ? 8 * VT : c.dim16, V16 = FULL ? 8 * VT : c.vdim16, LQ = D16 + 8, LV = V16 + 8, H = s.heads, group = H / s.kv_heads;
+    const int LQ = c.dim16 + 8, LV = c.vdim16 + 8, H = s.heads, group = H / s.kv_heads;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
     const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
@@ -689,13 +689,13 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
             for (int p = l16; p < width / 8; p += 16)
                 cp_async16_at(dst + (uint32_t)(row * ld + p * 8) * 2, src + (int64_t)row * c.ld + p * 8, row % KV_PAGE < live ? 16 : 0);
     };
-    auto fetch_k = [&](int v, int page) { fetch(v, page, 0, D16, tg.k, LQ); };
-    auto fetch_v = [&](int v, int page) { fetch(v, page, D16, V16, tg.v, LV); };
+    auto fetch_k = [&](int v, int page) { fetch(v, page, 0, c.dim16, tg.k, LQ); };
+    auto fetch_v = [&](int v, int page) { fetch(v, page, c.dim16, c.vdim16, tg.v, LV); };
     int next = id(1), after = id(2);  // places of pages v + 1 and v + 2
     for (int i = warp; i < nh * 16; i += MP_WARPS) {
         const int h = i / 16, r = i % 16;
         const bf16* src = q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * H + h0 + h) * c.dim16;
-        for (int p = lane; p < D16 / 8; p += 32) cp_async16_at(sm + (uint32_t)(tg.q + (i * LQ + p * 8) * 2), src + p * 8, 16);
+        for (int p = lane; p < c.dim16 / 8; p += 32) cp_async16_at(sm + (uint32_t)(tg.q + (i * LQ + p * 8) * 2), src + p * 8, 16);
     }
     const int page0 = id(0);
     fetch_k(0, page0);
@@ -743,35 +743,17 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
         for (int j = 0; j < HPW; ++j)
 #pragma unroll
             for (int e = 0; e < 8; ++e) sc[j][e >> 2][e & 3] = 0.f;
-        if (FULL) {
-            if (warp * HPW < nh) {
-                const uint32_t kp = ka[0] + odd * k_stage;
 #pragma unroll
-                for (int k = 0; k < 8 * VT; k += 16) {
-                    uint32_t b[4];
-                    ldsm_x4(b, kp + 2 * k);
-#pragma unroll
-                    for (int j = 0; j < HPW; ++j) {
-                        uint32_t a[4];
-                        ldsm_x4(a, qa[j] + 2 * k);
-                        mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                        mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                    }
-                }
-            }
-        } else {
-#pragma unroll
-            for (int j = 0; j < HPW; ++j) {
-                if (warp * HPW + j >= nh) continue;
-                const uint32_t kp = ka[j] + odd * k_stage;
+        for (int j = 0; j < HPW; ++j) {
+            if (warp * HPW + j >= nh) continue;
+            const uint32_t kp = ka[j] + odd * k_stage;
 #pragma unroll 4
-                for (int k = 0; k < c.dim16; k += 16) {
-                    uint32_t a[4], b[4];
-                    ldsm_x4(a, qa[j] + 2 * k);
-                    ldsm_x4(b, kp + 2 * k);
-                    mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                }
+            for (int k = 0; k < c.dim16; k += 16) {
+                uint32_t a[4], b[4];
+                ldsm_x4(a, qa[j] + 2 * k);
+                ldsm_x4(b, kp + 2 * k);
+                mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
         }
 #pragma unroll
@@ -843,38 +825,19 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
                 const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[j][i]));
                 r[j][i] = pack_bf16(u.x - back.x, u.y - back.y);
             }
-        if (FULL) {
-            const uint32_t vp = va[0] + odd * v_stage;
+#pragma unroll
+        for (int j = 0; j < HPW; ++j) {
+            if (warp * HPW + j >= nh) continue;
+            const uint32_t vp = va[j] + odd * v_stage;
 #pragma unroll
             for (int i = 0; i < VT; i += 2) {
-                uint32_t b[4];
-                ldsm_x4_t(b, vp + 2 * (i * 8));
-#pragma unroll
-                for (int j = 0; j < HPW; ++j) {
+                if (i * 8 < c.vdim16) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, vp + 2 * (i * 8));
                     mma_bf16(o[j][i], a[j][0], a[j][1], a[j][2], a[j][3], b[0], b[1]);
                     mma_bf16(o[j][i + 1], a[j][0], a[j][1], a[j][2], a[j][3], b[2], b[3]);
-                }
-#pragma unroll
-                for (int j = 0; j < HPW; ++j) {
                     mma_bf16(o[j][i], r[j][0], r[j][1], r[j][2], r[j][3], b[0], b[1]);
                     mma_bf16(o[j][i + 1], r[j][0], r[j][1], r[j][2], r[j][3], b[2], b[3]);
-                }
-            }
-        } else {
-#pragma unroll
-            for (int j = 0; j < HPW; ++j) {
-                if (warp * HPW + j >= nh) continue;
-                const uint32_t vp = va[j] + odd * v_stage;
-#pragma unroll
-                for (int i = 0; i < VT; i += 2) {
-                    if (i * 8 < c.vdim16) {
-                        uint32_t b[4];
-                        ldsm_x4_t(b, vp + 2 * (i * 8));
-                        mma_bf16(o[j][i], a[j][0], a[j][1], a[j][2], a[j][3], b[0], b[1]);
-                        mma_bf16(o[j][i + 1], a[j][0], a[j][1], a[j][2], a[j][3], b[2], b[3]);
-                        mma_bf16(o[j][i], r[j][0], r[j][1], r[j][2], r[j][3], b[0], b[1]);
-                        mma_bf16(o[j][i + 1], r[j][0], r[j][1], r[j][2], r[j][3], b[2], b[3]);
-                    }
                 }
             }
         }
@@ -899,17 +862,223 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
     if (tg.cluster > 1) cluster_sync();  // nobody leaves while a peer may still write here
 }
 
+// The same for keys and values of 8 VT coordinates (64 or 128), an even number of query heads per cached head and more than
+// eight of them: half of the warps make the weights of a page while the other half mixes and multiplies those of the page before.
+// Either half has two heads per warp that share the fragments of their cached head. At 128 coordinates the second half needs
+// registers that the first one gives up.
+constexpr int MX_THREADS = 2 * MP_WARPS * 32, MX_FEW = 72, MX_MANY = 184;
+static_assert(MX_FEW + MX_MANY == 2 * 128, "what the halves have together is what the block was launched with");
+
+template <int VT>
+__global__ void __launch_bounds__(MX_THREADS, 1)
+    mixed_prefill_halves_kernel(const bf16* __restrict__ q, const GroupedShape s, const GroupedCache c, const MixedTerms x, const MixedScratch m,
+                                const GroupedTile* __restrict__ tiles, bf16* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) uint8_t mp_sm[];
+    constexpr int D = 8 * VT, LD = D + 8;
+    const MixedTiling tg = mp_tiling(s, c, 2);
+    const int H = s.heads, group = H / s.kv_heads, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
+    const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
+    const uint32_t sm = smem_addr(mp_sm);
+    float2* const mix = reinterpret_cast<float2*>(mp_sm + tg.mix);  // [warp][head][2], twice side by side
+    for (int i = tid; i < MP_WARPS * 2 * H; i += MX_THREADS) {
+        const int e = i / 2 % H, h = i / 2 / H * 2 + i % 2;
+        const float f = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
+        mix[i] = make_float2(f, f);
+    }
+    pdl_wait();
+    pdl_trigger();
+    const GroupedTile tl = tiles[blockIdx.y];
+    const int hi = tl.pos0 + tl.n - 1;
+    const Visit vis(s, tl.pos0, hi);
+    const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages;
+    auto id = [&](int v) { return v < vis.pages ? pt[vis.page(v)] : 0; };
+    const int row0 = tid / VT, piece = tid % VT;  // a row's pieces are neighbouring threads
+    auto fetch = [&](int v, int page, int col, int base) {
+        if (v >= vis.pages) return;
+        const int live = hi - vis.page(v) * KV_PAGE + 1;
+        const bf16* src = reinterpret_cast<const bf16*>(c.pool) + (((int64_t)page * s.kv_heads + kv0) * KV_PAGE + row0) * c.ld + col + piece * 8;
+        uint32_t dst = sm + (uint32_t)(base + (((v & 1) * tg.kv * KV_PAGE + row0) * LD + piece * 8) * 2);
+        for (int row = row0; row < nkv * KV_PAGE; row += MX_THREADS / VT) {
+            cp_async16_at(dst, src, row % KV_PAGE < live ? 16 : 0);
+            src += (int64_t)(MX_THREADS / VT) * c.ld;
+            dst += (MX_THREADS / VT) * LD * 2;
+        }
+    };
+    auto fetch_k = [&](int v, int page) { fetch(v, page, 0, tg.k); };
+    auto fetch_v = [&](int v, int page) { fetch(v, page, D, tg.v); };
+    auto meet = [&] {
+        if (tg.cluster == 1) asm volatile("bar.sync 1, %0;\n" ::"n"(MX_THREADS) : "memory");
+        else cluster_sync();
+    };
+    int next = id(1), after = id(2);  // places of pages v + 1 and v + 2
+    const int page0 = id(0);
+    // what stands between two steps of the loop: everyone is done with keys v and values v - 1, keys v + 1 and values v are there
+    auto turn = [&](int v) {
+        cp_async_wait<0>();
+        meet();
+        fetch_k(v + 2, after);
+        fetch_v(v + 1, next);
+        cp_async_commit();
+        next = after;
+        after = id(v + 3);
+    };
+    for (int i = row0; i < nh * 16; i += MX_THREADS / VT) {
+        const int h = i / 16, r = i % 16;
+        cp_async16_at(sm + (uint32_t)(tg.q + (i * LD + piece * 8) * 2), q + ((int64_t)(tl.row0 + min(r, tl.n - 1)) * H + h0 + h) * D + piece * 8, 16);
+    }
+    fetch_k(0, page0);
+    cp_async_commit();
+    cp_async_wait<0>();
+    meet();  // (also: every peer has started)
+    fetch_k(1, next);
+    fetch_v(0, page0);
+    cp_async_commit();
+    const int pair = (warp % MP_WARPS) * 2, hp = min(pair, max(nh - 2, 0)), kv = (h0 + hp) / group - kv0;  // this warp's first head
+    const bool busy = pair < nh;
+    const uint32_t stage = (uint32_t)(tg.kv * KV_PAGE * LD * 2), w_stage = (uint32_t)(H * 16 * KV_PAGE * 4);
+    if (warp < MP_WARPS) {
+        if (VT > 8) asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;\n" ::"n"(MX_FEW));
+        const int ra = min(g, tl.n - 1), rb = min(g + 8, tl.n - 1), pa = tl.pos0 + ra, pb = tl.pos0 + rb;
+        float na[2], nb[2];  // of the two rows: what makes a score a weight
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int h = min(h0 + hp + j, H - 1);
+            na[j] = m.norm[(int64_t)(tl.row0 + ra) * H + h];
+            nb[j] = m.norm[(int64_t)(tl.row0 + rb) * H + h];
+        }
+        const Log2Score score(s);
+        const uint32_t qa = sm + (uint32_t)(tg.q + ((hp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2);
+        const uint32_t ka = sm + (uint32_t)(tg.k + ((kv * KV_PAGE + (lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2);
+        const uint32_t wd = sm + (uint32_t)(tg.w + (((h0 + hp) * 16 + g) * KV_PAGE + 2 * tq) * 4);
+        for (int v = 0; v <= vis.pages; ++v) {
+            if (busy && v < vis.pages) {
+                const int key0 = vis.page(v) * KV_PAGE;
+                const bool whole = key0 + KV_PAGE - 1 <= tl.pos0 && (hi - key0 < s.window || key0 + KV_PAGE <= s.keep);  // every row sees the page
+                const uint32_t kp = ka + (v & 1) * stage, wp = wd + (v & 1) * w_stage;
+                float sc[2][2][4] = {};
+#pragma unroll
+                for (int k = 0; k < D; k += 16) {
+                    uint32_t b[4];
+                    ldsm_x4(b, kp + 2 * k);
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        uint32_t a[4];
+                        ldsm_x4(a, qa + (uint32_t)(j * 16 * LD + k) * 2);
+                        mma_bf16(sc[j][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                        mma_bf16(sc[j][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    }
+                }
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int n = 0; n < 2; ++n) {
+                        float w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) w[e] = exp2_fast(score(sc[j][n][e], e < 2 ? na[j] : nb[j]));
+                        if (!whole) {
+                            const int key = key0 + 8 * n + 2 * tq;
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) w[e] = visible(s, key + (e & 1), e < 2 ? pa : pb) ? w[e] : 0.f;
+                        }
+                        const uint32_t d = wp + (uint32_t)(j * 16 * KV_PAGE + 8 * n) * 4;
+                        if (tg.cluster == 1) {
+                            *reinterpret_cast<float2*>(mp_sm + (d - sm)) = make_float2(w[0], w[1]);
+                            *reinterpret_cast<float2*>(mp_sm + (d - sm) + 8 * KV_PAGE * 4) = make_float2(w[2], w[3]);
+                        } else {
+                            for (int p = 0; p < tg.cluster; ++p) {
+                                const uint32_t a = peer_smem(d, p);
+                                st_peer(a, w[0], w[1]);
+                                st_peer(a + 8 * KV_PAGE * 4, w[2], w[3]);
+                            }
+                        }
+                    }
+            }
+            turn(v);
+        }
+    } else {
+        if (VT > 8) asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;\n" ::"n"(MX_MANY));
+        float o[2][VT][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < VT; ++i) o[j][i][0] = o[j][i][1] = o[j][i][2] = o[j][i][3] = 0.f;
+        const int v_key = 4 * ((lane & 7) >> 1) + (lane & 1) + 2 * ((lane >> 3) & 1);  // the key of the operand's row lane & 15
+        const uint32_t va = sm + (uint32_t)(tg.v + ((kv * KV_PAGE + v_key) * LD + (lane >> 4) * 8) * 2);
+        const uint8_t* const wr0 = mp_sm + tg.w + (g * KV_PAGE + 4 * tq) * 4;
+        const float2* const mr = mix + (warp % MP_WARPS) * H * 2;
+        turn(0);
+        for (int v = 0; v < vis.pages; ++v) {
+            if (busy) {
+                unsigned long long p[2][4];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8, in pairs
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) p[j][i] = 0ull;
+                const uint8_t* wr = wr0 + (v & 1) * w_stage;
+#pragma unroll 4
+                for (int e = 0; e < H; ++e) {
+                    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(wr + e * 16 * KV_PAGE * 4), b = *reinterpret_cast<const ulonglong2*>(wr + (e * 16 + 8) * KV_PAGE * 4);
+                    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(mr + e * 2);
+                    fma_pair(p[0][0], f.x, a.x); fma_pair(p[0][1], f.x, a.y); fma_pair(p[0][2], f.x, b.x); fma_pair(p[0][3], f.x, b.y);
+                    fma_pair(p[1][0], f.y, a.x); fma_pair(p[1][1], f.y, a.y); fma_pair(p[1][2], f.y, b.x); fma_pair(p[1][3], f.y, b.y);
+                }
+                uint32_t a[2][4], r[2][4];
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {  // as in mixed_prefill_kernel
+                        const float2 u = pair_of(p[j][2 * (i & 1) + (i >> 1)]);
+                        a[j][i] = pack_bf16(u.x, u.y);
+                        const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[j][i]));
+                        r[j][i] = pack_bf16(u.x - back.x, u.y - back.y);
+                    }
+                const uint32_t vp = va + (v & 1) * stage;
+#pragma unroll
+                for (int i = 0; i < VT; i += 2) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, vp + 2 * (i * 8));
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        mma_bf16(o[j][i], a[j][0], a[j][1], a[j][2], a[j][3], b[0], b[1]);
+                        mma_bf16(o[j][i + 1], a[j][0], a[j][1], a[j][2], a[j][3], b[2], b[3]);
+                    }
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        mma_bf16(o[j][i], r[j][0], r[j][1], r[j][2], r[j][3], b[0], b[1]);
+                        mma_bf16(o[j][i + 1], r[j][0], r[j][1], r[j][2], r[j][3], b[2], b[3]);
+                    }
+                }
+            }
+            turn(v + 1);
+        }
+        if (busy) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                bf16* d = out + (int64_t)tl.row0 * ldo + (int64_t)(h0 + pair + j) * D;
+#pragma unroll
+                for (int i = 0; i < VT; ++i) {
+                    const int col = i * 8 + 2 * tq;
+                    if (g < tl.n) *reinterpret_cast<uint32_t*>(d + (int64_t)g * ldo + col) = pack_bf16(o[j][i][0], o[j][i][1]);
+                    if (g + 8 < tl.n) *reinterpret_cast<uint32_t*>(d + (int64_t)(g + 8) * ldo + col) = pack_bf16(o[j][i][2], o[j][i][3]);
+                }
+            }
+        }
+    }
+    cp_async_wait<0>();
+    if (tg.cluster > 1) cluster_sync();  // nobody leaves while a peer may still write here
+}
+
 bool mixed_mma_supported(const GroupedShape& s, const GroupedCache& c) {
     return mp_heads_per_warp(s, c) > 0 && md_mix_smem(s, c) <= MD_CAP && (size_t)(16 + MD_WARPS * MD_STAGES * KV_PAGE) * (c.dim16 + 8) * 2 <= MD_CAP;
 }
 
 using MixedPrefillFn = void (*)(const bf16*, GroupedShape, GroupedCache, MixedTerms, MixedScratch, const GroupedTile*, bf16*, int);
-static MixedPrefillFn mp_kernel(int vdim16, int hpw, bool full) {
-    if (full) return vdim16 == 64 ? mixed_prefill_kernel<8, 2, true> : mixed_prefill_kernel<16, 2, true>;
-    if (vdim16 <= 32) return hpw == 2 ? mixed_prefill_kernel<4, 2, false> : mixed_prefill_kernel<4, 1, false>;
-    if (vdim16 <= 64) return hpw == 2 ? mixed_prefill_kernel<8, 2, false> : mixed_prefill_kernel<8, 1, false>;
-    if (vdim16 <= 128) return hpw == 2 ? mixed_prefill_kernel<16, 2, false> : mixed_prefill_kernel<16, 1, false>;
-    return mixed_prefill_kernel<32, 1, false>;
+static MixedPrefillFn mp_kernel(int vdim16, int hpw) {
+    if (vdim16 <= 32) return hpw == 2 ? mixed_prefill_kernel<4, 2> : mixed_prefill_kernel<4, 1>;
+    if (vdim16 <= 64) return hpw == 2 ? mixed_prefill_kernel<8, 2> : mixed_prefill_kernel<8, 1>;
+    if (vdim16 <= 128) return hpw == 2 ? mixed_prefill_kernel<16, 2> : mixed_prefill_kernel<16, 1>;
+    return mixed_prefill_kernel<32, 1>;
 }
 using MixedStatsFn = void (*)(const bf16*, GroupedShape, GroupedCache, MixedTerms, MixedScratch, const GroupedTile*);
 static MixedStatsFn mt_kernel(bool capped, int dim16) {
@@ -917,9 +1086,18 @@ static MixedStatsFn mt_kernel(bool capped, int dim16) {
     if (dim16 == 128) return capped ? mixed_stats_kernel<true, 128> : mixed_stats_kernel<false, 128>;
     return capped ? mixed_stats_kernel<true, 0> : mixed_stats_kernel<false, 0>;
 }
-// The variant with sizes at compile time: two heads per warp that have the same cached head, all of them there.
-static bool mp_full(const GroupedShape& s, const GroupedCache& c, int hpw) {
-    return hpw == 2 && (s.heads / s.kv_heads) % 2 == 0 && c.dim16 == c.vdim16 && (c.dim16 == 64 || c.dim16 == 128);
+// The kernel in halves: null where it does not fit, or was not compiled to start with the registers that the halves share out.
+static MixedPrefillFn mx_kernel(const GroupedShape& s, const GroupedCache& c, int hpw) {
+    if (hpw != 2 || (s.heads / s.kv_heads) % 2 || s.dim != s.vdim || (s.dim != 64 && s.dim != 128)) return nullptr;
+    const MixedPrefillFn f = s.dim == 64 ? mixed_prefill_halves_kernel<8> : mixed_prefill_halves_kernel<16>;
+    static std::atomic<int> regs[2];
+    int n = regs[s.dim == 128].load(std::memory_order_relaxed);
+    if (n == 0) {
+        cudaFuncAttributes a{};
+        n = cudaFuncGetAttributes(&a, (const void*)f) == cudaSuccess ? a.numRegs : -1;
+        regs[s.dim == 128].store(n, std::memory_order_relaxed);
+    }
+    return s.dim == 64 || n == (MX_FEW + MX_MANY) / 2 ? f : nullptr;
 }
 
 cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const GroupedCache& c, const MixedTerms& x, const MixedScratch& m,
@@ -930,7 +1108,7 @@ cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const Gro
     static PerDeviceOnce once;
     cudaError_t le = once.run([] {
         for (int i = 0; i < 9; ++i) {
-            const MixedPrefillFn f = i < 7 ? mp_kernel(32 << (i >> 1), 2 - (i & 1), false) : mp_kernel(64 << (i - 7), 2, true);
+            const MixedPrefillFn f = i < 7 ? mp_kernel(32 << (i >> 1), 2 - (i & 1)) : i < 8 ? mixed_prefill_halves_kernel<8> : mixed_prefill_halves_kernel<16>;
             const cudaError_t e = cudaFuncSetAttribute((const void*)f, cudaFuncAttributeMaxDynamicSharedMemorySize, MP_CAP);
             if (e != cudaSuccess) return e;
         }
@@ -945,7 +1123,9 @@ cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const Gro
     if (le == cudaSuccess) le = count_launch_and_check();
     if (le != cudaSuccess) return le;
     const MixedTiling t = mp_tiling(s, c, hpw);
-    le = launch_pdl_cluster(mp_kernel(c.vdim16, hpw, mp_full(s, c, hpw)), dim3(1, n_narrow, t.cluster), dim3(MP_WARPS * 32), t.smem, st, t.cluster, (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
+    const MixedPrefillFn halves = mx_kernel(s, c, hpw);
+    le = launch_pdl_cluster(halves ? halves : mp_kernel(c.vdim16, hpw), dim3(1, n_narrow, t.cluster), dim3(halves ? MX_THREADS : MP_WARPS * 32), t.smem, st, t.cluster,
+                            (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 

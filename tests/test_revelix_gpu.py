@@ -74,7 +74,10 @@ LEFT = [{"scale": 0.01}, {"scale": 1.5}, {"softcap": 0.5}, {"softcap": 1e4}, {"w
         {"scaling": {"factor": 2.5, "original": 100, "fast": 1.0, "slow": 0.9}, "rot": 20}, {"conv": 1}, {"conv": 2}, {"conv": 9}, {"conv": 32}, {"kv_heads": 1}, {"kv_heads": 6},
         {"heads": 1, "kv_heads": 1}, {"heads": 9, "kv_heads": 1}, {"heads": 9, "kv_heads": 9}, {"heads": 20, "kv_heads": 1}, {"heads": 20, "kv_heads": 4}, {"heads": 21, "kv_heads": 7},
         {"heads": 24, "kv_heads": 24}, {"heads": 34, "kv_heads": 2}, {"heads": 40, "kv_heads": 5}, {"heads": 96, "kv_heads": 12}, {"dim": 1, "rot": 0}, {"dim": 130}, {"dim": 256, "vdim": 256},
-        {"vdim": 1}, {"vdim": 2}, {"vdim": 33}, {"vdim": 70}, {"vdim": 150}, {"dim": 270}, {"vdim": 300}, {"heads": 40, "kv_heads": 20, "dim": 200, "vdim": 200}]
+        {"vdim": 1}, {"vdim": 2}, {"vdim": 33}, {"vdim": 70}, {"vdim": 150}, {"dim": 270}, {"vdim": 300}, {"heads": 40, "kv_heads": 20, "dim": 200, "vdim": 200},
+        {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 64}, {"heads": 10, "kv_heads": 1, "dim": 128, "vdim": 128}, {"heads": 24, "kv_heads": 12, "dim": 128, "vdim": 128, "rot": 128},
+        {"heads": 40, "kv_heads": 5, "dim": 64, "vdim": 64, "window": 50, "softcap": 90.0}, {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "window": 4000},
+        {"heads": 16, "kv_heads": 16, "dim": 128, "vdim": 128}, {"heads": 18, "kv_heads": 6, "dim": 64, "vdim": 64}]
 
 
 @pytest.mark.parametrize("change", LEFT, ids=lambda c: "-".join(f"{k}{v}" for k, v in c.items()))
