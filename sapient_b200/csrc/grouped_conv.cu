@@ -32,6 +32,7 @@ __device__ __forceinline__ void store_two(bf16* d, int a, int b, float u, float 
 }
 
 constexpr int CA_THREADS = 128;
+static_assert(MIXED_Q_TILE <= KV_PAGE, "a tile touches two pages at most");
 // CAP: taps at most; missing older ones weigh nothing.
 template <typename T, int CAP>
 __global__ void __launch_bounds__(CA_THREADS) conv_append_kernel(const float* __restrict__ proj, int ldp, const GroupedShape s, const GroupedCache c,
@@ -49,13 +50,13 @@ __global__ void __launch_bounds__(CA_THREADS) conv_append_kernel(const float* __
 #pragma unroll
     for (int j = 0; j < CAP; ++j) {
         const int tap = j - (CAP - in.taps);
-        wa[j] = tap >= 0 && on_a ? in.conv[(int64_t)tap * channels + ca] : 0.f;
-        wb[j] = tap >= 0 && on_b ? in.conv[(int64_t)tap * channels + cb] : 0.f;
+        wa[j] = tap >= 0 && on_a ? __ldg(in.conv + (int64_t)tap * channels + ca) : 0.f;
+        wb[j] = tap >= 0 && on_b ? __ldg(in.conv + (int64_t)tap * channels + cb) : 0.f;
         ha[j] = hb[j] = 0.f;
     }
-    const float bias_a = in.bias && on_a ? in.bias[ca] : 0.f, bias_b = in.bias && on_b ? in.bias[cb] : 0.f;
-    // one token: its projected values come in, everything goes out
-    auto token = [&](int t, int slot, int pos, float x, float y) {
+    const float bias_a = in.bias && on_a ? __ldg(in.bias + ca) : 0.f, bias_b = in.bias && on_b ? __ldg(in.bias + cb) : 0.f;
+    // one token: its projected values come in, everything goes out to d
+    auto token = [&](T* d, const float2& r, float x, float y) {
         float va = wa[CAP - 1] * x, vb = wb[CAP - 1] * y;
 #pragma unroll
         for (int j = 1; j < CAP; ++j) {
@@ -66,41 +67,55 @@ __global__ void __launch_bounds__(CA_THREADS) conv_append_kernel(const float* __
         for (int j = 1; j < CAP - 1; ++j) { ha[j] = ha[j + 1]; hb[j] = hb[j + 1]; }
         if (CAP > 1) { ha[CAP - 1] = x; hb[CAP - 1] = y; }
         if (turn) {
-            const float2 r = in.cs_key[(int64_t)pos * (s.rot / 2) + u];
             const float z = va * r.x - vb * r.y;
             vb = vb * r.x + va * r.y;
             va = z;
         }
-        if (!on) return;
-        T* d;
-        if (query) {
-            d = q + ((int64_t)t * s.heads + head) * c.dim16;
-        } else {
-            const int page = c.page_table[(int64_t)slot * c.max_pages + pos / KV_PAGE], g = value ? head : head - s.heads;
-            d = reinterpret_cast<T*>(c.pool) + (((int64_t)page * s.kv_heads + g) * KV_PAGE + pos % KV_PAGE) * c.ld + (value ? c.dim16 : 0);
-        }
-        store_two(d, a, b, va, vb);
+        if (on) store_two(d, a, b, va, vb);
     };
+    const int turn_ld = s.rot / 2, g = value ? head : head - s.heads;
+    auto query_row = [&](int t) { return q + ((int64_t)t * s.heads + head) * c.dim16; };
+    auto cache_page = [&](int page) { return reinterpret_cast<T*>(c.pool) + ((int64_t)page * s.kv_heads + g) * KV_PAGE * c.ld + (value ? c.dim16 : 0); };
+    auto angle = [&](int pos) { return __ldg(in.cs_key + (int64_t)pos * turn_ld + u); };
+    // Projected values as they are, and with the bias. Two neighbours are one load where rows and heads start on even elements.
+    const bool pairs = b == a + 1 && on_b && ((ldp | at) & 1) == 0 && (reinterpret_cast<uintptr_t>(proj) & 7) == 0;
+    auto two_of = [&](int t) { return *reinterpret_cast<const float2*>(proj + (int64_t)t * ldp + ca); };
+    auto each_of = [&](int t) { return make_float2(proj[(int64_t)t * ldp + ca], proj[(int64_t)t * ldp + cb]); };
     auto projected = [&](int t, float& x, float& y) {
-        x = on_a ? proj[(int64_t)t * ldp + ca] + bias_a : 0.f;
-        y = on_b ? proj[(int64_t)t * ldp + cb] + bias_b : 0.f;
+        const float2 v = pairs ? two_of(t) : each_of(t);
+        x = on_a ? v.x + bias_a : 0.f;
+        y = on_b ? v.y + bias_b : 0.f;
     };
     if (tiles) {
         pdl_wait();
         pdl_trigger();
         const GroupedTile tl = tiles[blockIdx.y];
         const float* tail = in.tail + tl.slot * in.tail_stride;
-        float x[MIXED_Q_TILE], y[MIXED_Q_TILE];
+        const int32_t* pt = c.page_table + (int64_t)tl.slot * c.max_pages + tl.pos0 / KV_PAGE;
+        const int in0 = tl.pos0 % KV_PAGE, page0 = pt[0], page1 = in0 + tl.n > KV_PAGE ? pt[1] : 0;  // (a tile is no longer than a page)
+        // everything the tile needs is requested at once, before anything is used
+        float2 x[MIXED_Q_TILE], r[MIXED_Q_TILE];
+        if (pairs) {
 #pragma unroll
-        for (int i = 0; i < MIXED_Q_TILE; ++i)
-            if (i < tl.n) projected(tl.row0 + i, x[i], y[i]);
-        int r = in.back[tl.row0], k = 0;  // rows of the slot before the tile, as far as they have been counted
+            for (int i = 0; i < MIXED_Q_TILE; ++i) x[i] = two_of(tl.row0 + min(i, tl.n - 1));
+        } else {
+#pragma unroll
+            for (int i = 0; i < MIXED_Q_TILE; ++i) x[i] = each_of(tl.row0 + min(i, tl.n - 1));
+        }
+        if (turn) {
+#pragma unroll
+            for (int i = 0; i < MIXED_Q_TILE; ++i) r[i] = angle(tl.pos0 + min(i, tl.n - 1));
+        }
+        int near[CAP];  // mostly the row before a row is the one above it: requested at once
+#pragma unroll
+        for (int d = 0; d < CAP - 1; ++d) near[d] = d < keep ? __ldg(in.back + max(tl.row0 - d, 0)) : -1;
+        int row = near[0], k = 0;  // rows of the slot before the tile, as far as they have been counted
 #pragma unroll
         for (int d = 1; d < CAP; ++d) {
             if (d > keep || tl.pos0 < d) continue;
-            if (r >= 0) {
-                projected(r, ha[CAP - d], hb[CAP - d]);
-                r = in.back[r];
+            if (row >= 0) {
+                projected(row, ha[CAP - d], hb[CAP - d]);
+                row = d < CAP - 1 && row == tl.row0 - d ? near[d] : in.back[row];
                 ++k;
             } else {
                 const int64_t place = (int64_t)(keep + k - d) * channels;
@@ -108,9 +123,15 @@ __global__ void __launch_bounds__(CA_THREADS) conv_append_kernel(const float* __
                 if (on_b) hb[CAP - d] = tail[place + cb];
             }
         }
+        const int64_t step = query ? (int64_t)s.heads * c.dim16 : c.ld;
+        T *d = query ? query_row(tl.row0) : cache_page(page0) + (int64_t)in0 * c.ld, *const d1 = query ? nullptr : cache_page(page1);
 #pragma unroll
         for (int i = 0; i < MIXED_Q_TILE; ++i)
-            if (i < tl.n) token(tl.row0 + i, tl.slot, tl.pos0 + i, x[i], y[i]);
+            if (i < tl.n) {
+                if (!query && in0 + i == KV_PAGE) d = d1;
+                token(d, r[i], on_a ? x[i].x + bias_a : 0.f, on_b ? x[i].y + bias_b : 0.f);
+                d += step;
+            }
         return;
     }
     const int t0 = blockIdx.y, lane = threadIdx.x & 31, rows_all = gridDim.y, mine = lane < rows_all ? tok_slot[lane] : -1, slot = tok_slot[t0], pos0 = tok_pos[t0];
@@ -123,13 +144,15 @@ __global__ void __launch_bounds__(CA_THREADS) conv_append_kernel(const float* __
         if (on_a) ha[CAP - d] = tail[(int64_t)(keep - d) * channels + ca];
         if (on_b) hb[CAP - d] = tail[(int64_t)(keep - d) * channels + cb];
     }
+    const int32_t* pt = c.page_table + (int64_t)slot * c.max_pages;
     pdl_wait();
     pdl_trigger();
     for (int i = 0; rows; rows &= rows - 1, ++i) {
         const int t = __ffs(rows) - 1;
         float x, y;
         projected(t, x, y);
-        token(t, slot, pos0 + i, x, y);
+        const int pos = pos0 + i;
+        token(query ? query_row(t) : cache_page(pt[pos / KV_PAGE]) + (int64_t)(pos % KV_PAGE) * c.ld, turn ? angle(pos) : make_float2(1.f, 0.f), x, y);
     }
 #pragma unroll
     for (int d = 1; d < CAP; ++d) {
