@@ -330,12 +330,15 @@ GroupedAttentionSpec read_talking_attention(const Cfg& c) {
     m.rot = read_rotary(c, m.dim);
     m.rot.neighbours = true;
     m.biases = m.sink = m.talk = true;
-    m.conv = c.size("conv");
-    m.score_softcap = (float)c.num("softcap");
-    m.window = c.sub("mask").size("size");
-    m.keep_first = c.sub("mask").size("keep_first", 0);
+    if (c.has("conv")) m.conv = c.size("conv");
+    if (c.has("softcap")) m.score_softcap = (float)c.num("softcap");
+    if (c.has("mask")) {
+        const Cfg mask = c.sub("mask");
+        if (mask.has("size")) m.window = mask.size("size");
+        if (mask.has("keep_first")) m.keep_first = mask.size("keep_first", 0);
+    }
     if (c.err->empty() && m.conv > CONV_MAX_TAPS) c.fail("conv is above " + std::to_string(CONV_MAX_TAPS));
-    if (c.err->empty() && m.score_softcap <= 0) c.fail("softcap must be positive");
+    if (c.err->empty() && c.has("softcap") && m.score_softcap <= 0) c.fail("softcap must be positive");
     return m;
 }
 
@@ -368,12 +371,12 @@ int read_revelix(const Json& cfg, ModelPlan* out) {
             l.mixer = MIX_BOTH;
             l.grouped = read_talking_attention(m.sub("left"));
             l.grouped.at = "mix.left.";
-            l.grouped.out_scale = (float)m.num("left_scale");
+            if (m.has("left_scale")) l.grouped.out_scale = (float)m.num("left_scale");
             l.state = read_state_mixer(m.sub("right"), STATE_FORGET);
             l.state.gain = STATE_GAIN_HEAD;
             l.state.gate = STATE_GATE_NONE;
             l.state.at = "mix.right.";
-            l.state.out_scale = (float)m.num("right_scale");
+            if (m.has("right_scale")) l.state.out_scale = (float)m.num("right_scale");
         } else {
             lc.fail("type is not a mixer of this design");
             break;

@@ -222,6 +222,9 @@ def test_configuration_is_read_from_the_file():
     plain = M.varied()
     del plain["logit_scale"], plain["layers"][0]["mlp"]
     assert create(plain)[0] == _lib.SP_OK
+    m = plain["layers"][0]["mixer"]
+    del m["left_scale"], m["right_scale"], m["left"]["mask"], m["left"]["softcap"], m["left"]["conv"], m["left"]["rot"]["scaling"]
+    assert create(plain)[0] == _lib.SP_OK
 
 
 LEFT = ["layers", 0, "mixer", "left"]
@@ -229,10 +232,10 @@ LEFT = ["layers", 0, "mixer", "left"]
 
 @pytest.mark.parametrize("path,value,word", [
     (["vocab"], None, "vocab"), (["width"], 0, "width"), (["norm"], None, "norm"), (["layers"], [], "layers"), (["logit_scale"], "x", "logit_scale"),
-    (["layers", 1, "type"], "attention", "type"), (["layers", 0, "mixer", "right"], None, "right"), (["layers", 0, "mixer", "left_scale"], None, "left_scale"),
+    (["layers", 1, "type"], "attention", "type"), (["layers", 0, "mixer", "right"], None, "right"), (["layers", 0, "mixer", "left_scale"], "x", "left_scale"),
     (["layers", 0, "mixer", "right_scale"], "x", "right_scale"), (["layers", 0, "mixer", "right", "dim"], 1000, "dim"), (LEFT + ["kv_heads"], 4, "kv_heads"),
     (LEFT + ["conv"], 0, "conv"), (LEFT + ["conv"], 33, "conv"), (LEFT + ["softcap"], 0, "softcap"), (LEFT + ["mask", "size"], 0, "size"),
-    (LEFT + ["mask", "keep_first"], None, "keep_first"), (LEFT + ["scale"], None, "scale"), (LEFT + ["rot", "dims"], 22, "rot"), (LEFT + ["rot", "dims"], 7, "rot"),
+    (LEFT + ["mask", "keep_first"], -1, "keep_first"), (LEFT + ["scale"], None, "scale"), (LEFT + ["rot", "dims"], 22, "rot"), (LEFT + ["rot", "dims"], 7, "rot"),
     (LEFT + ["rot", "scaling", "factor"], 0, "scaling"), (LEFT + ["rot", "scaling", "slow"], None, "slow"), (["layers", 1, "mixer", "decay"], [0.5], "decay"),
     (["layers", 1, "mixer", "rot"], None, "rot"), (["layers", 1, "mixer", "rot", "base"], None, "base"), (["layers", 1, "mixer", "heads"], 1.5, "heads"),
     (["layers", 0, "mlp", "kind"], "moe", "kind"), (["layers", 0, "mlp", "ff"], None, "ff")], ids=str)

@@ -149,6 +149,23 @@ def test_constants_of_the_stream_and_layers_out(change, dtype):
 
 
 @BOTH
+def test_what_a_configuration_may_leave_out(dtype):
+    """No window, kept keys, cap, convolution, scales: as values that change nothing."""
+    cfg = M.config([M.parallel(M.left(window=10 ** 6, keep=0, conv=1, softcap=1e6, scaling=None), left_scale=1.0, right_scale=1.0)])
+    W = M.weights(cfg, seed=10)
+    for n in ("q", "k", "v"):
+        W[f"l0.mix.left.{n}.conv"][:] = 1.0
+    ids = M.tokens(cfg, 80)
+    want, _ = L.forward(cfg, W, ids)
+    m = cfg["layers"][0]["mixer"]
+    del m["left_scale"], m["right_scale"], m["left"]["mask"], m["left"]["softcap"], m["left"]["conv"]
+    eng = engine(cfg, W, dtype)
+    check(all_logits(eng, ids), want, dtype)
+    check(in_portions(eng, ids, [33, 1, 2], slot=1), want, dtype)
+    eng.close()
+
+
+@BOTH
 def test_activation_far_from_zero(dtype):
     cfg = M.config([M.retention(ff=61)], width=64)
     W = M.only(M.weights(cfg, seed=9), "ff")
