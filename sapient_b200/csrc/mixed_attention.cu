@@ -653,6 +653,7 @@ __device__ __forceinline__ void st_peer(uint32_t addr, float a, float b) {
 __device__ __forceinline__ void fma_pair(unsigned long long& d, unsigned long long a, unsigned long long b) {
     asm("fma.rn.f32x2 %0, %1, %2, %0;\n" : "+l"(d) : "l"(a), "l"(b));
 }
+__device__ __forceinline__ unsigned long long both(float v) { return (unsigned long long)__float_as_uint(v) << 32 | __float_as_uint(v); }
 __device__ __forceinline__ float2 pair_of(unsigned long long v) { return make_float2(__uint_as_float((uint32_t)v), __uint_as_float((uint32_t)(v >> 32))); }
 
 template <int VT, int HPW>
@@ -864,10 +865,15 @@ __global__ void __launch_bounds__(MP_WARPS * 32, HPW == 1 && VT <= 16 ? 2 : 1)
 
 // The same for keys and values of 8 VT coordinates (64 or 128), an even number of query heads per cached head and more than
 // eight of them: half of the warps make the weights of a page while the other half mixes and multiplies those of the page before.
-// Either half has two heads per warp that share the fragments of their cached head. At 128 coordinates the second half needs
-// registers that the first one gives up.
+// The second half mixes together — a thread has two neighbouring keys of a row and eight output heads, so that a weight is read
+// twice and not once per warp — and passes the mixed weights on through shared memory, leading parts and remainders. Either half
+// has two heads per warp that share the fragments of their cached head. At 128 coordinates the second half needs registers that
+// the first one gives up.
 constexpr int MX_THREADS = 2 * MP_WARPS * 32, MX_FEW = 72, MX_MANY = 184;
 static_assert(MX_FEW + MX_MANY == 2 * 128, "what the halves have together is what the block was launched with");
+constexpr int MX_HEADS = 2 * MP_WARPS, MX_PART = MX_HEADS * 16 * KV_PAGE * 2;  // heads of a block; bytes of its mixed weights' leading parts
+// Shared memory behind mp_tiling's weights: the mixing matrix [head][output head], mixed weights [part][output head][16 rows][16 keys].
+static size_t mx_smem(const GroupedShape& s, const MixedTiling& t) { return (size_t)t.mix + (size_t)s.heads * MX_HEADS * 4 + 2 * MX_PART; }
 
 template <int VT>
 __global__ void __launch_bounds__(MX_THREADS, 1)
@@ -880,11 +886,10 @@ __global__ void __launch_bounds__(MX_THREADS, 1)
     const int h0 = blockIdx.z * tg.heads, nh = min(tg.heads, H - h0);  // (a cluster's last blocks may have none)
     const int kv0 = h0 / group, nkv = nh > 0 ? (h0 + nh - 1) / group - kv0 + 1 : 0;
     const uint32_t sm = smem_addr(mp_sm);
-    float2* const mix = reinterpret_cast<float2*>(mp_sm + tg.mix);  // [warp][head][2], twice side by side
-    for (int i = tid; i < MP_WARPS * 2 * H; i += MX_THREADS) {
-        const int e = i / 2 % H, h = i / 2 / H * 2 + i % 2;
-        const float f = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
-        mix[i] = make_float2(f, f);
+    float* const mix = reinterpret_cast<float*>(mp_sm + tg.mix);
+    for (int i = tid; i < H * MX_HEADS; i += MX_THREADS) {
+        const int e = i / MX_HEADS, h = i % MX_HEADS;
+        mix[i] = h < nh ? x.mix[(int64_t)(h0 + h) * H + e] : 0.f;
     }
     pdl_wait();
     pdl_trigger();
@@ -1003,36 +1008,54 @@ __global__ void __launch_bounds__(MX_THREADS, 1)
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int i = 0; i < VT; ++i) o[j][i][0] = o[j][i][1] = o[j][i][2] = o[j][i][3] = 0.f;
-        const int v_key = 4 * ((lane & 7) >> 1) + (lane & 1) + 2 * ((lane >> 3) & 1);  // the key of the operand's row lane & 15
-        const uint32_t va = sm + (uint32_t)(tg.v + ((kv * KV_PAGE + v_key) * LD + (lane >> 4) * 8) * 2);
-        const uint8_t* const wr0 = mp_sm + tg.w + (g * KV_PAGE + 4 * tq) * 4;
-        const float2* const mr = mix + (warp % MP_WARPS) * H * 2;
+        const uint32_t va = sm + (uint32_t)(tg.v + ((kv * KV_PAGE + (lane & 15)) * LD + (lane >> 4) * 8) * 2);
+        // mixing: eight output heads from m0, row mq, keys 2 mk and the next; a row's two runs of eight keys change places every
+        // four rows, so that reads of eight rows meet every bank once
+        const int m0 = (warp & 4) * 2, mq = (warp & 3) * 4 + (lane >> 3), mk = lane & 7;
+        const uint8_t* const wr0 = mp_sm + tg.w + (mq * KV_PAGE + 2 * mk) * 4;
+        uint8_t* const parts = mp_sm + tg.mix + H * MX_HEADS * 4;
+        uint8_t* const put = parts + m0 * 16 * KV_PAGE * 2 + mq * 32 + (((mk >> 2) ^ ((mq >> 2) & 1)) * 16) + (mk & 3) * 4;
+        const uint32_t pa = smem_addr(parts) + (uint32_t)(hp * 16 * KV_PAGE * 2 + (lane & 15) * 32 + (((lane >> 4) ^ ((lane >> 2) & 1)) * 16));
         turn(0);
         for (int v = 0; v < vis.pages; ++v) {
-            if (busy) {
-                unsigned long long p[2][4];  // row g: keys 4 tq .. 4 tq + 3, then row g + 8, in pairs
+            if (m0 < nh) {
+                unsigned long long p[2][4];  // two keys, pairs of heads
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
 #pragma unroll
                     for (int i = 0; i < 4; ++i) p[j][i] = 0ull;
                 const uint8_t* wr = wr0 + (v & 1) * w_stage;
+                const float* mr = mix + m0;
 #pragma unroll 4
                 for (int e = 0; e < H; ++e) {
-                    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(wr + e * 16 * KV_PAGE * 4), b = *reinterpret_cast<const ulonglong2*>(wr + (e * 16 + 8) * KV_PAGE * 4);
-                    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(mr + e * 2);
-                    fma_pair(p[0][0], f.x, a.x); fma_pair(p[0][1], f.x, a.y); fma_pair(p[0][2], f.x, b.x); fma_pair(p[0][3], f.x, b.y);
-                    fma_pair(p[1][0], f.y, a.x); fma_pair(p[1][1], f.y, a.y); fma_pair(p[1][2], f.y, b.x); fma_pair(p[1][3], f.y, b.y);
+                    const float2 w = *reinterpret_cast<const float2*>(wr + e * 16 * KV_PAGE * 4);
+                    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(mr + e * MX_HEADS), f2 = *reinterpret_cast<const ulonglong2*>(mr + e * MX_HEADS + 4);
+                    const unsigned long long wx = both(w.x), wy = both(w.y);
+                    fma_pair(p[0][0], f.x, wx); fma_pair(p[0][1], f.y, wx); fma_pair(p[0][2], f2.x, wx); fma_pair(p[0][3], f2.y, wx);
+                    fma_pair(p[1][0], f.x, wy); fma_pair(p[1][1], f.y, wy); fma_pair(p[1][2], f2.x, wy); fma_pair(p[1][3], f2.y, wy);
                 }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 x0 = pair_of(p[0][i]), x1 = pair_of(p[1][i]);
+#pragma unroll
+                    for (int k = 0; k < 2; ++k) {
+                        const float u = k ? x0.y : x0.x, w = k ? x1.y : x1.x;
+                        const uint32_t top = pack_bf16(u, w);
+                        const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&top));
+                        uint8_t* d = put + (2 * i + k) * 16 * KV_PAGE * 2;
+                        *reinterpret_cast<uint32_t*>(d) = top;
+                        *reinterpret_cast<uint32_t*>(d + MX_PART) = pack_bf16(u - back.x, w - back.y);
+                    }
+                }
+            }
+            asm volatile("bar.sync 2, %0;\n" ::"n"(MX_THREADS / 2) : "memory");  // this half alone
+            if (busy) {
                 uint32_t a[2][4], r[2][4];
 #pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {  // as in mixed_prefill_kernel
-                        const float2 u = pair_of(p[j][2 * (i & 1) + (i >> 1)]);
-                        a[j][i] = pack_bf16(u.x, u.y);
-                        const float2 back = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[j][i]));
-                        r[j][i] = pack_bf16(u.x - back.x, u.y - back.y);
-                    }
+                for (int j = 0; j < 2; ++j) {
+                    ldsm_x4(a[j], pa + j * 16 * KV_PAGE * 2);
+                    ldsm_x4(r[j], pa + j * 16 * KV_PAGE * 2 + MX_PART);
+                }
                 const uint32_t vp = va + (v & 1) * stage;
 #pragma unroll
                 for (int i = 0; i < VT; i += 2) {
@@ -1088,7 +1111,7 @@ static MixedStatsFn mt_kernel(bool capped, int dim16) {
 }
 // The kernel in halves: null where it does not fit, or was not compiled to start with the registers that the halves share out.
 static MixedPrefillFn mx_kernel(const GroupedShape& s, const GroupedCache& c, int hpw) {
-    if (hpw != 2 || (s.heads / s.kv_heads) % 2 || s.dim != s.vdim || (s.dim != 64 && s.dim != 128)) return nullptr;
+    if (hpw != 2 || (s.heads / s.kv_heads) % 2 || s.dim != s.vdim || (s.dim != 64 && s.dim != 128) || mx_smem(s, mp_tiling(s, c, hpw)) > MP_CAP) return nullptr;
     const MixedPrefillFn f = s.dim == 64 ? mixed_prefill_halves_kernel<8> : mixed_prefill_halves_kernel<16>;
     static std::atomic<int> regs[2];
     int n = regs[s.dim == 128].load(std::memory_order_relaxed);
@@ -1124,8 +1147,8 @@ cudaError_t launch_mixed_prefill(const void* q, const GroupedShape& s, const Gro
     if (le != cudaSuccess) return le;
     const MixedTiling t = mp_tiling(s, c, hpw);
     const MixedPrefillFn halves = mx_kernel(s, c, hpw);
-    le = launch_pdl_cluster(halves ? halves : mp_kernel(c.vdim16, hpw), dim3(1, n_narrow, t.cluster), dim3(halves ? MX_THREADS : MP_WARPS * 32), t.smem, st, t.cluster,
-                            (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
+    le = launch_pdl_cluster(halves ? halves : mp_kernel(c.vdim16, hpw), dim3(1, n_narrow, t.cluster), dim3(halves ? MX_THREADS : MP_WARPS * 32),
+                            halves ? mx_smem(s, t) : t.smem, st, t.cluster, (const bf16*)q, s, c, x, m, narrow, (bf16*)out, ldo);
     return le != cudaSuccess ? le : count_launch_and_check();
 }
 
