@@ -1,10 +1,12 @@
 // Grouped attention whose heads' softmax weights are mixed before they meet the values (plan_kernels.h). A head's mixture needs the
 // normalised weights of all heads, so scores and denominators come first, weights and values second:
-//   few rows    scores_kernel leaves scores (in powers of two, below their cap) and, per split of the keys, maximum and sum; mix_kernel makes the weights of all heads
-//               where it needs them, mixes them as a small product (16 output heads x heads x keys) whose accumulators are the A
-//               operand of the product with the values, and adds the splits' shares over a cluster.
-//   many rows   stats_kernel walks the keys of 64 query rows per head; prefill_kernel has 16 query rows of all heads (a cluster
-//               where one block cannot hold them): every warp makes its heads' weights for a page of keys, all read all of them.
+//   few rows    mixed_scores_kernel leaves scores (in powers of two, below their cap) and, per split of the keys, maximum and sum;
+//               mixed_mix_kernel makes the weights of all heads where it needs them, mixes them as a small product (16 output heads x
+//               heads x keys) whose accumulators are the A operand of the product with the values, and adds the splits' shares
+//               over a cluster.
+//   many rows   mixed_stats_kernel walks the keys of 64 query rows per head; mixed_prefill_kernel has 16 query rows of all heads (a
+//               cluster where one block cannot hold them): every warp makes its heads' weights for a page of keys, all read all of
+//               them. mixed_prefill_halves_kernel does that for common sizes with half of its warps a page ahead of the others.
 //   any sizes   simple_scores_kernel, simple_mix_kernel: plain arithmetic, rows in batches that the scratch holds.
 // The products' bf16 operands that stand for weights are a leading part plus its remainder; everything else is f32. Pages that hold
 // kept first keys and pages of the window are one run of visited pages.
