@@ -40,8 +40,10 @@ __device__ __forceinline__ float mat_act(int act, float z, const float (&arg)[2]
     }
 }
 
+// tanh z = 1 - 2 / (e^(2 z) + 1): no branches, an absolute error of a few 2^-24.
+__device__ __forceinline__ float tanh_by_exp(float z) { return fmaf(-2.f, __fdividef(1.f, __expf(2.f * z) + 1.f), 1.f); }
 // The same for several values at once in a product on bf16 operands: one decision for all, fast exponentials and divisions
-// (relative errors of a few 2^-22).
+// (errors of a few 2^-22). Short, since a decoded token's product is mostly the fetching of its weights and its code.
 template <int N>
 __device__ __forceinline__ void mat_act_fast(int act, float (&z)[N], const float (&arg)[2]) {
     switch (act) {
@@ -64,14 +66,19 @@ __device__ __forceinline__ void mat_act_fast(int act, float (&z)[N], const float
                 z[i] = fmaf(arg[0] * right, right, fmaf(arg[1], __expf(left) - 1.f - left, 0.5f * z[i]));
             }
             return;
-        default:
+        case MAT_TANH:
 #pragma unroll
-            for (int i = 0; i < N; ++i) z[i] = mat_act(act, z[i], arg);
+            for (int i = 0; i < N; ++i) z[i] = tanh_by_exp(z[i]);
+            return;
+        case MAT_SOFTCAP: {
+            const bool cap = arg[1] > 0.f;
+            const float scale = cap ? arg[0] / arg[1] : arg[0];
+#pragma unroll
+            for (int i = 0; i < N; ++i) z[i] = cap ? arg[1] * tanh_by_exp(z[i] * scale) : z[i] * scale;
+        }
     }
 }
 
-// tanh z = 1 - 2 / (e^(2 z) + 1): no branches, an absolute error of a few 2^-24.
-__device__ __forceinline__ float tanh_by_exp(float z) { return fmaf(-2.f, __fdividef(1.f, __expf(2.f * z) + 1.f), 1.f); }
 __device__ __forceinline__ float tanh_norm(const TanhNorm& n, float x, int c) { return fmaf(tanhf(n.alpha * x), n.w[c], n.b[c]); }
 
 // Sum over the block, the same value in every thread. sh: one float per warp.

@@ -134,6 +134,9 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
     for (; rows; rows &= rows - 1) {
         const int64_t row = __ffs(rows) - 1;
         const float* pr = a.proj + row * a.ldp;
+        // what the outputs are multiplied by after the norm, as far as there is a thread for each: ahead of the recurrence
+        const int n = max(nh, 0) * V;
+        const float factor = tid < n ? state_factor(a, pr + co.g, h0 * V + tid) : 0.f;
         for (int hh = 0; hh < nh; ++hh) {
             const int h = h0 + hh;
             if (DELTA) {
@@ -190,7 +193,6 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
             __syncthreads();
         }
         // every warp sums the squares for itself
-        const int n = max(nh, 0) * V;
         float ss = 0.f;
         for (int i = lane; i < n; i += 32) ss = fmaf(os[i], os[i], ss);
         ss = warp_sum(ss);
@@ -207,7 +209,7 @@ __global__ void __launch_bounds__(1024) state_step_kernel(const StateArgs a, int
         }
         const float r = rsqrtf(ss / (float)count + a.s.eps);
         T* out = reinterpret_cast<T*>(a.out) + row * a.ldo + (int64_t)h0 * V;
-        for (int i = tid; i < n; i += blockDim.x) out[i] = from_f32<T>(os[i] * r * state_factor(a, pr + co.g, h0 * V + i));
+        for (int i = tid; i < n; i += blockDim.x) out[i] = from_f32<T>(os[i] * r * (i == tid ? factor : state_factor(a, pr + co.g, h0 * V + i)));
         __syncthreads();
         fresh = false;
     }
